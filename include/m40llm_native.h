@@ -513,6 +513,118 @@ int m40llm_advance_positions_async(M40llmCudaContext* ctx, uint32_t* d_positions
 int m40llm_attention_last_token_f32_gqa_static_async(M40llmCudaContext* ctx, const M40llmKVCache* kv,
                                                      uint32_t seq_id, const void* d_q_f32, uint32_t q_heads,
                                                      uint32_t seq_len, void* d_out_f32);
+/* ---------------------------------------------------------------------
+ * Layer-stack mechanisms (no counterpart in the reference): the building blocks of models whose layers mix attention
+ * and recurrent mixers, with elementwise or RMS norms before and after each sublayer. All on the decode stream unless
+ * a stream kind is given; every size is an argument. Element types: */
+#define M40LLM_DT_F16 0u
+#define M40LLM_DT_F32 1u
+#define M40LLM_DT_BF16 2u
+/* Norm kinds. RMS: x / sqrt(mean(x^2) + eps) * w. DYT (dynamic tanh, no statistics): tanh(alpha * x) * w + b. */
+#define M40LLM_NORM_NONE 0u
+#define M40LLM_NORM_RMS 1u
+#define M40LLM_NORM_DYT 2u
+#define M40LLM_ACT_SILU 0u
+#define M40LLM_ACT_GELU_TANH 1u
+/* w and b are f32 device vectors; either may be null for DYT (1 and 0), b is unused by RMS. */
+typedef struct { uint32_t kind; float eps; float alpha; const void* w; const void* b; } M40llmNorm;
+/* y = pre(x) . w^T (rows [N][K]); with w2: y = act(pre(x) . w^T) * (pre(x) . w2^T); then
+ * out = cap(residual + post(y + bias)). out may alias residual, not x. Row pitch of x is ldx elements (0 = K), of out and
+ * residual N. `post` takes NONE or DYT. exact = 1: f32 multiply-adds only (no 16-bit operand, no tensor core); exact = 0:
+ * one row streams the weights through gemv_stream, more rows use the tensor cores on the activations split into 16-bit
+ * hi + lo parts, and shapes neither takes (K % 8, K < 64, alignment, f32 weights) fall back to the f32 kernels. */
+typedef struct {
+    const void* x;
+    const void* w;
+    const void* w2;
+    void* out;
+    const void* bias;
+    const void* residual;
+    M40llmNorm pre, post;
+    uint32_t rows, K, N, ldx, w_dtype, act, exact;
+    float soft_cap; /* > 0: cap * tanh(v / cap) on the result */
+} M40llmLinear;
+int m40llm_linear_async(M40llmCudaContext* ctx, const M40llmLinear* call, uint32_t stream_kind);
+
+/* The rows of one step. Every row is one token of one sequence; the rows of a sequence are consecutive and form a
+ * segment. A cache or state slot is sequence * slot_mul + slot_add, so that several layers of equal shape share one
+ * cache object. max_len bounds position + 1 over the rows (0: unknown, the cache capacity is assumed; a step that is
+ * captured once and replayed needs 0). */
+typedef struct {
+    uint32_t rows, segments, max_segment_rows, max_len, slot_mul, slot_add;
+    const uint32_t* row_seq;  /* device [rows] */
+    const uint32_t* row_pos;  /* device [rows] */
+    const uint32_t* row_len;  /* device [rows], position + 1 */
+    const uint32_t* seg;      /* device [segments][4]: first row, rows, sequence, position of the first row */
+} M40llmStepRows;
+
+/* Dense cache with separate key and value sizes and f16 or f32 elements. f16 with k_dim == v_dim is exactly
+ * m40llm_kvcache_create; any other combination is served by m40llm_attention_rotary_async only (the entry points above
+ * return their "no dense cache" code for it). */
+M40llmKVCache* m40llm_kvcache_create_typed(M40llmCudaContext* ctx, uint32_t max_seq_len, uint32_t slots, uint32_t kv_heads,
+                                           uint32_t k_dim, uint32_t v_dim, uint32_t elem_dtype);
+
+/* Softmax attention with rotary keys and, optionally, rotary values and a per-head output gate. `packed` holds per row
+ * q [q_heads * k_dim] | k [kv_heads * k_dim] | v [kv_heads * v_dim] | gate [q_heads] (row pitch ld, f32). Per row:
+ *   q, k <- RMS norm over the whole projection (weights q_norm / k_norm, null = none), then the first 2 * k_pairs
+ *   dimensions of each head turn (pair m with m + k_pairs) by pos * k_turns[m] turns, times k_amp;
+ *   v <- pairs (m, m + v_dim / 2) turn by pos * v_turns[m] (v_turns null = values pass unchanged);
+ *   k and v are appended to the cache at the row's position;
+ *   out = softmax(scale * q . k) v over positions 0 .. pos, turned back by pos when values are rotary, and multiplied by
+ *   sigmoid(gate) when has_gate. out f32 [rows][q_heads * v_dim].
+ * The tables are f64 (turns per position = frequency / 2 pi), so the angle is reduced exactly before sine and cosine. */
+typedef struct {
+    const void* packed;
+    const void* q_norm;
+    const void* k_norm;
+    const void* k_turns; /* f64 [k_pairs] */
+    const void* v_turns; /* f64 [v_dim / 2] or null */
+    void* out;
+    uint32_t ld, q_heads, k_pairs, has_gate;
+    float eps, k_amp, scale;
+} M40llmRotaryAttention;
+int m40llm_attention_rotary_async(M40llmCudaContext* ctx, M40llmKVCache* kv, const M40llmRotaryAttention* call,
+                                  const M40llmStepRows* rows);
+
+/* Recurrent matrix state: f32 [slot][heads][value dim][key dim]. A sequence's state is zero at position 0 whatever the
+ * slot held before, so a slot that is given back needs no clearing. */
+typedef struct M40llmStateCache M40llmStateCache;
+M40llmStateCache* m40llm_statecache_create(M40llmCudaContext* ctx, uint32_t slots, uint32_t heads, uint32_t dim);
+void m40llm_statecache_destroy(M40llmStateCache* st);
+/* One slot's state to host, [heads][key dim][value dim]. Synchronous, decode stream. */
+int m40llm_statecache_debug_read(M40llmCudaContext* ctx, M40llmStateCache* st, uint32_t slot, float* out_host);
+
+/* Generalised delta rule. `packed` holds per row r | k | v | g | a (heads * dim each) | z [rank] (row pitch ld, f32).
+ *   decay = exp(decay_scale * sigmoid(w2 . tanh(z) + w0)),  rate = sigmoid(a + a_bias),  u = k / sqrt(sum k^2 + unit_eps)
+ *   S <- diag(decay) S - (rate * u) (u^T S) + k v^T,  o = S^T r,
+ *   out = (o / sqrt(mean(o^2) + eps) per head) * norm * sigmoid(g).
+ * w2 [heads * dim][rank] of w_dtype; w0, a_bias, norm f32 [heads * dim]; out f32 [rows][heads * dim]. `decay_in`, when
+ * given, holds w2 . tanh(z) for every row (f32 [rows][heads * dim], for instance from m40llm_linear_async) and w2 / z are
+ * not read. The recurrence is f32 throughout. dim <= 256, rank <= 1024. */
+typedef struct {
+    const void* packed;
+    const void* w2;
+    const void* w0;
+    const void* a_bias;
+    const void* norm;
+    const void* decay_in;
+    void* out;
+    uint32_t ld, rank, w_dtype;
+    float decay_scale, unit_eps, eps;
+} M40llmDeltaRule;
+int m40llm_delta_rule_async(M40llmCudaContext* ctx, M40llmStateCache* st, const M40llmDeltaRule* call,
+                            const M40llmStepRows* rows);
+
+/* Token embedding gather for any table type (M40LLM_DT_*); an id >= vocab as in m40llm_embed_tokens_f16_async. */
+int m40llm_embed_tokens_async(M40llmCudaContext* ctx, const void* d_table, uint32_t table_dtype,
+                              const uint32_t* d_token_ids, void* d_out_f32, uint32_t rows, uint32_t hidden,
+                              uint32_t vocab);
+/* out[r] = [a[r] | b[r]], each half `dim` wide (f32). */
+int m40llm_concat_rows_async(M40llmCudaContext* ctx, const void* d_a, const void* d_b, void* d_out, uint32_t rows,
+                             uint32_t dim);
+/* out[i] = in[index[i]] for `count` rows of `dim` f32 values; an index >= rows_in yields zeros and status bit 8. */
+int m40llm_gather_rows_async(M40llmCudaContext* ctx, const void* d_in, const uint32_t* d_index, void* d_out,
+                             uint32_t count, uint32_t dim, uint32_t rows_in);
 /* Number of kernels this library has launched on `ctx` since creation (launch accounting for benchmarks). */
 int m40llm_context_launch_count(M40llmCudaContext* ctx, uint64_t* out_count);
 /* How many times a scratch arena of `ctx` has grown since creation. Growth happens only in eager (uncaptured)

@@ -309,7 +309,7 @@ void m40_attn_pick_chunk(const M40llmCudaContext* ctx, uint32_t rows, uint32_t k
 }
 
 int m40_attention_dense(M40llmCudaContext* ctx, const M40llmKVCache* kv, const M40DenseAttnCall& c) {
-    DenseAttnArgs a;
+    DenseAttnArgs a = {};
     a.K = kv->d_k;
     a.V = kv->d_v;
     a.q = c.q;

@@ -22,6 +22,7 @@ struct DenseAttnArgs {
     uint32_t chunk;           // tokens per split (multiple of 64); split s covers [begin + s*chunk, +chunk)
     uint32_t write_partials;  // 1: always write (m,l,o) partials
     float inv_sqrt;
+    uint32_t slot_mul, slot_add;  // cache slot = sequence id * slot_mul + slot_add (slot_mul 0: the id is the slot)
 };
 
 // Host-side description of one attention call.
@@ -65,10 +66,19 @@ int m40_attention_fused_row(M40llmCudaContext* ctx, M40llmKVCache* kv, const flo
                             const uint32_t* seq_lens, uint32_t rows, uint32_t q_heads, float freq_base,
                             float freq_scale, uint32_t layout, float* q_out, float* out);
 
+// Prompt attention over a dense f16 cache (head_dim 64 or 128) for the segments of a step whose keys and values are
+// already appended; f32 q [rows][q_heads][hd], out likewise. `turn_back` (float2 cos, sin [rows][hd / 2]) rotates each
+// head's output by the inverse of its position's value rotation, `gate` (row pitch gate_ld) multiplies it by
+// sigmoid(gate[row][head]); both optional. Decode stream. Returns 0, 1 for a shape it does not take, < 0 on failure.
+int m40_attention_prefill_cache(M40llmCudaContext* ctx, const M40llmKVCache* kv, const float* q, float* out,
+                                const M40llmStepRows& rows, uint32_t q_heads, float scale, const float2* turn_back,
+                                const float* gate, uint32_t gate_ld);
+
 // Token range of (row, split): shared by both kernels so partial layouts agree.
 __device__ __forceinline__ bool attn_resolve_row(const DenseAttnArgs& a, uint32_t row, uint32_t split, uint32_t* seq,
                                                  uint32_t* t0, uint32_t* t1) {
-    const uint32_t sid = a.seq_ids ? a.seq_ids[row] : a.seq_id;
+    uint32_t sid = a.seq_ids ? a.seq_ids[row] : a.seq_id;
+    if (a.slot_mul) sid = sid * a.slot_mul + a.slot_add;
     const uint32_t len = a.seq_lens ? a.seq_lens[row] : (a.seq_len_dev ? *a.seq_len_dev : a.seq_len);
     if (sid >= a.max_batch || len == 0 || len > a.max_seq_len) {
         if (a.seq_ids && a.status && threadIdx.x == 0 && split == 0 && blockIdx.y == 0) atomicOr(a.status, 1u);

@@ -11,8 +11,13 @@
 // shared memory while the previous tile is being used, S = Q K^T and O += P V run on mma.sync m16n8k16 with f32
 // accumulation (q split into f16 hi + lo so that the scores keep f32-level accuracy, P rounded to f16), and the
 // softmax is online, base 2, in registers. Every kv row is read once per 64 q rows instead of once per q row.
+//
+// The same kernel also reads K and V straight from a dense f16 cache (CACHE): a prompt portion whose rows are already
+// appended attends everything its sequence holds, and the output may be turned back and gated before it is stored.
+#include "attention.cuh"
 #include "attention_mma.cuh"
 #include "common.cuh"
+#include "stack_math.cuh"
 
 namespace {
 using namespace attn_mma;
@@ -32,14 +37,22 @@ __global__ void __launch_bounds__(256) prefill_pack_kv_kernel(const float* __res
     }
 }
 
-template <int HD>
+struct PrefillCache {
+    const uint32_t* seg;  // [segments][4]: first row, rows, sequence, position of the first row
+    const float2* turn_back;
+    const float* gate;
+    uint32_t* status;
+    uint32_t slot_mul, slot_add, slots, max_seq_len, gate_ld, rows;
+};
+
+template <int HD, bool CACHE>
 __global__ void __launch_bounds__(128, 2) prefill_varlen_kernel(const float* __restrict__ Q, const __half* __restrict__ K,
                                                                 const __half* __restrict__ V,
                                                                 const uint32_t* __restrict__ q_offsets,
                                                                 const uint32_t* __restrict__ kv_offsets,
                                                                 const uint32_t* __restrict__ q_lens,
                                                                 const uint32_t* __restrict__ kv_lens, uint32_t q_heads,
-                                                                uint32_t kv_heads, float inv_sqrt, float* __restrict__ Out) {
+                                                                uint32_t kv_heads, float inv_sqrt, float* __restrict__ Out, PrefillCache pc) {
     constexpr int KS = HD / 16;      // k-steps of Q K^T
     constexpr int NT = HD / 8;       // n8 tiles of the output
     constexpr int CHUNKS = HD / 8;   // 16-byte f16 pieces per row
@@ -47,12 +60,26 @@ __global__ void __launch_bounds__(128, 2) prefill_varlen_kernel(const float* __r
     constexpr uint32_t TILE_ELEMS = PF_TILE * HD;
     // the last q tiles of a sequence see the most kv rows: they are scheduled first (block index reversed)
     const uint32_t b = blockIdx.z, qh = blockIdx.y, r0 = (gridDim.x - 1u - blockIdx.x) * PF_TILE;
-    const uint32_t q_len = q_lens[b], kv_len = kv_lens[b];
+    if (CACHE) {
+        pdl_wait();
+        pdl_trigger();
+    }
+    const uint32_t q_len = CACHE ? pc.seg[4 * b + 1] : q_lens[b];
+    const uint32_t kv_len = CACHE ? pc.seg[4 * b + 3] + q_len : kv_lens[b];
     if (r0 >= q_len || q_len == 0 || kv_len == 0 || q_len > kv_len) return;
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
     const uint32_t g = lane >> 2, t4 = lane & 3u;
     const uint32_t kvh = qh / (q_heads / kv_heads);
-    const size_t q_row0 = (size_t)q_offsets[b] + r0, kv_row0 = kv_offsets[b];
+    const uint32_t slot = CACHE ? pc.seg[4 * b + 2] * pc.slot_mul + pc.slot_add : 0u;
+    if (CACHE && (slot >= pc.slots || kv_len > pc.max_seq_len || (uint64_t)pc.seg[4 * b] + q_len > pc.rows)) {
+        if (threadIdx.x == 0) atomicOr(pc.status, 1u);
+        return;
+    }
+    const size_t q_row0 = (size_t)(CACHE ? pc.seg[4 * b] : q_offsets[b]) + r0;
+    // K / V row t of this kv head: kv_base + t * kv_pitch
+    const size_t kv_pitch = CACHE ? HD : (size_t)kv_heads * HD;
+    const size_t kv_base = CACHE ? kv_row_offset(slot, kvh, 0, kv_heads, pc.max_seq_len, HD)
+                                 : ((size_t)kv_offsets[b] * kv_heads + kvh) * HD;
     const uint32_t shift = kv_len - q_len;  // q row i sees kv rows 0 .. shift + i
     // rows of this thread: r0 + warp * 16 + g and + 8
     const uint32_t row_a = r0 + warp * 16u + g, row_b = row_a + 8u;
@@ -102,7 +129,7 @@ __global__ void __launch_bounds__(128, 2) prefill_varlen_kernel(const float* __r
             const uint32_t r = idx / CHUNKS, ch = idx % CHUNKS;
             const uint32_t dst = r * HD + ((ch ^ (r & 7u)) * 8);
             const uint32_t row = min(base + r, kv_end - 1u);
-            const size_t src = ((kv_row0 + row) * kv_heads + kvh) * HD + ch * 8;
+            const size_t src = kv_base + row * kv_pitch + ch * 8;
             cp_async16(dK + dst, K + src);
             cp_async16(dV + dst, V + src);
         }
@@ -198,7 +225,30 @@ __global__ void __launch_bounds__(128, 2) prefill_varlen_kernel(const float* __r
         }
     }
     // ---- normalise and store
-    const float inv_a = 1.0f / (l_run[0] > 0.0f ? l_run[0] : 1.0f), inv_b = 1.0f / (l_run[1] > 0.0f ? l_run[1] : 1.0f);
+    float inv_a = 1.0f / (l_run[0] > 0.0f ? l_run[0] : 1.0f), inv_b = 1.0f / (l_run[1] > 0.0f ? l_run[1] : 1.0f);
+    if (CACHE) {
+        const size_t ra = q_row0 + warp * 16u + g;
+        if (pc.turn_back) {  // dims d and d + HD / 2 of a row sit in this thread's n-tiles n and n + NT / 2
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+                if ((h == 0 ? row_a : row_b) >= q_len) continue;
+                const float2* t = pc.turn_back + (ra + 8u * h) * (HD / 2);
+#pragma unroll
+                for (int n = 0; n < NT / 2; ++n)
+#pragma unroll
+                    for (int j = 0; j < 2; ++j) {
+                        const float2 cs = t[n * 8 + 2 * t4 + j];
+                        const float u = o[n][2 * h + j], v = o[n + NT / 2][2 * h + j];
+                        o[n][2 * h + j] = u * cs.x + v * cs.y;
+                        o[n + NT / 2][2 * h + j] = v * cs.x - u * cs.y;
+                    }
+            }
+        }
+        if (pc.gate) {
+            if (row_a < q_len) inv_a *= m40_sigmoid(pc.gate[ra * pc.gate_ld + qh]);
+            if (row_b < q_len) inv_b *= m40_sigmoid(pc.gate[(ra + 8u) * pc.gate_ld + qh]);
+        }
+    }
     float* oa = Out + ((q_row0 + warp * 16u + g) * q_heads + qh) * HD;
     float* ob = oa + (size_t)8 * q_heads * HD;
 #pragma unroll
@@ -208,7 +258,41 @@ __global__ void __launch_bounds__(128, 2) prefill_varlen_kernel(const float* __r
     }
 }
 
+// the hd-128 kernels need more dynamic shared memory than the default limit
+bool prefill_configure(int device_id) {
+    static unsigned long long configured = 0ull;
+    const unsigned long long bit = 1ull << (device_id & 63);
+    if (configured & bit) return true;
+    const int bytes = (int)(2 * 2 * PF_TILE * 128 * sizeof(__half));
+    if (cudaFuncSetAttribute(prefill_varlen_kernel<128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes) != cudaSuccess ||
+        cudaFuncSetAttribute(prefill_varlen_kernel<128, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes) != cudaSuccess)
+        return false;
+    configured |= bit;
+    return true;
+}
+
 }  // namespace
+
+int m40_attention_prefill_cache(M40llmCudaContext* ctx, const M40llmKVCache* kv, const float* q, float* out,
+                                const M40llmStepRows& rows, uint32_t q_heads, float scale, const float2* turn_back,
+                                const float* gate, uint32_t gate_ld) {
+    const uint32_t hd = kv->head_dim;
+    if ((hd != 64 && hd != 128) || !kv->d_k || !kv->d_v || !rows.seg) return 1;
+    if ((((uintptr_t)q) & 7u) != 0u || (((uintptr_t)out) & 7u) != 0u) return 1;
+    if (!prefill_configure(ctx->device_id)) return -4;
+    const PrefillCache pc = {rows.seg, turn_back, gate, ctx->d_status, rows.slot_mul, rows.slot_add, kv->max_batch_size,
+                             kv->max_seq_len, gate_ld, rows.rows};
+    const dim3 grid((rows.max_segment_rows + PF_TILE - 1) / PF_TILE, q_heads, rows.segments);
+    const size_t smem = (size_t)2 * 2 * PF_TILE * hd * sizeof(__half);
+    const uint32_t* none = nullptr;
+    const cudaError_t e =
+        hd == 128 ? m40_launch_dependent(prefill_varlen_kernel<128, true>, grid, dim3(128), smem, ctx->decode_stream, q, kv->d_k,
+                                         kv->d_v, none, none, none, none, q_heads, kv->num_heads, scale, out, pc)
+                  : m40_launch_dependent(prefill_varlen_kernel<64, true>, grid, dim3(128), smem, ctx->decode_stream, q, kv->d_k,
+                                         kv->d_v, none, none, none, none, q_heads, kv->num_heads, scale, out, pc);
+    M40_COUNT_LAUNCH(ctx);
+    return e == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
 
 extern "C" {
 
@@ -263,20 +347,13 @@ int m40llm_attention_prefill_f32_gqa_varlen_async(M40llmCudaContext* ctx, const 
     dim3 grid((max_q + PF_TILE - 1) / PF_TILE, q_heads, batch_size);
     const float inv_sqrt = attn_inv_sqrt(head_dim);
     const size_t smem = (size_t)2 * 2 * PF_TILE * head_dim * sizeof(__half);
-    static unsigned long long configured = 0ull;
-    const unsigned long long bit = 1ull << (ctx->device_id & 63);
-    if (!(configured & bit)) {
-        if (cudaFuncSetAttribute(prefill_varlen_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                 (int)(2 * 2 * PF_TILE * 128 * sizeof(__half))) != cudaSuccess)
-            return -4;
-        configured |= bit;
-    }
+    if (!prefill_configure(ctx->device_id)) return -4;
     if (head_dim == 128)
-        prefill_varlen_kernel<128><<<grid, 128, smem, s>>>((const float*)d_q_f32, kh, vh, d_q_offsets, d_kv_offsets, d_q_lens,
-                                                           d_kv_lens, q_heads, kv_heads, inv_sqrt, (float*)d_out_f32);
+        prefill_varlen_kernel<128, false><<<grid, 128, smem, s>>>((const float*)d_q_f32, kh, vh, d_q_offsets, d_kv_offsets, d_q_lens,
+                                                           d_kv_lens, q_heads, kv_heads, inv_sqrt, (float*)d_out_f32, PrefillCache{});
     else
-        prefill_varlen_kernel<64><<<grid, 128, smem, s>>>((const float*)d_q_f32, kh, vh, d_q_offsets, d_kv_offsets, d_q_lens,
-                                                          d_kv_lens, q_heads, kv_heads, inv_sqrt, (float*)d_out_f32);
+        prefill_varlen_kernel<64, false><<<grid, 128, smem, s>>>((const float*)d_q_f32, kh, vh, d_q_offsets, d_kv_offsets, d_q_lens,
+                                                          d_kv_lens, q_heads, kv_heads, inv_sqrt, (float*)d_out_f32, PrefillCache{});
     M40_COUNT_LAUNCH(ctx);
     return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

@@ -98,6 +98,12 @@ struct M40llmKVCache {
     uint32_t representatives;
     uint32_t representative_policy;
     uint32_t fp16_k_q4_v_backing;
+    // Dense caches whose values differ in size from the keys or whose elements are f32 (m40llm_kvcache_create_typed):
+    // head-major like d_k / d_v, which stay null so that the f16 entry points refuse such a cache.
+    void* d_typed_k;
+    void* d_typed_v;
+    uint32_t v_dim;      // 0: head_dim
+    uint32_t elem_f32;
 };
 
 // element offset of (slot, head, token, 0) in a head-major [slot][head][tokens][hd] array

@@ -17,6 +17,9 @@
 // SM are resident. Partials land in scratch and a small second kernel adds the K splits and applies the
 // epilogue (bias, residual, or SiLU(gate)*up).
 //
+// Prompt rows (M > 256) are cut into blocks of 128 on grid.z. Whenever one problem needs no K split, the epilogue warps
+// apply bias, post norm, residual and soft cap themselves and store the result: no partials, no second kernel.
+//
 // Every wait is bounded: a wait that runs out sets bit 2 of the context's device status word, the
 // CTA stops issuing work, frees its TMEM and returns.
 #include <cuda.h>
@@ -39,6 +42,16 @@ struct TcArgs {
     uint32_t kblocks_per_split, kblocks_total;
     uint32_t use_lo;           // 1: activations carry a lo part (second MMA)
     uint32_t stages;
+    uint32_t m_block;          // activation rows per grid.z block
+    uint32_t fmt_bits;         // operand type bits of the instruction descriptor (0: f16, see idesc_bf16())
+    // direct != 0: one problem, no K split; the result is finished and stored by the epilogue warps
+    uint32_t direct, n_out;
+    float* out;
+    const float* bias;
+    const float* residual;
+    const float* post_w;
+    const float* post_b;
+    M40Tail tail;
 };
 
 __global__ void __launch_bounds__(192, 1) gemm_tc_f16_kernel(const __grid_constant__ CUtensorMap tmW0,
@@ -51,6 +64,8 @@ __global__ void __launch_bounds__(192, 1) gemm_tc_f16_kernel(const __grid_consta
     unsigned char* smem = smem_unaligned + ((1024u - (smem_u32(smem_unaligned) & 1023u)) & 1023u);
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u;
     const uint32_t tile = blockIdx.x, ksplit = blockIdx.y;
+    const uint32_t m_base = blockIdx.z * a.m_block;
+    const uint32_t m_live = min(a.m_block, a.M - m_base);
     const uint32_t a_bytes = BLOCK_N * BLOCK_K * 2;                 // 16 KB
     const uint32_t b_bytes = a.M_pad * BLOCK_K * 2;                 // per hi / lo part
     const uint32_t stage_bytes = a_bytes + (a.use_lo ? 2u : 1u) * b_bytes;
@@ -108,8 +123,8 @@ __global__ void __launch_bounds__(192, 1) gemm_tc_f16_kernel(const __grid_consta
             for (uint32_t i = 0; i < pre; ++i) {
                 unsigned char* st = stage_base + i * stage_bytes;
                 const int kx = (int)((kb0 + i) * BLOCK_K);
-                tma_load_2d(st + a_bytes, &tmXh, &full[i], kx, 0);
-                if (a.use_lo) tma_load_2d(st + a_bytes + b_bytes, &tmXl, &full[i], kx, 0);
+                tma_load_2d(st + a_bytes, &tmXh, &full[i], kx, (int)m_base);
+                if (a.use_lo) tma_load_2d(st + a_bytes + b_bytes, &tmXl, &full[i], kx, (int)m_base);
             }
             for (uint32_t i = pre; i < n_kb; ++i) {
                 const uint32_t s = i % a.stages, round = i / a.stages;
@@ -119,14 +134,14 @@ __global__ void __launch_bounds__(192, 1) gemm_tc_f16_kernel(const __grid_consta
                 mbar_expect_tx(&full[s], stage_bytes);
                 const int kx = (int)((kb0 + i) * BLOCK_K);
                 tma_load_2d(st, tmW, &full[s], kx, (int)row0);
-                tma_load_2d(st + a_bytes, &tmXh, &full[s], kx, 0);
-                if (a.use_lo) tma_load_2d(st + a_bytes + b_bytes, &tmXl, &full[s], kx, 0);
+                tma_load_2d(st + a_bytes, &tmXh, &full[s], kx, (int)m_base);
+                if (a.use_lo) tma_load_2d(st + a_bytes + b_bytes, &tmXl, &full[s], kx, (int)m_base);
             }
         }
     } else if (warp == 1) {
         // ---------------- MMA issuer
         if (lane == 0) {
-            const uint32_t idesc = make_idesc(acc_cols);
+            const uint32_t idesc = make_idesc(acc_cols) | a.fmt_bits;
             bool ok = true;
             for (uint32_t i = 0; i < n_kb && ok; ++i) {
                 const uint32_t s = i % a.stages, round = i / a.stages;
@@ -155,7 +170,14 @@ __global__ void __launch_bounds__(192, 1) gemm_tc_f16_kernel(const __grid_consta
         ok = __all_sync(0xffffffffu, ok);  // tcgen05.ld is warp-collective
         tc_fence_after();
         const uint32_t n_glob = tile * BLOCK_N + lane_group * 32 + lane;
-        float* dst = a.partial + (size_t)ksplit * a.M * a.n_total + n_glob;
+        float* dst = a.partial + ((size_t)ksplit * a.M + m_base) * a.n_total + n_glob;
+        const bool n_ok = n_glob < a.n_out;  // direct mode: one problem, so the padded column is the output column
+        float bias = 0.0f, pw = 1.0f, pb = 0.0f;
+        if (a.direct && n_ok) {
+            if (a.bias) bias = a.bias[n_glob];
+            if (a.post_w) pw = a.post_w[n_glob];
+            if (a.post_b) pb = a.post_b[n_glob];
+        }
         for (uint32_t c = 0; c < a.M_pad; c += 8) {
             float v[8];
             if (ok) {
@@ -170,9 +192,22 @@ __global__ void __launch_bounds__(192, 1) gemm_tc_f16_kernel(const __grid_consta
 #pragma unroll
                 for (int j = 0; j < 8; ++j) v[j] = 0.0f;
             }
+            if (a.direct) {
+                float res[8];
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {  // unconditional loads (clamped), so that the eight go out together
+                    const uint32_t m = m_base + min(c + j, m_live - 1u);
+                    res[j] = a.residual ? a.residual[(size_t)m * a.n_out + (n_ok ? n_glob : 0u)] : 0.0f;
+                }
+#pragma unroll
+                for (int j = 0; j < 8; ++j)
+                    if (n_ok && c + j < m_live)
+                        a.out[(size_t)(m_base + c + j) * a.n_out + n_glob] = m40_tail(a.tail, v[j], bias, pw, pb, res[j]);
+                continue;
+            }
 #pragma unroll
             for (int j = 0; j < 8; ++j)
-                if (c + j < a.M) dst[(size_t)(c + j) * a.n_total] = v[j];
+                if (c + j < m_live) dst[(size_t)(c + j) * a.n_total] = v[j];
         }
     }
     if (*abort_flag && threadIdx.x == 64) atomicOr(a.status, 4u);
@@ -268,6 +303,69 @@ __global__ void __launch_bounds__(256) norm_split_rows_kernel(const float* __res
         split_store4(*reinterpret_cast<const float4*>(xr + k), norm_w4(w, w_f32, k), scale, hr + k, lr + k);
 }
 
+// Rows of any pitch -> hi / lo copies of type T, with an optional dynamic tanh or RMS norm. One CTA per row.
+template <typename T>
+__device__ __forceinline__ T to_half_type(float v);
+template <>
+__device__ __forceinline__ __half to_half_type<__half>(float v) { return __float2half_rn(v); }
+template <>
+__device__ __forceinline__ __nv_bfloat16 to_half_type<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
+struct SplitRowsArgs {
+    const float* x;
+    const void* w;
+    const float* b;
+    uint32_t K, ldx;
+    int kind;   // M40LLM_NORM_*
+    int w_f32;  // RMS weights: as in norm_split_rows_kernel
+    float eps, alpha;
+};
+template <typename T>
+__global__ void __launch_bounds__(256) split_rows_kernel(SplitRowsArgs a, T* __restrict__ hi, T* __restrict__ lo) {
+    __shared__ float red[8];
+    pdl_wait();
+    pdl_trigger();
+    const float* xr = a.x + (size_t)blockIdx.x * a.ldx;
+    T* hr = hi + (size_t)blockIdx.x * a.K;
+    T* lr = lo + (size_t)blockIdx.x * a.K;
+    float scale = 1.0f;
+    if (a.kind == (int)M40LLM_NORM_RMS) {
+        float ss = 0.0f;
+        for (uint32_t k = threadIdx.x * 4u; k < a.K; k += 1024u) {
+            const float4 v = *reinterpret_cast<const float4*>(xr + k);
+            ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        }
+        ss = warp_sum(ss);
+        if ((threadIdx.x & 31u) == 0u) red[threadIdx.x >> 5] = ss;
+        __syncthreads();
+        float tot = 0.0f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) tot += red[i];
+        scale = rsqrtf(tot / (float)a.K + a.eps);
+    }
+    const float* wf = reinterpret_cast<const float*>(a.w);
+    for (uint32_t k = threadIdx.x * 4u; k < a.K; k += 1024u) {
+        const float4 v = *reinterpret_cast<const float4*>(xr + k);
+        float y[4] = {v.x, v.y, v.z, v.w};
+        if (a.kind == (int)M40LLM_NORM_DYT) {
+            const float4 w = m40_vec4_or(wf, k, 1.0f), b = m40_vec4_or(a.b, k, 0.0f);
+            y[0] = tanhf(a.alpha * y[0]) * w.x + b.x, y[1] = tanhf(a.alpha * y[1]) * w.y + b.y;
+            y[2] = tanhf(a.alpha * y[2]) * w.z + b.z, y[3] = tanhf(a.alpha * y[3]) * w.w + b.w;
+        } else if (a.kind == (int)M40LLM_NORM_RMS) {
+            const float4 w = norm_w4(a.w, a.w_f32, k);
+            y[0] *= scale * w.x, y[1] *= scale * w.y, y[2] *= scale * w.z, y[3] *= scale * w.w;
+        }
+        T h[4], l[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            h[i] = to_half_type<T>(y[i]);
+            l[i] = to_half_type<T>(y[i] - m40_load_elem(&h[i]));
+        }
+        *reinterpret_cast<uint2*>(hr + k) = *reinterpret_cast<const uint2*>(h);
+        *reinterpret_cast<uint2*>(lr + k) = *reinterpret_cast<const uint2*>(l);
+    }
+}
+
 // Adds the K splits and applies the epilogue. Thread (n, lane of 2) walks 8 activation rows of one problem.
 // mode 0: C = sum (+ bias[n]) (+ residual[m][n]);  mode 1: problems 0/1 are gate/up, C = silu(gate) * up.
 struct EpiArgs {
@@ -280,6 +378,11 @@ struct EpiArgs {
     uint32_t problems, M, n_total, k_splits, mode;
     uint32_t rope_on;
     M40TcRopeAppend rope;
+    int act;             // mode 1
+    uint32_t tail_on;    // problem 0: bias, post norm, residual and soft cap in m40_tail's order
+    M40Tail tail;
+    const float* post_w;
+    const float* post_b;
 };
 
 __global__ void __launch_bounds__(256) gemm_tc_epilogue_kernel(EpiArgs e) {
@@ -327,7 +430,13 @@ __global__ void __launch_bounds__(256) gemm_tc_epilogue_kernel(EpiArgs e) {
         if (m >= e.M) continue;
         float r = acc[i];
         if (e.mode == 1) {
-            e.out[0][(size_t)m * e.N[0] + n] = (r / (1.0f + expf(-r))) * up[i];
+            e.out[0][(size_t)m * e.N[0] + n] = m40_act(e.act, r) * up[i];
+            continue;
+        }
+        if (e.tail_on) {
+            const size_t at = (size_t)m * e.N[0] + n;
+            e.out[0][at] = m40_tail(e.tail, r, e.bias[0] ? e.bias[0][n] : 0.0f, e.post_w ? e.post_w[n] : 1.0f,
+                                    e.post_b ? e.post_b[n] : 0.0f, e.residual[0] ? e.residual[0][at] : 0.0f);
             continue;
         }
         if (e.bias[p]) r += e.bias[p][n];
@@ -379,15 +488,15 @@ EncodeTiledFn get_encode() {
     return fn;
 }
 
-// 2D f16 tensor [rows][cols] row-major, box [box_rows][64], 128-byte swizzle, zero fill out of bounds.
-bool make_map_f16(CUtensorMap* map, const void* base, uint64_t rows, uint64_t cols, uint32_t box_rows) {
+// 2D f16 (or bf16) tensor [rows][cols] row-major, box [box_rows][64], 128-byte swizzle, zero fill out of bounds.
+bool make_map_f16(CUtensorMap* map, const void* base, uint64_t rows, uint64_t cols, uint32_t box_rows, bool bf16 = false) {
     EncodeTiledFn enc = get_encode();
     if (!enc) return false;
     const cuuint64_t dims[2] = {cols, rows};
     const cuuint64_t strides[1] = {cols * 2};
     const cuuint32_t box[2] = {BLOCK_K, box_rows};
     const cuuint32_t estr[2] = {1, 1};
-    return enc(map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
+    return enc(map, bf16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
                CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
                CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
@@ -420,14 +529,21 @@ bool m40_gemm_tc_supported(int M, int K, int problems, const void* const* W) {
 
 int m40_gemm_tc_f16(M40llmCudaContext* ctx, cudaStream_t s, uint32_t stream_kind, const float* X, int M, int K,
                     int problems, const __half* const* W, const int* N, float* const* out, const float* const* bias,
-                    const float* const* residual, int mode, const M40GemvNorm* norm, const M40TcRopeAppend* rope) {
+                    const float* const* residual, int mode, const M40GemvNorm* norm, const M40TcRopeAppend* rope,
+                    const M40TcExt* ext) {
+    const bool bf16 = ext && ext->bf16;
+    if (!ext && M > 256) return -2;
     if (rope) {
         if (problems != 3 || mode != 0 || rope->head_dim == 0 || rope->head_dim % 2 != 0) return -2;
         for (int p = 0; p < 3; ++p)
             if (N[p] % 128 != 0 || N[p] % (int)rope->head_dim != 0) return -2;
     }
-    const uint32_t M_pad = (uint32_t)((M + 15) / 16 * 16);
+    const uint32_t m_block = M > 256 ? 128u : (uint32_t)M;
+    const uint32_t m_blocks = ((uint32_t)M + m_block - 1) / m_block;
+    const uint32_t M_pad = (m_block + 15) / 16 * 16;
     TcArgs a = {};
+    a.m_block = m_block;
+    a.fmt_bits = bf16 ? idesc_bf16() : 0u;
     a.M = (uint32_t)M;
     a.M_pad = M_pad;
     a.K = (uint32_t)K;
@@ -452,18 +568,19 @@ int m40_gemm_tc_f16(M40llmCudaContext* ctx, cudaStream_t s, uint32_t stream_kind
     const size_t smem = (size_t)stages * stage_bytes + (2 * stages + 1) * 8 + 16 + 1024;
     const uint32_t ctas_per_sm = smem <= 110u * 1024u ? 2u : 1u;
     // K splits: fill about one wave of resident CTAs, keep at least 4 k-blocks per split
-    uint32_t ks = ((uint32_t)ctx->sm_count * ctas_per_sm) / tiles;
+    uint32_t ks = ((uint32_t)ctx->sm_count * ctas_per_sm) / (tiles * m_blocks);
     if (ks < 1) ks = 1;
     const uint32_t ks_max = a.kblocks_total / 4 ? a.kblocks_total / 4 : 1;
     if (ks > ks_max) ks = ks_max;
     if (ks > 16) ks = 16;
     a.kblocks_per_split = (a.kblocks_total + ks - 1) / ks;
     ks = (a.kblocks_total + a.kblocks_per_split - 1) / a.kblocks_per_split;
+    const bool direct = ext && ks == 1 && problems == 1 && mode == 0 && !rope;
 
     // scratch: [hi][lo] activation copies, then the partials
     const size_t act_elems = (size_t)M * K;
     const size_t act_bytes = ((act_elems * 2 + 255) / 256) * 256;
-    const size_t part_bytes = (size_t)ks * M * a.n_total * sizeof(float);
+    const size_t part_bytes = direct ? 0 : (size_t)ks * M * a.n_total * sizeof(float);
     unsigned char* scratch = (unsigned char*)m40_ensure_scratch(ctx, stream_kind, 2 * act_bytes + part_bytes);
     if (!scratch) return -2;
     __half* xh = (__half*)scratch;
@@ -474,12 +591,49 @@ int m40_gemm_tc_f16(M40llmCudaContext* ctx, cudaStream_t s, uint32_t stream_kind
     CUtensorMap mW[3], mXh, mXl;
     for (int p = 0; p < 3; ++p) {
         const int q = p < problems ? p : 0;
-        if (!make_map_f16(&mW[p], W[q], (uint64_t)N[q], (uint64_t)K, BLOCK_N)) return -2;
+        if (!make_map_f16(&mW[p], W[q], (uint64_t)N[q], (uint64_t)K, BLOCK_N, bf16)) return -2;
     }
-    if (!make_map_f16(&mXh, xh, (uint64_t)M, (uint64_t)K, M_pad)) return -2;
-    if (!make_map_f16(&mXl, a.use_lo ? xl : xh, (uint64_t)M, (uint64_t)K, M_pad)) return -2;
+    if (!make_map_f16(&mXh, xh, (uint64_t)M, (uint64_t)K, M_pad, bf16)) return -2;
+    if (!make_map_f16(&mXl, a.use_lo ? xl : xh, (uint64_t)M, (uint64_t)K, M_pad, bf16)) return -2;
 
-    if (m40_split_activations(ctx, s, X, xh, xl, M, K, norm) != 0) return -2;
+    if (ext) {
+        SplitRowsArgs sa = {};
+        sa.x = X;
+        sa.K = (uint32_t)K;
+        sa.ldx = ext->ldx ? (uint32_t)ext->ldx : (uint32_t)K;
+        if (K % 4 != 0 || sa.ldx % 4 != 0 || (((uintptr_t)X) & 15u) != 0u) return -2;
+        if (norm && norm->dyt) {
+            sa.kind = (int)M40LLM_NORM_DYT;
+            sa.w = norm->w;
+            sa.b = norm->b;
+            sa.alpha = norm->alpha;
+            if (((((uintptr_t)norm->w) | ((uintptr_t)norm->b)) & 15u) != 0u) return -2;
+        } else if (norm && norm->w) {
+            sa.kind = (int)M40LLM_NORM_RMS;
+            sa.w = norm->w;
+            sa.eps = norm->eps;
+            const bool w_vec = (((uintptr_t)norm->w) & (norm->w_is_f32 ? 15u : 7u)) == 0u;
+            sa.w_f32 = (norm->w_is_f32 ? 1 : 0) | (w_vec ? 0 : 2);
+        }
+        const cudaError_t es =
+            bf16 ? m40_launch_dependent(split_rows_kernel<__nv_bfloat16>, dim3((unsigned)M), dim3(256), 0, s, sa,
+                                        (__nv_bfloat16*)xh, (__nv_bfloat16*)xl)
+                 : m40_launch_dependent(split_rows_kernel<__half>, dim3((unsigned)M), dim3(256), 0, s, sa, xh, xl);
+        M40_COUNT_LAUNCH(ctx);
+        if (es != cudaSuccess) return -2;
+    } else if (m40_split_activations(ctx, s, X, xh, xl, M, K, norm) != 0) {
+        return -2;
+    }
+    if (ext) a.tail = ext->tail;
+    if (direct) {
+        a.direct = 1u;
+        a.n_out = (uint32_t)N[0];
+        a.out = out[0];
+        a.bias = bias ? bias[0] : nullptr;
+        a.residual = residual ? residual[0] : nullptr;
+        a.post_w = ext->post_w;
+        a.post_b = ext->post_b;
+    }
     static unsigned long long configured = 0ull;
     const unsigned long long bit = 1ull << (ctx->device_id & 63);
     if (!(configured & bit)) {
@@ -487,12 +641,20 @@ int m40_gemm_tc_f16(M40llmCudaContext* ctx, cudaStream_t s, uint32_t stream_kind
             return -2;
         configured |= bit;
     }
-    dim3 grid(tiles, ks);
+    dim3 grid(tiles, ks, m_blocks);
     m40_launch_dependent(gemm_tc_f16_kernel, grid, dim3(192), smem, s, mW[0], mW[1], mW[2], mXh, mXl, a);
     M40_COUNT_LAUNCH(ctx);
     if (cudaGetLastError() != cudaSuccess) return -2;
+    if (direct) return 0;
 
     EpiArgs e = {};
+    if (ext) {
+        e.act = ext->act;
+        e.tail_on = mode == 0 && problems == 1 ? 1u : 0u;
+        e.tail = ext->tail;
+        e.post_w = ext->post_w;
+        e.post_b = ext->post_b;
+    }
     e.partial = a.partial;
     uint32_t maxN = 0;
     for (int p = 0; p < problems; ++p) {

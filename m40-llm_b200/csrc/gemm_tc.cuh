@@ -21,14 +21,26 @@ struct M40TcRopeAppend {
 // True when the tcgen05 path can take this problem set (2 <= M <= 256, K % 8 == 0, 16-byte aligned weights).
 bool m40_gemm_tc_supported(int M, int K, int problems, const void* const* W);
 
+// What a call does beyond the Llama layer's projections. With it M may exceed 256: the rows are then cut into blocks that
+// share one launch (grid.z).
+struct M40TcExt {
+    int bf16;            // weights are bf16 and the activations are split into bf16 hi + lo (both MMA operands share a type)
+    int ldx;             // row pitch of X in elements (0: K)
+    int act;             // mode 1: M40LLM_ACT_*
+    M40Tail tail;
+    const float* post_w; // tail.post == DYT, problem 0 only; null: 1 and 0
+    const float* post_b;
+};
+
 // Up to three GGUF-layout f16 weight matrices W[p] ([N[p]][K]) applied to the same activations X [M][K] f32.
 // mode 0: out[p][m][n] = X.W[p]^T (+ bias[p][n]) (+ residual[p][m][n]); bias / residual arrays or entries may be null.
 // mode 1: two problems (gate, up) of equal N: out[0][m][n] = silu(X.Wg^T) * (X.Wu^T).
 int m40_gemm_tc_f16(M40llmCudaContext* ctx, cudaStream_t s, uint32_t stream_kind, const float* X, int M, int K,
                     int problems, const __half* const* W, const int* N, float* const* out, const float* const* bias,
                     const float* const* residual, int mode, const M40GemvNorm* norm = nullptr,
-                    const M40TcRopeAppend* rope = nullptr);
-// `norm` (optional): RMSNorm applied to X while it is split into f16 hi/lo (saves the separate norm pass).
+                    const M40TcRopeAppend* rope = nullptr, const M40TcExt* ext = nullptr);
+// `norm` (optional): RMSNorm (or, with ext, dynamic tanh) applied to X while it is split into 16-bit hi/lo (saves the
+// separate norm pass). With ext->bf16 the weight pointers are bf16 rows.
 
 // Two Q8_0 tensor-core calls chained through the f16 hi | lo copies the second one consumes (gate|up -> down): the
 // first call's epilogue writes its result already split, the second skips its split pass. Both calls request

@@ -11,7 +11,7 @@
 //   * sixteen consumer warps form groups of `cw` warps; a group owns every G-th stage, so the groups run
 //     decoupled from one another (no CTA-wide barrier in the steady state). A thread owns fixed column pieces of
 //     every row, so its slice of the activation vector stays in registers for the whole launch:
-//       - f16 weights: 16-byte pieces, f32 activations, f32 FMAs;
+//       - f16 or bf16 weights: 16-byte pieces, f32 activations, f32 FMAs;
 //       - Q8_0 weights: 68-byte pieces (two raw 34-byte GGUF blocks: 4-byte aligned although single blocks are
 //         not), int8 dot products with dp4a against the activations held as three signed 8-bit digits per value
 //         and one scale per 32-block (x = s/128 * (128 a + b + c/128), error <= 2^-22 of the block maximum, i.e.
@@ -21,7 +21,9 @@
 //   * row sums meet by warp shuffle, then across the warps of the group through shared memory in a fixed
 //     order (no atomics: results are deterministic).
 // Up to three matrices that share x go in one launch (Wq | Wk | Wv), gate and up are streamed side by side with
-// the SwiGLU epilogue, bias/residual are folded into the store, and the RMSNorm of x can be applied on the fly.
+// the SwiGLU epilogue, bias/residual are folded into the store, and the RMSNorm of x can be applied on the fly. The EXT
+// instantiations add a dynamic-tanh norm of x, another gate activation and an elementwise tail on the result (dynamic
+// tanh before the residual, soft cap after it).
 //
 // Every wait is bounded: a wait that runs out raises bit 4 of the context's status word, the CTA stops consuming
 // (all warps still pass the same barriers) and drains its own copies before it returns.
@@ -53,6 +55,8 @@ struct SegDev {
     int N;
     int group0;  // id of this matrix's first row group
     int R;       // rows per group of this matrix (the last group may hold fewer)
+    const float* post_w;
+    const float* post_b;
 };
 
 struct GemvArgs {
@@ -66,6 +70,10 @@ struct GemvArgs {
     int nseg, K, pieces, cw, R, nstages, total_groups;
     uint32_t row_bytes, stage_bytes, xq_off;
     int first_late;  // ring slots from this one on share their bytes with the activation digits
+    int dyt;         // EXT: the norm of x is a dynamic tanh
+    float alpha;
+    const float* norm_b;
+    M40GemvExt ext;
 };
 
 __device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
@@ -100,6 +108,21 @@ __device__ __forceinline__ float dot8(const uint4& w, const float* x) {
         acc = fmaf(x[2 * i + 1], f.y, acc);
     }
     return acc;
+}
+
+__device__ __forceinline__ float dot8_bf16(const uint4& w, const float* x) {
+    const uint32_t u[4] = {w.x, w.y, w.z, w.w};
+    float acc = 0.0f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {  // a bf16 is the upper half of the f32 with the same value
+        acc = fmaf(x[2 * i], __uint_as_float(u[i] << 16), acc);
+        acc = fmaf(x[2 * i + 1], __uint_as_float(u[i] & 0xffff0000u), acc);
+    }
+    return acc;
+}
+template <int FMT>
+__device__ __forceinline__ float dot8_fmt(const uint4& w, const float* x) {
+    return FMT == M40_GEMV_BF16 ? dot8_bf16(w, x) : dot8(w, x);
 }
 
 // Activations of one 64-value piece as three int8 digits per value (packed 4 per word) and a scale per 32-block.
@@ -161,21 +184,45 @@ __device__ __forceinline__ float q80_pair_dot(const uint32_t* wp, const Q80X& x)
     return fmaf(fmaf((float)sc, 1.0f / 128.0f, (float)(sa * 128 + sb)), d1 * x.s[1], r);
 }
 
-// bias[n] + residual[n]: loaded at the top of a stage so that the latency hides behind the dot products.
-__device__ __forceinline__ float load_addend(const SegDev& sg, int n) {
-    float add = 0.0f;
-    if (sg.bias) add = sg.bias[n];
-    if (sg.residual) add += sg.residual[n];
-    return add;
+// What is added to row n of the result: loaded at the top of a stage so that the latency hides behind the dot products.
+// Without EXT it is bias[n] + residual[n] in one number.
+template <int EXT>
+struct RowTail {
+    float add;
+};
+template <>
+struct RowTail<1> {
+    float bias, residual, pw, pb;
+};
+template <int EXT>
+__device__ __forceinline__ RowTail<EXT> load_tail(const SegDev& sg, int n) {
+    RowTail<EXT> t;
+    if constexpr (EXT) {
+        t.bias = sg.bias ? sg.bias[n] : 0.0f;
+        t.residual = sg.residual ? sg.residual[n] : 0.0f;
+        t.pw = sg.post_w ? sg.post_w[n] : 1.0f;
+        t.pb = sg.post_b ? sg.post_b[n] : 0.0f;
+    } else {
+        t.add = 0.0f;
+        if (sg.bias) t.add = sg.bias[n];
+        if (sg.residual) t.add += sg.residual[n];
+    }
+    return t;
 }
 
-template <int GATE_UP>
-__device__ __forceinline__ void store_row(const SegDev& sg, int n, float v, float v2, float add) {
-    if (GATE_UP) v = (v / (1.0f + expf(-v))) * v2;
-    sg.out[n] = v + add;
+template <int GATE_UP, int EXT>
+__device__ __forceinline__ void store_row(const GemvArgs& a, const SegDev& sg, int n, float v, float v2,
+                                          const RowTail<EXT>& t) {
+    if constexpr (EXT) {
+        if (GATE_UP) v = m40_act(a.ext.act, v) * v2;
+        sg.out[n] = m40_tail(a.ext.tail, v, t.bias, t.pw, t.pb, t.residual);
+    } else {
+        if (GATE_UP) v = (v / (1.0f + expf(-v))) * v2;
+        sg.out[n] = v + t.add;
+    }
 }
 
-template <int FMT, int GATE_UP, int CPT>
+template <int FMT, int GATE_UP, int CPT, int EXT>
 __global__ void __launch_bounds__(THREADS, 1) gemv_stream_kernel(const __grid_constant__ GemvArgs a) {
     extern __shared__ __align__(128) uint8_t ring[];
     __shared__ uint64_t full[MAX_STAGES], empty[MAX_STAGES], xq_done;
@@ -342,7 +389,8 @@ __global__ void __launch_bounds__(THREADS, 1) gemv_stream_kernel(const __grid_co
     } else {
         float4 sv[2] = {make_float4(0.f, 0.f, 0.f, 0.f), make_float4(0.f, 0.f, 0.f, 0.f)};
         float4 wr[CPT][2];
-        if (a.norm_w) {  // the loads of the sum-of-squares pass and of this thread's own pieces go out together
+        const bool rms = a.norm_w && !(EXT && a.dyt);
+        if (rms) {  // the loads of the sum-of-squares pass and of this thread's own pieces go out together
             const int k = tid * 4;
             if (k < a.K) sv[0] = *reinterpret_cast<const float4*>(a.x + k);
             if (k + CONSUMERS * 4 < a.K) sv[1] = *reinterpret_cast<const float4*>(a.x + k + CONSUMERS * 4);
@@ -359,13 +407,22 @@ __global__ void __launch_bounds__(THREADS, 1) gemv_stream_kernel(const __grid_co
                 const float4 t1 = *reinterpret_cast<const float4*>(a.x + k0 + 4);
                 xr[j][0] = t0.x, xr[j][1] = t0.y, xr[j][2] = t0.z, xr[j][3] = t0.w;
                 xr[j][4] = t1.x, xr[j][5] = t1.y, xr[j][6] = t1.z, xr[j][7] = t1.w;
-                if (a.norm_w) {
+                if (EXT && a.dyt) {
+                    const float* nw = reinterpret_cast<const float*>(a.norm_w);
+                    const float4 w0 = m40_vec4_or(nw, k0, 1.0f), w1 = m40_vec4_or(nw, k0 + 4, 1.0f);
+                    const float4 b0 = m40_vec4_or(a.norm_b, k0, 0.0f), b1 = m40_vec4_or(a.norm_b, k0 + 4, 0.0f);
+                    const float w8[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+                    const float b8[8] = {b0.x, b0.y, b0.z, b0.w, b1.x, b1.y, b1.z, b1.w};
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) xr[j][i] = tanhf(a.alpha * xr[j][i]) * w8[i] + b8[i];
+                }
+                if (rms) {
                     wr[j][0] = load_norm4(a.norm_w, a.norm_f32, k0);
                     wr[j][1] = load_norm4(a.norm_w, a.norm_f32, k0 + 4);
                 }
             }
         }
-        if (a.norm_w) {
+        if (rms) {
             float ss = sv[0].x * sv[0].x + sv[0].y * sv[0].y + sv[0].z * sv[0].z + sv[0].w * sv[0].w +
                        sv[1].x * sv[1].x + sv[1].y * sv[1].y + sv[1].z * sv[1].z + sv[1].w * sv[1].w;
             for (int k = tid * 4 + 2 * CONSUMERS * 4; k < a.K; k += CONSUMERS * 4) {
@@ -418,16 +475,17 @@ __global__ void __launch_bounds__(THREADS, 1) gemv_stream_kernel(const __grid_co
         locate_group(a, (int)blockIdx.x + i * (int)gridDim.x, &sidx, &row0, &rows);
         const SegDev& sg = a.seg[sidx];
         const uint8_t* st = ring + (size_t)s * a.stage_bytes;
-        float add_final = 0.0f;
-        if (cw > 1 && ok && c < rows) add_final = load_addend(sg, row0 + c);
+        RowTail<EXT> tail_final = {};
+        if (cw > 1 && ok && c < rows) tail_final = load_tail<EXT>(sg, row0 + c);
         if (ok) {
             for (int r = 0; r < rows; r += 2) {  // two rows per pass: independent chains for the shuffles
                 const bool two = r + 1 < rows;
                 const uint8_t* rowp = st + (size_t)r * a.row_bytes;
-                float acc[2] = {0.0f, 0.0f}, acc2[2] = {0.0f, 0.0f}, add[2] = {0.0f, 0.0f};
+                float acc[2] = {0.0f, 0.0f}, acc2[2] = {0.0f, 0.0f};
+                RowTail<EXT> tail[2] = {};
                 if (cw == 1 && lane == 0) {
-                    add[0] = load_addend(sg, row0 + r);
-                    if (two) add[1] = load_addend(sg, row0 + r + 1);
+                    tail[0] = load_tail<EXT>(sg, row0 + r);
+                    if (two) tail[1] = load_tail<EXT>(sg, row0 + r + 1);
                 }
 #pragma unroll
                 for (int j = 0; j < CPT; ++j) {
@@ -441,8 +499,8 @@ __global__ void __launch_bounds__(THREADS, 1) gemv_stream_kernel(const __grid_co
                                 acc[rr] += q80_pair_dot(reinterpret_cast<const uint32_t*>(pp), xq);
                                 if (GATE_UP) acc2[rr] += q80_pair_dot(reinterpret_cast<const uint32_t*>(pp + mat2_off), xq);
                             } else {
-                                acc[rr] += dot8(*reinterpret_cast<const uint4*>(pp), xr[j]);
-                                if (GATE_UP) acc2[rr] += dot8(*reinterpret_cast<const uint4*>(pp + mat2_off), xr[j]);
+                                acc[rr] += dot8_fmt<FMT>(*reinterpret_cast<const uint4*>(pp), xr[j]);
+                                if (GATE_UP) acc2[rr] += dot8_fmt<FMT>(*reinterpret_cast<const uint4*>(pp + mat2_off), xr[j]);
                             }
                         }
                     }
@@ -457,7 +515,7 @@ __global__ void __launch_bounds__(THREADS, 1) gemv_stream_kernel(const __grid_co
                     for (int rr = 0; rr < 2; ++rr) {
                         if (rr == 1 && !two) break;
                         if (cw == 1) {
-                            store_row<GATE_UP>(sg, row0 + r + rr, acc[rr], acc2[rr], add[rr]);
+                            store_row<GATE_UP, EXT>(a, sg, row0 + r + rr, acc[rr], acc2[rr], tail[rr]);
                         } else {
                             red[it & 1][0][r + rr][warp] = acc[rr];
                             if (GATE_UP) red[it & 1][1][r + rr][warp] = acc2[rr];
@@ -475,7 +533,7 @@ __global__ void __launch_bounds__(THREADS, 1) gemv_stream_kernel(const __grid_co
                     v += red[it & 1][0][c][grp * cw + k];
                     if (GATE_UP) v2 += red[it & 1][1][c][grp * cw + k];
                 }
-                store_row<GATE_UP>(sg, row0 + c, v, v2, add_final);
+                store_row<GATE_UP, EXT>(a, sg, row0 + c, v, v2, tail_final);
             }
         } else {
             __syncwarp();
@@ -484,28 +542,36 @@ __global__ void __launch_bounds__(THREADS, 1) gemv_stream_kernel(const __grid_co
     }
 }
 
-template <int FMT, int GATE_UP, int CPT>
+template <int FMT, int GATE_UP, int CPT, int EXT>
 int launch(M40llmCudaContext* ctx, cudaStream_t s, const GemvArgs& a, int grid, size_t smem) {
     static bool attr_set[64] = {};
     const int dev = ctx->device_id;
     if (dev < 0 || dev >= 64 || !attr_set[dev]) {
-        if (cudaFuncSetAttribute(gemv_stream_kernel<FMT, GATE_UP, CPT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        if (cudaFuncSetAttribute(gemv_stream_kernel<FMT, GATE_UP, CPT, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                  (int)SMEM_MAX) != cudaSuccess)
             return -2;
         if (dev >= 0 && dev < 64) attr_set[dev] = true;
     }
-    const cudaError_t e = m40_launch_dependent(gemv_stream_kernel<FMT, GATE_UP, CPT>, dim3(grid), dim3(THREADS), smem, s, a);
+    const cudaError_t e =
+        m40_launch_dependent(gemv_stream_kernel<FMT, GATE_UP, CPT, EXT>, dim3(grid), dim3(THREADS), smem, s, a);
     M40_COUNT_LAUNCH(ctx);
     return e == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
-template <int GATE_UP>
-int launch_fmt(M40llmCudaContext* ctx, cudaStream_t s, const GemvArgs& a, int grid, size_t smem, int fmt, int cpt) {
-    if (fmt == M40_GEMV_Q80) return launch<M40_GEMV_Q80, GATE_UP, 1>(ctx, s, a, grid, smem);
-    if (cpt == 1) return launch<M40_GEMV_F16, GATE_UP, 1>(ctx, s, a, grid, smem);
-    if (cpt == 2) return launch<M40_GEMV_F16, GATE_UP, 2>(ctx, s, a, grid, smem);
-    if (cpt == 4) return launch<M40_GEMV_F16, GATE_UP, 4>(ctx, s, a, grid, smem);
+template <int FMT, int GATE_UP, int EXT>
+int launch_cpt(M40llmCudaContext* ctx, cudaStream_t s, const GemvArgs& a, int grid, size_t smem, int cpt) {
+    if (cpt == 1) return launch<FMT, GATE_UP, 1, EXT>(ctx, s, a, grid, smem);
+    if (cpt == 2) return launch<FMT, GATE_UP, 2, EXT>(ctx, s, a, grid, smem);
+    if (cpt == 4) return launch<FMT, GATE_UP, 4, EXT>(ctx, s, a, grid, smem);
     return 1;
+}
+
+template <int GATE_UP>
+int launch_fmt(M40llmCudaContext* ctx, cudaStream_t s, const GemvArgs& a, int grid, size_t smem, int fmt, int cpt, bool ext) {
+    if (fmt == M40_GEMV_Q80) return launch<M40_GEMV_Q80, GATE_UP, 1, 0>(ctx, s, a, grid, smem);
+    if (fmt == M40_GEMV_BF16) return launch_cpt<M40_GEMV_BF16, GATE_UP, 1>(ctx, s, a, grid, smem, cpt);
+    return ext ? launch_cpt<M40_GEMV_F16, GATE_UP, 1>(ctx, s, a, grid, smem, cpt)
+               : launch_cpt<M40_GEMV_F16, GATE_UP, 0>(ctx, s, a, grid, smem, cpt);
 }
 
 bool aligned16(const void* p) { return (((uintptr_t)p) & 15u) == 0u; }
@@ -513,12 +579,14 @@ bool aligned16(const void* p) { return (((uintptr_t)p) & 15u) == 0u; }
 }  // namespace
 
 int m40_gemv_stream(M40llmCudaContext* ctx, cudaStream_t s, const float* x, int K, int fmt, int gate_up, int nseg,
-                    const M40GemvSeg* segs, const M40GemvNorm* norm) {
+                    const M40GemvSeg* segs, const M40GemvNorm* norm, const M40GemvExt* ext) {
     if (nseg < 1 || nseg > MAX_SEGS - 1 || K <= 0 || !aligned16(x)) return 1;
     GemvArgs a = {};
     int cpt_max;
     uint32_t xq_bytes = 0;
-    if (fmt == M40_GEMV_F16) {
+    const bool dyt = norm && norm->dyt;
+    if (fmt == M40_GEMV_Q80 && (ext || dyt)) return 1;
+    if (fmt == M40_GEMV_F16 || fmt == M40_GEMV_BF16) {
         if (K % 8 != 0) return 1;
         a.row_bytes = (uint32_t)K * 2u;
         a.pieces = K / 8;
@@ -540,6 +608,7 @@ int m40_gemv_stream(M40llmCudaContext* ctx, cudaStream_t s, const float* x, int 
         if (gate_up && (!segs[i].W2 || !aligned16(segs[i].W2))) return 1;
     }
     if (norm && norm->w && (!aligned16(norm->w) || (norm->xn_out && !aligned16(norm->xn_out)))) return 1;
+    if (dyt && (!aligned16(norm->b) || norm->xn_out)) return 1;
     if ((uint64_t)a.row_bytes * nmat > STAGE_MAX || xq_bytes + 2u * a.row_bytes * nmat > SMEM_MAX) return 1;
     // the digits are only needed until every consumer holds its slice in registers: the last ring slots reuse their bytes
 
@@ -633,6 +702,8 @@ int m40_gemv_stream(M40llmCudaContext* ctx, cudaStream_t s, const float* x, int 
             d.N = n;
             d.group0 = g;
             d.R = part == 0 ? a.R : a.R - 1;
+            d.post_w = segs[i].post_w ? segs[i].post_w + r0 : nullptr;
+            d.post_b = segs[i].post_b ? segs[i].post_b + r0 : nullptr;
             g += (n + d.R - 1) / d.R;
         }
     }
@@ -648,8 +719,16 @@ int m40_gemv_stream(M40llmCudaContext* ctx, cudaStream_t s, const float* x, int 
         a.eps = norm->eps;
         a.xn_out = norm->xn_out;
     }
+    if (dyt) {
+        a.dyt = 1;
+        a.alpha = norm->alpha;
+        a.norm_b = norm->b;
+    }
+    if (ext) a.ext = *ext;
     const int grid = g < grid_max ? g : grid_max;
     const size_t smem = smem_bytes;
-    return gate_up ? launch_fmt<1>(ctx, s, a, grid, smem, fmt, cpt) : launch_fmt<0>(ctx, s, a, grid, smem, fmt, cpt);
+    const bool use_ext = ext != nullptr || dyt;
+    return gate_up ? launch_fmt<1>(ctx, s, a, grid, smem, fmt, cpt, use_ext)
+                   : launch_fmt<0>(ctx, s, a, grid, smem, fmt, cpt, use_ext);
 }
 

@@ -6,6 +6,7 @@
 #include "gemm.cuh"
 #include "gemm_tc.cuh"
 #include "gemv_stream.cuh"
+#include "stack_math.cuh"
 
 int m40_rms_norm_rows(M40llmCudaContext* ctx, const void* in, const void* w, void* out, uint32_t rows, uint32_t dim,
                       float eps, uint32_t wdtype);
@@ -13,17 +14,42 @@ int m40_rms_norm_rows(M40llmCudaContext* ctx, const void* in, const void* w, voi
 namespace {
 
 // out[r][:] = f32(table[ids[r]][:]); an id outside the table raises status bit 8 and yields zeros.
-__global__ void __launch_bounds__(256) embed_rows_f16_kernel(const __half* __restrict__ table,
-                                                             const uint32_t* __restrict__ ids, float* __restrict__ out,
-                                                             uint32_t hidden, uint32_t vocab, uint32_t* status) {
+template <typename T>
+__global__ void __launch_bounds__(256) embed_rows_kernel(const T* __restrict__ table, const uint32_t* __restrict__ ids,
+                                                         float* __restrict__ out, uint32_t hidden, uint32_t vocab,
+                                                         uint32_t* status) {
     pdl_wait();
     pdl_trigger();
     const uint32_t r = blockIdx.x, id = ids[r];
     const bool ok = id < vocab;
     if (!ok && threadIdx.x == 0) atomicOr(status, 8u);
-    const __half* src = table + (size_t)(ok ? id : 0u) * hidden;
+    const T* src = table + (size_t)(ok ? id : 0u) * hidden;
     float* dst = out + (size_t)r * hidden;
-    for (uint32_t i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = ok ? __half2float(src[i]) : 0.0f;
+    for (uint32_t i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = ok ? m40_load_elem(src + i) : 0.0f;
+}
+
+// out[r] = [a[r] | b[r]]
+__global__ void __launch_bounds__(256) concat_rows_kernel(const float* __restrict__ a, const float* __restrict__ b,
+                                                          float* __restrict__ out, uint32_t dim) {
+    pdl_wait();
+    pdl_trigger();
+    const size_t r = blockIdx.x;
+    for (uint32_t i = threadIdx.x; i < dim; i += blockDim.x) {
+        out[2 * r * dim + i] = a[r * dim + i];
+        out[(2 * r + 1) * dim + i] = b[r * dim + i];
+    }
+}
+
+__global__ void __launch_bounds__(256) gather_rows_kernel(const float* __restrict__ in, const uint32_t* __restrict__ index,
+                                                          float* __restrict__ out, uint32_t dim, uint32_t rows_in,
+                                                          uint32_t* status) {
+    pdl_wait();
+    pdl_trigger();
+    const uint32_t i = index[blockIdx.x];
+    const bool ok = i < rows_in;
+    if (!ok && threadIdx.x == 0) atomicOr(status, 8u);
+    for (uint32_t c = threadIdx.x; c < dim; c += blockDim.x)
+        out[(size_t)blockIdx.x * dim + c] = ok ? in[(size_t)i * dim + c] : 0.0f;
 }
 
 // Greedy choice per row: the first index of the largest value under strict '>' from -inf, so NaN is never chosen
@@ -79,14 +105,53 @@ __global__ void advance_rows_kernel(uint32_t* __restrict__ positions, uint32_t* 
 
 extern "C" {
 
-int m40llm_embed_tokens_f16_async(M40llmCudaContext* ctx, const void* d_table_f16, const uint32_t* d_token_ids,
-                                  void* d_out_f32, uint32_t rows, uint32_t hidden, uint32_t vocab) {
-    if (!ctx || !d_table_f16 || !d_token_ids || !d_out_f32) return -1;
+int m40llm_embed_tokens_async(M40llmCudaContext* ctx, const void* d_table, uint32_t table_dtype,
+                              const uint32_t* d_token_ids, void* d_out_f32, uint32_t rows, uint32_t hidden,
+                              uint32_t vocab) {
+    if (!ctx || !d_table || !d_token_ids || !d_out_f32) return -1;
     if (rows == 0 || hidden == 0 || vocab == 0) return -2;
     if (m40_ensure_device(ctx) != 0) return -1;
-    const cudaError_t e = m40_launch_dependent(embed_rows_f16_kernel, dim3(rows), dim3(256), 0, ctx->decode_stream,
-                                               (const __half*)d_table_f16, d_token_ids, (float*)d_out_f32, hidden,
-                                               vocab, ctx->d_status);
+    cudaStream_t s = ctx->decode_stream;
+    float* out = (float*)d_out_f32;
+    cudaError_t e;
+    if (table_dtype == M40LLM_DT_F16)
+        e = m40_launch_dependent(embed_rows_kernel<__half>, dim3(rows), dim3(256), 0, s, (const __half*)d_table, d_token_ids, out,
+                                 hidden, vocab, ctx->d_status);
+    else if (table_dtype == M40LLM_DT_BF16)
+        e = m40_launch_dependent(embed_rows_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, s, (const __nv_bfloat16*)d_table,
+                                 d_token_ids, out, hidden, vocab, ctx->d_status);
+    else if (table_dtype == M40LLM_DT_F32)
+        e = m40_launch_dependent(embed_rows_kernel<float>, dim3(rows), dim3(256), 0, s, (const float*)d_table, d_token_ids, out,
+                                 hidden, vocab, ctx->d_status);
+    else
+        return -4;
+    M40_COUNT_LAUNCH(ctx);
+    return e == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+int m40llm_embed_tokens_f16_async(M40llmCudaContext* ctx, const void* d_table_f16, const uint32_t* d_token_ids,
+                                  void* d_out_f32, uint32_t rows, uint32_t hidden, uint32_t vocab) {
+    return m40llm_embed_tokens_async(ctx, d_table_f16, M40LLM_DT_F16, d_token_ids, d_out_f32, rows, hidden, vocab);
+}
+
+int m40llm_concat_rows_async(M40llmCudaContext* ctx, const void* d_a, const void* d_b, void* d_out, uint32_t rows,
+                             uint32_t dim) {
+    if (!ctx || !d_a || !d_b || !d_out) return -1;
+    if (rows == 0 || dim == 0) return -2;
+    if (m40_ensure_device(ctx) != 0) return -1;
+    const cudaError_t e = m40_launch_dependent(concat_rows_kernel, dim3(rows), dim3(256), 0, ctx->decode_stream,
+                                               (const float*)d_a, (const float*)d_b, (float*)d_out, dim);
+    M40_COUNT_LAUNCH(ctx);
+    return e == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+int m40llm_gather_rows_async(M40llmCudaContext* ctx, const void* d_in, const uint32_t* d_index, void* d_out,
+                             uint32_t count, uint32_t dim, uint32_t rows_in) {
+    if (!ctx || !d_in || !d_index || !d_out) return -1;
+    if (count == 0 || dim == 0 || rows_in == 0) return -2;
+    if (m40_ensure_device(ctx) != 0) return -1;
+    const cudaError_t e = m40_launch_dependent(gather_rows_kernel, dim3(count), dim3(256), 0, ctx->decode_stream,
+                                               (const float*)d_in, d_index, (float*)d_out, dim, rows_in, ctx->d_status);
     M40_COUNT_LAUNCH(ctx);
     return e == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -3;
 }

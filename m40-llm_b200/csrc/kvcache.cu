@@ -174,6 +174,33 @@ M40llmKVCache* m40llm_kvcache_create(M40llmCudaContext* ctx, uint32_t max_seq_le
     return kv;
 }
 
+M40llmKVCache* m40llm_kvcache_create_typed(M40llmCudaContext* ctx, uint32_t max_seq_len, uint32_t slots, uint32_t kv_heads,
+                                           uint32_t k_dim, uint32_t v_dim, uint32_t elem_dtype) {
+    if (!ctx || max_seq_len == 0 || slots == 0 || kv_heads == 0 || k_dim == 0 || v_dim == 0) return nullptr;
+    if (elem_dtype != M40LLM_DT_F16 && elem_dtype != M40LLM_DT_F32) return nullptr;
+    if (elem_dtype == M40LLM_DT_F16 && k_dim == v_dim) return m40llm_kvcache_create(ctx, max_seq_len, slots, kv_heads, k_dim);
+    if (m40_ensure_device(ctx) != 0) return nullptr;
+    M40llmKVCache* kv = (M40llmKVCache*)calloc(1, sizeof(M40llmKVCache));
+    if (!kv) return nullptr;
+    kv->device_id = ctx->device_id;
+    kv->max_seq_len = max_seq_len;
+    kv->max_batch_size = slots;
+    kv->num_heads = kv_heads;
+    kv->head_dim = k_dim;
+    kv->v_dim = v_dim;
+    kv->elem_f32 = elem_dtype == M40LLM_DT_F32 ? 1u : 0u;
+    const size_t rows = (size_t)max_seq_len * slots * kv_heads, es = kv->elem_f32 ? 4u : 2u;
+    bool ok = dev_alloc_zero((uint8_t**)&kv->d_typed_k, rows * k_dim * es);
+    ok = ok && dev_alloc_zero((uint8_t**)&kv->d_typed_v, rows * v_dim * es);
+    ok = ok && dev_alloc_zero(&kv->d_seq_map, slots);
+    ok = ok && cudaStreamSynchronize(cudaStreamLegacy) == cudaSuccess;  // as in m40llm_kvcache_create
+    if (!ok) {
+        m40llm_kvcache_destroy(kv);
+        return nullptr;
+    }
+    return kv;
+}
+
 M40llmKVCache* m40llm_kvcache_create_compressed(M40llmCudaContext* ctx, uint32_t max_seq_len, uint32_t max_batch_size,
                                                 uint32_t num_heads, uint32_t head_dim, uint32_t recent_window,
                                                 uint32_t block_size, uint32_t top_blocks, uint32_t representatives,
@@ -228,6 +255,8 @@ void m40llm_kvcache_destroy(M40llmKVCache* kv) {
     if (kv->d_old_k) cudaFree(kv->d_old_k);
     if (kv->d_q4_v) cudaFree(kv->d_q4_v);
     if (kv->d_q4_scale) cudaFree(kv->d_q4_scale);
+    if (kv->d_typed_k) cudaFree(kv->d_typed_k);
+    if (kv->d_typed_v) cudaFree(kv->d_typed_v);
     free(kv);
 }
 
@@ -499,6 +528,7 @@ int m40llm_kvcache_debug_write_range(M40llmCudaContext* ctx, M40llmKVCache* kv, 
                                      uint32_t count, const void* k_f16_host, const void* v_f16_host,
                                      uint32_t final_seq_len) {
     if (!ctx || !kv || !k_f16_host || !v_f16_host) return -1;
+    if (!kv->compressed && (!kv->d_k || !kv->d_v)) return -4;
     if (seq_id >= kv->max_batch_size) return -2;
     if ((uint64_t)tok_begin + count > kv->max_seq_len || final_seq_len > kv->max_seq_len ||
         (uint64_t)tok_begin + count > final_seq_len)

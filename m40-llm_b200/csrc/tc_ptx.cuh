@@ -87,6 +87,8 @@ __device__ __forceinline__ uint32_t make_idesc(uint32_t n) {
     return (1u << 4) | ((n >> 3) << 17) | ((uint32_t)(BLOCK_N >> 4) << 24);
 }
 
+// Added to the above when both operands are bf16 (type code 1 in the A and B format fields).
+__device__ __host__ __forceinline__ constexpr uint32_t idesc_bf16() { return (1u << 7) | (1u << 10); }
 
 // Wide TMEM loads: N consecutive 32-bit columns of this thread's lane. Issue, then tmem_ld_wait() once.
 __device__ __forceinline__ void tmem_ld_x4(uint32_t taddr, uint32_t* r) {

@@ -1,0 +1,170 @@
+"""Plain, slow float64 statement of the layer-stack mechanisms (numpy), one function per mechanism.
+
+TEST INFRASTRUCTURE ONLY, like oracle.py: the product never imports it and it shares no code with it. Everything works
+on one sequence at a time, token rows first: h [T, width]. State that outlives a call (keys, values, the recurrent
+matrix) is passed in and out explicitly, so the same functions run a whole prompt, a portion of it or one token.
+"""
+from __future__ import annotations
+
+import math
+
+import numpy as np
+
+F = np.float64
+
+
+def sigmoid(x):
+    return 1.0 / (1.0 + np.exp(-np.asarray(x, F)))
+
+
+def gelu_tanh(z):
+    z = np.asarray(z, F)
+    return 0.5 * z * (1.0 + np.tanh(math.sqrt(2.0 / math.pi) * (z + 0.044715 * z ** 3)))
+
+
+def rms_norm(x, w, eps):
+    x = np.asarray(x, F)
+    return x / np.sqrt(np.mean(x * x, axis=-1, keepdims=True) + eps) * np.asarray(w, F)
+
+
+def dyt_norm(x, alpha, w, b):
+    """Dynamic tanh: elementwise, no statistics."""
+    return np.tanh(float(alpha) * np.asarray(x, F)) * np.asarray(w, F) + np.asarray(b, F)
+
+
+def rope_freqs(base, dims, scaling=None):
+    """(frequencies [dims/2], amplitude). `scaling` = dict(factor, original, fast, slow) switches YaRN on."""
+    f = np.array([float(base) ** (-2.0 * i / dims) for i in range(dims // 2)], F)
+    if not scaling:
+        return f, 1.0
+    def dim_of(turns):
+        return dims * math.log(scaling["original"] / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+    lo = max(math.floor(dim_of(scaling["fast"])), 0)
+    hi = min(math.ceil(dim_of(scaling["slow"])), dims - 1)
+    ramp = np.clip((np.arange(dims // 2) - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+    return f / scaling["factor"] * ramp + f * (1.0 - ramp), 0.1 * math.log(scaling["factor"]) + 1.0
+
+
+def rotate_half(x, pos, freqs, amp=1.0, sign=1.0):
+    """x [T, heads, d]: the pair (m, m + n) of the first 2n = 2 len(freqs) dimensions turns by sign * pos * freqs[m]."""
+    n = len(freqs)
+    ang = sign * np.asarray(pos, F)[:, None] * freqs[None, :]
+    c, s = (np.cos(ang) * amp)[:, None, :], (np.sin(ang) * amp)[:, None, :]
+    u, v = x[..., :n], x[..., n:2 * n]
+    return np.concatenate([u * c - v * s, v * c + u * s, x[..., 2 * n:]], axis=-1)
+
+
+def gated_attention(h, pos0, K, V, w, m, eps):
+    """w: q k v o g q.norm k.norm; m: heads kv_heads dim vdim scale rot. K [n, G, dim], V [n, G, vdim] hold the earlier
+    tokens (keys normalised and turned, values turned). Returns (out [T, width], K, V) with the new rows appended."""
+    h = np.asarray(h, F)
+    T, H, G, D, VD = len(h), m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    pos = np.arange(pos0, pos0 + T)
+    q = rms_norm(h @ w["q"].T, w["q.norm"], eps).reshape(T, H, D)
+    k = rms_norm(h @ w["k"].T, w["k.norm"], eps).reshape(T, G, D)
+    v = (h @ w["v"].T).reshape(T, G, VD)
+    f, amp = rope_freqs(m["rot"]["base"], m["rot"]["dims"], m["rot"].get("scaling"))
+    fv, _ = rope_freqs(m["rot"]["base"], VD)
+    q, k = rotate_half(q, pos, f, amp), rotate_half(k, pos, f, amp)
+    v = rotate_half(v, pos, fv)
+    K, V = np.concatenate([K, k]), np.concatenate([V, v])
+    out = np.zeros((T, H, VD), F)
+    for t in range(T):
+        n = pos0 + t + 1
+        for head in range(H):
+            g = head // (H // G)
+            s = K[:n, g] @ q[t, head] * m["scale"]
+            p = np.exp(s - s.max())
+            out[t, head] = (p / p.sum()) @ V[:n, g]
+    out = rotate_half(out, pos, fv, sign=-1.0)
+    out = out * sigmoid(h @ w["g"].T)[:, :, None]
+    return out.reshape(T, H * VD) @ w["o"].T, K, V
+
+
+def general_delta(h, S, w, m, eps):
+    """S [heads, dim (key), dim (value)]; w: r k v g a a.b w0 w1 w2 norm o. Returns (out [T, width], S)."""
+    h = np.asarray(h, F)
+    T, H, D = len(h), m["heads"], m["dim"]
+    shape = (T, H, D)
+    r, k, v = ((h @ w[n].T).reshape(shape) for n in ("r", "k", "v"))
+    decay = np.exp(-math.exp(-0.5) * sigmoid(np.tanh(h @ w["w1"].T) @ w["w2"].T + w["w0"])).reshape(shape)
+    a = sigmoid(h @ w["a"].T + w["a.b"]).reshape(shape)
+    u = k / np.sqrt(np.sum(k * k, axis=-1, keepdims=True) + 1e-6)
+    S = np.array(S, F)
+    o = np.zeros(shape, F)
+    for t in range(T):
+        for head in range(H):
+            old = S[head]
+            S[head] = decay[t, head][:, None] * old - np.outer(a[t, head] * u[t, head], u[t, head] @ old) \
+                + np.outer(k[t, head], v[t, head])
+            o[t, head] = r[t, head] @ S[head]
+    o = o / np.sqrt(np.mean(o * o, axis=-1, keepdims=True) + eps)
+    y = o.reshape(T, H * D) * w["norm"] * sigmoid(h @ w["g"].T)
+    return y @ w["o"].T, S
+
+
+def gated_mlp(h, gate, up, down, act=gelu_tanh):
+    h = np.asarray(h, F)
+    return (act(h @ gate.T) * (h @ up.T)) @ down.T
+
+
+def soft_cap(x, cap):
+    return cap * np.tanh(np.asarray(x, F) / cap)
+
+
+class StackOracle:
+    """A whole model: `cfg` as in config.json, `weights` = {tensor name: array}. One sequence, any portions."""
+
+    def __init__(self, cfg, weights):
+        self.cfg = cfg
+        self.w = {n: np.asarray(a, F) for n, a in weights.items()}
+        lp = cfg.get("loop")
+        n = len(cfg["layers"])
+        self.runs = []  # (layer, pass or None at its first layer)
+        if lp:
+            self.runs += [(i, None) for i in range(lp["start"])]
+            for t in range(lp["times"]):
+                self.runs += [(i, t if i == lp["start"] else None) for i in range(lp["start"], lp["stop"])]
+            self.runs += [(i, None) for i in range(lp["stop"], n)]
+        else:
+            self.runs = [(i, None) for i in range(n)]
+        self.reset()
+
+    def reset(self):
+        self.pos = 0
+        self.state = []
+        for i, _ in self.runs:
+            ly = self.cfg["layers"][i]
+            m = ly["mixer"]
+            if ly["type"] == "attention":
+                self.state.append([np.zeros((0, m["kv_heads"], m["dim"])), np.zeros((0, m["kv_heads"], m["vdim"]))])
+            else:
+                self.state.append(np.zeros((m["heads"], m["dim"], m["dim"])))
+
+    def norm(self, name, x):
+        return dyt_norm(x, self.w[name + ".alpha"], self.w[name], self.w[name + ".b"])
+
+    def step(self, tokens, layer_out=None):
+        cfg, eps = self.cfg, self.cfg["norm"]["eps"]
+        x0 = self.w["embed"][np.asarray(tokens)]
+        x = x0
+        for at, (i, t) in enumerate(self.runs):
+            ly = cfg["layers"][i]
+            if t is not None:
+                x = np.concatenate([x, x0], axis=-1) @ self.w["loop.in"].T + self.w["loop.step"][t]
+            p = f"l{i}."
+            mw = {n[len(p) + 4:]: a for n, a in self.w.items() if n.startswith(p + "mix.")}
+            h = self.norm(p + "norm1", x)
+            if ly["type"] == "attention":
+                y, K, V = gated_attention(h, self.pos, *self.state[at], mw, ly["mixer"], eps)
+                self.state[at] = [K, V]
+            else:
+                y, self.state[at] = general_delta(h, self.state[at], mw, ly["mixer"], eps)
+            x = x + self.norm(p + "norm1b", y)
+            if ly["mlp"]:
+                h = self.norm(p + "norm2", x)
+                x = x + self.norm(p + "norm2b", gated_mlp(h, *(self.w[p + "mlp." + n] for n in ("gate", "up", "down"))))
+            if layer_out is not None:
+                layer_out.append(x)
+        self.pos += len(tokens)
+        return soft_cap(self.norm("final.norm", x) @ self.w["head"].T, cfg["logit_softcap"])
