@@ -7,6 +7,8 @@ import os
 
 import numpy as np
 
+from .native import Norm
+
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "libm40llm_host.so")
 
@@ -28,6 +30,28 @@ class Weights(C.Structure):
 
 class ModelHead(C.Structure):
     _fields_ = [("embeddings", C.c_void_p), ("output_norm", C.c_void_p), ("lm_head", C.c_void_p), ("vocab", C.c_uint32)]
+
+
+class StackCfg(C.Structure):
+    """m40host_stack_cfg."""
+    _fields_ = ([(n, C.c_uint32) for n in ("hidden", "vocab", "w_dtype", "exact", "sequences", "max_len", "max_rows")] +
+                [("soft_cap", C.c_float), ("embeddings", C.c_void_p), ("lm_head", C.c_void_p), ("norm", Norm)])
+
+
+MIXER_ROTARY_ATTENTION, MIXER_DELTA_RULE = 1, 2
+
+
+class StackLayerDesc(C.Structure):
+    """StackLayerDesc of host/model_layer.hpp."""
+    _fields_ = ([(n, C.c_uint32) for n in ("mixer", "n_in")] + [(n, Norm) for n in ("norm1", "norm1b", "norm2", "norm2b")] +
+                [("w_in", C.c_void_p), ("w_out", C.c_void_p), ("eps", C.c_float)] +
+                [(n, C.c_uint32) for n in ("q_heads", "kv_heads", "k_dim", "v_dim", "k_pairs", "has_gate")] +
+                [("k_amp", C.c_float), ("scale", C.c_float)] +
+                [(n, C.c_void_p) for n in ("q_norm", "k_norm", "k_turns", "v_turns")] +
+                [(n, C.c_uint32) for n in ("heads", "dim", "rank")] +
+                [("decay_scale", C.c_float), ("unit_eps", C.c_float)] +
+                [(n, C.c_void_p) for n in ("w2", "w0", "a_bias", "o_norm")] +
+                [("ff", C.c_uint32), ("act", C.c_uint32)] + [(n, C.c_void_p) for n in ("gate", "up", "down")])
 
 
 class KvCfg(C.Structure):
@@ -60,7 +84,20 @@ def lib() -> C.CDLL:
         L.m40host_model_create.restype = C.c_void_p
         L.m40host_model_create.argtypes = [C.c_void_p, C.POINTER(LayerCfg), C.c_uint32, C.POINTER(Weights),
                                            C.POINTER(ModelHead), C.c_void_p, C.c_uint32]
+        L.m40host_model_create_rows.restype = C.c_void_p
+        L.m40host_model_create_rows.argtypes = L.m40host_model_create.argtypes + [C.c_uint32]
         L.m40host_model_destroy.argtypes = [C.c_void_p]
+        L.m40host_model_acquire.argtypes = [C.c_void_p]
+        L.m40host_model_release.argtypes = [C.c_void_p, C.c_uint32]
+        L.m40host_model_length.restype = C.c_uint32
+        L.m40host_model_length.argtypes = [C.c_void_p, C.c_uint32]
+        L.m40host_model_step.argtypes = [C.c_void_p, C.c_uint32] + [C.c_void_p] * 3 + [C.c_uint32] + [C.c_void_p] * 4
+        L.m40host_model_begin_sequences.argtypes = [C.c_void_p, C.c_uint32, C.c_void_p, C.c_void_p]
+        L.m40host_stack_create.restype = C.c_void_p
+        L.m40host_stack_create.argtypes = [C.c_void_p, C.POINTER(StackCfg)]
+        L.m40host_stack_add_layer.argtypes = [C.c_void_p, C.POINTER(StackCfg), C.POINTER(StackLayerDesc)]
+        L.m40host_stack_add_join.argtypes = [C.c_void_p, C.POINTER(StackCfg), C.c_void_p, C.c_void_p]
+        L.m40host_stack_finish.argtypes = [C.c_void_p]
         L.m40host_model_begin.argtypes = [C.c_void_p, C.c_void_p, C.c_void_p]
         L.m40host_model_generate.argtypes = [C.c_void_p, C.c_uint32, C.c_uint32, C.c_void_p, C.c_void_p]
         L.m40host_model_graph_replays.restype = C.c_uint64
@@ -157,18 +194,42 @@ class DecodeLayer:
             self.handle = None
 
 
-class DecodeModel:
-    """Greedy decode of a whole layer stack (embedding -> layers -> logits head -> arg-max on the device); mirror of the
-    reference's session loop (src/decode_session.rs:637-954, src/infer/logits.rs:57-116, src/sampling.rs:95-108).
-    `kv` is a dense cache with sequences * layers slots (slot = sequence * layers + layer, src/infer/kv.rs:109)."""
+class Model:
+    """What every model of the framework does once it is built (host/decode_model.hpp): a table of sequence slots, step()
+    over any portions of live sequences, and greedy generate() for a fixed set of them."""
 
-    def __init__(self, ctx, cfg: LayerCfg, layers, head: ModelHead, kv, sequences: int):
-        arr = (Weights * len(layers))(*layers)
-        self._keep = (arr, head, cfg)
-        self.sequences, self.vocab = sequences, int(head.vocab)
-        self.h = lib().m40host_model_create(ctx, C.byref(cfg), len(layers), arr, C.byref(head), kv, sequences)
-        if not self.h:
+    h = None
+    sequences = vocab = hidden = 0
+    layers = 0      # layers whose residual a traced step returns
+
+    def acquire(self) -> int:
+        s = lib().m40host_model_acquire(self.h)
+        if s < 0:
             raise RuntimeError(last_error())
+        return s
+
+    def release(self, sequence: int):
+        if lib().m40host_model_release(self.h, sequence) != 0:
+            raise RuntimeError(last_error())
+
+    def length(self, sequence: int) -> int:
+        return int(lib().m40host_model_length(self.h, sequence))
+
+    def step(self, entries, want=(), want_logits: bool = True, want_next: bool = False, trace_layers: bool = False):
+        """entries: [(sequence, token ids)], want: ascending row indexes into the concatenated tokens. Returns a dict with
+        `logits` [len(want), vocab], `next` (greedy ids after the wanted rows) and `layers` [layers, rows, hidden]."""
+        seqs = np.array([e[0] for e in entries], np.uint32)
+        counts = np.array([len(e[1]) for e in entries], np.uint32)
+        toks = np.ascontiguousarray(np.concatenate([np.asarray(e[1], np.uint32) for e in entries]))
+        want = np.ascontiguousarray(want, np.uint32)
+        logits = np.empty((len(want), self.vocab), np.float32) if want_logits else None
+        nxt = np.empty(len(want), np.uint32) if want_next else None
+        trace = np.empty((self.layers, len(toks), self.hidden), np.float32) if trace_layers else None
+        p = lambda a: None if a is None else a.ctypes.data_as(C.c_void_p)
+        if lib().m40host_model_step(self.h, len(entries), p(seqs), p(counts), p(toks), len(want), p(want), p(logits), p(nxt),
+                                    p(trace)) != 0:
+            raise RuntimeError(last_error())
+        return {"logits": logits, "next": nxt, "layers": trace}
 
     def begin(self, token_ids, positions):
         t = np.ascontiguousarray(token_ids, dtype=np.uint32)
@@ -176,11 +237,21 @@ class DecodeModel:
         assert t.shape == (self.sequences,) and p.shape == (self.sequences,)
         if lib().m40host_model_begin(self.h, t.ctypes.data_as(C.c_void_p), p.ctypes.data_as(C.c_void_p)) != 0:
             raise RuntimeError(last_error())
+        self.rows = self.sequences
+
+    def begin_sequences(self, sequences, token_ids):
+        """Next input tokens of some live sequences; generate() then advances exactly these."""
+        s = np.ascontiguousarray(sequences, dtype=np.uint32)
+        t = np.ascontiguousarray(token_ids, dtype=np.uint32)
+        assert s.shape == t.shape
+        if lib().m40host_model_begin_sequences(self.h, len(s), s.ctypes.data_as(C.c_void_p), t.ctypes.data_as(C.c_void_p)) != 0:
+            raise RuntimeError(last_error())
+        self.rows = len(s)
 
     def generate(self, steps: int, use_graph: bool = True, want_ids: bool = True, want_logits: bool = False):
-        """Returns (ids [steps, sequences] or None, logits of the last step [sequences, vocab] or None)."""
-        ids = np.empty((steps, self.sequences), np.uint32) if want_ids else None
-        logits = np.empty((self.sequences, self.vocab), np.float32) if want_logits else None
+        """Returns (ids [steps, rows] or None, logits of the last step [rows, vocab] or None)."""
+        ids = np.empty((steps, self.rows), np.uint32) if want_ids else None
+        logits = np.empty((self.rows, self.vocab), np.float32) if want_logits else None
         rc = lib().m40host_model_generate(self.h, steps, 1 if use_graph else 0,
                                           ids.ctypes.data_as(C.c_void_p) if want_ids else None,
                                           logits.ctypes.data_as(C.c_void_p) if want_logits else None)
@@ -198,3 +269,41 @@ class DecodeModel:
         if self.h:
             lib().m40host_model_destroy(self.h)
             self.h = None
+
+
+class DecodeModel(Model):
+    """The reference's layer stack (embedding -> layers -> logits head -> arg-max on the device); mirror of its
+    session loop (src/decode_session.rs:637-954, src/infer/logits.rs:57-116, src/sampling.rs:95-108).
+    `kv` is a dense cache with sequences * layers slots (slot = sequence * layers + layer, src/infer/kv.rs:109).
+    max_rows > 0 gives step() room for prompt portions of that many tokens per pass."""
+
+    def __init__(self, ctx, cfg: LayerCfg, layers, head: ModelHead, kv, sequences: int, max_rows: int = 0):
+        arr = (Weights * len(layers))(*layers)
+        self._keep = (arr, head, cfg)
+        self.sequences, self.vocab, self.hidden, self.layers = sequences, int(head.vocab), int(cfg.hidden), len(layers)
+        self.h = lib().m40host_model_create_rows(ctx, C.byref(cfg), len(layers), arr, C.byref(head), kv, sequences, max_rows)
+        if not self.h:
+            raise RuntimeError(last_error())
+
+
+class StackModel(Model):
+    """A stack of mixer layers and joins in running order; caches and states belong to the model. `runs` holds
+    StackLayerDesc objects and (weights pointer, bias pointer) pairs for joins."""
+
+    def __init__(self, ctx, cfg: StackCfg, runs):
+        self._keep = (cfg, runs)
+        self.sequences, self.vocab, self.hidden = int(cfg.sequences), int(cfg.vocab), int(cfg.hidden)
+        L = lib()
+        self.h = L.m40host_stack_create(ctx, C.byref(cfg))
+        if not self.h:
+            raise RuntimeError(last_error())
+        for run in runs:
+            if isinstance(run, StackLayerDesc):
+                rc = L.m40host_stack_add_layer(self.h, C.byref(cfg), C.byref(run))
+                self.layers += 1
+            else:
+                rc = L.m40host_stack_add_join(self.h, C.byref(cfg), run[0], run[1])
+            if rc != 0:
+                raise RuntimeError(last_error())
+        if L.m40host_stack_finish(self.h) != 0:
+            raise RuntimeError(last_error())

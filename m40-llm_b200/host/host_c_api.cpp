@@ -2,12 +2,14 @@
 // negative code and m40host_last_error() gives the text.
 #include <string.h>
 
+#include <memory>
 #include <string>
 
 #include "decode_batch.hpp"
 #include "decode_layer.hpp"
 #include "decode_model.hpp"
 #include "kv_compression.hpp"
+#include "model_layer.hpp"
 
 using namespace m40host;
 
@@ -141,9 +143,10 @@ struct m40host_model_head {
     uint32_t vocab;
 };
 
-void* m40host_model_create(M40llmCudaContext* ctx, const m40host_layer_cfg* c, uint32_t n_layers,
+// max_rows: room for prompt portions of that many tokens per pass (0: token steps only).
+void* m40host_model_create_rows(M40llmCudaContext* ctx, const m40host_layer_cfg* c, uint32_t n_layers,
                            const m40host_weights* layers, const m40host_model_head* head, M40llmKVCache* kv,
-                           uint32_t sequences) {
+                           uint32_t sequences, uint32_t max_rows) {
     if (!ctx || !c || !layers || !head || !kv || n_layers == 0) {
         g_err = "m40host_model_create: null argument";
         return nullptr;
@@ -162,13 +165,106 @@ void* m40host_model_create(M40llmCudaContext* ctx, const m40host_layer_cfg* c, u
     }
     ModelHead h;
     h.embeddings = head->embeddings, h.output_norm = head->output_norm, h.lm_head = head->lm_head, h.vocab = head->vocab;
-    DecodeModel* dm = new DecodeModel(ctx, m, lw, h, kv, sequences);
+    DecodeModel* dm = new DecodeModel(ctx, m, lw, h, kv, sequences, max_rows);
     if (!dm->ok()) {
         g_err = "m40host_model_create: device allocation failed or bad arguments";
         delete dm;
         return nullptr;
     }
     return dm;
+}
+
+void* m40host_model_create(M40llmCudaContext* ctx, const m40host_layer_cfg* c, uint32_t n_layers,
+                           const m40host_weights* layers, const m40host_model_head* head, M40llmKVCache* kv,
+                           uint32_t sequences) {
+    return m40host_model_create_rows(ctx, c, n_layers, layers, head, kv, sequences, 0);
+}
+
+// ---- layer stacks: create, add joins and layers in running order, finish; then as any model
+struct m40host_stack_cfg {
+    uint32_t hidden, vocab, w_dtype, exact, sequences, max_len, max_rows;
+    float soft_cap;
+    const void *embeddings, *lm_head;
+    M40llmNorm norm;
+};
+
+void* m40host_stack_create(M40llmCudaContext* ctx, const m40host_stack_cfg* c) {
+    if (!ctx || !c || !c->embeddings || !c->lm_head || c->hidden == 0 || c->vocab == 0 || c->sequences == 0 || c->max_len == 0) {
+        g_err = "m40host_stack_create: null or zero argument";
+        return nullptr;
+    }
+    ModelHead h;
+    h.embeddings = c->embeddings, h.lm_head = c->lm_head, h.vocab = c->vocab, h.table_dtype = c->w_dtype;
+    h.generic = true, h.norm = c->norm, h.soft_cap = c->soft_cap, h.exact = c->exact != 0;
+    return new DecodeModel(ctx, c->hidden, h, c->sequences, c->max_len, c->max_rows,
+                           c->exact ? M40LLM_DT_F32 : M40LLM_DT_F16);
+}
+int m40host_stack_add_layer(void* model, const m40host_stack_cfg* c, const StackLayerDesc* d) {
+    DecodeModel* dm = (DecodeModel*)model;
+    const bool delta = d->mixer == (uint32_t)MixerKind::DeltaRule;
+    if (!delta && d->mixer != (uint32_t)MixerKind::RotaryAttention) {
+        g_err = "stack layer: unknown mixer kind " + std::to_string(d->mixer);
+        return -1;
+    }
+    const uint64_t need = delta ? 5ull * d->heads * d->dim + d->rank
+                                : (uint64_t)d->q_heads * d->k_dim + (uint64_t)d->kv_heads * (d->k_dim + d->v_dim) +
+                                      (d->has_gate ? d->q_heads : 0u);
+    if (!d->w_in || !d->w_out || d->n_in != need || (!delta && (d->kv_heads == 0 || d->q_heads % d->kv_heads != 0)) ||
+        (d->ff && (!d->gate || !d->up || !d->down))) {
+        g_err = "stack layer: sizes or weights are inconsistent";
+        return -1;
+    }
+    dm->add_layer(std::unique_ptr<ModelLayer>(new StackLayer(dm->hidden(), c->w_dtype, c->exact != 0, *d, &dm->store())));
+    return 0;
+}
+int m40host_stack_add_join(void* model, const m40host_stack_cfg* c, const void* w, const void* bias) {
+    DecodeModel* dm = (DecodeModel*)model;
+    if (!w) {
+        g_err = "stack join: no weights";
+        return -1;
+    }
+    dm->add_layer(std::unique_ptr<ModelLayer>(new JoinLayer(dm->hidden(), c->w_dtype, c->exact != 0, w, bias)));
+    return 0;
+}
+int m40host_stack_finish(void* model) {
+    DecodeModel* dm = (DecodeModel*)model;
+    const int rc = dm->finish();
+    if (rc != 0) g_err = "stack model: " + dm->failed_step();
+    return rc;
+}
+
+// ---- sequences and steps of any model
+int m40host_model_acquire(void* model) {
+    const long s = ((DecodeModel*)model)->store().acquire();
+    if (s < 0) g_err = "no free sequence slot";
+    return (int)s;
+}
+int m40host_model_release(void* model, uint32_t sequence) {
+    const int rc = ((DecodeModel*)model)->store().release(sequence);
+    if (rc != 0) g_err = "release of a sequence that is not live";
+    return rc;
+}
+uint32_t m40host_model_length(void* model, uint32_t sequence) {
+    SequenceStore& st = ((DecodeModel*)model)->store();
+    return st.live(sequence) ? st.length(sequence) : 0u;
+}
+// See DecodeModel::step; layer_trace (or null) as in DecodeModel::trace_layers.
+int m40host_model_step(void* model, uint32_t n_entries, const uint32_t* sequences, const uint32_t* counts, const uint32_t* tokens,
+                       uint32_t n_want, const uint32_t* want, float* out_logits, uint32_t* out_next, float* layer_trace) {
+    DecodeModel* dm = (DecodeModel*)model;
+    std::vector<StepEntry> e(n_entries);
+    for (uint32_t i = 0; i < n_entries; ++i) e[i] = {sequences[i], counts[i]};
+    dm->trace_layers(layer_trace);
+    const int rc = dm->step(e, tokens, std::vector<uint32_t>(want, want + n_want), out_logits, out_next);
+    dm->trace_layers(nullptr);
+    if (rc != 0) g_err = "model step failed at " + dm->failed_step() + " rc=" + std::to_string(rc);
+    return rc;
+}
+int m40host_model_begin_sequences(void* model, uint32_t n, const uint32_t* sequences, const uint32_t* token_ids) {
+    DecodeModel* dm = (DecodeModel*)model;
+    const int rc = dm->begin_sequences(n, sequences, token_ids);
+    if (rc != 0) g_err = "model begin failed at " + dm->failed_step() + " rc=" + std::to_string(rc);
+    return rc;
 }
 
 void m40host_model_destroy(void* model) { delete (DecodeModel*)model; }

@@ -20,6 +20,42 @@ HEADER_PATH = os.path.join(_HERE, "..", "include", "m40llm_native.h")
 ERR_UNSUPPORTED = -100
 ERR_LIMIT = -101
 
+DT_F16, DT_F32, DT_BF16 = 0, 1, 2
+NORM_NONE, NORM_RMS, NORM_DYT = 0, 1, 2
+ACT_SILU, ACT_GELU_TANH = 0, 1
+
+
+class Norm(C.Structure):
+    """M40llmNorm."""
+    _fields_ = [("kind", C.c_uint32), ("eps", C.c_float), ("alpha", C.c_float), ("w", C.c_void_p), ("b", C.c_void_p)]
+
+
+class Linear(C.Structure):
+    """M40llmLinear."""
+    _fields_ = ([(n, C.c_void_p) for n in ("x", "w", "w2", "out", "bias", "residual")] + [("pre", Norm), ("post", Norm)] +
+                [(n, C.c_uint32) for n in ("rows", "K", "N", "ldx", "w_dtype", "act", "exact")] + [("soft_cap", C.c_float)])
+
+
+class StepRows(C.Structure):
+    """M40llmStepRows."""
+    _fields_ = ([(n, C.c_uint32) for n in ("rows", "segments", "max_segment_rows", "max_len", "slot_mul", "slot_add")] +
+                [(n, C.c_void_p) for n in ("row_seq", "row_pos", "row_len", "seg")])
+
+
+class RotaryAttention(C.Structure):
+    """M40llmRotaryAttention."""
+    _fields_ = ([(n, C.c_void_p) for n in ("packed", "q_norm", "k_norm", "k_turns", "v_turns", "out")] +
+                [(n, C.c_uint32) for n in ("ld", "q_heads", "k_pairs", "has_gate")] +
+                [(n, C.c_float) for n in ("eps", "k_amp", "scale")])
+
+
+class DeltaRule(C.Structure):
+    """M40llmDeltaRule."""
+    _fields_ = ([(n, C.c_void_p) for n in ("packed", "w2", "w0", "a_bias", "norm", "decay_in", "out")] +
+                [(n, C.c_uint32) for n in ("ld", "rank", "w_dtype")] +
+                [(n, C.c_float) for n in ("decay_scale", "unit_eps", "eps")])
+
+
 _SCALARS = {
     "int": C.c_int, "uint32_t": C.c_uint32, "uint64_t": C.c_uint64, "size_t": C.c_size_t, "float": C.c_float,
 }
