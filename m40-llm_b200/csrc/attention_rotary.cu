@@ -225,10 +225,16 @@ __global__ void __launch_bounds__(128) rotary_rows_kernel(RotArgs a) {
         for (int i = 0; i < MAX_VDIM / 128; ++i) {
             const uint32_t d = tid + 128u * i;
             if (d >= a.vd) break;
-            float x = acc[i] * corr;
+            // the tile's sum on its own, in two chains, before it meets the running one: fewer roundings in a row
+            float x0 = 0.0f, x1 = 0.0f;
             const ET* vp = V + (size_t)t0 * a.vd + d;
-            for (uint32_t t = 0; t < m; ++t) x = fmaf(sp[t], m40_load_elem(vp + (size_t)t * a.vd), x);
-            acc[i] = x;
+            uint32_t t = 0;
+            for (; t + 2u <= m; t += 2u) {
+                x0 = fmaf(sp[t], m40_load_elem(vp + (size_t)t * a.vd), x0);
+                x1 = fmaf(sp[t + 1u], m40_load_elem(vp + (size_t)(t + 1u) * a.vd), x1);
+            }
+            if (t < m) x0 = fmaf(sp[t], m40_load_elem(vp + (size_t)t * a.vd), x0);
+            acc[i] = fmaf(acc[i], corr, x0 + x1);
         }
         __syncthreads();  // sp, red and red2 are rewritten by the next tile
     }

@@ -61,8 +61,9 @@ def bf16_to_f32(bits: np.ndarray) -> np.ndarray:
 
 
 def f32_to_bf16(x: np.ndarray) -> np.ndarray:
-    u = np.ascontiguousarray(x, np.float32).view(np.uint32)
-    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
+    x = np.asarray(x, np.float32)
+    u = np.ascontiguousarray(x).view(np.uint32)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16).reshape(x.shape)
 
 
 def write(path: str, tensors: dict[str, np.ndarray]):

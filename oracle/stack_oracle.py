@@ -167,4 +167,5 @@ class StackOracle:
             if layer_out is not None:
                 layer_out.append(x)
         self.pos += len(tokens)
-        return soft_cap(self.norm("final.norm", x) @ self.w["head"].T, cfg["logit_softcap"])
+        logits = self.norm("final.norm", x) @ self.w["head"].T
+        return soft_cap(logits, cfg["logit_softcap"]) if cfg.get("logit_softcap") else logits
