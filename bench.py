@@ -696,6 +696,277 @@ def prefill_case(nat, ev, reps=10):
                     "the call also reads the lengths back to the host as the reference does"}
 
 
+# ---------------------------------------------------------------------------------------------------- layer stacks
+STACK_SIZES = {
+    # name: width, ff, q heads, kv heads, head dim, delta heads, delta dim, rank, layers (attention at 0, 4, ...; vocabulary
+    # 32000); the Llama stack of the same name has the same width, ff, heads and number of layers
+    "tinyllama-sized": (2048, 5632, 32, 4, 64, 32, 64, 64, 8),
+    "llama3-8b-sized": (4096, 14336, 32, 8, 128, 64, 64, 128, 4),
+}
+STACK_VOCAB, STACK_PROMPT = 32000, 2048
+
+
+def _torch_stack_weights(pkg, nat, rank):
+    """Random bf16 weights made on the device, with the interface the model builder expects."""
+    import torch
+    from m40_llm_b200 import native as N
+    from m40_llm_b200.models.stack import StackWeights
+
+    class Random(StackWeights):
+        def __init__(self):
+            super().__init__(nat, None)
+            self.keep = []
+            self.gen = torch.Generator(device="cuda")
+            self.gen.manual_seed(23)
+
+        def shape(self, name):
+            return (rank,)          # only asked for the low-rank projection
+
+        def matrix(self, *names, shapes=None):
+            if names not in self._mat:
+                n, k = sum(sh[0] for sh in shapes or [(1, 1)]), shapes[0][1] if shapes else None
+                if shapes is None:
+                    raise ValueError(names)
+                t = (torch.randn(n, k, generator=self.gen, device="cuda") / k ** 0.5).to(torch.bfloat16)
+                self.keep.append(t)
+                self._mat[names] = t.data_ptr()
+            return self._mat[names]
+
+        def vector(self, name, size, row=None):
+            key = (name, row)
+            if key not in self._vec:
+                t = 1.0 + 0.1 * torch.randn(size, generator=self.gen, device="cuda")
+                self.keep.append(t)
+                self._vec[key] = t.data_ptr()
+            return self._vec[key]
+
+        def dynamic_tanh(self, name, size):
+            return N.Norm(N.NORM_DYT, 0.0, 0.8, self.vector(name, size), self.vector(name + ".b", size))
+
+    return Random()
+
+
+def stack_model(pkg, nat, name, sequences, max_len):
+    W, F, QH_, KVH_, HD_, DH, DD, R, NL = STACK_SIZES[name]
+    from m40_llm_b200 import models
+    att = {"type": "attention", "mlp": {"kind": "dense", "ff": F},
+           "mixer": {"heads": QH_, "kv_heads": KVH_, "dim": HD_, "vdim": HD_, "scale": HD_ ** -0.5,
+                     "rot": {"base": 1e6, "dims": HD_ // 2, "scaling": {"factor": 8.0, "fast": 32.0, "original": 4096, "slow": 1.0}}}}
+    dl = {"type": "general_delta", "mlp": {"kind": "dense", "ff": F}, "mixer": {"heads": DH, "dim": DD}}
+    spec = models.read_config({"architecture": "Lamutar", "width": W, "vocab": STACK_VOCAB, "norm": {"eps": 1e-5},
+                               "logit_softcap": 30.0, "layers": [att if i % 4 == 0 else dl for i in range(NL)]})
+    return spec.build(nat, _torch_stack_weights(pkg, nat, R), sequences=sequences, max_len=max_len, max_rows=STACK_PROMPT)
+
+
+def llama_model(pkg, nat, name, sequences, max_len, keep):
+    """The framework's closest existing model at the same sizes: f16 weights, Llama layers, dense f16 cache. Its projections
+    take up to 256 rows per call, so prompts run in portions of 256."""
+    import torch
+    W, F, QH_, KVH_, HD_, _, _, _, NL = STACK_SIZES[name]
+    host = pkg.host
+    g = torch.Generator(device="cuda")
+    g.manual_seed(29)
+
+    def rnd(n, k):
+        t = (torch.randn(n, k, generator=g, device="cuda") / k ** 0.5).to(torch.float16)
+        keep.append(t)
+        return t.data_ptr()
+
+    ones = torch.ones(W, device="cuda")
+    keep.append(ones)
+    lw = []
+    for _ in range(NL):
+        w = host.Weights()
+        w.attn_norm = w.ffn_norm = ones.data_ptr()
+        w.wq, w.wk, w.wv, w.wo = rnd(QH_ * HD_, W), rnd(KVH_ * HD_, W), rnd(KVH_ * HD_, W), rnd(W, QH_ * HD_)
+        w.wg, w.wu, w.wd, w.ffn_q80 = rnd(F, W), rnd(F, W), rnd(W, F), 0
+        lw.append(w)
+    head = host.ModelHead(rnd(STACK_VOCAB, W), ones.data_ptr(), rnd(STACK_VOCAB, W), STACK_VOCAB)
+    kv = nat.kv_dense(max_len, sequences * NL, KVH_, HD_)
+    m = host.DecodeModel(nat.ctx, host.LayerCfg(W, QH_, KVH_, HD_, F, 0, 1e-5, 1e4, 1.0), lw, head, kv, sequences, max_rows=256)
+    return m, kv
+
+
+def stack_ops_case(nat, ev, name, reps=20):
+    """Single calls of the layer-stack mechanisms at one size, each beside the like kernel of the Llama path."""
+    import torch
+    from m40_llm_b200 import native as N
+    W, F, QH_, KVH_, HD_, DH, DD, R, _ = STACK_SIZES[name]
+    L, ctx = nat.lib, nat.ctx
+    peak, _ = measured_peak_gbs()
+    peak_tf = 1636.2
+    try:
+        peak_tf = float(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"])
+    except Exception:
+        pass
+    keep, out = [], {}
+
+    def dev(*shape, dtype=torch.float32, std=1.0):
+        t = (torch.randn(*shape, device="cuda") * std).to(dtype)
+        keep.append(t)
+        return t.data_ptr()
+
+    def timed(call):
+        for _ in range(3):
+            assert call(0) == 0
+        nat.sync(1)
+        ev.start()
+        for i in range(reps):
+            assert call(i) == 0
+        return ev.stop_ms() / reps
+
+    def put(key, ms, flops=None, bytes_=None):
+        rec = {"us": ms * 1e3}
+        if flops:
+            rec["frac_of_bf16_tensor_peak"] = flops / (ms * 1e-3) / 1e12 / peak_tf
+        if bytes_:
+            rec["frac_of_hbm_peak"] = bytes_ / (ms * 1e-3) / 1e9 / peak
+        out[key] = rec
+
+    T = STACK_PROMPT
+    one = dev(max(W, F))
+    norm = N.Norm(N.NORM_DYT, 0.0, 0.8, one, one)
+    SETS = 4                                        # weight sets in rotation, so that one row streams from HBM
+    wqkv_n = 5 * DH * DD + R
+    mats = {"mixer_in": (wqkv_n, W), "mixer_out": (W, DH * DD), "mlp_down": (W, F)}
+    for rows in (1, 32, 256, T):
+        x, y, res = dev(rows, max(W, F)), dev(rows, max(wqkv_n, F)), dev(rows, W)
+        for key, (n, k) in mats.items():
+            ws = [dev(n, k, dtype=torch.bfloat16, std=k ** -0.5) for _ in range(SETS)]
+            post = key != "mixer_in"
+
+            def call(i):
+                c = N.Linear(x=x, w=ws[i % SETS], out=res if post else y, residual=res if post else None, pre=norm if not post else N.Norm(),
+                             post=norm if post else N.Norm(), rows=rows, K=k, N=n, w_dtype=N.DT_BF16)
+                return L.m40llm_linear_async(ctx, C.byref(c), 1)
+            put(f"{key} rows {rows}", timed(call), 2.0 * rows * n * k, n * k * 2 if rows <= 256 else None)
+            if rows <= 256:
+                hs = [dev(n, k, dtype=torch.float16, std=k ** -0.5) for _ in range(SETS)]
+                put(f"like {key}: f16 gguf gemm rows {rows}",
+                    timed(lambda i: L.m40llm_gemm_f32xf16_gguf_f32_async(ctx, x, hs[i % SETS], y, rows, n, k, 1)), 2.0 * rows * n * k, n * k * 2)
+            keep[:] = keep[:4] if rows == 1 else keep
+        wg = [(dev(F, W, dtype=torch.bfloat16, std=W ** -0.5), dev(F, W, dtype=torch.bfloat16, std=W ** -0.5)) for _ in range(SETS)]
+
+        def gate_up(i):
+            c = N.Linear(x=x, w=wg[i % SETS][0], w2=wg[i % SETS][1], out=y, pre=norm, rows=rows, K=W, N=F, w_dtype=N.DT_BF16,
+                         act=N.ACT_GELU_TANH)
+            return L.m40llm_linear_async(ctx, C.byref(c), 1)
+        put(f"mlp gate|up rows {rows}", timed(gate_up), 4.0 * rows * F * W, 4 * F * W if rows <= 256 else None)
+        if rows <= 256:
+            wh = [tuple(dev(a, b, dtype=torch.float16, std=b ** -0.5) for a, b in ((F, W), (F, W), (W, F))) for _ in range(2)]
+            put(f"like: f16 swiglu ffn (gate|up and down) rows {rows}",
+                timed(lambda i: L.m40llm_ffn_swiglu_f16_f32_async(ctx, x, *wh[i % 2], res, y, res, rows, W, F, 1)), 6.0 * rows * F * W, 6 * F * W)
+
+    def step_rows(segments):
+        seq, pos, seg = [], [], []
+        for s, p0, n in segments:
+            seg += [len(seq), n, s, p0]
+            seq += [s] * n
+            pos += list(range(p0, p0 + n))
+        u = lambda a: nat.buf(np.array(a, np.uint32)).ptr
+        return N.StepRows(len(seq), len(segments), max(s[2] for s in segments), 0, 1, 0, u(seq), u(pos), u(np.array(pos) + 1), u(seg))
+
+    # ---- rotary attention: one 2048-token prompt, and decoding at context 2047 / 8191
+    ctxs = 8192
+    for rows, segs, key in ((T, [(0, 0, T)], "prompt 2048"), (1, [(0, ctxs - 1, 1)], "decode 1 x 8192"),
+                            (32, [(s, 2047, 1) for s in range(32)], "decode 32 x 2048")):
+        max_len = ctxs if rows == 1 else 2048
+        kv = L.m40llm_kvcache_create_typed(ctx, max_len, len(segs), KVH_, HD_, HD_, N.DT_F16)
+        ld = QH_ * HD_ + 2 * KVH_ * HD_ + QH_
+        kt, vt = nat.buf(np.full(HD_ // 4, 0.01)).ptr, nat.buf(np.full(HD_ // 2, 0.01)).ptr
+        packed, o, r = dev(rows, ld), dev(rows, QH_ * HD_), step_rows(segs)
+        c = N.RotaryAttention(packed, dev(QH_ * HD_), dev(KVH_ * HD_), kt, vt, o, ld, QH_, HD_ // 4, 1, 1e-5, 1.2, HD_ ** -0.5)
+        ms = timed(lambda i: L.m40llm_attention_rotary_async(ctx, kv, C.byref(c), C.byref(r)))
+        tokens = sum(p0 + n for _, p0, n in segs)
+        if rows == T:
+            put(f"rotary attention, {key}", ms, 4.0 * HD_ * QH_ * T * (T + 1) / 2)
+            q, k, v = dev(T, QH_, HD_), dev(T, KVH_, HD_), dev(T, KVH_, HD_)
+            z, ln = nat.buf(np.zeros(1, np.uint32)).ptr, nat.buf(np.array([T], np.uint32)).ptr
+            for _ in range(2):
+                assert L.m40llm_attention_prefill_f32_gqa_varlen_async(ctx, q, k, v, z, z, ln, ln, 1, QH_, KVH_, HD_, o) == 0
+            nat.sync(0)
+            e0, e1, m = C.c_void_p(), C.c_void_p(), C.c_float()
+            L.m40llm_cuda_event_create(ctx, C.byref(e0)), L.m40llm_cuda_event_create(ctx, C.byref(e1))
+            L.m40llm_cuda_event_record(ctx, e0, 0)
+            for _ in range(reps):
+                assert L.m40llm_attention_prefill_f32_gqa_varlen_async(ctx, q, k, v, z, z, ln, ln, 1, QH_, KVH_, HD_, o) == 0
+            L.m40llm_cuda_event_record(ctx, e1, 0)
+            L.m40llm_cuda_event_elapsed_sync(ctx, e0, e1, C.byref(m))
+            put(f"like: prefill attention, {key}", m.value / reps, 4.0 * HD_ * QH_ * T * (T + 1) / 2)
+        else:
+            put(f"rotary attention, {key}", ms, None, tokens * KVH_ * HD_ * 4)
+            q = dev(rows, QH_ * HD_)
+            put(f"like: batched attention, {key}",
+                timed(lambda i: L.m40llm_attention_last_token_f32_gqa_batched_async(ctx, kv, r.row_seq, r.row_len, rows, q, QH_, o)),
+                None, tokens * KVH_ * HD_ * 4)
+        nat.sync(1)
+        L.m40llm_kvcache_destroy(kv)
+
+    # ---- delta rule: the same prompt, and one token for 1 / 32 sequences
+    HD2 = DH * DD
+    for rows, segs, key in ((T, [(0, 0, T)], "prompt 2048"), (1, [(0, 5, 1)], "decode 1"), (32, [(s, 5, 1) for s in range(32)], "decode 32")):
+        st = L.m40llm_statecache_create(ctx, len(segs), DH, DD)
+        r = step_rows(segs)
+        c = N.DeltaRule(dev(rows, wqkv_n), dev(HD2, R, dtype=torch.bfloat16, std=R ** -0.5), one, one, one, dev(rows, HD2) if rows == T else None,
+                        dev(rows, HD2), wqkv_n, R, N.DT_BF16, -0.6065, 1e-6, 1e-5)
+        ms = timed(lambda i: L.m40llm_delta_rule_async(ctx, st, C.byref(c), C.byref(r)))
+        io = rows * HD2 * 4 * 7 + 2 * len(segs) * HD2 * DD * 4      # r k v g a, decay in, result; state in and out
+        put(f"delta rule, {key}", ms, None, io)
+        nat.sync(1)
+        L.m40llm_statecache_destroy(st)
+    nat.free_all()
+    return out
+
+
+def stack_case(nat, pkg, name, steps):
+    """Prefill and greedy decode of the layer-stack model beside the Llama stack of equal size (random weights)."""
+    ev = Events(nat)
+    rec = {"sizes": dict(zip(("width", "ff", "q_heads", "kv_heads", "head_dim", "delta_heads", "delta_dim", "rank", "layers"),
+                             STACK_SIZES[name]))}
+    rng = np.random.default_rng(3)
+    prompt = rng.integers(0, STACK_VOCAB, STACK_PROMPT)
+    for kind in ("stack", "llama"):
+        keep, kv, r = [], None, {}
+        for batch in (1, 32):
+            max_len = STACK_PROMPT + 3 * steps + 16 if batch == 1 else 256 + 3 * steps + 16
+            if kind == "stack":
+                m = stack_model(pkg, nat, name, batch, max_len)
+            else:
+                m, kv = llama_model(pkg, nat, name, batch, max_len, keep)
+            if batch == 1:
+                for i in range(3):
+                    s = m.acquire()
+                    nat.sync(1)
+                    ev.start()
+                    first = m.step([(s, prompt)], [len(prompt) - 1], want_logits=False, want_next=True)["next"]
+                    ms = ev.stop_ms()
+                    if i < 2:
+                        m.release(s)
+                r["prefill_ms"], r["prefill_tokens_per_s"] = ms, STACK_PROMPT / ms * 1e3
+                slots = [s]
+            else:
+                slots = [m.acquire() for _ in range(batch)]
+                first = np.zeros(batch, np.uint32)
+                for s in slots:
+                    m.step([(s, prompt[:256])], [255], want_logits=False)
+            m.begin_sequences(slots, first)
+            m.generate(4, want_ids=False)
+            nat.sync(1)
+            ev.start()
+            m.generate(steps, want_ids=False)
+            ms = ev.stop_ms() / steps
+            r[f"decode_batch{batch}"] = {"ms_per_token": ms, "tokens_per_s": batch / ms * 1e3, "launches_per_step": m.launches_per_step()}
+            m.close()
+            if kv:
+                nat.lib.m40llm_kvcache_destroy(kv)
+                kv = None
+            nat.free_all()
+        rec[kind] = r
+    rec["stack_over_llama"] = {"prefill": rec["stack"]["prefill_tokens_per_s"] / rec["llama"]["prefill_tokens_per_s"],
+                               **{b: rec["stack"][b]["tokens_per_s"] / rec["llama"][b]["tokens_per_s"] for b in ("decode_batch1", "decode_batch32")}}
+    return rec
+
+
 def run_reference_arm(args, rank, world):
     """`--impl reference`: the reference's CPU path is Rust and cannot be built here (no cargo/rustc, no network),
     so the timed stand-in is the oracle port of that math, on all host threads. Rank 0 only. It is ONE CPU process on
@@ -747,9 +1018,10 @@ def main():
                     help="small case for a profiler: the 32K compressed attention call alone")
     ap.add_argument("--prefill-only", action="store_true",
                     help="small case for a profiler: the packed varlen prefill attention call alone")
-    ap.add_argument("--workload", default="layer", choices=["layer", "splitk"],
+    ap.add_argument("--workload", default="layer", choices=["layer", "splitk", "stack"],
                     help="layer: the batched decode layer (the contract's line); splitk: one 32K sequence, split-K over "
-                         "the ranks (its own JSON line)")
+                         "the ranks (its own JSON line); stack: the Lamutar layer stack at several sizes beside the Llama "
+                         "stack of equal size, whole models and single calls (its own JSON line, one GPU)")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
     rank = int(os.environ.get("RANK", "0"))
@@ -789,6 +1061,16 @@ def main():
 
     if args.prefill_only:
         print(json.dumps({"case": "prefill_varlen", **prefill_case(nat, Events(nat), reps=max(args.steps, 1))}), flush=True)
+        return
+
+    if args.workload == "stack":
+        clk = ClockSampler(local_rank)
+        clk.start()
+        clk.wait_first_sample()
+        rec = {n: {**stack_case(nat, pkg, n, min(args.steps, 100)), "calls": stack_ops_case(nat, Events(nat), n)} for n in STACK_SIZES}
+        print(json.dumps({"metric": "stack_prefill_and_decode_tokens_per_s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic",
+                          "config": {"prompt": STACK_PROMPT, "l2": "inputs larger than L2 (weights in rotation)"},
+                          "clocks": clk.stop(), "models": rec}), flush=True)
         return
 
     if args.workload == "splitk":

@@ -48,7 +48,7 @@ class LamutarSpec:
               max_rows: int = 2048) -> host.StackModel:
         if dtype not in ("bfloat16", "float32"):
             raise ValueError(f"dtype {dtype!r}")
-        w = StackWeights(nat, tensors)
+        w = tensors if isinstance(tensors, StackWeights) else StackWeights(nat, tensors)
         W, V = self.width, self.vocab
         cfg = host.StackCfg(hidden=W, vocab=V, w_dtype=native.DT_BF16, exact=1 if dtype == "float32" else 0,
                             sequences=sequences, max_len=max_len, max_rows=max_rows, soft_cap=self.soft_cap,
@@ -82,7 +82,7 @@ class LamutarSpec:
             d.k_pairs, d.k_turns, d.k_amp, d.scale = len(turns), w.table(turns), amp, float(m["scale"])
             d.v_turns = w.table(rotary_tables(rot["base"], V, None)[0])   # values turn unscaled over all their dimensions
         else:
-            D, R = int(m["dim"]), w.t.shape(mix + "w1")[0]
+            D, R = int(m["dim"]), w.shape(mix + "w1")[0]
             HD = H * D
             d.mixer = host.MIXER_DELTA_RULE
             d.w_in = w.matrix(*(mix + n for n in ("r", "k", "v", "g", "a", "w1")), shapes=[(HD, W)] * 5 + [(R, W)])

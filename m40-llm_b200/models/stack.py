@@ -40,6 +40,9 @@ class StackWeights:
         self._mat: dict[tuple, int] = {}
         self._vec: dict[tuple, int] = {}
 
+    def shape(self, name: str) -> tuple[int, ...]:
+        return self.t.shape(name)
+
     def matrix(self, *names: str, shapes=None) -> int:
         """bf16 rows of the named [out, in] matrices, one after the other."""
         if names not in self._mat:
