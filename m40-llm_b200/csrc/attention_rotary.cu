@@ -1,8 +1,9 @@
 // Softmax attention with whole-projection query / key norms, partial rotary keys with a scaled frequency table, rotary
 // values and a per-head output gate: m40llm_attention_rotary_async.
 //
-//   rotary_prepare_kernel  CTA = row: both norms, all rotations, the cache append, and the row's value-rotation table
-//                          (cos, sin), which the last step needs to turn the output back.
+//   rotary_prepare_kernel  CTA = (row, share of the heads): both norms, all rotations, the cache append, and the row's
+//                          value-rotation table (cos, sin), which the last step needs to turn the output back. With few
+//                          rows the heads are dealt to many CTAs, each summing the squares of the whole projection itself.
 //   attention              one of
 //     decode tiles  (attention_tiled.cu)   f16 cache, head sizes 64 / 128, few rows: token splits over the whole GPU, then
 //                                          rotary_merge_kernel merges them and finishes (turn back, gate);
@@ -36,6 +37,21 @@ struct RotArgs {
     float eps, k_amp, scale;
 };
 
+// sum of squares of x[0 .. n), this thread's share; eight loads in flight
+__device__ __forceinline__ float squares_256(const float* __restrict__ x, uint32_t n) {
+    float s0 = 0.0f, s1 = 0.0f;
+    uint32_t i = threadIdx.x;
+    for (; i + 7u * 256u < n; i += 8u * 256u) {
+        float v[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] = x[i + 256u * j];
+#pragma unroll
+        for (int j = 0; j < 8; j += 2) s0 = fmaf(v[j], v[j], s0), s1 = fmaf(v[j + 1], v[j + 1], s1);
+    }
+    for (; i < n; i += 256u) s0 = fmaf(x[i], x[i], s0);
+    return s0 + s1;
+}
+
 // sine and cosine of `pos * turns` full turns; the whole turns are dropped in double, where the product is exact enough
 __device__ __forceinline__ float2 turn_cs(uint32_t pos, double turns) {
     const double t = (double)pos * turns;
@@ -64,7 +80,7 @@ __global__ void __launch_bounds__(256) rotary_prepare_kernel(RotArgs a) {
     const uint32_t row = blockIdx.x, tid = threadIdx.x;
     const uint32_t pos = a.row_pos[row], slot = a.row_seq[row] * a.slot_mul + a.slot_add;
     if (slot >= a.slots || pos >= a.max_seq_len) {
-        if (tid == 0) atomicOr(a.status, 2u);
+        if (tid == 0 && blockIdx.y == 0) atomicOr(a.status, 2u);
         return;
     }
     const uint32_t QD = a.q_heads * a.kd, KD = a.kv_heads * a.kd, VD = a.kv_heads * a.vd, half_v = a.vd / 2u;
@@ -80,13 +96,9 @@ __global__ void __launch_bounds__(256) rotary_prepare_kernel(RotArgs a) {
     if (a.v_turns)
         for (uint32_t i = tid; i < half_v; i += 256u) {
             tv[i] = turn_cs(pos, a.v_turns[i]);
-            a.turn[(size_t)row * half_v + i] = tv[i];
+            if (blockIdx.y == 0) a.turn[(size_t)row * half_v + i] = tv[i];
         }
-    float sq = 0.0f, sk = 0.0f;
-    if (a.q_norm)
-        for (uint32_t i = tid; i < QD; i += 256u) sq = fmaf(q[i], q[i], sq);
-    if (a.k_norm)
-        for (uint32_t i = tid; i < KD; i += 256u) sk = fmaf(k[i], k[i], sk);
+    float sq = a.q_norm ? squares_256(q, QD) : 0.0f, sk = a.k_norm ? squares_256(k, KD) : 0.0f;
     sq = block_sum_256(sq, red);  // its barriers also publish the tables
     sk = block_sum_256(sk, red);
     const float nq = a.q_norm ? 1.0f / sqrtf(sq / (float)QD + a.eps) : 1.0f;
@@ -102,13 +114,16 @@ __global__ void __launch_bounds__(256) rotary_prepare_kernel(RotArgs a) {
         const float2 cs = tk[low ? d : d - a.k_pairs];
         return low ? own * cs.x - other * cs.y : own * cs.x + other * cs.y;
     };
-    for (uint32_t e = tid; e < QD; e += 256u) a.q[(size_t)row * QD + e] = turned(q, a.q_norm, nq, e);
+    // this CTA's share of the elements of each projection
+    const uint32_t step = gridDim.y * 256u, first = blockIdx.y * 256u + tid;
+#pragma unroll 2
+    for (uint32_t e = first; e < QD; e += step) a.q[(size_t)row * QD + e] = turned(q, a.q_norm, nq, e);
     ET* K = reinterpret_cast<ET*>(a.K);
     ET* V = reinterpret_cast<ET*>(a.V);
-    for (uint32_t e = tid; e < KD; e += 256u)
+    for (uint32_t e = first; e < KD; e += step)
         m40_store_elem(K + kv_row_offset(slot, e / a.kd, pos, a.kv_heads, a.max_seq_len, a.kd) + e % a.kd,
                        turned(k, a.k_norm, nk, e));
-    for (uint32_t e = tid; e < VD; e += 256u) {
+    for (uint32_t e = first; e < VD; e += step) {
         const uint32_t d = e % a.vd;
         float y = v[e];
         if (a.v_turns && d < 2u * half_v) {
@@ -119,7 +134,7 @@ __global__ void __launch_bounds__(256) rotary_prepare_kernel(RotArgs a) {
         }
         m40_store_elem(V + kv_row_offset(slot, e / a.vd, pos, a.kv_heads, a.max_seq_len, a.vd) + d, y);
     }
-    if (tid == 0 && a.seq_map) a.seq_map[slot] = pos + 1u;
+    if (tid == 0 && blockIdx.y == 0 && a.seq_map) a.seq_map[slot] = pos + 1u;
 }
 
 // Output element d of one head, given the head's attention output o[vd] in shared memory.
@@ -138,40 +153,57 @@ __device__ __forceinline__ float gate_of(const RotArgs& a, uint32_t row, uint32_
     return m40_sigmoid(a.packed[(size_t)row * a.ld + (size_t)a.q_heads * a.kd + (size_t)a.kv_heads * (a.kd + a.vd) + head]);
 }
 
-// Merge of the decode tiles' partials [row][head][split] (splits <= 128), then the finish. grid (q_heads, rows), block 128.
-__global__ void __launch_bounds__(128) rotary_merge_kernel(RotArgs a, const float* __restrict__ pm, const float* __restrict__ pl,
+// Merge of the decode tiles' partials [row][head][split] (splits <= 128, vd 64 or 128), then the finish.
+// grid (q_heads, rows), block 256: eight groups of 32 float4 lanes share the splits.
+__global__ void __launch_bounds__(256) rotary_merge_kernel(RotArgs a, const float* __restrict__ pm, const float* __restrict__ pl,
                                                            const float* __restrict__ po, uint32_t splits) {
-    __shared__ float sw[128], so[MAX_VDIM], red[4], red2[4];
+    __shared__ __align__(16) float so[128];
+    __shared__ float sw[128], red[4], red2[4];
+    __shared__ float4 sacc[8][32];
     pdl_wait();
     pdl_trigger();
     const uint32_t head = blockIdx.x, row = blockIdx.y, tid = threadIdx.x, lane = tid & 31u, warp = tid >> 5;
     const size_t base = ((size_t)row * a.q_heads + head) * splits;
+    const float gate = gate_of(a, row, head);
     const float l = tid < splits ? pl[base + tid] : 0.0f;
     const float m = l > 0.0f ? pm[base + tid] : -INFINITY;
-    float M = warp_max(m);
-    if (lane == 0) red[warp] = M;
+    const float wm = warp_max(m);
+    if (lane == 0 && warp < 4u) red[warp] = wm;
     __syncthreads();
-    M = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
+    const float M = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
     const float e = l > 0.0f ? expf(m - M) : 0.0f;
-    sw[tid] = e;
+    if (tid < 128u) sw[tid] = e;
     const float part = warp_sum(l * e);
-    if (lane == 0) red2[warp] = part;
+    if (lane == 0 && warp < 4u) red2[warp] = part;
     __syncthreads();
     const float L = (red2[0] + red2[1]) + (red2[2] + red2[3]);
     const float inv = 1.0f / (L > 0.0f ? L : 1.0f);
-    for (uint32_t d = tid; d < a.vd; d += 128u) {
-        float acc = 0.0f;
+    const uint32_t vl = a.vd / 4u;
+    float4 acc = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (lane < vl) {
 #pragma unroll 4
-        for (uint32_t s = 0; s < splits; ++s) {
-            const float w = sw[s], x = po[(base + s) * a.vd + d];
-            acc = w != 0.0f ? fmaf(w, x, acc) : acc;  // empty splits may hold anything
+        for (uint32_t s = warp; s < splits; s += 8u) {
+            const float w = sw[s];
+            const float4 x = *reinterpret_cast<const float4*>(po + (base + s) * a.vd + 4u * lane);
+            if (w != 0.0f) {  // empty splits may hold anything
+                acc.x = fmaf(w, x.x, acc.x), acc.y = fmaf(w, x.y, acc.y);
+                acc.z = fmaf(w, x.z, acc.z), acc.w = fmaf(w, x.w, acc.w);
+            }
         }
-        so[d] = acc * inv;
+    }
+    sacc[warp][lane] = acc;
+    __syncthreads();
+    if (warp == 0 && lane < vl) {
+        float4 t = sacc[0][lane];
+#pragma unroll
+        for (int i = 1; i < 8; ++i) {
+            const float4 u = sacc[i][lane];
+            t.x += u.x, t.y += u.y, t.z += u.z, t.w += u.w;
+        }
+        *reinterpret_cast<float4*>(so + 4u * lane) = make_float4(t.x * inv, t.y * inv, t.z * inv, t.w * inv);
     }
     __syncthreads();
-    const float gate = gate_of(a, row, head);
-    for (uint32_t d = tid; d < a.vd; d += 128u)
-        a.out[((size_t)row * a.q_heads + head) * a.vd + d] = finished(a, so, row, head, d, gate);
+    if (tid < a.vd) a.out[((size_t)row * a.q_heads + head) * a.vd + tid] = finished(a, so, row, head, tid, gate);
 }
 
 // Any head sizes, f16 or f32 cache, f32 arithmetic. grid (q_heads, rows), block 128: a thread scores one key of a
@@ -307,13 +339,16 @@ extern "C" int m40llm_attention_rotary_async(M40llmCudaContext* ctx, M40llmKVCac
     float* part = nullptr;
     if (decode) {
         m40_attn_pick_chunk(ctx, r->rows, kv->num_heads, bound, &chunk, &splits);
+        // o first (16-byte aligned rows for the merge), then m and l
         part = (float*)m40_ensure_scratch(ctx, 1, (size_t)r->rows * c->q_heads * splits * (2 + (size_t)vd) * sizeof(float), 0);
         if (!part) return -5;
     }
 
     const size_t table_bytes = ((size_t)c->k_pairs + vd / 2u) * sizeof(float2);
-    cudaError_t e = kv->elem_f32 ? m40_launch_dependent(rotary_prepare_kernel<float>, dim3(r->rows), dim3(256), table_bytes, s, a)
-                                 : m40_launch_dependent(rotary_prepare_kernel<__half>, dim3(r->rows), dim3(256), table_bytes, s, a);
+    const uint32_t shares_max = (c->q_heads * kd + 255u) / 256u, shares_want = (uint32_t)ctx->sm_count / r->rows;
+    const dim3 pgrid(r->rows, shares_want < 1u ? 1u : (shares_want < shares_max ? shares_want : shares_max));
+    cudaError_t e = kv->elem_f32 ? m40_launch_dependent(rotary_prepare_kernel<float>, pgrid, dim3(256), table_bytes, s, a)
+                                 : m40_launch_dependent(rotary_prepare_kernel<__half>, pgrid, dim3(256), table_bytes, s, a);
     M40_COUNT_LAUNCH(ctx);
     if (e != cudaSuccess) return -6;
 
@@ -325,9 +360,9 @@ extern "C" int m40llm_attention_rotary_async(M40llmCudaContext* ctx, M40llmKVCac
         d.seq_ids = r->row_seq;
         d.seq_lens = r->row_len;
         const size_t n = (size_t)r->rows * c->q_heads * splits;
-        d.part_m = part;
-        d.part_l = part + n;
-        d.part_o = part + 2 * n;
+        d.part_o = part;
+        d.part_m = part + n * vd;
+        d.part_l = d.part_m + n;
         d.status = ctx->d_status;
         d.max_seq_len = kv->max_seq_len;
         d.max_batch = kv->max_batch_size;
@@ -342,7 +377,7 @@ extern "C" int m40llm_attention_rotary_async(M40llmCudaContext* ctx, M40llmKVCac
         d.slot_add = r->slot_add;
         const int rc = m40_attention_dense_tiled(ctx, d, r->rows);
         if (rc != 0) return rc < 0 ? rc : -6;
-        e = m40_launch_dependent(rotary_merge_kernel, dim3(c->q_heads, r->rows), dim3(128), 0, s, a, d.part_m, d.part_l, d.part_o,
+        e = m40_launch_dependent(rotary_merge_kernel, dim3(c->q_heads, r->rows), dim3(256), 0, s, a, d.part_m, d.part_l, d.part_o,
                                  splits);
         M40_COUNT_LAUNCH(ctx);
         return e == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -6;

@@ -11,7 +11,7 @@
 //
 //   delta_scan_kernel    portions of several tokens: CTA = (32 columns, head, segment), four consumer warps walk the tokens
 //                        while four producer warps make the next chunk's vectors (gates, decays, unit keys) in shared
-//                        memory; delta_finish_kernel then applies the per-head norm and the output gate.
+//                        memory and fetch the raw values of the one after it; delta_finish_kernel then applies the per-head norm and the output gate.
 //   delta_decode_kernel  one token per sequence: CTA = (head, row) does everything, the low-rank decay projection
 //                        included, in one launch; bound by reading and writing the state once.
 // A chunked (matrix-product) form is not used: its products of decays and of removals would have to leave f32, or lose the
@@ -154,20 +154,40 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS) delta_scan_ke
     float4 s[NI];
     if (consumer) load_column<NI>(colp, D, l4, pos0 == 0 || col >= D, s);
 
-    auto produce = [&](uint32_t chunk) {
-        const uint32_t pw = (tid - SCAN_CONSUMERS) >> 5, lane = tid & 31u;
-        float* buf = ring + (size_t)(chunk & 1u) * CHUNK * TOK;
-        for (uint32_t t = pw; t < CHUNK; t += SCAN_PRODUCERS / 32) {
-            const uint32_t row = chunk * CHUNK + t;
-            if (row >= n) break;
-            const float* p = a.packed + (size_t)(row0 + row) * a.ld + head * D;
-            float* dst = buf + (size_t)t * TOK;
-            float k[CPL], ss = 0.0f;
+    // Producers: a warp owns tokens pw, pw + 4, ... of every chunk. The raw values of its tokens of one chunk are fetched
+    // into registers a whole chunk ahead (the loads fly while the consumers work), then turned into the staged vectors.
+    constexpr int TPW = CHUNK / (SCAN_PRODUCERS / 32);  // tokens per producer warp and chunk
+    const uint32_t pw = (tid - SCAN_CONSUMERS) >> 5, lane = tid & 31u;
+    float raw[TPW][4 * CPL + 1], w0[CPL], ab[CPL];
+    auto fetch = [&](uint32_t chunk) {
+#pragma unroll
+        for (int j = 0; j < TPW; ++j) {
+            const uint32_t row = chunk * CHUNK + pw + j * (SCAN_PRODUCERS / 32);
+            const size_t at = row0 + (row < n ? row : n - 1u);
+            const float* p = a.packed + at * a.ld + head * D;
 #pragma unroll
             for (int i = 0; i < CPL; ++i) {
-                const uint32_t ch = lane + 32u * i;
-                k[i] = ch < D ? p[HD + ch] : 0.0f;
-                ss = fmaf(k[i], k[i], ss);
+                const uint32_t ch = lane + 32u * i, cc = ch < D ? ch : D - 1u;  // clamped: every load is unconditional
+                raw[j][4 * i] = p[cc];
+                raw[j][4 * i + 1] = p[HD + cc];
+                raw[j][4 * i + 2] = p[4 * (size_t)HD + cc];
+                raw[j][4 * i + 3] = a.decay_in ? a.decay_in[at * HD + head * D + cc] : 0.0f;
+            }
+            raw[j][4 * CPL] = p[2 * (size_t)HD + (col0 + lane < D ? col0 + lane : D - 1u)];  // SCAN_COLS == 32
+        }
+    };
+    auto stage = [&](uint32_t chunk) {
+        float* buf = ring + (size_t)(chunk & 1u) * CHUNK * TOK;
+#pragma unroll
+        for (int j = 0; j < TPW; ++j) {
+            const uint32_t t = pw + j * (SCAN_PRODUCERS / 32), row = chunk * CHUNK + t;
+            if (row >= n) break;
+            float* dst = buf + (size_t)t * TOK;
+            float ss = 0.0f;
+#pragma unroll
+            for (int i = 0; i < CPL; ++i) {
+                const float k = lane + 32u * i < D ? raw[j][4 * i + 1] : 0.0f;
+                ss = fmaf(k, k, ss);
             }
             ss = warp_sum(ss) + a.unit_eps;
             const float len = sqrtf(ss), inv = 1.0f / len;
@@ -175,32 +195,33 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS) delta_scan_ke
             for (int i = 0; i < CPL; ++i) {
                 const uint32_t ch = lane + 32u * i;
                 if (ch >= DP) break;
-                float w = 0.0f, rate = 0.0f, r = 0.0f;
-                if (ch < D) {
-                    float z;
-                    if (a.decay_in) {
-                        z = a.decay_in[(size_t)(row0 + row) * HD + head * D + ch];
-                    } else {
-                        const float* zp = a.packed + (size_t)(row0 + row) * a.ld + 5 * (size_t)HD;
-                        z = 0.0f;
-                        for (uint32_t q = 0; q < a.rank; ++q)
-                            z = fmaf(w2_elem(a, (size_t)(head * D + ch) * a.rank + q), tanhf(zp[q]), z);
-                    }
-                    w = decay_of(a, z + a.w0[head * D + ch]);
-                    rate = m40_sigmoid(p[4 * (size_t)HD + ch] + a.a_bias[head * D + ch]);
-                    r = p[ch];
+                const bool in = ch < D;
+                float z = raw[j][4 * i + 3];
+                if (!a.decay_in && in) {
+                    const float* zp = a.packed + (size_t)(row0 + row) * a.ld + 5 * (size_t)HD;
+                    for (uint32_t q = 0; q < a.rank; ++q)
+                        z = fmaf(w2_elem(a, (size_t)(head * D + ch) * a.rank + q), tanhf(zp[q]), z);
                 }
-                dst[ch] = w;
-                dst[DP + ch] = k[i] * inv;
-                dst[2 * DP + ch] = rate;
-                dst[3 * DP + ch] = r;
+                dst[ch] = in ? decay_of(a, z + w0[i]) : 0.0f;
+                dst[DP + ch] = in ? raw[j][4 * i + 1] * inv : 0.0f;
+                dst[2 * DP + ch] = in ? m40_sigmoid(raw[j][4 * i + 2] + ab[i]) : 0.0f;
+                dst[3 * DP + ch] = in ? raw[j][4 * i] : 0.0f;
             }
-            for (uint32_t j = lane; j < SCAN_COLS; j += 32u)
-                dst[4 * DP + j] = col0 + j < D ? len * p[2 * (size_t)HD + col0 + j] : 0.0f;
+            dst[4 * DP + lane] = col0 + lane < D ? len * raw[j][4 * CPL] : 0.0f;
         }
     };
     const uint32_t chunks = (n + CHUNK - 1) / CHUNK;
-    if (!consumer) produce(0);
+    if (!consumer) {
+#pragma unroll
+        for (int i = 0; i < CPL; ++i) {
+            const uint32_t ch = lane + 32u * i, cc = ch < D ? ch : D - 1u;
+            w0[i] = a.w0[head * D + cc];
+            ab[i] = a.a_bias[head * D + cc];
+        }
+        fetch(0);
+        stage(0);
+        if (chunks > 1) fetch(1);
+    }
     __syncthreads();
     for (uint32_t ch = 0; ch < chunks; ++ch) {
         if (consumer) {
@@ -213,7 +234,8 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS) delta_scan_ke
                 if (l4 == 0 && col < D) o[(size_t)t * HD] = v;
             }
         } else if (ch + 1 < chunks) {
-            produce(ch + 1);
+            stage(ch + 1);
+            if (ch + 2 < chunks) fetch(ch + 2);
         }
         __syncthreads();
     }
