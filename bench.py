@@ -918,6 +918,26 @@ def stack_ops_case(nat, ev, name, reps=20):
     return out
 
 
+def delta_only_case(nat, args):
+    """Small case for a profiler: the delta rule over one 2048-token prompt at the llama3-8b size."""
+    from m40_llm_b200 import native as N
+    _, _, _, _, _, H, D, R, _ = STACK_SIZES["llama3-8b-sized"]
+    T, HD2, ld = STACK_PROMPT, H * D, 5 * H * D + R
+    rng = np.random.default_rng(1)
+    up = lambda *shape: nat.buf(rng.standard_normal(shape, dtype=np.float32)).ptr
+    st = nat.lib.m40llm_statecache_create(nat.ctx, 1, H, D)
+    u = lambda a: nat.buf(np.array(a, np.uint32)).ptr
+    r = N.StepRows(T, 1, T, 0, 1, 0, u([0] * T), u(range(T)), u(range(1, T + 1)), u([0, T, 0, 0]))
+    c = N.DeltaRule(up(T, ld), None, up(HD2), up(HD2), up(HD2), up(T, HD2), nat.buf(T * HD2 * 4).ptr, ld, R, N.DT_BF16, -0.6065, 1e-6, 1e-5)
+    ev = Events(nat)
+    for i in range(3 + max(args.steps, 1)):
+        if i == 3:
+            nat.sync(1)
+            ev.start()
+        assert nat.lib.m40llm_delta_rule_async(nat.ctx, st, C.byref(c), C.byref(r)) == 0
+    print(json.dumps({"case": "delta_rule_prompt2048", "us_per_call": ev.stop_ms() * 1e3 / max(args.steps, 1)}), flush=True)
+
+
 def stack_case(nat, pkg, name, steps):
     """Prefill and greedy decode of the layer-stack model beside the Llama stack of equal size (random weights)."""
     ev = Events(nat)
@@ -1018,6 +1038,8 @@ def main():
                     help="small case for a profiler: the 32K compressed attention call alone")
     ap.add_argument("--prefill-only", action="store_true",
                     help="small case for a profiler: the packed varlen prefill attention call alone")
+    ap.add_argument("--delta-only", action="store_true",
+                    help="small case for a profiler: the delta rule over one 2048-token prompt alone")
     ap.add_argument("--workload", default="layer", choices=["layer", "splitk", "stack"],
                     help="layer: the batched decode layer (the contract's line); splitk: one 32K sequence, split-K over "
                          "the ranks (its own JSON line); stack: the Lamutar layer stack at several sizes beside the Llama "
@@ -1061,6 +1083,10 @@ def main():
 
     if args.prefill_only:
         print(json.dumps({"case": "prefill_varlen", **prefill_case(nat, Events(nat), reps=max(args.steps, 1))}), flush=True)
+        return
+
+    if args.delta_only:
+        delta_only_case(nat, args)
         return
 
     if args.workload == "stack":

@@ -49,7 +49,7 @@ def trace_main(argv=None) -> int:
     ap.add_argument("--out", required=True)
     ap.add_argument("--max-tokens", type=int, default=4096, help="most tokens that live requests hold at any time")
     a = ap.parse_args(argv)
-    nat, model = _open(a.model, a.dtype, 8, max(a.max_tokens, 1))
+    nat, model = _open(a.model, a.dtype, 4, max(a.max_tokens, 1))
     slots: dict[str, int] = {}
     for line in sys.stdin:
         if not line.strip():

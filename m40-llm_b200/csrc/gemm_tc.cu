@@ -18,7 +18,9 @@
 // epilogue (bias, residual, or SiLU(gate)*up).
 //
 // Prompt rows (M > 256) are cut into blocks of 128 on grid.z. Whenever one problem needs no K split, the epilogue warps
-// apply bias, post norm, residual and soft cap themselves and store the result: no partials, no second kernel.
+// apply bias, post norm, residual and soft cap themselves and store the result: no partials, no second kernel. Gate and up
+// projections without a K split are paired: a weight tile is 64 gate rows over 64 up rows, and the epilogue warps that
+// hold the up half hand it to the others through shared memory, which store act(gate) * up.
 //
 // Every wait is bounded: a wait that runs out sets bit 2 of the context's device status word, the
 // CTA stops issuing work, frees its TMEM and returns.
@@ -46,6 +48,8 @@ struct TcArgs {
     uint32_t fmt_bits;         // operand type bits of the instruction descriptor (0: f16, see idesc_bf16())
     // direct != 0: one problem, no K split; the result is finished and stored by the epilogue warps
     uint32_t direct, n_out;
+    uint32_t paired;  // direct gate|up: problems 0 and 1 share every tile, 64 rows each
+    int act;
     float* out;
     const float* bias;
     const float* residual;
@@ -88,7 +92,7 @@ __global__ void __launch_bounds__(192, 1) gemm_tc_f16_kernel(const __grid_consta
     uint32_t problem = 0;
     while (problem + 1 < a.problems && tile >= a.tile_begin[problem + 1]) ++problem;
     const CUtensorMap* tmW = problem == 0 ? &tmW0 : (problem == 1 ? &tmW1 : &tmW2);
-    const uint32_t row0 = (tile - a.tile_begin[problem]) * BLOCK_N;
+    const uint32_t row0 = a.paired ? tile * (BLOCK_N / 2) : (tile - a.tile_begin[problem]) * BLOCK_N;
     const uint32_t kb0 = ksplit * a.kblocks_per_split;
     uint32_t kb1 = kb0 + a.kblocks_per_split;
     if (kb1 > a.kblocks_total) kb1 = a.kblocks_total;
@@ -118,6 +122,8 @@ __global__ void __launch_bounds__(192, 1) gemm_tc_f16_kernel(const __grid_consta
             for (uint32_t i = 0; i < pre; ++i) {
                 mbar_expect_tx(&full[i], stage_bytes);
                 tma_load_2d(stage_base + i * stage_bytes, tmW, &full[i], (int)((kb0 + i) * BLOCK_K), (int)row0);
+                if (a.paired)
+                    tma_load_2d(stage_base + i * stage_bytes + a_bytes / 2, &tmW1, &full[i], (int)((kb0 + i) * BLOCK_K), (int)row0);
             }
             pdl_wait();
             for (uint32_t i = 0; i < pre; ++i) {
@@ -134,6 +140,7 @@ __global__ void __launch_bounds__(192, 1) gemm_tc_f16_kernel(const __grid_consta
                 mbar_expect_tx(&full[s], stage_bytes);
                 const int kx = (int)((kb0 + i) * BLOCK_K);
                 tma_load_2d(st, tmW, &full[s], kx, (int)row0);
+                if (a.paired) tma_load_2d(st + a_bytes / 2, &tmW1, &full[s], kx, (int)row0);
                 tma_load_2d(st + a_bytes, &tmXh, &full[s], kx, (int)m_base);
                 if (a.use_lo) tma_load_2d(st + a_bytes + b_bytes, &tmXl, &full[s], kx, (int)m_base);
             }
@@ -170,6 +177,36 @@ __global__ void __launch_bounds__(192, 1) gemm_tc_f16_kernel(const __grid_consta
         ok = __all_sync(0xffffffffu, ok);  // tcgen05.ld is warp-collective
         tc_fence_after();
         const uint32_t n_glob = tile * BLOCK_N + lane_group * 32 + lane;
+        if (a.paired) {
+            // lanes 0..63 of the accumulator hold gate rows, 64..127 the up rows of the same outputs; the ring is free
+            float* xs = reinterpret_cast<float*>(smem);  // [M_pad][64]
+            const uint32_t r = (lane_group & 1u) * 32u + lane;
+            const uint32_t n = tile * (BLOCK_N / 2) + r;
+            for (uint32_t half = 0; half < 2; ++half) {
+                if (half == 1) asm volatile("bar.sync 1, 128;" ::: "memory");
+                if ((lane_group >= 2u) != (half == 0)) continue;  // up warps first, then gate warps
+                for (uint32_t c = 0; c < a.M_pad; c += 8) {
+                    float v[8];
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) v[j] = 0.0f;
+                    if (ok) {
+                        tmem_ld8(tmem_base + ((lane_group * 32u) << 16) + c, v);
+                        if (stacked) {
+                            float w[8];
+                            tmem_ld8(tmem_base + ((lane_group * 32u) << 16) + a.M_pad + c, w);
+#pragma unroll
+                            for (int j = 0; j < 8; ++j) v[j] += w[j];
+                        }
+                    }
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) {
+                        if (half == 0) xs[(c + j) * 64u + r] = v[j];
+                        else if (n < a.n_out && c + j < m_live)
+                            a.out[(size_t)(m_base + c + j) * a.n_out + n] = m40_act(a.act, v[j]) * xs[(c + j) * 64u + r];
+                    }
+                }
+            }
+        }
         float* dst = a.partial + ((size_t)ksplit * a.M + m_base) * a.n_total + n_glob;
         const bool n_ok = n_glob < a.n_out;  // direct mode: one problem, so the padded column is the output column
         float bias = 0.0f, pw = 1.0f, pb = 0.0f;
@@ -178,7 +215,7 @@ __global__ void __launch_bounds__(192, 1) gemm_tc_f16_kernel(const __grid_consta
             if (a.post_w) pw = a.post_w[n_glob];
             if (a.post_b) pb = a.post_b[n_glob];
         }
-        for (uint32_t c = 0; c < a.M_pad; c += 8) {
+        for (uint32_t c = a.paired ? a.M_pad : 0u; c < a.M_pad; c += 8) {
             float v[8];
             if (ok) {
                 tmem_ld8(tmem_base + ((lane_group * 32u) << 16) + c, v);
@@ -552,11 +589,20 @@ int m40_gemm_tc_f16(M40llmCudaContext* ctx, cudaStream_t s, uint32_t stream_kind
     // so the lo part is always carried; above ~128 rows this makes the kernel tensor-bound instead of HBM-bound.
     a.use_lo = 1u;
     uint32_t tiles = 0;
-    for (int p = 0; p < problems; ++p) {
+    // Gate|up of prompt rows in paired tiles when those alone fill the machine: no K split, and none of the M x 2N partials
+    // (up to 256 rows the separate tiles and their epilogue kernel measured faster).
+    a.paired = ext && mode == 1 && problems == 2 && N[0] == N[1] && M > 256 &&
+                       (uint32_t)((N[0] + BLOCK_N / 2 - 1) / (BLOCK_N / 2)) * m_blocks >= (uint32_t)ctx->sm_count
+                   ? 1u : 0u;
+    for (int p = 0; p < (a.paired ? 0 : problems); ++p) {
         a.tile_begin[p] = tiles;
         tiles += (uint32_t)((N[p] + BLOCK_N - 1) / BLOCK_N);
     }
-    for (int p = problems; p < 4; ++p) a.tile_begin[p] = tiles;
+    for (int p = a.paired ? 4 : problems; p < 4; ++p) a.tile_begin[p] = tiles;
+    if (a.paired) {
+        tiles = (uint32_t)((N[0] + BLOCK_N / 2 - 1) / (BLOCK_N / 2));
+        a.tile_begin[1] = a.tile_begin[2] = a.tile_begin[3] = tiles;
+    }
     a.n_total = tiles * BLOCK_N;
     a.kblocks_total = (uint32_t)((K + BLOCK_K - 1) / BLOCK_K);
     // stages from the shared-memory budget; two CTAs per SM when the stage is small
@@ -569,13 +615,13 @@ int m40_gemm_tc_f16(M40llmCudaContext* ctx, cudaStream_t s, uint32_t stream_kind
     const uint32_t ctas_per_sm = smem <= 110u * 1024u ? 2u : 1u;
     // K splits: fill about one wave of resident CTAs, keep at least 4 k-blocks per split
     uint32_t ks = ((uint32_t)ctx->sm_count * ctas_per_sm) / (tiles * m_blocks);
-    if (ks < 1) ks = 1;
+    if (ks < 1 || a.paired) ks = 1;
     const uint32_t ks_max = a.kblocks_total / 4 ? a.kblocks_total / 4 : 1;
     if (ks > ks_max) ks = ks_max;
     if (ks > 16) ks = 16;
     a.kblocks_per_split = (a.kblocks_total + ks - 1) / ks;
     ks = (a.kblocks_total + a.kblocks_per_split - 1) / a.kblocks_per_split;
-    const bool direct = ext && ks == 1 && problems == 1 && mode == 0 && !rope;
+    const bool direct = ext && ks == 1 && !rope && (a.paired || (problems == 1 && mode == 0));
 
     // scratch: [hi][lo] activation copies, then the partials
     const size_t act_elems = (size_t)M * K;
@@ -591,7 +637,7 @@ int m40_gemm_tc_f16(M40llmCudaContext* ctx, cudaStream_t s, uint32_t stream_kind
     CUtensorMap mW[3], mXh, mXl;
     for (int p = 0; p < 3; ++p) {
         const int q = p < problems ? p : 0;
-        if (!make_map_f16(&mW[p], W[q], (uint64_t)N[q], (uint64_t)K, BLOCK_N, bf16)) return -2;
+        if (!make_map_f16(&mW[p], W[q], (uint64_t)N[q], (uint64_t)K, a.paired ? BLOCK_N / 2 : BLOCK_N, bf16)) return -2;
     }
     if (!make_map_f16(&mXh, xh, (uint64_t)M, (uint64_t)K, M_pad, bf16)) return -2;
     if (!make_map_f16(&mXl, a.use_lo ? xl : xh, (uint64_t)M, (uint64_t)K, M_pad, bf16)) return -2;
@@ -633,6 +679,7 @@ int m40_gemm_tc_f16(M40llmCudaContext* ctx, cudaStream_t s, uint32_t stream_kind
         a.residual = residual ? residual[0] : nullptr;
         a.post_w = ext->post_w;
         a.post_b = ext->post_b;
+        a.act = ext->act;
     }
     static unsigned long long configured = 0ull;
     const unsigned long long bit = 1ull << (ctx->device_id & 63);

@@ -73,7 +73,7 @@ def test_linear_pre_post_residual_cap(nat, rows, n, k, wdt, exact):
 
 
 @pytest.mark.parametrize("rows", [1, 3, 70, 150, 400])
-@pytest.mark.parametrize("n,k", [(200, 192), (72, 1024), (33, 50)])
+@pytest.mark.parametrize("n,k", [(200, 192), (72, 1024), (33, 50), (9570, 136)])
 @pytest.mark.parametrize("act,fn", [(N.ACT_GELU_TANH, S.gelu_tanh), (N.ACT_SILU, lambda z: z * S.sigmoid(z))])
 def test_linear_gated(nat, rows, n, k, act, fn):
     rng = np.random.default_rng(rows + n)
@@ -364,8 +364,9 @@ def test_delta_rule_portions_and_decode(nat, H, D, R):
     d = Delta(nat, H, D, R, seed=D)
     rng = np.random.default_rng(D + R)
     p0 = {0: 0, 2: 0}
-    # portions around the 16-token staging, mixed segments, single tokens; the low-rank product inside or outside
-    for i, step in enumerate([[(0, 15)], [(0, 2)], [(2, 16), (0, 1)], [(0, 1), (2, 1)], [(2, 17)], [(0, 33), (2, 2)], [(0, 1)], [(2, 1)]]):
+    # portions around the 16- or 32-token staging, mixed segments, single tokens; the low-rank product inside or outside
+    for i, step in enumerate([[(0, 15)], [(0, 2)], [(2, 16), (0, 1)], [(0, 1), (2, 1)], [(2, 17)], [(0, 33), (2, 2)], [(0, 1)], [(2, 1)],
+                              [(0, 32)], [(2, 31), (0, 65)], [(2, 140)]]):
         segs = []
         for s, n in step:
             segs.append((s, p0[s], n))
