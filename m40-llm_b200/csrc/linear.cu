@@ -85,7 +85,8 @@ __global__ void __launch_bounds__(256) linear_f32_rows_kernel(F32Args a) {
     }
 }
 
-// Many rows: 64 x 64 output tile, 16-deep k tiles in shared memory, 4 x 4 outputs per thread.
+// Many rows: 64 x 64 output tile, 16-deep k tiles in shared memory, 4 x 4 outputs per thread. A k tile is summed on its own
+// before it joins the running sum, so that the rounding error grows with K / 16, not K.
 template <typename WT>
 __global__ void __launch_bounds__(256) linear_f32_tile_kernel(F32Args a) {
     constexpr int BM = 64, BN = 64, BK = 16;
@@ -107,6 +108,7 @@ __global__ void __launch_bounds__(256) linear_f32_tile_kernel(F32Args a) {
             if (w2) su[kk][r] = in ? m40_load_elem(w2 + (size_t)(n0 + r) * a.K + k) : 0.0f;
         }
         __syncthreads();
+        float part[4][4] = {}, part2[4][4] = {};
 #pragma unroll
         for (int kk = 0; kk < BK; ++kk) {
             const float4 xv = *reinterpret_cast<const float4*>(&sx[kk][tm]);
@@ -115,16 +117,20 @@ __global__ void __launch_bounds__(256) linear_f32_tile_kernel(F32Args a) {
 #pragma unroll
             for (int i = 0; i < 4; ++i)
 #pragma unroll
-                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(xa[i], wa[j], acc[i][j]);
+                for (int j = 0; j < 4; ++j) part[i][j] = fmaf(xa[i], wa[j], part[i][j]);
             if (w2) {
                 const float4 uv = *reinterpret_cast<const float4*>(&su[kk][tn]);
                 const float ua[4] = {uv.x, uv.y, uv.z, uv.w};
 #pragma unroll
                 for (int i = 0; i < 4; ++i)
 #pragma unroll
-                    for (int j = 0; j < 4; ++j) acc2[i][j] = fmaf(xa[i], ua[j], acc2[i][j]);
+                    for (int j = 0; j < 4; ++j) part2[i][j] = fmaf(xa[i], ua[j], part2[i][j]);
             }
         }
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) acc[i][j] += part[i][j], acc2[i][j] += part2[i][j];
         __syncthreads();
     }
 #pragma unroll
