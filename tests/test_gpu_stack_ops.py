@@ -140,7 +140,6 @@ class Attn:
         self.fv = S.rope_freqs(base, V)[0] if turn_values else None
         kt, amp = rotary_tables(base, dims, scaling)
         assert abs(amp - self.amp) < 1e-12
-        self.kt = nat.lib  # keep the library alive
         self.kv = nat.lib.m40llm_kvcache_create_typed(nat.ctx, max_len, slots * mul, G, D, V, N.DT_F32 if f32 else N.DT_F16)
         assert self.kv
         self.tabs = (kt, rotary_tables(base, V, None)[0] if turn_values else None)
