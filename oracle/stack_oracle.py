@@ -9,6 +9,7 @@ from __future__ import annotations
 import math
 
 import numpy as np
+from scipy.special import erf
 
 F = np.float64
 
@@ -169,3 +170,164 @@ class StackOracle:
         self.pos += len(tokens)
         logits = self.norm("final.norm", x) @ self.w["head"].T
         return soft_cap(logits, cfg["logit_softcap"]) if cfg.get("logit_softcap") else logits
+
+
+# ---------------------------------------------------------------------------------------- Sidalorn's mechanisms
+def gelu_erf(z):
+    z = np.asarray(z, F)
+    return 0.5 * z * (1.0 + erf(z / math.sqrt(2.0)))
+
+
+def softplus(z):
+    return np.logaddexp(0.0, np.asarray(z, F))
+
+
+def group_rms_norm(x, w, eps, groups):
+    """Every one of `groups` consecutive parts of a row is divided by its own root mean square."""
+    x = np.asarray(x, F)
+    parts = x.reshape(*x.shape[:-1], groups, -1)
+    parts = parts / np.sqrt(np.mean(parts * parts, axis=-1, keepdims=True) + eps)
+    return parts.reshape(x.shape) * np.asarray(w, F)
+
+
+def causal_conv(x, past, w, bias=None):
+    """x [T, channels], past [taps - 1, channels] the inputs before it, w [channels, taps], the last column being the
+    current token's. Returns (out, new past)."""
+    taps = w.shape[1]
+    seq = np.concatenate([past, np.asarray(x, F)])
+    out = np.zeros_like(np.asarray(x, F))
+    for t in range(len(out)):
+        for j in range(taps):
+            out[t] += w[:, j] * seq[t + j]
+        if bias is not None:
+            out[t] += bias
+    return out, seq[len(seq) - (taps - 1):]
+
+
+def latent_attention(h, C, w, m, eps):
+    """w: q dkv dkv.norm uk uv sink o; m: heads dim vdim kv_rank scale. C [n, kv_rank] the earlier tokens' latents.
+    Returns (out [T, width], C with the new rows)."""
+    h = np.asarray(h, F)
+    H, D, V = m["heads"], m["dim"], m["vdim"]
+    n0 = len(C)
+    C = np.concatenate([C, rms_norm(h @ w["dkv"].T, w["dkv.norm"], eps)])
+    q = (h @ w["q"].T).reshape(-1, H, D)
+    k, v = (C @ w["uk"].T).reshape(-1, H, D), (C @ w["uv"].T).reshape(-1, H, V)
+    out = np.zeros((len(h), H, V), F)
+    for t in range(len(h)):
+        for head in range(H):
+            s = k[:n0 + t + 1, head] @ q[t, head] * m["scale"]
+            top = max(s.max(), w["sink"][head])
+            p = np.exp(s - top)
+            out[t, head] = (p / (p.sum() + np.exp(w["sink"][head] - top))) @ v[:n0 + t + 1, head]
+    return out.reshape(len(h), H * V) @ w["o"].T, C
+
+
+def rglru(h, S, past, w, m):
+    """w: y y.b x x.b conv conv.b ra ra.b ri ri.b lam o; S [width] the state, past [taps - 1, width] earlier inputs of the
+    convolution. Returns (out [T, model width], S, past)."""
+    h = np.asarray(h, F)
+    B = m["blocks"]
+    y = gelu_tanh(h @ w["y"].T + w["y.b"])
+    u, past = causal_conv(h @ w["x"].T + w["x.b"], past, w["conv"], w["conv.b"])
+    parts = u.reshape(len(u), B, -1)
+    r = sigmoid(np.einsum("tbi,boi->tbo", parts, w["ra"]) + w["ra.b"]).reshape(u.shape)
+    i = sigmoid(np.einsum("tbi,boi->tbo", parts, w["ri"]) + w["ri.b"]).reshape(u.shape)
+    a = np.exp(-8.0 * r * softplus(w["lam"]))
+    S, out = np.array(S, F), np.zeros_like(u)
+    for t in range(len(u)):
+        S = a[t] * S + np.sqrt(1.0 - a[t] * a[t]) * i[t] * u[t]
+        out[t] = S * y[t]
+    return out @ w["o"].T, S, past
+
+
+def poly_norm(z, coef, eps):
+    """a N(z) + b N(z^2) + c N(z^3) + e, N dividing a row by its root mean square."""
+    z = np.asarray(z, F)
+    n = lambda x: x / np.sqrt(np.mean(x * x, axis=-1, keepdims=True) + eps)
+    a, b, c, e = coef
+    return a * n(z) + b * n(z * z) + c * n(z ** 3) + e
+
+
+def route(z, correction, r):
+    """Router logits z -> chosen experts and their weights per token: (ids [T, top], weights [T, top]).
+    r: top scale groups."""
+    z = np.asarray(z, F)
+    s = np.exp(z - z.max(-1, keepdims=True))
+    s /= s.sum(-1, keepdims=True)
+    choice = s + correction
+    if r.get("groups"):
+        parts = choice.reshape(len(z), r["groups"]["count"], -1)
+        best = np.argsort(-parts.max(-1), axis=-1, kind="stable")[:, :r["groups"]["keep"]]
+        keep = np.zeros(parts.shape[:2], bool)
+        np.put_along_axis(keep, best, True, axis=1)
+        choice = np.where(keep[:, :, None], parts, -np.inf).reshape(choice.shape)
+    ids = np.argsort(-choice, axis=-1, kind="stable")[:, :r["top"]]
+    got = np.take_along_axis(s, ids, axis=1)
+    return ids, got / (got.sum(-1, keepdims=True) + 1e-20) * r["scale"]
+
+
+def moe(h, w, spec):
+    """w: router correction e<i>.up e<i>.down and, with spec["shared"], shared.up shared.down."""
+    h = np.asarray(h, F)
+    r = spec["router"]
+    ids, weights = route(h @ w["router"].T, w["correction"], r)
+    out = np.zeros_like(h)
+    for t in range(len(h)):
+        for e, g in zip(ids[t], weights[t]):
+            if e >= r["experts"]:
+                out[t] += g * h[t]
+            else:
+                out[t] += g * (w[f"e{e}.down"] @ gelu_erf(w[f"e{e}.up"] @ h[t]))
+    if spec.get("shared"):
+        out += gelu_erf(h @ w["shared.up"].T) @ w["shared.down"].T
+    return out
+
+
+class SidalornOracle:
+    """A whole model, as StackOracle: one sequence, any portions."""
+
+    def __init__(self, cfg, weights):
+        self.cfg = cfg
+        self.w = {n: np.asarray(a, F) for n, a in weights.items()}
+        self.reset()
+
+    def part(self, prefix):
+        return {n[len(prefix):]: a for n, a in self.w.items() if n.startswith(prefix)}
+
+    def reset(self):
+        taps, width = self.cfg["canon"]["taps"], self.cfg["width"]
+        self.state = []
+        for ly in self.cfg["layers"]:
+            m, st = ly["mixer"], {"canon": np.zeros((taps - 1, width))}
+            if ly["type"] == "latent_attention":
+                st["C"] = np.zeros((0, m["kv_rank"]))
+            else:
+                st["S"], st["past"] = np.zeros(m["width"]), np.zeros((m["conv"] - 1, m["width"]))
+            self.state.append(st)
+
+    def norm(self, name, x):
+        return group_rms_norm(x, self.w[name], self.cfg["norm"]["eps"], self.cfg["norm"]["groups"])
+
+    def step(self, tokens, layer_out=None):
+        eps = self.cfg["norm"]["eps"]
+        x = self.w["embed"][np.asarray(tokens)]
+        for i, (ly, st) in enumerate(zip(self.cfg["layers"], self.state)):
+            p = f"l{i}."
+            mw = self.part(p + "mix.")
+            conv, st["canon"] = causal_conv(x, st["canon"], self.w[p + "canon1"])
+            if ly["type"] == "latent_attention":
+                y, st["C"] = latent_attention(x + conv, st["C"], mw, ly["mixer"], eps)
+            else:
+                y, st["S"], st["past"] = rglru(x + conv, st["S"], st["past"], mw, ly["mixer"])
+            x = x + self.norm(p + "norm1", y)
+            if ly["mlp"]:
+                fw = self.part(p + "mlp.")
+                if ly["mlp"]["kind"] == "dense":
+                    y = poly_norm(x @ fw["up"].T, fw["act"], eps) @ fw["down"].T
+                else:
+                    y = moe(x, fw, ly["mlp"])
+                x = x + self.norm(p + "norm2", y)
+            if layer_out is not None:
+                layer_out.append(x)
+        return self.norm("final.norm", x) @ self.w["head"].T
