@@ -520,17 +520,29 @@ int m40llm_attention_last_token_f32_gqa_static_async(M40llmCudaContext* ctx, con
 #define M40LLM_DT_F16 0u
 #define M40LLM_DT_F32 1u
 #define M40LLM_DT_BF16 2u
-/* Norm kinds. RMS: x / sqrt(mean(x^2) + eps) * w. DYT (dynamic tanh, no statistics): tanh(alpha * x) * w + b. */
+/* Norm kinds. RMS: x / sqrt(mean(x^2) + eps) * w, the mean over each of `groups` equal consecutive parts (0 = 1 part).
+ * DYT (dynamic tanh, no statistics): tanh(alpha * x) * w + b. POLY: w[0] R(x) + w[1] R(x^2) + w[2] R(x^3) + w[3], powers
+ * element by element, R(z) = z / sqrt(mean(z^2) + eps) over the row. ACT: the activation `act`, element by element. */
 #define M40LLM_NORM_NONE 0u
 #define M40LLM_NORM_RMS 1u
 #define M40LLM_NORM_DYT 2u
+#define M40LLM_NORM_POLY 3u
+#define M40LLM_NORM_ACT 4u
 #define M40LLM_ACT_SILU 0u
 #define M40LLM_ACT_GELU_TANH 1u
-/* w and b are f32 device vectors; either may be null for DYT (1 and 0), b is unused by RMS. */
-typedef struct { uint32_t kind; float eps; float alpha; const void* w; const void* b; } M40llmNorm;
+#define M40LLM_ACT_GELU_ERF 2u
+/* w and b are f32 device vectors; either may be null for DYT (1 and 0), b is unused by RMS and POLY, both by ACT. */
+typedef struct {
+    uint32_t kind;
+    float eps;
+    float alpha;
+    const void* w;
+    const void* b;
+    uint32_t groups, act;
+} M40llmNorm;
 /* y = pre(x) . w^T (rows [N][K]); with w2: y = act(pre(x) . w^T) * (pre(x) . w2^T); then
  * out = cap(residual + post(y + bias)). out may alias residual, not x. Row pitch of x is ldx elements (0 = K), of out and
- * residual N. `post` takes NONE or DYT. exact = 1: f32 multiply-adds only (no 16-bit operand, no tensor core); exact = 0:
+ * residual N. `post` takes NONE, DYT or RMS. exact = 1: f32 multiply-adds only (no 16-bit operand, no tensor core); exact = 0:
  * one row streams the weights through gemv_stream, more rows use the tensor cores on the activations split into 16-bit
  * hi + lo parts, and shapes neither takes (K % 8, K < 64, alignment, f32 weights) fall back to the f32 kernels. */
 typedef struct {
@@ -556,10 +568,12 @@ typedef struct {
     const uint32_t* row_pos;  /* device [rows] */
     const uint32_t* row_len;  /* device [rows], position + 1 */
     const uint32_t* seg;      /* device [segments][4]: first row, rows, sequence, position of the first row */
+    const uint32_t* seg_host; /* the same on the host, or null: calls that would pick a form per segment then take one for all */
 } M40llmStepRows;
 
-/* Dense cache with separate key and value sizes and f16 or f32 elements. f16 with k_dim == v_dim is exactly
- * m40llm_kvcache_create; any other combination is served by m40llm_attention_rotary_async only (the entry points above
+/* Dense cache with separate key and value sizes and f16 or f32 elements; v_dim 0 keeps one array only (latents, for
+ * m40llm_attention_latent_async). f16 with k_dim == v_dim is exactly m40llm_kvcache_create; any other combination with
+ * values is served by m40llm_attention_rotary_async only (the entry points above
  * return their "no dense cache" code for it). */
 M40llmKVCache* m40llm_kvcache_create_typed(M40llmCudaContext* ctx, uint32_t max_seq_len, uint32_t slots, uint32_t kv_heads,
                                            uint32_t k_dim, uint32_t v_dim, uint32_t elem_dtype);
@@ -614,6 +628,89 @@ typedef struct {
 } M40llmDeltaRule;
 int m40llm_delta_rule_async(M40llmCudaContext* ctx, M40llmStateCache* st, const M40llmDeltaRule* call,
                             const M40llmStepRows* rows);
+
+/* Per-slot recurrent values of any shape: `values` f32 per slot (rings of a causal convolution, vector states). */
+M40llmStateCache* m40llm_statecache_create_values(M40llmCudaContext* ctx, uint32_t slots, uint32_t values);
+/* One slot's `values` floats to host. Synchronous, decode stream. */
+int m40llm_statecache_debug_read_values(M40llmCudaContext* ctx, M40llmStateCache* st, uint32_t slot, float* out_host);
+
+/* Causal convolution over time, one filter per channel: out_t = (add_input ? x_t : 0) + sum_j w[c][j] x_(t - taps + 1 + j)
+ * + bias[c], inputs before a sequence's start being zero. x f32 [rows][ldx] (0 = dim), out f32 [rows][dim] (not x), w f32
+ * [dim][taps], bias f32 [dim] or null. The last inputs of every sequence live in `ring` (taps * dim values per slot, the input
+ * of position p at p % taps; null when taps == 1). taps <= 32. */
+typedef struct {
+    const void* x;
+    const void* w;
+    const void* bias;
+    void* out;
+    uint32_t ldx, dim, taps, add_input;
+} M40llmShortConv;
+int m40llm_short_conv_async(M40llmCudaContext* ctx, M40llmStateCache* ring, const M40llmShortConv* call,
+                            const M40llmStepRows* rows);
+
+/* Real-gated linear recurrence with its convolution. `packed` holds per row y [width] | x [width] (row pitch ld, f32).
+ *   u = causal convolution of x (conv_w f32 [width][taps], conv_b f32 [width] or null),
+ *   r = sigmoid(ra . u + ra_b), i = sigmoid(ri . u + ri_b), where ra and ri are block diagonal: `blocks` square matrices
+ *   [out][in] of w_dtype one after the other; log a = -decay * r * softplus(lam), a = exp(log a),
+ *   S <- a S + sqrt(1 - a^2) i u,   out = S * gelu_tanh(y).      out f32 [rows][width]
+ * `state` holds per slot S [width], then the convolution's ring [taps][width] (the input of position p at p % taps). All of the
+ * recurrence is f32; exact = 1 keeps the gates' products off the tensor cores too. width / blocks <= 1024, taps <= 32. */
+typedef struct {
+    const void* packed;
+    const void* conv_w;
+    const void* conv_b;
+    const void* ra;
+    const void* ra_b;
+    const void* ri;
+    const void* ri_b;
+    const void* lam;
+    void* out;
+    uint32_t ld, width, blocks, taps, w_dtype, exact;
+    float decay;
+} M40llmRgLru;
+int m40llm_rglru_async(M40llmCudaContext* ctx, M40llmStateCache* state, const M40llmRgLru* call, const M40llmStepRows* rows);
+
+/* Attention over a compressed (latent) cache, without positions. `packed` holds per row q [heads * dim] | c [rank] (row pitch
+ * ld, f32). c <- RMS norm (c_norm f32 [rank], eps), appended to the cache at the row's position; per head k = uk c,
+ * v = uv c (uk [heads * dim][rank], uv [heads * vdim][rank], of w_dtype);
+ *   out = sum_j p_j v_j, p = exp(scale * q . k_j) / (sum over positions 0 .. pos + exp(sink[head])); sink f32 or null.
+ * out f32 [rows][heads * vdim]. The cache is m40llm_kvcache_create_typed with one head, k_dim = rank and v_dim = 0. Keys and
+ * values of the heads are made only for long portions; otherwise uk meets the query and uv the weighted latents.
+ * rank <= 1024. */
+typedef struct {
+    const void* packed;
+    const void* c_norm;
+    const void* uk;
+    const void* uv;
+    const void* sink;
+    void* out;
+    uint32_t ld, heads, dim, vdim, w_dtype;
+    float eps, scale;
+} M40llmLatentAttention;
+int m40llm_attention_latent_async(M40llmCudaContext* ctx, M40llmKVCache* kv, const M40llmLatentAttention* call,
+                                  const M40llmStepRows* rows);
+
+/* Mixture of experts. Per row: s = softmax(logits) over experts + identity outputs; the choice is made on s + correction:
+ * of `groups` equal groups of neighbours the `keep` with the largest best choice count (groups <= 1: all), and among their
+ * members the `top` largest are chosen (ties: the lower index); weights = s of the chosen / (their sum + 1e-20) * scale.
+ *   y = sum over the chosen: weight * (expert < experts ? down_e . act(up_e . x) : x)  + add,
+ *   out = residual + post(y), post NONE, DYT or RMS. out may alias residual and x.
+ * logits f32 [rows][ld_logits]; up [experts][ff][K] and down [experts][K][ff] of w_dtype; add, residual f32 [rows][K] or
+ * null; correction f32 [experts + identity] or null. experts + identity <= 1024, top <= 32. */
+typedef struct {
+    const void* x;
+    const void* logits;
+    const void* correction;
+    const void* up;
+    const void* down;
+    const void* add;
+    const void* residual;
+    void* out;
+    M40llmNorm post;
+    uint32_t rows, K, ff, experts, identity, top, groups, keep, ld_logits, w_dtype, act, exact;
+    float scale;
+} M40llmMoe;
+int m40llm_moe_async(M40llmCudaContext* ctx, const M40llmMoe* call, uint32_t stream_kind);
 
 /* Token embedding gather for any table type (M40LLM_DT_*); an id >= vocab as in m40llm_embed_tokens_f16_async. */
 int m40llm_embed_tokens_async(M40llmCudaContext* ctx, const void* d_table, uint32_t table_dtype,

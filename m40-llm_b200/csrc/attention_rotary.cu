@@ -288,7 +288,7 @@ extern "C" int m40llm_attention_rotary_async(M40llmCudaContext* ctx, M40llmKVCac
     if (r->rows == 0 || r->segments == 0 || r->max_segment_rows == 0) return -2;
     if (c->q_heads == 0 || kv->num_heads == 0 || c->q_heads % kv->num_heads != 0) return -3;
     const bool typed = kv->d_typed_k != nullptr;
-    if (kv->compressed || (!typed && (!kv->d_k || !kv->d_v))) return -4;
+    if (kv->compressed || (typed ? !kv->d_typed_v : (!kv->d_k || !kv->d_v))) return -4;
     const uint32_t kd = kv->head_dim, vd = typed && kv->v_dim ? kv->v_dim : kd;
     if (2u * c->k_pairs > kd || kd > 1024u || vd > (uint32_t)MAX_VDIM) return -3;
     const uint64_t need = (uint64_t)c->q_heads * kd + (uint64_t)kv->num_heads * (kd + vd) + (c->has_gate ? c->q_heads : 0u);

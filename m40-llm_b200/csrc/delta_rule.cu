@@ -21,17 +21,10 @@
 //
 // The scan's waits are bounded like the tensor-core kernels': a wait that runs out raises status bit 4, the CTA stops,
 // waits (bounded) for its copies in flight and returns.
-#include <stdlib.h>
-
 #include "common.cuh"
 #include "stack_math.cuh"
+#include "state_cache.cuh"
 #include "tc_ptx.cuh"
-
-struct M40llmStateCache {
-    int device_id;
-    uint32_t slots, heads, dim;
-    float* d_state;  // [slot][head][value][key]
-};
 
 namespace {
 
@@ -498,56 +491,11 @@ int run_scan(M40llmCudaContext* ctx, const DeltaArgs& a, uint32_t segments, uint
 
 extern "C" {
 
-M40llmStateCache* m40llm_statecache_create(M40llmCudaContext* ctx, uint32_t slots, uint32_t heads, uint32_t dim) {
-    if (!ctx || slots == 0 || heads == 0 || dim == 0 || dim > 256) return nullptr;
-    if (m40_ensure_device(ctx) != 0) return nullptr;
-    M40llmStateCache* st = (M40llmStateCache*)calloc(1, sizeof(M40llmStateCache));
-    if (!st) return nullptr;
-    st->device_id = ctx->device_id;
-    st->slots = slots;
-    st->heads = heads;
-    st->dim = dim;
-    const size_t bytes = (size_t)slots * heads * dim * dim * sizeof(float);
-    if (cudaMalloc((void**)&st->d_state, bytes) != cudaSuccess || cudaMemset(st->d_state, 0, bytes) != cudaSuccess ||
-        cudaStreamSynchronize(cudaStreamLegacy) != cudaSuccess) {
-        cudaGetLastError();
-        m40llm_statecache_destroy(st);
-        return nullptr;
-    }
-    return st;
-}
-
-void m40llm_statecache_destroy(M40llmStateCache* st) {
-    if (!st) return;
-    cudaSetDevice(st->device_id);
-    if (st->d_state) cudaFree(st->d_state);
-    free(st);
-}
-
-int m40llm_statecache_debug_read(M40llmCudaContext* ctx, M40llmStateCache* st, uint32_t slot, float* out_host) {
-    if (!ctx || !st || !out_host) return -1;
-    if (slot >= st->slots) return -2;
-    if (m40_ensure_device(ctx) != 0) return -1;
-    const size_t per = (size_t)st->heads * st->dim * st->dim;
-    float* tmp = (float*)malloc(per * sizeof(float));
-    if (!tmp) return -5;
-    int rc = 0;
-    if (cudaMemcpyAsync(tmp, st->d_state + slot * per, per * sizeof(float), cudaMemcpyDeviceToHost, ctx->decode_stream) !=
-            cudaSuccess ||
-        cudaStreamSynchronize(ctx->decode_stream) != cudaSuccess)
-        rc = -4;
-    for (size_t h = 0; rc == 0 && h < st->heads; ++h)
-        for (size_t v = 0; v < st->dim; ++v)
-            for (size_t k = 0; k < st->dim; ++k)
-                out_host[(h * st->dim + k) * st->dim + v] = tmp[(h * st->dim + v) * st->dim + k];
-    free(tmp);
-    return rc;
-}
-
 int m40llm_delta_rule_async(M40llmCudaContext* ctx, M40llmStateCache* st, const M40llmDeltaRule* c,
                             const M40llmStepRows* rows) {
     if (!ctx || !st || !c || !rows || !c->packed || !c->w0 || !c->a_bias || !c->norm || !c->out) return -1;
     if (!c->decay_in && (!c->w2 || c->rank == 0 || c->rank > 1024)) return -2;
+    if (st->dim == 0) return -3;  // a cache of plain values
     if (rows->rows == 0 || rows->segments == 0 || rows->max_segment_rows == 0) return -2;
     if (rows->max_segment_rows == 1 ? (!rows->row_seq || !rows->row_pos) : !rows->seg) return -1;
     if (c->w_dtype > M40LLM_DT_BF16) return -3;

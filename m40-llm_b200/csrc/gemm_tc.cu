@@ -354,12 +354,13 @@ struct SplitRowsArgs {
     const float* b;
     uint32_t K, ldx;
     int kind;   // M40LLM_NORM_*
+    int act;    // M40LLM_NORM_ACT
     int w_f32;  // RMS weights: as in norm_split_rows_kernel
     float eps, alpha;
 };
 template <typename T>
 __global__ void __launch_bounds__(256) split_rows_kernel(SplitRowsArgs a, T* __restrict__ hi, T* __restrict__ lo) {
-    __shared__ float red[8];
+    __shared__ float red[8], red2[8], red3[8];
     pdl_wait();
     pdl_trigger();
     const float* xr = a.x + (size_t)blockIdx.x * a.ldx;
@@ -381,6 +382,26 @@ __global__ void __launch_bounds__(256) split_rows_kernel(SplitRowsArgs a, T* __r
         scale = rsqrtf(tot / (float)a.K + a.eps);
     }
     const float* wf = reinterpret_cast<const float*>(a.w);
+    float4 poly = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (a.kind == (int)M40LLM_NORM_POLY) {
+        float s1 = 0.0f, s2 = 0.0f, s3 = 0.0f;
+        for (uint32_t k = threadIdx.x * 4u; k < a.K; k += 1024u) {
+            const float4 v = *reinterpret_cast<const float4*>(xr + k);
+            const float z[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float q = z[i] * z[i], c = q * z[i];
+                s1 += q, s2 = fmaf(q, q, s2), s3 = fmaf(c, c, s3);
+            }
+        }
+        s1 = warp_sum(s1), s2 = warp_sum(s2), s3 = warp_sum(s3);
+        if ((threadIdx.x & 31u) == 0u) red[threadIdx.x >> 5] = s1, red2[threadIdx.x >> 5] = s2, red3[threadIdx.x >> 5] = s3;
+        __syncthreads();
+        s1 = s2 = s3 = 0.0f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) s1 += red[i], s2 += red2[i], s3 += red3[i];
+        poly = m40_poly_scales(wf, s1, s2, s3, (float)a.K, a.eps);
+    }
     for (uint32_t k = threadIdx.x * 4u; k < a.K; k += 1024u) {
         const float4 v = *reinterpret_cast<const float4*>(xr + k);
         float y[4] = {v.x, v.y, v.z, v.w};
@@ -391,6 +412,12 @@ __global__ void __launch_bounds__(256) split_rows_kernel(SplitRowsArgs a, T* __r
         } else if (a.kind == (int)M40LLM_NORM_RMS) {
             const float4 w = norm_w4(a.w, a.w_f32, k);
             y[0] *= scale * w.x, y[1] *= scale * w.y, y[2] *= scale * w.z, y[3] *= scale * w.w;
+        } else if (a.kind == (int)M40LLM_NORM_POLY) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) y[i] = m40_poly(poly, y[i]);
+        } else if (a.kind == (int)M40LLM_NORM_ACT) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) y[i] = m40_act(a.act, y[i]);
         }
         T h[4], l[4];
 #pragma unroll
@@ -648,7 +675,12 @@ int m40_gemm_tc_f16(M40llmCudaContext* ctx, cudaStream_t s, uint32_t stream_kind
         sa.K = (uint32_t)K;
         sa.ldx = ext->ldx ? (uint32_t)ext->ldx : (uint32_t)K;
         if (K % 4 != 0 || sa.ldx % 4 != 0 || (((uintptr_t)X) & 15u) != 0u) return -2;
-        if (norm && norm->dyt) {
+        if (norm && norm->special) {
+            sa.kind = norm->special;
+            sa.act = norm->act;
+            sa.w = norm->w;
+            sa.eps = norm->eps;
+        } else if (norm && norm->dyt) {
             sa.kind = (int)M40LLM_NORM_DYT;
             sa.w = norm->w;
             sa.b = norm->b;

@@ -71,6 +71,8 @@ struct GemvArgs {
     uint32_t row_bytes, stage_bytes, xq_off;
     int first_late;  // ring slots from this one on share their bytes with the activation digits
     int dyt;         // EXT: the norm of x is a dynamic tanh
+    int special;     // EXT: M40LLM_NORM_POLY (coefficients in norm_w) or M40LLM_NORM_ACT
+    int pre_act;
     float alpha;
     const float* norm_b;
     M40GemvExt ext;
@@ -227,7 +229,7 @@ __global__ void __launch_bounds__(THREADS, 1) gemv_stream_kernel(const __grid_co
     extern __shared__ __align__(128) uint8_t ring[];
     __shared__ uint64_t full[MAX_STAGES], empty[MAX_STAGES], xq_done;
     __shared__ float red[2][2][MAX_ROWS][CWARPS];  // [parity][matrix][row][consumer warp]
-    __shared__ float ssq[CWARPS];
+    __shared__ float ssq[EXT ? 3 : 1][CWARPS];
     __shared__ volatile uint32_t abort_flag;
     // use number (ring index / nstages) the producer last armed each slot for: a parity wait can only tell adjacent
     // uses of a slot apart, and a group may reach a slot that another group used last
@@ -334,11 +336,11 @@ __global__ void __launch_bounds__(THREADS, 1) gemv_stream_kernel(const __grid_co
                 for (int p = 0; p < UR; ++p)
                     ss += xv[p].x * xv[p].x + xv[p].y * xv[p].y + xv[p].z * xv[p].z + xv[p].w * xv[p].w;
                 ss = warp_sum(ss);
-                if (lane == 0) ssq[warp] = ss;
+                if (lane == 0) ssq[0][warp] = ss;
                 consumer_barrier();
                 float tot = 0.0f;
 #pragma unroll
-                for (int i = 0; i < CWARPS; ++i) tot += ssq[i];
+                for (int i = 0; i < CWARPS; ++i) tot += ssq[0][i];
                 scale = rsqrtf(tot / (float)a.K + a.eps);
             }
 #pragma unroll
@@ -389,7 +391,7 @@ __global__ void __launch_bounds__(THREADS, 1) gemv_stream_kernel(const __grid_co
     } else {
         float4 sv[2] = {make_float4(0.f, 0.f, 0.f, 0.f), make_float4(0.f, 0.f, 0.f, 0.f)};
         float4 wr[CPT][2];
-        const bool rms = a.norm_w && !(EXT && a.dyt);
+        const bool rms = a.norm_w && !(EXT && (a.dyt || a.special));
         if (rms) {  // the loads of the sum-of-squares pass and of this thread's own pieces go out together
             const int k = tid * 4;
             if (k < a.K) sv[0] = *reinterpret_cast<const float4*>(a.x + k);
@@ -416,6 +418,10 @@ __global__ void __launch_bounds__(THREADS, 1) gemv_stream_kernel(const __grid_co
 #pragma unroll
                     for (int i = 0; i < 8; ++i) xr[j][i] = tanhf(a.alpha * xr[j][i]) * w8[i] + b8[i];
                 }
+                if (EXT && a.special == (int)M40LLM_NORM_ACT) {
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) xr[j][i] = m40_act(a.pre_act, xr[j][i]);
+                }
                 if (rms) {
                     wr[j][0] = load_norm4(a.norm_w, a.norm_f32, k0);
                     wr[j][1] = load_norm4(a.norm_w, a.norm_f32, k0 + 4);
@@ -430,11 +436,11 @@ __global__ void __launch_bounds__(THREADS, 1) gemv_stream_kernel(const __grid_co
                 ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
             }
             ss = warp_sum(ss);
-            if (lane == 0) ssq[warp] = ss;
+            if (lane == 0) ssq[0][warp] = ss;
             consumer_barrier();
             float tot = 0.0f;
 #pragma unroll
-            for (int i = 0; i < CWARPS; ++i) tot += ssq[i];
+            for (int i = 0; i < CWARPS; ++i) tot += ssq[0][i];
             scale = rsqrtf(tot / (float)a.K + a.eps);
 #pragma unroll
             for (int j = 0; j < CPT; ++j) {
@@ -449,6 +455,33 @@ __global__ void __launch_bounds__(THREADS, 1) gemv_stream_kernel(const __grid_co
                     *reinterpret_cast<float4*>(a.xn_out + k0 + 4) = make_float4(xr[j][4], xr[j][5], xr[j][6], xr[j][7]);
                 }
             }
+        }
+    }
+
+    if constexpr (EXT && FMT != M40_GEMV_Q80) {
+        if (a.special == (int)M40LLM_NORM_POLY) {
+            float s1 = 0.0f, s2 = 0.0f, s3 = 0.0f;
+            auto add = [&](const float4& v) {
+                const float z[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const float q = z[i] * z[i], c = q * z[i];
+                    s1 += q, s2 = fmaf(q, q, s2), s3 = fmaf(c, c, s3);
+                }
+            };
+#pragma unroll 4
+            for (int k = tid * 4; k < a.K; k += CONSUMERS * 4) add(*reinterpret_cast<const float4*>(a.x + k));
+            s1 = warp_sum(s1), s2 = warp_sum(s2), s3 = warp_sum(s3);
+            if (lane == 0) ssq[0][warp] = s1, ssq[1][warp] = s2, ssq[2][warp] = s3;
+            consumer_barrier();
+            s1 = s2 = s3 = 0.0f;
+#pragma unroll
+            for (int i = 0; i < CWARPS; ++i) s1 += ssq[0][i], s2 += ssq[1][i], s3 += ssq[2][i];
+            const float4 pn = m40_poly_scales(reinterpret_cast<const float*>(a.norm_w), s1, s2, s3, (float)a.K, a.eps);
+#pragma unroll
+            for (int j = 0; j < CPT; ++j)
+#pragma unroll
+                for (int i = 0; i < 8; ++i) xr[j][i] = m40_poly(pn, xr[j][i]);
         }
     }
 
@@ -585,7 +618,8 @@ int m40_gemv_stream(M40llmCudaContext* ctx, cudaStream_t s, const float* x, int 
     int cpt_max;
     uint32_t xq_bytes = 0;
     const bool dyt = norm && norm->dyt;
-    if (fmt == M40_GEMV_Q80 && (ext || dyt)) return 1;
+    const bool special = norm && norm->special;
+    if (fmt == M40_GEMV_Q80 && (ext || dyt || special)) return 1;
     if (fmt == M40_GEMV_F16 || fmt == M40_GEMV_BF16) {
         if (K % 8 != 0) return 1;
         a.row_bytes = (uint32_t)K * 2u;
@@ -607,7 +641,7 @@ int m40_gemv_stream(M40llmCudaContext* ctx, cudaStream_t s, const float* x, int 
         if (segs[i].N <= 0 || !segs[i].W || !segs[i].out || !aligned16(segs[i].W)) return 1;
         if (gate_up && (!segs[i].W2 || !aligned16(segs[i].W2))) return 1;
     }
-    if (norm && norm->w && (!aligned16(norm->w) || (norm->xn_out && !aligned16(norm->xn_out)))) return 1;
+    if (norm && norm->w && !special && (!aligned16(norm->w) || (norm->xn_out && !aligned16(norm->xn_out)))) return 1;
     if (dyt && (!aligned16(norm->b) || norm->xn_out)) return 1;
     if ((uint64_t)a.row_bytes * nmat > STAGE_MAX || xq_bytes + 2u * a.row_bytes * nmat > SMEM_MAX) return 1;
     // the digits are only needed until every consumer holds its slice in registers: the last ring slots reuse their bytes
@@ -724,10 +758,15 @@ int m40_gemv_stream(M40llmCudaContext* ctx, cudaStream_t s, const float* x, int 
         a.alpha = norm->alpha;
         a.norm_b = norm->b;
     }
+    if (special) {
+        a.special = norm->special;
+        a.pre_act = norm->act;
+        a.eps = norm->eps;
+    }
     if (ext) a.ext = *ext;
     const int grid = g < grid_max ? g : grid_max;
     const size_t smem = smem_bytes;
-    const bool use_ext = ext != nullptr || dyt;
+    const bool use_ext = ext != nullptr || dyt || special;
     return gate_up ? launch_fmt<1>(ctx, s, a, grid, smem, fmt, cpt, use_ext)
                    : launch_fmt<0>(ctx, s, a, grid, smem, fmt, cpt, use_ext);
 }

@@ -18,7 +18,8 @@ struct M40GemvSeg {
 };
 
 // Optional norm applied to x on the fly (each CTA normalises its own copy): RMS, x <- x * rsqrt(mean(x^2)+eps) * w, or
-// dynamic tanh (`dyt`), x <- tanh(alpha * x) * w + b with f32 w and b, either of which may be null (1 and 0).
+// dynamic tanh (`dyt`), x <- tanh(alpha * x) * w + b with f32 w and b, either of which may be null (1 and 0), or (`special`)
+// a PolyNorm with its four f32 coefficients in w, or the bare activation `act` (w null).
 struct M40GemvNorm {
     const void* w;    // null: no normalisation
     int w_is_f32;     // 1: f32 weights, 0: f16
@@ -27,6 +28,8 @@ struct M40GemvNorm {
     int dyt;
     float alpha;
     const float* b;
+    int special;  // 0, M40LLM_NORM_POLY or M40LLM_NORM_ACT
+    int act;
 };
 
 // What a launch does beyond the Llama layer's norm / bias / residual / SiLU: see stack_math.cuh.

@@ -176,7 +176,7 @@ M40llmKVCache* m40llm_kvcache_create(M40llmCudaContext* ctx, uint32_t max_seq_le
 
 M40llmKVCache* m40llm_kvcache_create_typed(M40llmCudaContext* ctx, uint32_t max_seq_len, uint32_t slots, uint32_t kv_heads,
                                            uint32_t k_dim, uint32_t v_dim, uint32_t elem_dtype) {
-    if (!ctx || max_seq_len == 0 || slots == 0 || kv_heads == 0 || k_dim == 0 || v_dim == 0) return nullptr;
+    if (!ctx || max_seq_len == 0 || slots == 0 || kv_heads == 0 || k_dim == 0) return nullptr;
     if (elem_dtype != M40LLM_DT_F16 && elem_dtype != M40LLM_DT_F32) return nullptr;
     if (elem_dtype == M40LLM_DT_F16 && k_dim == v_dim) return m40llm_kvcache_create(ctx, max_seq_len, slots, kv_heads, k_dim);
     if (m40_ensure_device(ctx) != 0) return nullptr;
@@ -191,7 +191,7 @@ M40llmKVCache* m40llm_kvcache_create_typed(M40llmCudaContext* ctx, uint32_t max_
     kv->elem_f32 = elem_dtype == M40LLM_DT_F32 ? 1u : 0u;
     const size_t rows = (size_t)max_seq_len * slots * kv_heads, es = kv->elem_f32 ? 4u : 2u;
     bool ok = dev_alloc_zero((uint8_t**)&kv->d_typed_k, rows * k_dim * es);
-    ok = ok && dev_alloc_zero((uint8_t**)&kv->d_typed_v, rows * v_dim * es);
+    if (v_dim) ok = ok && dev_alloc_zero((uint8_t**)&kv->d_typed_v, rows * v_dim * es);
     ok = ok && dev_alloc_zero(&kv->d_seq_map, slots);
     ok = ok && cudaStreamSynchronize(cudaStreamLegacy) == cudaSuccess;  // as in m40llm_kvcache_create
     if (!ok) {

@@ -2,10 +2,13 @@
 //   one row      the weight-streaming GEMV (gemv_stream.cu), norm, activation and tail folded into the launch;
 //   more rows    the tcgen05 GEMM (gemm_tc.cu), norm folded into the 16-bit hi/lo split, tail into the epilogue;
 //   f32          the kernels below: f32 multiply-adds only. They are the exact mode and take every shape and alignment.
+// Norms that a route does not fold in (grouped RMS; any norm on the f32 route) and an RMS norm of the result, which needs
+// whole rows, run as passes of norm_rows.cu.
 #include "common.cuh"
 #include "gemm.cuh"
 #include "gemm_tc.cuh"
 #include "gemv_stream.cuh"
+#include "norm_rows.cuh"
 #include "stack_math.cuh"
 
 namespace {
@@ -29,33 +32,6 @@ __device__ __forceinline__ void f32_finish(const F32Args& a, uint32_t m, uint32_
     const size_t at = (size_t)m * a.N + n;
     a.out[at] = m40_tail(a.tail, y, a.bias ? a.bias[n] : 0.0f, a.post_w ? a.post_w[n] : 1.0f, a.post_b ? a.post_b[n] : 0.0f,
                          a.residual ? a.residual[at] : 0.0f);
-}
-
-// Rows of x -> norm(x), tightly packed. One CTA per row.
-__global__ void __launch_bounds__(256) norm_rows_f32_kernel(const float* __restrict__ x, uint32_t ldx, float* __restrict__ out,
-                                                            uint32_t K, int kind, const float* __restrict__ w,
-                                                            const float* __restrict__ b, float eps, float alpha) {
-    __shared__ float red[8];
-    pdl_wait();
-    pdl_trigger();
-    const float* xr = x + (size_t)blockIdx.x * ldx;
-    float* o = out + (size_t)blockIdx.x * K;
-    float scale = 1.0f;
-    if (kind == (int)M40LLM_NORM_RMS) {
-        float ss = 0.0f;
-        for (uint32_t k = threadIdx.x; k < K; k += 256u) ss = fmaf(xr[k], xr[k], ss);
-        ss = warp_sum(ss);
-        if ((threadIdx.x & 31u) == 0u) red[threadIdx.x >> 5] = ss;
-        __syncthreads();
-        float tot = 0.0f;
-#pragma unroll
-        for (int i = 0; i < 8; ++i) tot += red[i];
-        scale = 1.0f / sqrtf(tot / (float)K + eps);
-    }
-    for (uint32_t k = threadIdx.x; k < K; k += 256u) {
-        const float wk = w ? w[k] : 1.0f;
-        o[k] = kind == (int)M40LLM_NORM_DYT ? tanhf(alpha * xr[k]) * wk + (b ? b[k] : 0.0f) : xr[k] * scale * wk;
-    }
 }
 
 // A few rows: one warp per weight row (pair), lanes stride K.
@@ -156,85 +132,128 @@ int launch_f32(M40llmCudaContext* ctx, cudaStream_t s, const F32Args& a) {
 
 bool al16(const void* p) { return (((uintptr_t)p) & 15u) == 0u; }
 
-}  // namespace
+bool tc_takes(const M40llmLinear& c) {
+    const void* wp[2] = {c.w, c.w2};
+    const bool tail_used = c.post.kind != M40LLM_NORM_NONE || c.soft_cap > 0.0f || c.bias || c.residual;
+    return c.rows >= 2 && (!c.w2 || !tail_used) && al16(c.x) && c.ldx % 4 == 0 &&
+           m40_gemm_tc_supported(c.rows > 256 ? 256 : (int)c.rows, (int)c.K, c.w2 ? 2 : 1, wp);
+}
 
-extern "C" int m40llm_linear_async(M40llmCudaContext* ctx, const M40llmLinear* c, uint32_t stream_kind) {
-    if (!ctx || !c || !c->x || !c->w || !c->out || stream_kind > 1) return -1;
-    if (c->rows == 0 || c->K == 0 || c->N == 0) return -2;
-    if (c->w_dtype > M40LLM_DT_BF16 || c->act > M40LLM_ACT_GELU_TANH) return -3;
-    if (c->pre.kind > M40LLM_NORM_DYT || (c->pre.kind == M40LLM_NORM_RMS && !c->pre.w)) return -4;
-    if (c->post.kind != M40LLM_NORM_NONE && c->post.kind != M40LLM_NORM_DYT) return -4;
-    const uint32_t ldx = c->ldx ? c->ldx : c->K;
-    if (ldx < c->K) return -2;
-    if (m40_ensure_device(ctx) != 0) return -1;
-    cudaStream_t s = m40_stream(ctx, stream_kind);
-    const M40Tail tail = {(int)c->post.kind, c->post.alpha, c->soft_cap};
-    const float *post_w = (const float*)c->post.w, *post_b = (const float*)c->post.b;
-    const float *bias = (const float*)c->bias, *residual = (const float*)c->residual;
+// Whether the route the call takes applies its norm of x itself. (The streaming kernel declines a few shapes only when it is
+// called; project() then runs the norm as a pass.)
+bool folds_norm(const M40llmLinear& c) {
+    if (c.exact || c.w_dtype == M40LLM_DT_F32 || (c.pre.kind == M40LLM_NORM_RMS && c.pre.groups > 1)) return false;
+    if (c.pre.kind <= M40LLM_NORM_DYT && (!al16(c.pre.w) || !al16(c.pre.b))) return false;
+    return c.rows == 1 ? c.K % 8 == 0 && al16(c.x) : tc_takes(c);
+}
+
+// The projection itself: pre is NONE or one that the route folds in, post NONE or DYT.
+int project(M40llmCudaContext* ctx, cudaStream_t s, uint32_t stream_kind, const M40llmLinear& c) {
+    const M40Tail tail = {(int)c.post.kind, c.post.alpha, c.soft_cap};
+    const float *post_w = (const float*)c.post.w, *post_b = (const float*)c.post.b;
+    const float *bias = (const float*)c.bias, *residual = (const float*)c.residual;
     M40GemvNorm norm = {};
-    norm.w = c->pre.w;
+    norm.w = c.pre.kind == M40LLM_NORM_ACT ? nullptr : c.pre.w;
     norm.w_is_f32 = 1;
-    norm.eps = c->pre.eps;
-    norm.dyt = c->pre.kind == M40LLM_NORM_DYT ? 1 : 0;
-    norm.alpha = c->pre.alpha;
-    norm.b = (const float*)c->pre.b;
-    const M40GemvNorm* np = c->pre.kind != M40LLM_NORM_NONE ? &norm : nullptr;
-    const bool half_weights = c->w_dtype != M40LLM_DT_F32;
-    const bool tail_used = tail.post != (int)M40LLM_NORM_NONE || tail.soft_cap > 0.0f || bias || residual;
+    norm.eps = c.pre.eps;
+    norm.dyt = c.pre.kind == M40LLM_NORM_DYT ? 1 : 0;
+    norm.alpha = c.pre.alpha;
+    norm.b = (const float*)c.pre.b;
+    norm.special = c.pre.kind >= M40LLM_NORM_POLY ? (int)c.pre.kind : 0;
+    norm.act = (int)c.pre.act;
+    const M40GemvNorm* np = c.pre.kind != M40LLM_NORM_NONE ? &norm : nullptr;
+    const bool fast = !c.exact && c.w_dtype != M40LLM_DT_F32;
 
-    if (!c->exact && half_weights && c->rows == 1) {
-        const M40GemvSeg seg = {c->w, c->w2, (float*)c->out, bias, residual, (int)c->N, post_w, post_b};
-        const M40GemvExt ext = {(int)c->act, tail};
-        const int rc = m40_gemv_stream(ctx, s, (const float*)c->x, (int)c->K,
-                                       c->w_dtype == M40LLM_DT_BF16 ? M40_GEMV_BF16 : M40_GEMV_F16, c->w2 ? 1 : 0, 1, &seg,
-                                       np, &ext);
+    if (fast && c.rows == 1) {
+        const M40GemvSeg seg = {c.w, c.w2, (float*)c.out, bias, residual, (int)c.N, post_w, post_b};
+        const M40GemvExt ext = {(int)c.act, tail};
+        const int rc = m40_gemv_stream(ctx, s, (const float*)c.x, (int)c.K,
+                                       c.w_dtype == M40LLM_DT_BF16 ? M40_GEMV_BF16 : M40_GEMV_F16, c.w2 ? 1 : 0, 1, &seg, np, &ext);
         if (rc != 1) return rc;
     }
-    const void* wp[2] = {c->w, c->w2};
-    if (!c->exact && half_weights && c->rows >= 2 && (!c->w2 || !tail_used) && al16(c->x) && ldx % 4 == 0 &&
-        (!np || (al16(norm.w) && al16(norm.b))) &&
-        m40_gemm_tc_supported(c->rows > 256 ? 256 : (int)c->rows, (int)c->K, c->w2 ? 2 : 1, wp)) {
+    if (fast && tc_takes(c)) {
         M40TcExt ext = {};
-        ext.bf16 = c->w_dtype == M40LLM_DT_BF16 ? 1 : 0;
-        ext.ldx = (int)ldx;
-        ext.act = (int)c->act;
+        ext.bf16 = c.w_dtype == M40LLM_DT_BF16 ? 1 : 0;
+        ext.ldx = (int)c.ldx;
+        ext.act = (int)c.act;
         ext.tail = tail;
         ext.post_w = post_w;
         ext.post_b = post_b;
-        const __half* w[2] = {(const __half*)c->w, (const __half*)c->w2};
-        const int n[2] = {(int)c->N, (int)c->N};
-        float* o[2] = {(float*)c->out, nullptr};
+        const __half* w[2] = {(const __half*)c.w, (const __half*)c.w2};
+        const int n[2] = {(int)c.N, (int)c.N};
+        float* o[2] = {(float*)c.out, nullptr};
         const float* b[2] = {bias, nullptr};
         const float* r[2] = {residual, nullptr};
-        return m40_gemm_tc_f16(ctx, s, stream_kind, (const float*)c->x, (int)c->rows, (int)c->K, c->w2 ? 2 : 1, w, n, o, b, r,
-                               c->w2 ? 1 : 0, np, nullptr, &ext);
+        return m40_gemm_tc_f16(ctx, s, stream_kind, (const float*)c.x, (int)c.rows, (int)c.K, c.w2 ? 2 : 1, w, n, o, b, r,
+                               c.w2 ? 1 : 0, np, nullptr, &ext);
     }
 
     F32Args a = {};
-    a.x = (const float*)c->x;
-    a.ldx = ldx;
-    if (np) {  // f32 route: the norm is a pass of its own (level-1 arena: this is a composite call)
-        float* xn = (float*)m40_ensure_scratch(ctx, stream_kind, (size_t)c->rows * c->K * sizeof(float), 1);
+    a.x = (const float*)c.x;
+    a.ldx = c.ldx;
+    if (np) {
+        float* xn = (float*)m40_ensure_scratch(ctx, stream_kind, (size_t)c.rows * c.K * sizeof(float));
         if (!xn) return -5;
-        const cudaError_t e = m40_launch_dependent(norm_rows_f32_kernel, dim3(c->rows), dim3(256), 0, s, a.x, ldx, xn, c->K,
-                                                   (int)c->pre.kind, (const float*)norm.w, norm.b, norm.eps, norm.alpha);
-        M40_COUNT_LAUNCH(ctx);
-        if (e != cudaSuccess) return -6;
+        const M40NormRows first = {a.x, xn, nullptr, c.pre, c.rows, c.K, c.ldx, 0.0f};
+        const int rc = m40_norm_rows(ctx, s, first);
+        if (rc != 0) return rc;
         a.x = xn;
-        a.ldx = c->K;
+        a.ldx = c.K;
     }
-    a.w = c->w;
-    a.w2 = c->w2;
-    a.out = (float*)c->out;
+    a.w = c.w;
+    a.w2 = c.w2;
+    a.out = (float*)c.out;
     a.bias = bias;
     a.residual = residual;
     a.post_w = post_w;
     a.post_b = post_b;
-    a.M = c->rows;
-    a.N = c->N;
-    a.K = c->K;
-    a.act = (int)c->act;
+    a.M = c.rows;
+    a.N = c.N;
+    a.K = c.K;
+    a.act = (int)c.act;
     a.tail = tail;
-    if (c->w_dtype == M40LLM_DT_F32) return launch_f32<float>(ctx, s, a);
-    return c->w_dtype == M40LLM_DT_BF16 ? launch_f32<__nv_bfloat16>(ctx, s, a) : launch_f32<__half>(ctx, s, a);
+    if (c.w_dtype == M40LLM_DT_F32) return launch_f32<float>(ctx, s, a);
+    return c.w_dtype == M40LLM_DT_BF16 ? launch_f32<__nv_bfloat16>(ctx, s, a) : launch_f32<__half>(ctx, s, a);
+}
+
+}  // namespace
+
+extern "C" int m40llm_linear_async(M40llmCudaContext* ctx, const M40llmLinear* call, uint32_t stream_kind) {
+    if (!ctx || !call || !call->x || !call->w || !call->out || stream_kind > 1) return -1;
+    if (call->rows == 0 || call->K == 0 || call->N == 0) return -2;
+    if (call->w_dtype > M40LLM_DT_BF16 || call->act > M40LLM_ACT_GELU_ERF) return -3;
+    if (!m40_norm_valid(call->pre, call->K) || !m40_norm_valid(call->post, call->N)) return -4;
+    if (call->post.kind > M40LLM_NORM_DYT) return -4;
+    M40llmLinear c = *call;
+    if (c.ldx == 0) c.ldx = c.K;
+    if (c.ldx < c.K) return -2;
+    if (m40_ensure_device(ctx) != 0) return -1;
+    cudaStream_t s = m40_stream(ctx, stream_kind);
+
+    // passes of their own: rows of pre(x), rows of the plain result (level-1 arena: this is a composite call)
+    const bool rms_after = c.post.kind == M40LLM_NORM_RMS;
+    const bool norm_first = c.pre.kind != M40LLM_NORM_NONE && !folds_norm(c);
+    const size_t pre_elems = norm_first ? ((size_t)c.rows * c.K + 3) & ~(size_t)3 : 0;
+    const size_t post_elems = rms_after ? (size_t)c.rows * c.N : 0;
+    float* work = nullptr;
+    if (pre_elems + post_elems) {
+        work = (float*)m40_ensure_scratch(ctx, stream_kind, (pre_elems + post_elems) * sizeof(float), 1);
+        if (!work) return -5;
+    }
+    if (norm_first) {
+        const M40NormRows first = {(const float*)c.x, work, nullptr, c.pre, c.rows, c.K, c.ldx, 0.0f};
+        const int rc = m40_norm_rows(ctx, s, first);
+        if (rc != 0) return rc;
+        c.x = work;
+        c.ldx = c.K;
+        c.pre = M40llmNorm{};
+    }
+    if (!rms_after) return project(ctx, s, stream_kind, c);
+    const M40NormRows after = {work + pre_elems, (float*)c.out, (const float*)c.residual, c.post, c.rows, c.N, c.N, c.soft_cap};
+    c.out = work + pre_elems;
+    c.residual = nullptr;
+    c.post = M40llmNorm{};
+    c.soft_cap = 0.0f;
+    const int rc = project(ctx, s, stream_kind, c);
+    return rc != 0 ? rc : m40_norm_rows(ctx, s, after);
 }

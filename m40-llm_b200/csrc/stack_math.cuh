@@ -10,6 +10,7 @@ __device__ __forceinline__ float m40_sigmoid(float x) { return 1.0f / (1.0f + ex
 __device__ __forceinline__ float m40_act(int act, float v) {
     if (act == (int)M40LLM_ACT_GELU_TANH)  // 0.5 v (1 + tanh(sqrt(2/pi) (v + 0.044715 v^3)))
         return 0.5f * v * (1.0f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
+    if (act == (int)M40LLM_ACT_GELU_ERF) return 0.5f * v * (1.0f + erff(0.7071067811865476f * v));
     return v / (1.0f + expf(-v));  // SiLU
 }
 
@@ -35,4 +36,25 @@ __device__ __forceinline__ void m40_store_elem(__half* p, float v) { *p = __floa
 
 __device__ __forceinline__ float4 m40_vec4_or(const float* p, uint32_t k, float fallback) {
     return p ? *reinterpret_cast<const float4*>(p + k) : make_float4(fallback, fallback, fallback, fallback);
+}
+
+// PolyNorm of a row with K values and sums s1 = sum z^2, s2 = sum z^4, s3 = sum z^6: (x, y, z, w) such that the result is
+// x z + y z^2 + z z^3 + w.
+__device__ __forceinline__ float4 m40_poly_scales(const float* coef, float s1, float s2, float s3, float K, float eps) {
+    return make_float4(coef[0] / sqrtf(s1 / K + eps), coef[1] / sqrtf(s2 / K + eps), coef[2] / sqrtf(s3 / K + eps), coef[3]);
+}
+__device__ __forceinline__ float m40_poly(const float4& n, float z) { return fmaf(z, fmaf(z, fmaf(z, n.z, n.y), n.x), n.w); }
+
+// Eight consecutive values of a 16-bit type (16-byte aligned), or of f32, as f32.
+template <typename WT>
+__device__ __forceinline__ void m40_load8(const WT* p, float* v) {
+    const uint4 r = *reinterpret_cast<const uint4*>(p);
+    const WT* h = reinterpret_cast<const WT*>(&r);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = m40_load_elem(h + i);
+}
+template <>
+__device__ __forceinline__ void m40_load8<float>(const float* p, float* v) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = p[i];
 }

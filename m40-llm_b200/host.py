@@ -38,7 +38,7 @@ class StackCfg(C.Structure):
                 [("soft_cap", C.c_float), ("embeddings", C.c_void_p), ("lm_head", C.c_void_p), ("norm", Norm)])
 
 
-MIXER_ROTARY_ATTENTION, MIXER_DELTA_RULE = 1, 2
+MIXER_ROTARY_ATTENTION, MIXER_DELTA_RULE, MIXER_LATENT_ATTENTION, MIXER_RGLRU = 1, 2, 3, 4
 
 
 class StackLayerDesc(C.Structure):
@@ -51,7 +51,14 @@ class StackLayerDesc(C.Structure):
                 [(n, C.c_uint32) for n in ("heads", "dim", "rank")] +
                 [("decay_scale", C.c_float), ("unit_eps", C.c_float)] +
                 [(n, C.c_void_p) for n in ("w2", "w0", "a_bias", "o_norm")] +
-                [("ff", C.c_uint32), ("act", C.c_uint32)] + [(n, C.c_void_p) for n in ("gate", "up", "down")])
+                [("ff", C.c_uint32), ("act", C.c_uint32)] + [(n, C.c_void_p) for n in ("gate", "up", "down")] + [("mid", Norm)] +
+                [(n, C.c_uint32) for n in ("experts", "identity", "top", "groups", "keep")] +
+                [("router_scale", C.c_float), ("shared_ff", C.c_uint32), ("n_router", C.c_uint32)] +
+                [(n, C.c_void_p) for n in ("w_router", "shared_down", "correction")] +
+                [("conv_taps", C.c_uint32), ("conv_w", C.c_void_p), ("in_bias", C.c_void_p), ("rank_kv", C.c_uint32)] +
+                [(n, C.c_void_p) for n in ("c_norm", "uk", "uv", "sink")] +
+                [(n, C.c_uint32) for n in ("rg_width", "rg_blocks", "rg_taps")] + [("rg_decay", C.c_float)] +
+                [(n, C.c_void_p) for n in ("rg_conv", "rg_conv_b", "ra", "ra_b", "ri", "ri_b", "lam")])
 
 
 class KvCfg(C.Structure):

@@ -46,7 +46,7 @@ int DecodeModel::allocate() {
     bool good = get(r * h * 4, &buf_.x) && get(r * h * 4, &buf_.spare) && get(r * h * 4, &buf_.x1) &&
                 get(r * needs_.packed * 4, &buf_.packed) && get(r * needs_.att * 4, &buf_.att) &&
                 get(r * needs_.hid * 4, &buf_.hid) && get(r * needs_.low * 4, &buf_.low) &&
-                get(needs_.x0 ? r * h * 4 : 0, &buf_.x0) && get((size_t)max_want_ * h * 4, &d_want_x_) &&
+                get(needs_.x0 ? r * h * 4 : 0, &buf_.x0) && get(needs_.conv ? r * h * 4 : 0, &buf_.conv) && get((size_t)max_want_ * h * 4, &d_want_x_) &&
                 get((size_t)max_want_ * head_.vocab * 4, &d_logits_) && get((9 * r + max_want_) * 4, &d_plan_) &&
                 get((size_t)flat_layers_ * r * 4, (void**)&d_flat_) && get((size_t)kHistory * seqs_ * 4, &d_history_);
     if (!good) return -1;
@@ -61,7 +61,7 @@ DecodeModel::~DecodeModel() {
     m40llm_stream_synchronize(ctx_, 1);
     for (auto& g : graphs_)
         if (g.second) m40llm_cuda_graph_destroy(g.second);
-    void* bufs[] = {buf_.x, buf_.spare, buf_.x0, buf_.packed, buf_.att, buf_.x1, buf_.hid, buf_.low,
+    void* bufs[] = {buf_.x, buf_.spare, buf_.x0, buf_.packed, buf_.att, buf_.x1, buf_.hid, buf_.low, buf_.conv,
                     d_want_x_, d_logits_, d_plan_, d_flat_, d_history_};
     for (void* b : bufs)
         if (b) m40llm_device_free(ctx_, b);
@@ -74,7 +74,7 @@ int DecodeModel::fail(int rc, const std::string& step) {
 
 StepBatch DecodeModel::batch(uint32_t rows, uint32_t segments, uint32_t max_segment_rows, uint32_t max_len) const {
     StepBatch b;
-    b.rows = {rows, segments, max_segment_rows, max_len, 1u, 0u, d_seq_, d_pos_, d_lens_, d_seg_};
+    b.rows = {rows, segments, max_segment_rows, max_len, 1u, 0u, d_seq_, d_pos_, d_lens_, d_seg_, max_len ? seg_host_.data() : nullptr};
     b.flat_slots = d_flat_;
     b.flat_stride = max_rows_;
     return b;
@@ -93,6 +93,7 @@ int DecodeModel::upload_rows(uint32_t rows, const std::vector<uint32_t>& tokens,
     }
     std::copy(want.begin(), want.end(), host.begin() + 4 * r);
     std::copy(seg.begin(), seg.end(), host.begin() + 5 * r);
+    seg_host_ = seg;
     int rc = m40llm_stream_synchronize(ctx_, 1);
     if (rc != 0) return fail(rc, "stream_synchronize");
     if ((rc = m40llm_memcpy_h2d(ctx_, d_plan_, host.data(), host.size() * 4)) != 0) return fail(rc, "upload_plan");

@@ -113,6 +113,7 @@ private:
     void* d_history_ = nullptr;   // u32 [kHistory][sequences]: ids generated by the steps of one generate() call
     uint32_t rows_ = 0;           // rows of the current token step
     std::vector<uint32_t> row_sequences_;
+    std::vector<uint32_t> seg_host_;  // segments of the last upload
     std::map<uint32_t, M40llmCudaGraphExec*> graphs_;  // by rows
     std::map<uint32_t, bool> capture_tried_;
     float* layer_trace_ = nullptr;

@@ -201,16 +201,32 @@ void* m40host_stack_create(M40llmCudaContext* ctx, const m40host_stack_cfg* c) {
 }
 int m40host_stack_add_layer(void* model, const m40host_stack_cfg* c, const StackLayerDesc* d) {
     DecodeModel* dm = (DecodeModel*)model;
-    const bool delta = d->mixer == (uint32_t)MixerKind::DeltaRule;
-    if (!delta && d->mixer != (uint32_t)MixerKind::RotaryAttention) {
-        g_err = "stack layer: unknown mixer kind " + std::to_string(d->mixer);
-        return -1;
+    uint64_t need = 0;
+    bool good = d->w_in && d->w_out;
+    switch ((MixerKind)d->mixer) {
+        case MixerKind::DeltaRule: need = 5ull * d->heads * d->dim + d->rank; break;
+        case MixerKind::RotaryAttention:
+            need = (uint64_t)d->q_heads * d->k_dim + (uint64_t)d->kv_heads * (d->k_dim + d->v_dim) + (d->has_gate ? d->q_heads : 0u);
+            good = good && d->kv_heads && d->q_heads % d->kv_heads == 0;
+            break;
+        case MixerKind::LatentAttention:
+            need = (uint64_t)d->q_heads * d->k_dim + d->rank_kv;
+            good = good && d->rank_kv && d->c_norm && d->uk && d->uv;
+            break;
+        case MixerKind::RgLru:
+            need = 2ull * d->rg_width;
+            good = good && d->rg_blocks && d->rg_width % d->rg_blocks == 0 && d->rg_taps && d->rg_conv && d->ra && d->ri && d->lam;
+            break;
+        default:
+            g_err = "stack layer: unknown mixer kind " + std::to_string(d->mixer);
+            return -1;
     }
-    const uint64_t need = delta ? 5ull * d->heads * d->dim + d->rank
-                                : (uint64_t)d->q_heads * d->k_dim + (uint64_t)d->kv_heads * (d->k_dim + d->v_dim) +
-                                      (d->has_gate ? d->q_heads : 0u);
-    if (!d->w_in || !d->w_out || d->n_in != need || (!delta && (d->kv_heads == 0 || d->q_heads % d->kv_heads != 0)) ||
-        (d->ff && (!d->gate || !d->up || !d->down))) {
+    // padding rows may follow (they keep the row pitch aligned)
+    good = good && d->n_in >= need && need && (!d->ff || (d->up && d->down)) && (!d->conv_taps || d->conv_w);
+    if (d->experts)
+        good = good && d->ff && d->w_router && (uint64_t)d->shared_ff + d->experts + d->identity <= d->n_router &&
+               (!d->shared_ff || d->shared_down);
+    if (!good) {
         g_err = "stack layer: sizes or weights are inconsistent";
         return -1;
     }

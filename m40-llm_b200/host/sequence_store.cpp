@@ -23,12 +23,15 @@ size_t SequenceStore::add(bool is_state, uint32_t heads, uint32_t a, uint32_t b)
 }
 
 size_t SequenceStore::add_kv(uint32_t kv_heads, uint32_t k_dim, uint32_t v_dim) { return add(false, kv_heads, k_dim, v_dim); }
+size_t SequenceStore::add_latent(uint32_t rank) { return add(false, 1u, rank, 0u); }
 size_t SequenceStore::add_state(uint32_t heads, uint32_t dim) { return add(true, heads, dim, 0u); }
+size_t SequenceStore::add_values(uint32_t values) { return add(true, 0u, values, 0u); }
 
 int SequenceStore::allocate() {
     for (Group& g : groups_) {
         const uint32_t slots = (uint32_t)length_.size() * g.members;
-        if (g.is_state) g.state = m40llm_statecache_create(ctx_, slots, g.heads, g.a);
+        if (g.is_state) g.state = g.heads ? m40llm_statecache_create(ctx_, slots, g.heads, g.a)
+                                          : m40llm_statecache_create_values(ctx_, slots, g.a);
         else g.kv = m40llm_kvcache_create_typed(ctx_, max_len_, slots, g.heads, g.a, g.b, elem_dtype_);
         if (!g.kv && !g.state) return -1;
     }

@@ -24,7 +24,9 @@ public:
 
     // Registers one cache-bearing layer (before allocate()) and returns its handle.
     size_t add_kv(uint32_t kv_heads, uint32_t k_dim, uint32_t v_dim);
+    size_t add_latent(uint32_t rank);                    // one array of `rank` values per token (kv())
     size_t add_state(uint32_t heads, uint32_t dim);
+    size_t add_values(uint32_t values);                  // f32 values per sequence (state())
     int allocate();  // 0, or -1 when a cache could not be made
 
     M40llmKVCache* kv(size_t handle) const { return groups_[members_[handle].group].kv; }
@@ -45,7 +47,7 @@ public:
 private:
     struct Group {
         bool is_state;
-        uint32_t heads, a, b;  // kv: k_dim, v_dim; state: dim, 0
+        uint32_t heads, a, b;  // kv: k_dim, v_dim (0: latents); state: dim, 0, or heads = 0 and the number of values
         uint32_t members;
         M40llmKVCache* kv;
         M40llmStateCache* state;

@@ -38,4 +38,4 @@ def load(nat, directory: str, **options):
     return spec.build(nat, TensorFile(os.path.join(directory, "model.safetensors")), **options)
 
 
-from . import lamutar  # noqa: E402,F401  (registers itself)
+from . import lamutar, sidalorn  # noqa: E402,F401  (they register themselves)

@@ -43,14 +43,32 @@ class StackWeights:
     def shape(self, name: str) -> tuple[int, ...]:
         return self.t.shape(name)
 
-    def matrix(self, *names: str, shapes=None) -> int:
-        """bf16 rows of the named [out, in] matrices, one after the other."""
+    def matrix(self, *names: str, shapes=None, rows: int = 0) -> int:
+        """bf16 rows of the named [out, in] matrices, one after the other; zero rows follow up to `rows` of them."""
         if names not in self._mat:
             for n, shape in zip(names, shapes or ()):
                 if self.t.shape(n) != tuple(shape):
                     raise ValueError(f"tensor {n}: shape {self.t.shape(n)}, expected {tuple(shape)}")
-            self._mat[names] = self.nat.buf(np.concatenate([self.t.bf16(n) for n in names])).ptr
+            parts = [self.t.bf16(n) for n in names]
+            missing = rows - sum(len(p) for p in parts)
+            if missing > 0:
+                parts.append(np.zeros((missing, *parts[0].shape[1:]), np.uint16))
+            self._mat[names] = self.nat.buf(np.concatenate(parts)).ptr
         return self._mat[names]
+
+    def vectors(self, names, sizes, total: int) -> int:
+        """f32 copies of several vectors, one after the other, zeros up to `total` values."""
+        key = ("vectors", *names)
+        if key not in self._vec:
+            out, at = np.zeros(total, np.float32), 0
+            for n, size in zip(names, sizes):
+                a = self.t.f32(n).reshape(-1)
+                if a.size != size:
+                    raise ValueError(f"tensor {n}: {a.size} values, expected {size}")
+                out[at:at + size] = a
+                at += size
+            self._vec[key] = self.nat.buf(out).ptr
+        return self._vec[key]
 
     def vector(self, name: str, size: int, row: int | None = None) -> int:
         """f32 copy of a vector, or of one row of a matrix."""
@@ -68,6 +86,9 @@ class StackWeights:
         if key not in self._vec:
             self._vec[key] = self.nat.buf(np.ascontiguousarray(values, np.float64)).ptr
         return self._vec[key]
+
+    def rms(self, name: str, size: int, eps: float, groups: int = 1) -> native.Norm:
+        return native.Norm(native.NORM_RMS, eps, 0.0, self.vector(name, size), None, groups, 0)
 
     def dynamic_tanh(self, name: str, size: int) -> native.Norm:
         alpha = self.t.f32(name + ".alpha").reshape(-1)

@@ -21,13 +21,14 @@ ERR_UNSUPPORTED = -100
 ERR_LIMIT = -101
 
 DT_F16, DT_F32, DT_BF16 = 0, 1, 2
-NORM_NONE, NORM_RMS, NORM_DYT = 0, 1, 2
-ACT_SILU, ACT_GELU_TANH = 0, 1
+NORM_NONE, NORM_RMS, NORM_DYT, NORM_POLY, NORM_ACT = 0, 1, 2, 3, 4
+ACT_SILU, ACT_GELU_TANH, ACT_GELU_ERF = 0, 1, 2
 
 
 class Norm(C.Structure):
     """M40llmNorm."""
-    _fields_ = [("kind", C.c_uint32), ("eps", C.c_float), ("alpha", C.c_float), ("w", C.c_void_p), ("b", C.c_void_p)]
+    _fields_ = [("kind", C.c_uint32), ("eps", C.c_float), ("alpha", C.c_float), ("w", C.c_void_p), ("b", C.c_void_p),
+                ("groups", C.c_uint32), ("act", C.c_uint32)]
 
 
 class Linear(C.Structure):
@@ -39,7 +40,7 @@ class Linear(C.Structure):
 class StepRows(C.Structure):
     """M40llmStepRows."""
     _fields_ = ([(n, C.c_uint32) for n in ("rows", "segments", "max_segment_rows", "max_len", "slot_mul", "slot_add")] +
-                [(n, C.c_void_p) for n in ("row_seq", "row_pos", "row_len", "seg")])
+                [(n, C.c_void_p) for n in ("row_seq", "row_pos", "row_len", "seg", "seg_host")])
 
 
 class RotaryAttention(C.Structure):
@@ -54,6 +55,32 @@ class DeltaRule(C.Structure):
     _fields_ = ([(n, C.c_void_p) for n in ("packed", "w2", "w0", "a_bias", "norm", "decay_in", "out")] +
                 [(n, C.c_uint32) for n in ("ld", "rank", "w_dtype")] +
                 [(n, C.c_float) for n in ("decay_scale", "unit_eps", "eps")])
+
+
+class ShortConv(C.Structure):
+    """M40llmShortConv."""
+    _fields_ = ([(n, C.c_void_p) for n in ("x", "w", "bias", "out")] +
+                [(n, C.c_uint32) for n in ("ldx", "dim", "taps", "add_input")])
+
+
+class RgLru(C.Structure):
+    """M40llmRgLru."""
+    _fields_ = ([(n, C.c_void_p) for n in ("packed", "conv_w", "conv_b", "ra", "ra_b", "ri", "ri_b", "lam", "out")] +
+                [(n, C.c_uint32) for n in ("ld", "width", "blocks", "taps", "w_dtype", "exact")] + [("decay", C.c_float)])
+
+
+class LatentAttention(C.Structure):
+    """M40llmLatentAttention."""
+    _fields_ = ([(n, C.c_void_p) for n in ("packed", "c_norm", "uk", "uv", "sink", "out")] +
+                [(n, C.c_uint32) for n in ("ld", "heads", "dim", "vdim", "w_dtype")] + [("eps", C.c_float), ("scale", C.c_float)])
+
+
+class Moe(C.Structure):
+    """M40llmMoe."""
+    _fields_ = ([(n, C.c_void_p) for n in ("x", "logits", "correction", "up", "down", "add", "residual", "out")] +
+                [("post", Norm)] +
+                [(n, C.c_uint32) for n in ("rows", "K", "ff", "experts", "identity", "top", "groups", "keep", "ld_logits",
+                                          "w_dtype", "act", "exact")] + [("scale", C.c_float)])
 
 
 _SCALARS = {
