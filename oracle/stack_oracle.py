@@ -267,6 +267,26 @@ def route(z, correction, r):
     return ids, got / (got.sum(-1, keepdims=True) + 1e-20) * r["scale"]
 
 
+def choice_margin(z, correction, r):
+    """Per token, how far the choice is from another one: the smallest gap, in choice scores, between what is taken and what is
+    left out, among groups and among outputs."""
+    z = np.asarray(z, F)
+    s = np.exp(z - z.max(-1, keepdims=True))
+    choice = s / s.sum(-1, keepdims=True) + correction
+    gaps = np.full(len(z), np.inf)
+    if r.get("groups"):
+        parts = choice.reshape(len(z), r["groups"]["count"], -1)
+        best, keep = np.sort(parts.max(-1), axis=-1)[:, ::-1], r["groups"]["keep"]
+        if keep < best.shape[1]:
+            gaps = np.minimum(gaps, best[:, keep - 1] - best[:, keep])
+        order = np.argsort(-parts.max(-1), axis=-1, kind="stable")[:, :keep]
+        choice = np.take_along_axis(parts, order[:, :, None], axis=1).reshape(len(z), -1)
+    top = np.sort(choice, axis=-1)[:, ::-1]
+    if r["top"] < top.shape[1]:
+        gaps = np.minimum(gaps, top[:, r["top"] - 1] - top[:, r["top"]])
+    return gaps
+
+
 def moe(h, w, spec):
     """w: router correction e<i>.up e<i>.down and, with spec["shared"], shared.up shared.down."""
     h = np.asarray(h, F)
@@ -312,6 +332,7 @@ class SidalornOracle:
     def step(self, tokens, layer_out=None):
         eps = self.cfg["norm"]["eps"]
         x = self.w["embed"][np.asarray(tokens)]
+        self.margin = np.full(len(x), np.inf)   # how clear the experts' choices were, per token of this call
         for i, (ly, st) in enumerate(zip(self.cfg["layers"], self.state)):
             p = f"l{i}."
             mw = self.part(p + "mix.")
@@ -327,6 +348,8 @@ class SidalornOracle:
                     y = poly_norm(x @ fw["up"].T, fw["act"], eps) @ fw["down"].T
                 else:
                     y = moe(x, fw, ly["mlp"])
+                    z = x @ fw["router"].T
+                    self.margin = np.minimum(self.margin, choice_margin(z, fw["correction"], ly["mlp"]["router"]))
                 x = x + self.norm(p + "norm2", y)
             if layer_out is not None:
                 layer_out.append(x)

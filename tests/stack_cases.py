@@ -1,6 +1,7 @@
 """Random layer-stack models for the tests: small configurations, weights already rounded to bfloat16."""
 from __future__ import annotations
 
+import copy
 import json
 import os
 
@@ -110,4 +111,133 @@ CASES = {
                         loop={"start": 0, "stop": 2, "times": 1}),
     # recurrent layers only
     "delta_only": config([delta(1, 128), delta(4, 17)], width=128, vocab=300),
+}
+
+
+# ------------------------------------------------------------------------------------------------------- Sidalorn
+def latent(heads, dim, vdim, rank, scale=None, mlp=None):
+    return {"type": "latent_attention", "mlp": mlp, "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "kv_rank": rank,
+                                                              "scale": dim ** -0.5 if scale is None else scale}}
+
+
+def rglru(width, blocks, conv, mlp=None):
+    return {"type": "rglru", "mlp": mlp, "mixer": {"width": width, "blocks": blocks, "conv": conv}}
+
+
+def dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def experts(n, identity, top, ff, groups=None, scale=1.0, shared=None):
+    r = {"experts": n, "identity": identity, "top": top, "scale": scale}
+    if groups:
+        r["groups"] = {"count": groups[0], "keep": groups[1]}
+    spec = {"kind": "moe", "expert": {"ff": ff}, "router": r}
+    if shared:
+        spec["shared"] = {"ff": shared}
+    return spec
+
+
+def sidalorn(layers, width, vocab, taps, groups=1, eps=1e-5):
+    return {"architecture": "Sidalorn", "canon": {"taps": taps}, "layers": layers, "norm": {"eps": eps, "groups": groups},
+            "vocab": vocab, "width": width}
+
+
+def sidalorn_weights(cfg, seed):
+    """Random tensors rounded to bfloat16; sinks and corrections are large enough to matter."""
+    helpers.load_package()
+    from m40_llm_b200.weights import bf16_to_f32, f32_to_bf16
+    rng = np.random.default_rng(seed)
+    out = {}
+
+    def put(name, a):
+        out[name] = bf16_to_f32(f32_to_bf16(np.asarray(a, np.float32)))
+
+    def mat(name, n, k, gain=1.0):
+        put(name, rng.standard_normal((n, k)) * gain / np.sqrt(k))
+
+    def near_one(name, *shape):
+        put(name, 1.0 + 0.3 * rng.standard_normal(shape))
+
+    W = cfg["width"]
+    put("embed", rng.standard_normal((cfg["vocab"], W)))
+    mat("head", cfg["vocab"], W, 3.0)
+    near_one("final.norm", W)
+    for i, ly in enumerate(cfg["layers"]):
+        p, m, mlp = f"l{i}.", ly["mixer"], ly["mlp"]
+        put(p + "canon1", 0.4 * rng.standard_normal((W, cfg["canon"]["taps"])))
+        near_one(p + "norm1", W)
+        if ly["type"] == "latent_attention":
+            H, D, V, R = m["heads"], m["dim"], m["vdim"], m["kv_rank"]
+            mat(p + "mix.q", H * D, W, 1.5)
+            mat(p + "mix.dkv", R, W)
+            near_one(p + "mix.dkv.norm", R)
+            mat(p + "mix.uk", H * D, R, 1.5)
+            mat(p + "mix.uv", H * V, R)
+            put(p + "mix.sink", rng.uniform(-1.0, 3.0, H))
+            mat(p + "mix.o", W, H * V)
+        else:
+            D, B = m["width"], m["blocks"]
+            for n in "yx":
+                mat(p + "mix." + n, D, W, 1.5)
+                put(p + f"mix.{n}.b", 0.3 * rng.standard_normal(D))
+            put(p + "mix.conv", 0.5 * rng.standard_normal((D, m["conv"])))
+            put(p + "mix.conv.b", 0.3 * rng.standard_normal(D))
+            for n in ("ra", "ri"):
+                put(p + "mix." + n, 1.5 * rng.standard_normal((B, D // B, D // B)) / np.sqrt(D // B))
+                put(p + f"mix.{n}.b", rng.standard_normal((B, D // B)))
+            put(p + "mix.lam", rng.uniform(-9.0, 0.5, D))
+            mat(p + "mix.o", W, D)
+        if not mlp:
+            continue
+        near_one(p + "norm2", W)
+        if mlp["kind"] == "dense":
+            mat(p + "mlp.up", mlp["ff"], W)
+            mat(p + "mlp.down", W, mlp["ff"])
+            put(p + "mlp.act", rng.uniform(0.3, 1.0, 4) * rng.choice([-1, 1], 4))
+            continue
+        r, F = mlp["router"], mlp["expert"]["ff"]
+        n = r["experts"] + r["identity"]
+        for e in range(r["experts"]):
+            mat(p + f"mlp.e{e}.up", F, W, 1.5)
+            mat(p + f"mlp.e{e}.down", W, F, 1.5)
+        mat(p + "mlp.router", n, W, 1.5)
+        put(p + "mlp.correction", 0.3 * rng.standard_normal(n))
+        if mlp.get("shared"):
+            mat(p + "mlp.shared.up", mlp["shared"]["ff"], W, 1.5)
+            mat(p + "mlp.shared.down", W, mlp["shared"]["ff"], 1.5)
+    return out
+
+
+def clear_tokens(oracle, n, rng, margin=0.01):
+    """Random tokens at which no choice of experts is a close call, so that 16-bit rounding cannot turn one; `oracle` is a
+    SidalornOracle, reset before and after."""
+    oracle.reset()
+    out = []
+    while len(out) < n:
+        before = copy.deepcopy(oracle.state)
+        t = int(rng.integers(0, oracle.cfg["vocab"]))
+        oracle.step([t])
+        if oracle.margin[0] >= margin:
+            out.append(t)
+        else:
+            oracle.state = before
+    oracle.reset()
+    return np.array(out)
+
+
+SIDALORN = {
+    # shapes of the tensor-core kernels; experts, groups and a shared expert; a layer without a feed-forward
+    "tiles": sidalorn([latent(6, 64, 64, 128, mlp=experts(10, 2, 3, 64, groups=(3, 2), scale=1.7, shared=96)),
+                       rglru(320, 5, 4, mlp=dense(200)), latent(2, 128, 128, 256), rglru(128, 2, 2, mlp=experts(5, 0, 1, 72))],
+                      width=192, vocab=210, taps=4, groups=3),
+    # more than 16 heads, key and value sizes differ, one filter tap, one block, every output chosen, no correction to speak of
+    "wide_heads": sidalorn([latent(20, 32, 48, 80, scale=0.3, mlp=dense(136)), rglru(96, 1, 1, mlp=experts(3, 1, 4, 40, shared=24)),
+                            latent(3, 96, 16, 512, mlp=experts(6, 3, 2, 48, groups=(9, 4)))],
+                           width=160, vocab=99, taps=1, groups=1, eps=1e-3),
+    # nothing is a multiple of 8: the f32 kernels in every mode
+    "unaligned": sidalorn([rglru(42, 3, 3, mlp=experts(7, 1, 2, 19, groups=(2, 1), scale=0.5, shared=13)),
+                           latent(3, 10, 14, 21, mlp=dense(33))], width=54, vocab=61, taps=7, groups=6),
+    # recurrent layers only
+    "recurrent": sidalorn([rglru(256, 4, 4, mlp=dense(144)), rglru(64, 8, 6)], width=128, vocab=150, taps=2, groups=8),
 }

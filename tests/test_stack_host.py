@@ -179,3 +179,82 @@ def test_scheduler_on_a_fake_model():
     assert max(sum(n for _, n in s) for s in m.steps) <= 8 + 2        # a portion plus the decode rows
     with pytest.raises(ValueError):
         e.submit([], 3)
+
+
+# ------------------------------------------------------------------------------------------------------- Sidalorn
+def test_sidalorn_registry():
+    assert "Sidalorn" in models.architectures()
+    spec = models.read_config(SC.SIDALORN["tiles"])
+    assert (spec.width, spec.vocab, spec.taps, spec.groups) == (192, 210, 4, 3)
+    for at, key, bad, msg in ((("layers", 0), "type", "convolution", "unknown type"),
+                              (("layers", 0, "mlp"), "kind", "sparse", "unknown feed-forward"), (("norm",), "groups", 7, "do not divide")):
+        cfg = json.loads(json.dumps(SC.SIDALORN["tiles"]))
+        d = cfg
+        for k in at:
+            d = d[k]
+        d[key] = bad
+        with pytest.raises(ValueError, match=msg):
+            models.read_config(cfg)
+
+
+@pytest.mark.parametrize("name", sorted(SC.SIDALORN))
+def test_sidalorn_oracle_portions_agree(name):
+    cfg = SC.SIDALORN[name]
+    w = SC.sidalorn_weights(cfg, 1)
+    t = np.random.default_rng(1).integers(0, cfg["vocab"], 20)
+    m = S.SidalornOracle(cfg, w)
+    whole = m.step(t)
+    m.reset()
+    assert np.allclose(np.concatenate([m.step(t[:7]), m.step(t[7:9]), m.step(t[9:10]), m.step(t[10:])]), whole, atol=1e-9)
+
+
+def test_oracle_grouped_and_polynomial_norms_by_hand():
+    x = np.array([[3.0, 4.0, 0.0, 2.0]])
+    got = S.group_rms_norm(x, np.array([1.0, 2.0, 1.0, 1.0]), 0.5, 2)
+    a, b = math.sqrt(12.5 + 0.5), math.sqrt(2.0 + 0.5)
+    assert np.allclose(got, [[3 / a, 8 / a, 0.0, 2 / b]])
+    z = np.array([[1.0, -2.0]])
+    n = [math.sqrt(5 / 2 + 0.1), math.sqrt(17 / 2 + 0.1), math.sqrt(65 / 2 + 0.1)]
+    assert np.allclose(S.poly_norm(z, (2.0, 3.0, 5.0, 7.0), 0.1),
+                       [[2 / n[0] + 3 / n[1] + 5 / n[2] + 7, -4 / n[0] + 12 / n[1] - 40 / n[2] + 7]])
+
+
+def test_oracle_convolution_by_hand():
+    w = np.array([[2.0, 3.0, 5.0]])
+    out, past = S.causal_conv(np.array([[1.0], [10.0], [100.0]]), np.zeros((2, 1)), w)
+    assert out.ravel().tolist() == [5.0, 53.0, 532.0] and past.ravel().tolist() == [10.0, 100.0]
+    out, past = S.causal_conv(np.array([[7.0]]), past, w, np.array([1.0]))
+    assert out.ravel().tolist() == [20.0 + 300.0 + 35.0 + 1.0] and past.ravel().tolist() == [100.0, 7.0]
+
+
+def test_oracle_recurrence_by_hand():
+    one = lambda v: np.array([v])
+    w = {"y": np.array([[1.0]]), "y.b": one(0.5), "x": np.array([[2.0]]), "x.b": one(0.0), "conv": np.array([[1.0]]), "conv.b": one(0.0),
+         "ra": np.array([[[0.3]]]), "ra.b": np.array([[0.1]]), "ri": np.array([[[-0.2]]]), "ri.b": np.array([[0.4]]), "lam": one(-1.0),
+         "o": np.array([[1.0]])}
+    s = 0.0
+    for h in (0.7, -1.1):
+        u = 2 * h
+        r, i = 1 / (1 + math.exp(-(0.3 * u + 0.1))), 1 / (1 + math.exp(-(-0.2 * u + 0.4)))
+        a = math.exp(-8 * r * math.log(1 + math.exp(-1.0)))
+        s = a * s + math.sqrt(1 - a * a) * i * u
+    out, S2, _ = S.rglru(np.array([[0.7], [-1.1]]), np.zeros(1), np.zeros((0, 1)), w, {"blocks": 1})
+    assert S2[0] == pytest.approx(s) and out[1, 0] == pytest.approx(s * S.gelu_tanh(-0.6))
+
+
+def test_oracle_sink_takes_weight_once():
+    """Two equal keys and a sink with the same score: each gets a third, and the sink brings no value."""
+    eye = np.eye(2)
+    w = {"q": np.zeros((2, 2)), "dkv": eye, "dkv.norm": np.ones(2), "uk": eye, "uv": eye, "sink": np.zeros(1), "o": eye}
+    out, C = S.latent_attention(np.array([[1.0, 1.0], [1.0, -1.0]]), np.zeros((0, 2)), w, {"heads": 1, "dim": 2, "vdim": 2, "scale": 5.0}, 0.0)
+    assert np.allclose(out, [[0.5, 0.5], [2 / 3, 0.0]]) and C.shape == (2, 2)
+
+
+def test_oracle_route_groups_and_weights():
+    s = np.array([[0.1, 0.2, 0.3, 0.4]])
+    ids, w = S.route(np.log(s), np.array([0.0, 0.0, -1.0, -1.0]), {"top": 1, "scale": 2.0})
+    assert ids.tolist() == [[1]] and np.allclose(w, 2.0)
+    r = {"top": 2, "scale": 1.0, "groups": {"count": 2, "keep": 1}}
+    ids, w = S.route(np.log(s), np.array([0.31, 0.0, 0.0, 0.0]), r)      # the group of 0.41 wins over that of 0.4
+    assert ids.tolist() == [[0, 1]] and np.allclose(w, [[1 / 3, 2 / 3]])
+    assert S.choice_margin(np.log(s), np.array([0.31, 0.0, 0.0, 0.0]), r) == pytest.approx(0.01)
