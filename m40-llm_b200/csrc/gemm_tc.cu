@@ -567,6 +567,10 @@ bool make_map_f16(CUtensorMap* map, const void* base, uint64_t rows, uint64_t co
 
 }  // namespace
 
+bool m40_tc_map(CUtensorMap* map, const void* base, uint64_t rows, uint64_t cols, uint32_t box_rows, bool bf16) {
+    return make_map_f16(map, base, rows, cols, box_rows, bf16);
+}
+
 int m40_split_activations(M40llmCudaContext* ctx, cudaStream_t s, const float* X, __half* hi, __half* lo, int M, int K,
                           const M40GemvNorm* norm) {
     if (norm && norm->w) {

@@ -1,5 +1,7 @@
 // Tensor-core (tcgen05) weight-streaming GEMM for batched decode rows; see gemm_tc.cu.
 #pragma once
+#include <cuda.h>
+
 #include "common.cuh"
 #include "gemv_stream.cuh"  // M40GemvNorm
 
@@ -17,6 +19,9 @@ struct M40TcRopeAppend {
     float freq_base, freq_scale;
     const float* inv_freq;  // host-made inverse-frequency table [head_dim / 2] or null (see m40_rope_inv_freq)
 };
+
+// Tensor map of a row-major 16-bit matrix [rows][cols] for 128-byte-swizzled boxes of box_rows x 64, zeros out of bounds.
+bool m40_tc_map(CUtensorMap* map, const void* base, uint64_t rows, uint64_t cols, uint32_t box_rows, bool bf16);
 
 // True when the tcgen05 path can take this problem set (2 <= M <= 256, K % 8 == 0, 16-byte aligned weights).
 bool m40_gemm_tc_supported(int M, int K, int problems, const void* const* W);

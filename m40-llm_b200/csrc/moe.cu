@@ -4,15 +4,22 @@
 //   moe_up_kernel      hid[row, slot] = act(up_e x), moe_down_kernel y[row] = sum_slot weight * down_e hid + identity + add:
 //                      f32 multiply-adds on streamed weight rows, any shape. They serve one row (every chosen expert's weights
 //                      are read once), the exact mode and the shapes the tensor path does not take;
+//   tensor path          moe_sort_kernel deals the chosen slots to experts (rows sorted by expert, each expert's share padded to
+//                      whole tiles) and writes the tile table, moe_scatter_kernel copies the rows there as hi + lo, two grouped
+//                      GEMMs (gemm_tc_grouped.cu; act and the next split in the first one's epilogue), moe_gather_kernel adds a
+//                      row's slots up. No host round trip: the table and its length stay on the device;
 //   then post norm and residual (norm_rows.cu).
 #include "moe.cuh"
 
+#include "gemm_tc_grouped.cuh"
 #include "norm_rows.cuh"
 
 namespace {
 
 constexpr uint32_t MAX_OUTPUTS = 1024, MAX_TOP = 32;
 constexpr int ROUTE_WARPS = 4;
+constexpr uint32_t TENSOR_ROWS = 2;               // rows from which the tensor path is taken
+constexpr uint64_t PASS_SLOTS = 32768;            // slots of one pass of it
 
 // Largest value of v[0 .. n) and the lowest index that holds it, over the warp.
 __device__ __forceinline__ uint32_t warp_argmax(const float* v, uint32_t n, uint32_t lane) {
@@ -175,6 +182,150 @@ __global__ void __launch_bounds__(256) moe_down_kernel(M40MoeArgs a) {
     if (lane == 0) a.y[at] = fmaf(own, a.x[at], y) + (a.add ? a.add[at] : 0.0f);
 }
 
+// One CTA. Slots are counted per expert, shares padded to tiles, tiles listed; then every slot draws its place. The order
+// within a share follows from atomics, which changes no result: a row's values do not depend on its place.
+__global__ void __launch_bounds__(1024) moe_sort_kernel(M40MoeArgs a) {
+    extern __shared__ uint32_t count[];  // [experts] counts, then next places
+    __shared__ uint32_t warp_sum_tiles[32], total_tiles;
+    pdl_wait();
+    pdl_trigger();
+    const uint32_t tid = threadIdx.x, lane = tid & 31u, warp = tid >> 5, slots = a.rows * a.top, E = a.experts;
+    for (uint32_t e = tid; e < E; e += 1024u) count[e] = 0u;
+    __syncthreads();
+    for (uint32_t i = tid; i < slots; i += 1024u) {
+        const uint32_t e = a.ids[i];
+        if (e < E) atomicAdd(&count[e], 1u);
+    }
+    __syncthreads();
+    // exclusive sum of the experts' tiles; experts <= 1024: one per thread
+    const uint32_t n = tid < E ? count[tid] : 0u, t = (n + a.tile_rows - 1u) / a.tile_rows;
+    uint32_t inc = t;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const uint32_t v = __shfl_up_sync(0xffffffffu, inc, o);
+        if (lane >= (uint32_t)o) inc += v;
+    }
+    if (lane == 31u) warp_sum_tiles[warp] = inc;
+    __syncthreads();
+    if (warp == 0) {
+        uint32_t w = warp_sum_tiles[lane], own = w;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const uint32_t v = __shfl_up_sync(0xffffffffu, w, o);
+            if (lane >= (uint32_t)o) w += v;
+        }
+        warp_sum_tiles[lane] = w - own;
+        if (lane == 31u) total_tiles = w;
+    }
+    __syncthreads();
+    const uint32_t first = warp_sum_tiles[warp] + inc - t;
+    if (tid < E) {
+        count[tid] = first * a.tile_rows;
+        for (uint32_t i = 0; i < t; ++i)
+            a.tiles[first + i] = M40GroupTile{tid, (first + i) * a.tile_rows, min(a.tile_rows, n - i * a.tile_rows), 0u};
+    }
+    if (tid == 0) *a.n_tiles = total_tiles;
+    __syncthreads();
+    for (uint32_t i = tid; i < slots; i += 1024u) {
+        const uint32_t e = a.ids[i];
+        if (e < E) a.place[i] = atomicAdd(&count[e], 1u);
+    }
+}
+
+// CTA = row: its hi and lo parts to every place that reads it.
+template <typename T>
+__global__ void __launch_bounds__(256) moe_scatter_kernel(M40MoeArgs a) {
+    pdl_wait();
+    pdl_trigger();
+    const uint32_t row = blockIdx.x;
+    const float* x = a.x + (size_t)row * a.K;
+    for (uint32_t k = threadIdx.x * 4u; k < a.K; k += 1024u) {
+        const float4 v = *reinterpret_cast<const float4*>(x + k);
+        const float y[4] = {v.x, v.y, v.z, v.w};
+        T h[4], l[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            h[i] = (T)y[i];
+            l[i] = (T)(y[i] - m40_load_elem(&h[i]));
+        }
+        for (uint32_t j = 0; j < a.top; ++j) {
+            if (a.ids[(size_t)row * a.top + j] >= a.experts) continue;
+            const size_t at = (size_t)a.place[(size_t)row * a.top + j] * a.K + k;
+            *reinterpret_cast<uint2*>(reinterpret_cast<T*>(a.xs[0]) + at) = *reinterpret_cast<const uint2*>(h);
+            *reinterpret_cast<uint2*>(reinterpret_cast<T*>(a.xs[1]) + at) = *reinterpret_cast<const uint2*>(l);
+        }
+    }
+}
+
+// CTA = (row, 1024 columns): y = sum of the slots' results (in the slots' order) + identity + add.
+__global__ void __launch_bounds__(256) moe_gather_kernel(M40MoeArgs a) {
+    __shared__ float sw[MAX_TOP];
+    __shared__ uint32_t sp[MAX_TOP];
+    pdl_wait();
+    pdl_trigger();
+    const uint32_t row = blockIdx.y, k = blockIdx.x * 1024u + threadIdx.x * 4u;
+    if (threadIdx.x < a.top) {
+        const size_t i = (size_t)row * a.top + threadIdx.x;
+        sw[threadIdx.x] = a.weights[i];
+        sp[threadIdx.x] = a.ids[i] < a.experts ? a.place[i] : 0xffffffffu;
+    }
+    __syncthreads();
+    if (k >= a.K) return;
+    const size_t at = (size_t)row * a.K + k;
+    const float4 x = *reinterpret_cast<const float4*>(a.x + at);
+    float4 y = a.add ? *reinterpret_cast<const float4*>(a.add + at) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (uint32_t j = 0; j < a.top; ++j) {
+        const float4 v = sp[j] == 0xffffffffu ? x : *reinterpret_cast<const float4*>(a.ys + (size_t)sp[j] * a.K + k);
+        y.x = fmaf(sw[j], v.x, y.x), y.y = fmaf(sw[j], v.y, y.y), y.z = fmaf(sw[j], v.z, y.z), y.w = fmaf(sw[j], v.w, y.w);
+    }
+    *reinterpret_cast<float4*>(a.y + at) = y;
+}
+
+// Rows of a tile: about the rows an expert gets, so that an expert's weights are read once and tiles are mostly full.
+uint32_t pick_tile_rows(uint32_t slots, uint32_t experts) {
+    const uint32_t avg = (slots + experts - 1) / experts;
+    return avg <= 16 ? 16 : (avg <= 32 ? 32 : (avg <= 96 ? 64 : 128));
+}
+
+int run_tensor(M40llmCudaContext* ctx, cudaStream_t s, const M40MoeArgs& a, uint32_t max_tiles) {
+    cudaError_t e = m40_launch_dependent(moe_sort_kernel, dim3(1), dim3(1024), a.experts * sizeof(uint32_t), s, a);
+    M40_COUNT_LAUNCH(ctx);
+    if (e != cudaSuccess) return -6;
+    e = a.bf16 ? m40_launch_dependent(moe_scatter_kernel<__nv_bfloat16>, dim3(a.rows), dim3(256), 0, s, a)
+               : m40_launch_dependent(moe_scatter_kernel<__half>, dim3(a.rows), dim3(256), 0, s, a);
+    M40_COUNT_LAUNCH(ctx);
+    if (e != cudaSuccess) return -6;
+    M40GroupedCall c = {};
+    c.w = a.up;
+    c.x[0] = a.xs[0], c.x[1] = a.xs[1];
+    c.parts = 2;
+    c.bf16 = a.bf16;
+    c.groups = a.experts;
+    c.N = a.ff;
+    c.K = c.ldx = a.K;
+    c.x_rows = max_tiles * a.tile_rows;
+    c.tile_rows = a.tile_rows;
+    c.tiles = a.tiles;
+    c.n_tiles = a.n_tiles;
+    c.max_tiles = max_tiles;
+    c.kind = M40_GROUPED_ACT_SPLIT;
+    c.act = a.act;
+    c.hi = a.hs[0], c.lo = a.hs[1];
+    int rc = m40_gemm_tc_grouped(ctx, s, c);
+    if (rc != 0) return rc;
+    c.w = a.down;
+    c.x[0] = a.hs[0], c.x[1] = a.hs[1];
+    c.N = a.K;
+    c.K = c.ldx = a.ff;
+    c.kind = M40_GROUPED_F32;
+    c.out = a.ys;
+    if ((rc = m40_gemm_tc_grouped(ctx, s, c)) != 0) return rc;
+    e = m40_launch_dependent(moe_gather_kernel, dim3((a.K + 1023) / 1024, a.rows), dim3(256), 0, s, a);
+    M40_COUNT_LAUNCH(ctx);
+    return e == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -6;
+}
+
 template <typename WT>
 int run_rows(M40llmCudaContext* ctx, cudaStream_t s, const M40MoeArgs& a) {
     constexpr int NR = 2;
@@ -222,31 +373,61 @@ extern "C" int m40llm_moe_async(M40llmCudaContext* ctx, const M40llmMoe* c, uint
     a.wide_down = c->w_dtype != M40LLM_DT_F32 && c->ff % 8 == 0 && al16(c->down);
     a.rows = c->rows;
 
-    // level-1 arena: chosen ids, weights, sums, hidden values (16-byte aligned pieces). Rows go in passes whose slots fit the
-    // grid.
-    const uint32_t pass = 65535u / c->top < c->rows ? 65535u / c->top : c->rows;
-    auto pad = [](size_t v) { return (v + 3) & ~(size_t)3; };
-    const size_t n_sel = pad((size_t)c->rows * c->top), n_y = pad((size_t)c->rows * c->K), n_hid = (size_t)pass * c->top * c->ff;
-    float* work = (float*)m40_ensure_scratch(ctx, stream_kind, (2 * n_sel + n_y + n_hid) * sizeof(float), 1);
+    a.bf16 = c->w_dtype == M40LLM_DT_BF16;
+    const bool tensor = !c->exact && c->rows >= TENSOR_ROWS && c->w_dtype != M40LLM_DT_F32 && al16(c->x) && al16(c->add) &&
+                        m40_gemm_tc_grouped_supported(c->up, c->ff, c->K, c->K, 0) &&
+                        m40_gemm_tc_grouped_supported(c->down, c->K, c->ff, c->ff, 0);
+
+    // level-1 arena: chosen ids, weights, sums; hidden values, or the sorted rows and their results (256-byte aligned pieces).
+    // Rows go in passes whose slots fit the grid and whose sorted rows stay within a fixed work space.
+    uint64_t pass = 65535u / c->top;
+    if (tensor && pass > PASS_SLOTS / c->top) pass = PASS_SLOTS / c->top;
+    if (pass > c->rows) pass = c->rows;
+    const uint64_t slots = pass * c->top;
+    a.tile_rows = pick_tile_rows((uint32_t)slots, c->experts);
+    const uint32_t max_tiles = (uint32_t)(slots / a.tile_rows + (c->experts < slots ? c->experts : slots));
+    const uint64_t sorted = (uint64_t)max_tiles * a.tile_rows;
+    size_t used = 0;
+    auto take = [&](size_t bytes) {
+        const size_t at = used;
+        used += (bytes + 255) & ~(size_t)255;
+        return at;
+    };
+    const size_t at_ids = take((size_t)c->rows * c->top * 4), at_weights = take((size_t)c->rows * c->top * 4);
+    const size_t at_y = take((size_t)c->rows * c->K * 4), at_hid = take(tensor ? 0 : slots * c->ff * 4);
+    size_t at_place = 0, at_tiles = 0, at_n = 0, at_x[2] = {}, at_h[2] = {}, at_ys = 0;
+    if (tensor) {
+        at_place = take(slots * 4), at_tiles = take((size_t)max_tiles * sizeof(M40GroupTile)), at_n = take(4);
+        for (int p = 0; p < 2; ++p) at_x[p] = take(sorted * c->K * 2), at_h[p] = take(sorted * c->ff * 2);
+        at_ys = take(sorted * c->K * 4);
+    }
+    unsigned char* work = (unsigned char*)m40_ensure_scratch(ctx, stream_kind, used + 256, 1);
     if (!work) return -5;
-    a.ids = (uint32_t*)work;
-    a.weights = work + n_sel;
-    a.y = work + 2 * n_sel;
-    a.hid = a.y + n_y;
+    work = (unsigned char*)(((uintptr_t)work + 255) & ~(uintptr_t)255);
+    a.ids = (uint32_t*)(work + at_ids);
+    a.weights = (float*)(work + at_weights);
+    a.y = (float*)(work + at_y);
+    a.hid = (float*)(work + at_hid);
+    a.place = (uint32_t*)(work + at_place);
+    a.tiles = (M40GroupTile*)(work + at_tiles);
+    a.n_tiles = (uint32_t*)(work + at_n);
+    for (int p = 0; p < 2; ++p) a.xs[p] = work + at_x[p], a.hs[p] = work + at_h[p];
+    a.ys = (float*)(work + at_ys);
 
     const size_t smem = (size_t)ROUTE_WARPS * (2 * n + G) * sizeof(float);
     cudaError_t e = m40_launch_dependent(moe_route_kernel, dim3((c->rows + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(32 * ROUTE_WARPS), smem, s, a);
     M40_COUNT_LAUNCH(ctx);
     if (e != cudaSuccess) return -6;
-    for (uint32_t at = 0; at < c->rows; at += pass) {
+    for (uint32_t at = 0; at < c->rows; at += (uint32_t)pass) {
         M40MoeArgs p = a;
-        p.rows = c->rows - at < pass ? c->rows - at : pass;
+        p.rows = c->rows - at < pass ? c->rows - at : (uint32_t)pass;
         p.x += (size_t)at * c->K;
         if (p.add) p.add += (size_t)at * c->K;
         p.y += (size_t)at * c->K;
         p.ids += (size_t)at * c->top;
         p.weights += (size_t)at * c->top;
-        const int rc = c->w_dtype == M40LLM_DT_F32 ? run_rows<float>(ctx, s, p)
+        const int rc = tensor ? run_tensor(ctx, s, p, max_tiles)
+                       : c->w_dtype == M40LLM_DT_F32 ? run_rows<float>(ctx, s, p)
                        : c->w_dtype == M40LLM_DT_BF16 ? run_rows<__nv_bfloat16>(ctx, s, p) : run_rows<__half>(ctx, s, p);
         if (rc != 0) return rc;
     }

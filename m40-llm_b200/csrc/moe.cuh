@@ -13,6 +13,14 @@ struct M40MoeArgs {
     float* weights;          // [rows][top]
     float* hid;              // [rows * top][ff]
     float* y;                // [rows][K]
+    // tensor path: rows sorted by expert, every expert's share padded to whole tiles
+    uint32_t* place;         // [rows][top]: sorted row of the slot
+    struct M40GroupTile* tiles;
+    uint32_t* n_tiles;
+    void* xs[2];             // [sorted rows][K] hi, lo of the weights' type
+    void* hs[2];             // [sorted rows][ff]
+    float* ys;               // [sorted rows][K]
+    uint32_t tile_rows, bf16;
     uint32_t rows, K, ff, experts, identity, top, groups, keep, ld_logits, wide_up, wide_down;
     int act;
     float scale;

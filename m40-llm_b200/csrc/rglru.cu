@@ -6,13 +6,16 @@
 //                         gates, the state and the output gate in one launch; a weight row is read once per RG rows.
 //   portions:
 //     short convolution   u (short_conv.cu);
-//     gates               a and b = sqrt(1 - a^2) i u per (row, channel): the block-diagonal products on f32 multiply-adds;
+//     gates               a and b = sqrt(1 - a^2) i u per (row, channel). The block-diagonal products run on the tensor cores
+//                         (gemm_tc_grouped.cu) with u cut into three bf16 parts, whose sum is the f32 value and whose products
+//                         with bf16 weights are exact in f32, or on f32 multiply-adds: 32-bit arithmetic either way;
 //     rglru_scan_kernel   CTA = (32 channels, segment), a warp per piece of the portion: every piece is folded into one
 //                         (product of a, sum) pair, the pairs are chained from the slot's state, and the pieces are walked
 //                         again from their starting states.
 // 1 - a^2 is taken as -expm1(2 log a), which keeps its accuracy when a is close to one.
 #include "rglru.cuh"
 
+#include "gemm_tc_grouped.cuh"
 #include "short_conv.cuh"
 
 namespace {
@@ -286,8 +289,12 @@ template <typename WT>
 int run_portion(M40llmCudaContext* ctx, RgArgs g, uint32_t blocks, const M40llmStepRows& rows) {
     cudaStream_t s = ctx->decode_stream;
     const size_t n = ((size_t)g.rows * g.width + 3) & ~(size_t)3;
-    float* work = (float*)m40_ensure_scratch(ctx, 1, 3 * n * sizeof(float), 1);
+    const bool tensor = g.tensor && m40_gemm_tc_grouped_supported(g.ra, g.bs, g.bs, g.width, g.bs) &&
+                        m40_gemm_tc_grouped_supported(g.ri, g.bs, g.bs, g.width, g.bs);
+    const size_t part = (n * 2 + 255) / 256 * 256;
+    float* work = (float*)m40_ensure_scratch(ctx, 1, 3 * n * sizeof(float) + (tensor ? 256 + 3 * part : 0), 1);
     if (!work) return -5;
+    unsigned char* parts = (unsigned char*)(((uintptr_t)(work + 3 * n) + 255) & ~(uintptr_t)255);
     g.u = work, g.a = work + n, g.b = work + 2 * n;
     M40ConvArgs c = {};
     c.x = g.packed + g.width;
@@ -300,12 +307,31 @@ int run_portion(M40llmCudaContext* ctx, RgArgs g, uint32_t blocks, const M40llmS
     c.row_seq = g.row_seq, c.row_pos = g.row_pos, c.seg = g.seg;
     c.ldx = g.ld, c.dim = g.width, c.taps = g.taps;
     c.slot_mul = g.slot_mul, c.slot_add = g.slot_add, c.slots = g.slots, c.rows = g.rows;
+    for (int p = 0; tensor && p < 3; ++p) c.parts[p] = parts + p * part;
     int rc = m40_short_conv(ctx, s, c, rows);
     if (rc != 0) return rc;
-    const dim3 grid((g.bs + 63) / 64, (g.rows + 63) / 64, blocks);
-    cudaError_t e = m40_launch_dependent(rglru_gates_f32_kernel<WT>, grid, dim3(256), 0, s, g);
-    M40_COUNT_LAUNCH(ctx);
-    if (e != cudaSuccess) return -6;
+    cudaError_t e;
+    if (tensor) {
+        M40GroupedCall q = {};
+        q.w = g.ra;
+        q.w2 = g.ri;
+        for (int p = 0; p < 3; ++p) q.x[p] = c.parts[p];
+        q.parts = 3;
+        q.bf16 = 1;
+        q.groups = blocks;
+        q.N = q.K = q.group_k = g.bs;
+        q.x_rows = g.rows;
+        q.ldx = g.width;
+        q.tile_rows = g.rows > 32 ? 64 : 32;
+        q.kind = M40_GROUPED_RG;
+        q.rg = g;
+        if ((rc = m40_gemm_tc_grouped(ctx, s, q)) != 0) return rc;
+    } else {
+        const dim3 grid((g.bs + 63) / 64, (g.rows + 63) / 64, blocks);
+        e = m40_launch_dependent(rglru_gates_f32_kernel<WT>, grid, dim3(256), 0, s, g);
+        M40_COUNT_LAUNCH(ctx);
+        if (e != cudaSuccess) return -6;
+    }
     e = m40_launch_dependent(rglru_scan_kernel, dim3((g.width + 31) / 32, rows.segments), dim3(1024), 0, s, g);
     M40_COUNT_LAUNCH(ctx);
     return e == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -6;
@@ -353,6 +379,7 @@ extern "C" int m40llm_rglru_async(M40llmCudaContext* ctx, M40llmStateCache* stat
     g.rows = r->rows;
     g.decay = c->decay;
     g.wide = c->w_dtype != M40LLM_DT_F32 && g.bs % 8 == 0 && (((uintptr_t)c->ra | (uintptr_t)c->ri) & 15u) == 0;
+    g.tensor = c->w_dtype == M40LLM_DT_BF16 && !c->exact;
     if (c->w_dtype == M40LLM_DT_F32) return run<float>(ctx, g, c->blocks, *r);
     return c->w_dtype == M40LLM_DT_BF16 ? run<__nv_bfloat16>(ctx, g, c->blocks, *r) : run<__half>(ctx, g, c->blocks, *r);
 }

@@ -21,7 +21,7 @@ struct M40RgArgs {
     const uint32_t* row_seq;
     const uint32_t* row_pos;
     const uint32_t* seg;
-    uint32_t ld, width, bs, taps, slot_mul, slot_add, slots, rows, wide;
+    uint32_t ld, width, bs, taps, slot_mul, slot_add, slots, rows, wide, tensor;
     float decay;
 };
 

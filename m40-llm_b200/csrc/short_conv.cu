@@ -6,9 +6,23 @@
 // write the portion's last inputs to it when they are done, so a channel's ring is touched by one thread per launch.
 #include "short_conv.cuh"
 
+#include <cuda_bf16.h>
+
 namespace {
 
 constexpr uint32_t PIECE = 32, MAX_TAPS = 32;
+
+__device__ __forceinline__ void store_out(const M40ConvArgs& a, size_t at, float y) {
+    a.out[at] = y;
+    if (a.parts[0]) {
+        const __nv_bfloat16 p0 = __float2bfloat16_rn(y);
+        const float r1 = y - __bfloat162float(p0);
+        const __nv_bfloat16 p1 = __float2bfloat16_rn(r1);
+        reinterpret_cast<__nv_bfloat16*>(a.parts[0])[at] = p0;
+        reinterpret_cast<__nv_bfloat16*>(a.parts[1])[at] = p1;
+        reinterpret_cast<__nv_bfloat16*>(a.parts[2])[at] = __float2bfloat16_rn(r1 - __bfloat162float(p1));
+    }
+}
 
 // TAPS > 0: a window of the last inputs stays in registers; 0: any number of taps, inputs read again.
 template <bool DECODE, int TAPS>
@@ -39,7 +53,7 @@ __global__ void __launch_bounds__(128) short_conv_kernel(M40ConvArgs a) {
     }
     if (c >= a.dim) return;
     const float* x = a.x + (size_t)row0 * a.ldx + c;
-    float* out = a.out + (size_t)row0 * a.dim + c;
+    const size_t out0 = (size_t)row0 * a.dim + c;
     float* ring = a.ring ? a.ring + (size_t)slot * a.slot_stride + c : nullptr;
     const uint32_t last = min(first + PIECE, n);
     // the input `back` tokens before token t of the portion
@@ -60,13 +74,13 @@ __global__ void __launch_bounds__(128) short_conv_kernel(M40ConvArgs a) {
             float y = bias;
 #pragma unroll
             for (int j = 0; j < TAPS; ++j) y = fmaf(wv[j], win[j], y);
-            out[(size_t)t * a.dim] = a.add_input ? win[TAPS ? TAPS - 1 : 0] + y : y;
+            store_out(a, out0 + (size_t)t * a.dim, a.add_input ? win[TAPS ? TAPS - 1 : 0] + y : y);
         }
     } else {
         for (uint32_t t = first; t < last; ++t) {
             float y = bias;
             for (uint32_t back = taps; back-- > 0u;) y = fmaf(w[taps - 1u - back], input(t, back), y);
-            out[(size_t)t * a.dim] = a.add_input ? x[(size_t)t * a.ldx] + y : y;
+            store_out(a, out0 + (size_t)t * a.dim, a.add_input ? x[(size_t)t * a.ldx] + y : y);
         }
     }
     if (first == 0u && taps > 1u) {

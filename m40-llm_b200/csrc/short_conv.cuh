@@ -7,6 +7,7 @@ struct M40ConvArgs {
     const float* w;      // [dim][taps]
     const float* bias;
     float* out;
+    void* parts[3];      // optional: out cut into three bf16 parts whose sum is the f32 value, [rows][dim] each
     float* ring;         // [taps][dim] of slot 0: the input of position p at p % taps
     uint32_t* status;
     const uint32_t* row_seq;
