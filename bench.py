@@ -722,15 +722,20 @@ def _torch_stack_weights(pkg, nat, rank):
         def shape(self, name):
             return (rank,)          # only asked for the low-rank projection
 
-        def matrix(self, *names, shapes=None):
+        def matrix(self, *names, shapes=None, rows=0):
             if names not in self._mat:
-                n, k = sum(sh[0] for sh in shapes or [(1, 1)]), shapes[0][1] if shapes else None
                 if shapes is None:
                     raise ValueError(names)
-                t = (torch.randn(n, k, generator=self.gen, device="cuda") / k ** 0.5).to(torch.bfloat16)
+                n, rest = max(rows, sum(sh[0] for sh in shapes)), shapes[0][1:]
+                t = torch.empty(n, *rest, dtype=torch.bfloat16, device="cuda")
+                for i in range(0, n, 8192):     # in pieces: the f32 draft of a large layer's experts would not be small
+                    t[i:i + 8192] = torch.randn(min(8192, n - i), *rest, generator=self.gen, device="cuda") / rest[-1] ** 0.5
                 self.keep.append(t)
                 self._mat[names] = t.data_ptr()
             return self._mat[names]
+
+        def vectors(self, names, sizes, total):
+            return self.vector(names, total)
 
         def vector(self, name, size, row=None):
             key = (name, row)
@@ -918,6 +923,177 @@ def stack_ops_case(nat, ev, name, reps=20):
     return out
 
 
+# ---------------------------------------------------------------------------------------------------- Sidalorn
+SIDALORN_SIZES = {
+    # name (a layer stack of STACK_SIZES with the same width and feed-forward size): heads, head dim, latent size, recurrence
+    # blocks, experts, identity outputs, groups (count, keep), chosen, expert ff, shared ff, layers. An expert layer's active
+    # feed-forward (chosen * ff + shared) is about the dense layers' ff.
+    "tinyllama-sized": (16, 128, 512, 16, 60, 4, (8, 4), 6, 704, 1408, 8),
+    "llama3-8b-sized": (32, 128, 512, 16, 60, 4, (8, 4), 6, 1792, 3584, 4),
+}
+
+
+def sidalorn_model(pkg, nat, name, sequences, max_len):
+    from m40_llm_b200 import models
+    H, D, R, B, E, I, G, top, F, FS, NL = SIDALORN_SIZES[name]
+    W, FF = STACK_SIZES[name][:2]
+    moe = {"kind": "moe", "expert": {"ff": F}, "shared": {"ff": FS},
+           "router": {"experts": E, "identity": I, "top": top, "scale": 2.5, "groups": {"count": G[0], "keep": G[1]}}}
+    dense = {"kind": "dense", "ff": FF}
+    lat = {"type": "latent_attention", "mixer": {"heads": H, "dim": D, "vdim": D, "kv_rank": R, "scale": D ** -0.5}}
+    rec = {"type": "rglru", "mixer": {"width": W, "blocks": B, "conv": 4}}
+    cycle = [{**lat, "mlp": dense}, {**rec, "mlp": moe}, {**rec, "mlp": dense}, {**lat, "mlp": moe}]
+    spec = models.read_config({"architecture": "Sidalorn", "width": W, "vocab": STACK_VOCAB, "norm": {"eps": 1e-5, "groups": 8},
+                               "canon": {"taps": 4}, "layers": [cycle[i % 4] for i in range(NL)]})
+    return spec.build(nat, _torch_stack_weights(pkg, nat, 0), sequences=sequences, max_len=max_len, max_rows=STACK_PROMPT)
+
+
+def sidalorn_ops_case(nat, ev, name, reps=20):
+    """Single calls of Sidalorn's mechanisms at one size, each beside the like call of the Lamutar stack (or of itself where
+    there is none). Fractions: algorithmic bytes over the measured copy bandwidth, or operations over the measured bf16 rate."""
+    import torch
+    from m40_llm_b200 import native as N
+    H, D, R, B, E, I, G, top, F, FS, _ = SIDALORN_SIZES[name]
+    W, FF, QH_, KVH_, HD_, DH, DD, RK, _ = STACK_SIZES[name]
+    L, ctx = nat.lib, nat.ctx
+    peak, _ = measured_peak_gbs()
+    peak_tf = 1636.2
+    try:
+        peak_tf = float(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"])
+    except Exception:
+        pass
+    out, keep, T = {}, [], STACK_PROMPT
+
+    def dev(*shape, dtype=torch.float32, std=1.0):
+        t = (torch.randn(*shape, device="cuda") * std).to(dtype)
+        keep.append(t)
+        return t.data_ptr()
+
+    def timed(call):
+        for i in range(3):
+            assert call(i) == 0
+        nat.sync(1)
+        ev.start()
+        for i in range(reps):
+            assert call(i) == 0
+        return ev.stop_ms() / reps
+
+    def put(key, ms, flops=None, bytes_=None):
+        rec = {"us": ms * 1e3}
+        if flops:
+            rec["frac_of_bf16_tensor_peak"] = flops / (ms * 1e-3) / 1e12 / peak_tf
+        if bytes_:
+            rec["frac_of_hbm_peak"] = bytes_ / (ms * 1e-3) / 1e9 / peak
+        out[key] = rec
+
+    def step_rows(segments):
+        seq, pos, seg = [], [], []
+        for s, p0, n in segments:
+            seg += [len(seq), n, s, p0]
+            seq += [s] * n
+            pos += list(range(p0, p0 + n))
+        u = lambda a: nat.buf(np.array(a, np.uint32)).ptr
+        host = np.array(seg, np.uint32)
+        r = N.StepRows(len(seq), len(segments), max(s[2] for s in segments), 0, 1, 0, u(seq), u(pos), u(np.array(pos) + 1), u(seg))
+        if r.max_segment_rows > 1:
+            r.seg_host = host.ctypes.data
+        return r, host
+
+    bf = torch.bfloat16
+    cases = ((T, [(0, 0, T)], "prompt 2048"), (1, [(0, 8191, 1)], "decode 1 x 8192"), (32, [(s, 2047, 1) for s in range(32)], "decode 32 x 2048"))
+    # ---- latent attention beside rotary attention
+    cn, uk, uv, sink = dev(R), dev(H * D, R, dtype=bf, std=R ** -0.5), dev(H * D, R, dtype=bf, std=R ** -0.5), dev(H)
+    for rows, segs, key in cases:
+        max_len, tokens = (8192 if rows == 1 else 2048), sum(p0 + n for _, p0, n in segs)
+        r, host = step_rows(segs)
+        kv = L.m40llm_kvcache_create_typed(ctx, max_len, len(segs), 1, R, 0, N.DT_F16)
+        c = N.LatentAttention(dev(rows, H * D + R), cn, uk, uv, sink, dev(rows, H * D), H * D + R, H, D, D, N.DT_BF16, 1e-5, D ** -0.5)
+        ms = timed(lambda i: L.m40llm_attention_latent_async(ctx, kv, C.byref(c), C.byref(r)))
+        if rows == T:   # scores and values, and making the heads' keys and values once
+            put(f"latent attention, {key}", ms, 4.0 * D * H * T * (T + 1) / 2 + 4.0 * T * R * H * D)
+        else:           # the latents once, uk and uv once
+            put(f"latent attention, {key}", ms, None, tokens * R * 2 + 2 * H * D * R * 2)
+        nat.sync(1)
+        L.m40llm_kvcache_destroy(kv)
+        kv = L.m40llm_kvcache_create_typed(ctx, max_len, len(segs), KVH_, HD_, HD_, N.DT_F16)
+        ld = QH_ * HD_ + 2 * KVH_ * HD_ + QH_
+        kt, vt = nat.buf(np.full(HD_ // 4, 0.01)).ptr, nat.buf(np.full(HD_ // 2, 0.01)).ptr
+        c = N.RotaryAttention(dev(rows, ld), dev(QH_ * HD_), dev(KVH_ * HD_), kt, vt, dev(rows, QH_ * HD_), ld, QH_, HD_ // 4, 1, 1e-5, 1.2, HD_ ** -0.5)
+        ms = timed(lambda i: L.m40llm_attention_rotary_async(ctx, kv, C.byref(c), C.byref(r)))
+        put(f"like: rotary attention, {key}", ms, 4.0 * HD_ * QH_ * T * (T + 1) / 2 if rows == T else None,
+            None if rows == T else tokens * KVH_ * HD_ * 4)
+        nat.sync(1)
+        L.m40llm_kvcache_destroy(kv)
+    # ---- real-gated recurrence beside the delta rule
+    bs = W // B
+    wts = [dev(W, 4), dev(W), dev(B, bs, bs, dtype=bf, std=bs ** -0.5), dev(W), dev(B, bs, bs, dtype=bf, std=bs ** -0.5), dev(W), dev(W)]
+    for rows, segs, key in ((T, [(0, 0, T)], "prompt 2048"), (1, [(0, 5, 1)], "decode 1"), (32, [(s, 5, 1) for s in range(32)], "decode 32")):
+        r, host = step_rows(segs)
+        st = L.m40llm_statecache_create_values(ctx, len(segs), 5 * W)
+        c = N.RgLru(dev(rows, 2 * W), *wts, dev(rows, W), 2 * W, W, B, 4, N.DT_BF16, 0, 8.0)
+        ms = timed(lambda i: L.m40llm_rglru_async(ctx, st, C.byref(c), C.byref(r)))
+        put(f"recurrence, {key}", ms, None, rows * W * 4 * 3 + 2 * W * bs * 2 + len(segs) * W * 4 * 6)
+        nat.sync(1)
+        L.m40llm_statecache_destroy(st)
+        st, HD2, ld = L.m40llm_statecache_create(ctx, len(segs), DH, DD), DH * DD, 5 * DH * DD + RK
+        one = dev(HD2)
+        c = N.DeltaRule(dev(rows, ld), dev(HD2, RK, dtype=bf, std=RK ** -0.5), one, one, one, dev(rows, HD2) if rows == T else None,
+                        dev(rows, HD2), ld, RK, N.DT_BF16, -0.6065, 1e-6, 1e-5)
+        ms = timed(lambda i: L.m40llm_delta_rule_async(ctx, st, C.byref(c), C.byref(r)))
+        put(f"like: delta rule, {key}", ms, None, rows * HD2 * 4 * 7 + 2 * len(segs) * HD2 * DD * 4)
+        nat.sync(1)
+        L.m40llm_statecache_destroy(st)
+    # ---- experts beside a gated feed-forward of the same active size; two sets of weights in rotation
+    up, down = [dev(E, F, W, dtype=bf, std=W ** -0.5) for _ in range(2)], [dev(E, W, F, dtype=bf, std=F ** -0.5) for _ in range(2)]
+    FA = top * F
+    wd = [(dev(FA, W, dtype=bf, std=W ** -0.5), dev(W, FA, dtype=bf, std=FA ** -0.5)) for _ in range(4)]
+    nw, coef = dev(W), dev(4)
+    rng = np.random.default_rng(11)
+    for rows in (1, 32, 256, T):
+        z = (rng.standard_normal((rows, E + I))).astype(np.float32)
+        # what the choice will be, for the byte counts
+        s = np.exp(z) / np.exp(z).sum(1, keepdims=True)
+        gm = s.reshape(rows, G[0], -1).max(2)
+        kept = np.zeros_like(gm, bool)
+        np.put_along_axis(kept, np.argsort(-gm, 1)[:, :G[1]], True, 1)
+        ids = np.argsort(-np.where(np.repeat(kept, (E + I) // G[0], 1), s, -1), 1)[:, :top]
+        live, used = int((ids < E).sum()), len(np.unique(ids[ids < E]))
+        x, y, zl = dev(rows, W), dev(rows, W), nat.buf(z).ptr
+        calls = [N.Moe(x=x, logits=zl, up=up[i], down=down[i], out=y, post=N.Norm(N.NORM_RMS, 1e-5, 0.0, nw, None, 8, 0), rows=rows, K=W, ff=F,
+                       experts=E, identity=I, top=top, groups=G[0], keep=G[1], ld_logits=E + I, w_dtype=N.DT_BF16, act=N.ACT_GELU_ERF,
+                       scale=2.5) for i in range(2)]
+        ms = timed(lambda i: L.m40llm_moe_async(ctx, C.byref(calls[i % 2]), 1))
+        put(f"experts rows {rows}", ms, 4.0 * live * F * W, used * F * W * 4 if rows <= 256 else None)
+        hid = dev(rows, FA)
+
+        def ffn(i):
+            a, b = wd[i % 4]
+            c = N.Linear(x=x, w=a, out=hid, rows=rows, K=W, N=FA, w_dtype=N.DT_BF16)
+            rc = L.m40llm_linear_async(ctx, C.byref(c), 1)
+            c = N.Linear(x=hid, w=b, out=y, pre=N.Norm(N.NORM_DYT, 0.0, 0.8, None, None), post=N.Norm(N.NORM_DYT, 0.0, 0.8, nw, None), rows=rows,
+                         K=FA, N=W, w_dtype=N.DT_BF16)
+            return rc or L.m40llm_linear_async(ctx, C.byref(c), 1)
+        put(f"like: dense up and down of the active size, rows {rows}", timed(ffn), 4.0 * rows * FA * W, FA * W * 4 if rows <= 256 else None)
+
+        def poly(i):
+            a, b = wd[i % 4]
+            c = N.Linear(x=x, w=a, out=hid, rows=rows, K=W, N=FA, w_dtype=N.DT_BF16)
+            rc = L.m40llm_linear_async(ctx, C.byref(c), 1)
+            c = N.Linear(x=hid, w=b, out=y, pre=N.Norm(N.NORM_POLY, 1e-5, 0.0, coef, None), post=N.Norm(N.NORM_RMS, 1e-5, 0.0, nw, None, 8, 0),
+                         rows=rows, K=FA, N=W, w_dtype=N.DT_BF16)
+            return rc or L.m40llm_linear_async(ctx, C.byref(c), 1)
+        put(f"PolyNorm up and down, grouped norm, rows {rows}", timed(poly), 4.0 * rows * FA * W, FA * W * 4 if rows <= 256 else None)
+        # ---- input convolution
+        r, host = step_rows([(0, 0, T)] if rows == T else [(s, 9, 1) for s in range(rows)])
+        st = L.m40llm_statecache_create_values(ctx, 1 if rows == T else rows, 4 * W)
+        c = N.ShortConv(x, wts[0], None, y, 0, W, 4, 1)
+        put(f"input convolution rows {rows}", timed(lambda i: L.m40llm_short_conv_async(ctx, st, C.byref(c), C.byref(r))), None, rows * W * 8)
+        nat.sync(1)
+        L.m40llm_statecache_destroy(st)
+    nat.free_all()
+    return out
+
+
 def delta_only_case(nat, args):
     """Small case for a profiler: the delta rule over one 2048-token prompt at the llama3-8b size."""
     from m40_llm_b200 import native as N
@@ -938,19 +1114,20 @@ def delta_only_case(nat, args):
     print(json.dumps({"case": "delta_rule_prompt2048", "us_per_call": ev.stop_ms() * 1e3 / max(args.steps, 1)}), flush=True)
 
 
-def stack_case(nat, pkg, name, steps):
-    """Prefill and greedy decode of the layer-stack model beside the Llama stack of equal size (random weights)."""
+def stack_case(nat, pkg, name, steps, kinds=("stack", "llama")):
+    """Prefill and greedy decode of the first of two models beside the second, of equal size (random weights): "stack" the
+    Lamutar stack, "llama" the Llama stack, "sidalorn"."""
     ev = Events(nat)
     rec = {"sizes": dict(zip(("width", "ff", "q_heads", "kv_heads", "head_dim", "delta_heads", "delta_dim", "rank", "layers"),
                              STACK_SIZES[name]))}
     rng = np.random.default_rng(3)
     prompt = rng.integers(0, STACK_VOCAB, STACK_PROMPT)
-    for kind in ("stack", "llama"):
+    for kind in kinds:
         keep, kv, r = [], None, {}
         for batch in (1, 32):
             max_len = STACK_PROMPT + 3 * steps + 16 if batch == 1 else 256 + 3 * steps + 16
-            if kind == "stack":
-                m = stack_model(pkg, nat, name, batch, max_len)
+            if kind != "llama":
+                m = (stack_model if kind == "stack" else sidalorn_model)(pkg, nat, name, batch, max_len)
             else:
                 m, kv = llama_model(pkg, nat, name, batch, max_len, keep)
             if batch == 1:
@@ -982,8 +1159,9 @@ def stack_case(nat, pkg, name, steps):
                 kv = None
             nat.free_all()
         rec[kind] = r
-    rec["stack_over_llama"] = {"prefill": rec["stack"]["prefill_tokens_per_s"] / rec["llama"]["prefill_tokens_per_s"],
-                               **{b: rec["stack"][b]["tokens_per_s"] / rec["llama"][b]["tokens_per_s"] for b in ("decode_batch1", "decode_batch32")}}
+    one, two = kinds
+    rec[f"{one}_over_{two}"] = {"prefill": rec[one]["prefill_tokens_per_s"] / rec[two]["prefill_tokens_per_s"],
+                                **{b: rec[one][b]["tokens_per_s"] / rec[two][b]["tokens_per_s"] for b in ("decode_batch1", "decode_batch32")}}
     return rec
 
 
@@ -1040,7 +1218,7 @@ def main():
                     help="small case for a profiler: the packed varlen prefill attention call alone")
     ap.add_argument("--delta-only", action="store_true",
                     help="small case for a profiler: the delta rule over one 2048-token prompt alone")
-    ap.add_argument("--workload", default="layer", choices=["layer", "splitk", "stack"],
+    ap.add_argument("--workload", default="layer", choices=["layer", "splitk", "stack", "sidalorn"],
                     help="layer: the batched decode layer (the contract's line); splitk: one 32K sequence, split-K over "
                          "the ranks (its own JSON line); stack: the Lamutar layer stack at several sizes beside the Llama "
                          "stack of equal size, whole models and single calls (its own JSON line, one GPU)")
@@ -1087,6 +1265,21 @@ def main():
 
     if args.delta_only:
         delta_only_case(nat, args)
+        return
+
+    if args.workload == "sidalorn":
+        clk = ClockSampler(local_rank)
+        clk.start()
+        clk.wait_first_sample()
+        rec = {}
+        for n in SIDALORN_SIZES:
+            rec[n] = stack_case(nat, pkg, n, min(args.steps, 100), ("sidalorn", "stack"))
+            rec[n]["sidalorn_sizes"] = dict(zip(("heads", "head_dim", "latent", "blocks", "experts", "identity", "groups", "top", "expert_ff",
+                                                 "shared_ff", "layers"), SIDALORN_SIZES[n]))
+            rec[n]["calls"] = sidalorn_ops_case(nat, Events(nat), n)
+        print(json.dumps({"metric": "sidalorn_prefill_and_decode_tokens_per_s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic",
+                          "config": {"prompt": STACK_PROMPT, "l2": "inputs larger than L2 (weights in rotation)"},
+                          "clocks": clk.stop(), "models": rec}), flush=True)
         return
 
     if args.workload == "stack":

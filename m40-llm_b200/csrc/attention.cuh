@@ -66,13 +66,25 @@ int m40_attention_fused_row(M40llmCudaContext* ctx, M40llmKVCache* kv, const flo
                             const uint32_t* seq_lens, uint32_t rows, uint32_t q_heads, float freq_base,
                             float freq_scale, uint32_t layout, float* q_out, float* out);
 
-// Prompt attention over a dense f16 cache (head_dim 64 or 128) for the segments of a step whose keys and values are
-// already appended; f32 q [rows][q_heads][hd], out likewise. `turn_back` (float2 cos, sin [rows][hd / 2]) rotates each
-// head's output by the inverse of its position's value rotation, `gate` (row pitch gate_ld) multiplies it by
-// sigmoid(gate[row][head]); both optional. Decode stream. Returns 0, 1 for a shape it does not take, < 0 on failure.
-int m40_attention_prefill_cache(M40llmCudaContext* ctx, const M40llmKVCache* kv, const float* q, float* out,
-                                const M40llmStepRows& rows, uint32_t q_heads, float scale, const float2* turn_back,
-                                const float* gate, uint32_t gate_ld);
+// Prompt attention over head-major f16 keys and values [slot][kv_heads][max_seq_len][hd] (hd 64 or 128) for the segments of
+// a step whose keys and values are already there; f32 q, row pitch q_ld, q_dim <= hd values per head (the keys' further
+// dimensions are zero), f32 out, row pitch out_ld, v_dim <= hd values per head. Decode stream. Returns 0, 1 for a shape it
+// does not take, < 0 on failure.
+struct M40PrefillCall {
+    const __half* K;
+    const __half* V;
+    const float* q;
+    float* out;
+    const uint32_t* seg;      // device [segments][4]: first row, rows, sequence, position of the first row
+    const float2* turn_back;  // optional (cos, sin) [rows][hd / 2]: the output turns by the inverse of its value rotation
+    const float* gate;        // optional, row pitch gate_ld: the output is multiplied by sigmoid(gate[row][head])
+    const float* sink;        // optional [q_heads]: exp(sink) joins the denominator
+    uint32_t segments, max_segment_rows, rows;
+    uint32_t hd, q_heads, kv_heads, q_ld, q_dim, out_ld, v_dim, gate_ld;
+    uint32_t slot_mul, slot_add, slots, max_seq_len;
+    float scale;
+};
+int m40_attention_prefill(M40llmCudaContext* ctx, const M40PrefillCall& c);
 
 // Token range of (row, split): shared by both kernels so partial layouts agree.
 __device__ __forceinline__ bool attn_resolve_row(const DenseAttnArgs& a, uint32_t row, uint32_t split, uint32_t* seq,

@@ -4,9 +4,17 @@
 // with uk folded into the query every head attends the same rows c, which are key and value at once.
 //
 //   latent_prepare_kernel  uk^T q per head (absorbed query), and the latent's norm and append;
-//   attention over latents latent_rows_kernel: any rank, f16 or f32 cache, f32 arithmetic, CTA = (head, row, token split);
+//   attention over latents, one of
+//     latent_tiles_kernel  f16 cache, rank a multiple of 16 up to 512: CTA = (row, 16 heads, token split). The tokens' latents
+//                          stream once through shared memory and serve all 16 heads, as keys and as values;
+//     latent_rows_kernel   any rank, f16 or f32 cache, f32 arithmetic: CTA = (head, row, token split);
 //   latent_merge_kernel    merges the token splits and the sink, then uv.
+// Long portions (segments of EXPAND_ROWS rows or more, f16 cache) do less work with the heads' keys and values in hand: they
+// are made once per portion from the cached latents by the grouped tcgen05 GEMM, f16 and head-major, and the prompt kernel of
+// attention_prefill.cu attends them.
 #include "attention.cuh"
+#include "attention_mma.cuh"
+#include "gemm_tc_grouped.cuh"
 #include "stack_math.cuh"
 
 namespace {
@@ -14,6 +22,8 @@ namespace {
 constexpr uint32_t MAX_RANK = 1024;
 constexpr uint32_t COLS = 64;        // latent columns per absorbing CTA
 constexpr uint32_t RUN_ROWS = 512;   // rows per pass of the absorbed form (bounds the work space)
+constexpr uint32_t EXPAND_ROWS = 64;
+constexpr size_t EXPAND_BYTES = (size_t)1 << 30;  // work space for one portion's keys and values
 
 struct LatArgs {
     const float* packed;   // of the pass's first row
@@ -196,6 +206,197 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(LatArgs a) {
     }
 }
 
+// Tensor-core form. Eight warps; warp w owns UW units of 16 latent columns. Per tile of 64 tokens: every warp multiplies the
+// absorbed queries of 16 heads with the tile over its own columns (mma.sync, query split into f16 hi + lo), the eight partial
+// score tiles are added in shared memory, two heads per warp run the online softmax (base 2), and every warp adds P c for its
+// columns. So a latent is read from shared memory once as key and once as value, whatever the number of heads.
+constexpr int LT = 64;
+constexpr int SC_PITCH = 72, P_PITCH = 72;
+__host__ __device__ constexpr size_t latent_tile_bytes(uint32_t rank) { return (size_t)LT * (rank + 8u) * 2u; }
+constexpr size_t LT_FIXED = (size_t)8 * 16 * SC_PITCH * 4 + (size_t)16 * P_PITCH * 2 + 16 * 4;
+
+template <int UW>
+__global__ void __launch_bounds__(256, UW <= 2 ? 2 : 1) latent_tiles_kernel(LatArgs a, uint32_t stages) {
+    using namespace attn_mma;
+    extern __shared__ __align__(128) unsigned char lt_smem[];
+    float* sc = reinterpret_cast<float*>(lt_smem);                              // [8][16][SC_PITCH]
+    __half* sp = reinterpret_cast<__half*>(sc + 8 * 16 * SC_PITCH);             // [16][P_PITCH]
+    float* scorr = reinterpret_cast<float*>(sp + 16 * P_PITCH);                 // [16]
+    __half* ring = reinterpret_cast<__half*>(lt_smem + (LT_FIXED + 127) / 128 * 128);
+    pdl_wait();
+    pdl_trigger();
+    const uint32_t split = blockIdx.x, h0 = blockIdx.y * 16u, row = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
+    const uint32_t g = lane >> 2, t4 = lane & 3u, jm = lane >> 3, NU = a.rank / 16u, pitch = a.rank + 8u;
+    const uint32_t pos = a.row_pos[row], slot = a.row_seq[row] * a.slot_mul + a.slot_add;
+    const uint32_t lo = split * a.chunk, hi = min(lo + a.chunk, pos + 1u), heads = min(16u, a.heads - h0);
+    if (slot >= a.slots || pos >= a.max_seq_len || lo >= hi) {  // empty partials
+        if (tid < heads) {
+            const size_t pi = ((size_t)row * a.heads + h0 + tid) * a.splits + split;
+            a.pm[pi] = -INFINITY, a.pl[pi] = 0.0f;
+        }
+        return;
+    }
+    const __half* C = reinterpret_cast<const __half*>(a.C) + (size_t)slot * a.max_seq_len * a.rank;
+    const uint32_t n_tiles = (hi - lo + LT - 1u) / LT, pieces = a.rank / 8u;
+    auto load_tile = [&](uint32_t tile) {
+        __half* dst = ring + (size_t)(tile % stages) * LT * pitch;
+        const uint32_t base = lo + tile * LT;
+        for (uint32_t i = tid; i < LT * pieces; i += 256u) {
+            const uint32_t r = i / pieces, ch = i % pieces;
+            // rows past the end repeat the last visible one: masked below, and their bytes are finite
+            cp_async16(dst + r * pitch + ch * 8u, C + (size_t)min(base + r, hi - 1u) * a.rank + ch * 8u);
+        }
+    };
+    for (uint32_t t = 0; t + 1u < stages; ++t) {
+        if (t < n_tiles) load_tile(t);
+        cp_async_commit();
+    }
+    // query fragments of this warp's columns
+    uint32_t qhi[UW][4], qlo[UW][4];
+    const float qs = a.scale * LOG2E;
+#pragma unroll
+    for (int i = 0; i < UW; ++i) {
+        const uint32_t u = warp * UW + i, k0 = u * 16u + 2u * t4;
+        float2 x[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {  // rows g, g + 8 of columns k0, then of k0 + 8
+            const uint32_t h = g + (j & 1) * 8u;
+            x[j] = u < NU && h < heads
+                       ? *reinterpret_cast<const float2*>(a.qa + ((size_t)row * a.heads + h0 + h) * a.rank + k0 + (j >> 1) * 8u)
+                       : make_float2(0.f, 0.f);
+            split_h2(x[j].x * qs, x[j].y * qs, &qhi[i][j], &qlo[i][j]);
+        }
+    }
+    float o[UW][2][4];
+#pragma unroll
+    for (int i = 0; i < UW; ++i)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) o[i][j >> 2][j & 3] = 0.0f;
+    float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};  // heads 2 * warp and 2 * warp + 1
+    const uint32_t busy = (NU + UW - 1u) / UW;                         // warps that own columns
+
+    for (uint32_t tile = 0; tile < n_tiles; ++tile) {
+        if (stages == 2u) cp_async_wait<0>();
+        else if (stages == 3u) cp_async_wait<1>();
+        else cp_async_wait<2>();
+        __syncthreads();
+        if (tile + stages - 1u < n_tiles) load_tile(tile + stages - 1u);
+        cp_async_commit();
+        const __half* tc = ring + (size_t)(tile % stages) * LT * pitch;
+        if (warp < busy) {
+            float s[8][4];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.0f;
+#pragma unroll
+            for (int i = 0; i < UW; ++i) {
+                const uint32_t u = warp * UW + i;
+                if (u >= NU) break;
+#pragma unroll
+                for (int p = 0; p < 4; ++p) {
+                    const uint32_t r = p * 16 + (jm >> 1) * 8 + (lane & 7u);
+                    uint32_t b[4];
+                    ldmatrix_x4(b, tc + r * pitch + u * 16u + (jm & 1u) * 8u);
+                    mma16816(s[2 * p], qhi[i][0], qhi[i][1], qhi[i][2], qhi[i][3], b[0], b[1]);
+                    mma16816(s[2 * p], qlo[i][0], qlo[i][1], qlo[i][2], qlo[i][3], b[0], b[1]);
+                    mma16816(s[2 * p + 1], qhi[i][0], qhi[i][1], qhi[i][2], qhi[i][3], b[2], b[3]);
+                    mma16816(s[2 * p + 1], qlo[i][0], qlo[i][1], qlo[i][2], qlo[i][3], b[2], b[3]);
+                }
+            }
+            float* mine = sc + (size_t)warp * 16 * SC_PITCH;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                *reinterpret_cast<float2*>(mine + g * SC_PITCH + j * 8 + 2 * t4) = make_float2(s[j][0], s[j][1]);
+                *reinterpret_cast<float2*>(mine + (g + 8) * SC_PITCH + j * 8 + 2 * t4) = make_float2(s[j][2], s[j][3]);
+            }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const uint32_t h = 2u * warp + e;
+            float v0 = 0.0f, v1 = 0.0f;
+            for (uint32_t w = 0; w < busy; ++w) {
+                v0 += sc[((size_t)w * 16 + h) * SC_PITCH + lane];
+                v1 += sc[((size_t)w * 16 + h) * SC_PITCH + lane + 32u];
+            }
+            const uint32_t t = lo + tile * LT + lane;
+            if (t >= hi) v0 = -INFINITY;
+            if (t + 32u >= hi) v1 = -INFINITY;
+            const float m_new = fmaxf(m_run[e], warp_max(fmaxf(v0, v1)));  // the tile's first token is visible: finite
+            const float corr = fast_exp2(m_run[e] - m_new), p0 = fast_exp2(v0 - m_new), p1 = fast_exp2(v1 - m_new);
+            l_run[e] = l_run[e] * corr + warp_sum(p0 + p1);
+            m_run[e] = m_new;
+            sp[h * P_PITCH + lane] = __float2half_rn(p0);
+            sp[h * P_PITCH + lane + 32u] = __float2half_rn(p1);
+            if (lane == 0) scorr[h] = corr;
+        }
+        __syncthreads();
+        if (warp < busy) {
+            const float ca = scorr[g], cb = scorr[g + 8];
+#pragma unroll
+            for (int i = 0; i < UW; ++i)
+#pragma unroll
+                for (int n = 0; n < 2; ++n) o[i][n][0] *= ca, o[i][n][1] *= ca, o[i][n][2] *= cb, o[i][n][3] *= cb;
+#pragma unroll
+            for (int kk = 0; kk < 4; ++kk) {
+                uint32_t pa[4];
+                ldmatrix_x4(pa, sp + (lane & 15u) * P_PITCH + kk * 16 + (lane >> 4) * 8u);
+                const uint32_t r = kk * 16 + (jm & 1u) * 8 + (lane & 7u);
+#pragma unroll
+                for (int i = 0; i < UW; ++i) {
+                    const uint32_t u = warp * UW + i;
+                    if (u >= NU) break;
+                    uint32_t b[4];
+                    ldmatrix_x4_trans(b, tc + r * pitch + u * 16u + (jm >> 1) * 8u);
+                    mma16816(o[i][0], pa[0], pa[1], pa[2], pa[3], b[0], b[1]);
+                    mma16816(o[i][1], pa[0], pa[1], pa[2], pa[3], b[2], b[3]);
+                }
+            }
+        }
+    }
+    cp_async_wait<0>();
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+        const uint32_t h = 2u * warp + e;
+        if (lane == 0 && h < heads) {
+            const size_t pi = ((size_t)row * a.heads + h0 + h) * a.splits + split;
+            a.pm[pi] = m_run[e] * LN2;  // natural-log domain, as in the other form
+            a.pl[pi] = l_run[e];
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < UW; ++i) {
+        const uint32_t u = warp * UW + i;
+        if (u >= NU) break;
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+            const uint32_t h = g + 8u * j;
+            if (h >= heads) continue;
+            float* dst = a.po + (((size_t)row * a.heads + h0 + h) * a.splits + split) * a.rank + u * 16u + 2u * t4;
+#pragma unroll
+            for (int n = 0; n < 2; ++n) *reinterpret_cast<float2*>(dst + n * 8) = make_float2(o[i][n][2 * j], o[i][n][2 * j + 1]);
+        }
+    }
+}
+
+// Cached f16 latents -> hi + lo in bf16 (exact: 8 + 8 significant bits cover 11).
+__global__ void __launch_bounds__(256) latent_split_kernel(const __half* __restrict__ c, __nv_bfloat16* __restrict__ hi,
+                                                           __nv_bfloat16* __restrict__ lo, size_t n) {
+    pdl_wait();
+    pdl_trigger();
+    for (size_t i = ((size_t)blockIdx.x * 256u + threadIdx.x) * 8u; i < n; i += (size_t)gridDim.x * 2048u) {
+        float v[8];
+        m40_load8(c + i, v);
+        __nv_bfloat16 h[8], l[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            h[j] = __float2bfloat16_rn(v[j]);
+            l[j] = __float2bfloat16_rn(v[j] - __bfloat162float(h[j]));
+        }
+        *reinterpret_cast<uint4*>(hi + i) = *reinterpret_cast<const uint4*>(h);
+        *reinterpret_cast<uint4*>(lo + i) = *reinterpret_cast<const uint4*>(l);
+    }
+}
+
 // grid (heads, row groups of RG, slices of the values): splits and sink -> the head's weighted latent, then uv.
 template <typename WT, int RG>
 __global__ void __launch_bounds__(256) latent_merge_kernel(LatArgs a) {
@@ -292,20 +493,32 @@ cudaError_t prepare(cudaStream_t s, const LatArgs& a, bool f32, bool append) {
     return f32 ? launch_prepare<WT, float>(s, a, append) : launch_prepare<WT, __half>(s, a, append);
 }
 
+template <int UW>
+cudaError_t launch_tiles(M40llmCudaContext* ctx, const LatArgs& a) {
+    static unsigned long long configured = 0ull;
+    const unsigned long long bit = 1ull << (ctx->device_id & 63);
+    constexpr size_t fixed = (LT_FIXED + 127) / 128 * 128, budget = UW <= 2 ? 112u * 1024u : 200u * 1024u;
+    if (!(configured & bit)) {
+        const cudaError_t e = cudaFuncSetAttribute(latent_tiles_kernel<UW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)budget);
+        if (e != cudaSuccess) return e;
+        configured |= bit;
+    }
+    size_t stages = (budget - fixed) / latent_tile_bytes(a.rank);
+    if (stages > 4) stages = 4;
+    const dim3 grid(a.splits, (a.heads + 15) / 16, a.rows);
+    return m40_launch_dependent(latent_tiles_kernel<UW>, grid, dim3(256), fixed + stages * latent_tile_bytes(a.rank),
+                                ctx->decode_stream, a, (uint32_t)stages);
+}
+static_assert((LT_FIXED + 127) / 128 * 128 + 2 * latent_tile_bytes(256) <= 112u * 1024u, "two tiles of rank 256, two CTAs per SM");
+static_assert((LT_FIXED + 127) / 128 * 128 + 2 * latent_tile_bytes(512) <= 200u * 1024u, "two tiles of rank 512");
+
+// Absorbed form over the rows of `all`; append: the latents are not in the cache yet.
 template <typename WT>
-int run(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs& all, uint32_t bound) {
+int run_absorbed(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs& all, uint32_t bound, bool append) {
     cudaStream_t s = ctx->decode_stream;
     const uint32_t slices = (all.rank + COLS - 1) / COLS;
+    const bool tiles = !kv->elem_f32 && all.rank % 16 == 0 && all.rank <= 512;
     cudaError_t e;
-    // one pass does everything in one prepare launch; several append first, so that every pass sees the whole step
-    const bool one = all.rows <= RUN_ROWS;
-    if (!one) {
-        LatArgs a = all;
-        a.absorb_ctas = 0;
-        e = prepare<WT>(s, a, kv->elem_f32, true);
-        M40_COUNT_LAUNCH(ctx);
-        if (e != cudaSuccess) return -6;
-    }
     for (uint32_t at = 0; at < all.rows; at += RUN_ROWS) {
         LatArgs a = all;
         a.rows = all.rows - at < RUN_ROWS ? all.rows - at : RUN_ROWS;
@@ -313,7 +526,7 @@ int run(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs& all, uin
         a.out += (size_t)at * a.heads * a.vdim;
         a.row_seq += at;
         a.row_pos += at;
-        m40_attn_pick_chunk(ctx, a.rows, a.heads, bound, &a.chunk, &a.splits);
+        m40_attn_pick_chunk(ctx, a.rows, tiles ? (a.heads + 15) / 16 : a.heads, bound, &a.chunk, &a.splits);
         const size_t nh = (size_t)a.rows * a.heads, np = nh * a.splits;
         auto pad = [](size_t v) { return (v + 3) & ~(size_t)3; };
         float* work = (float*)m40_ensure_scratch(ctx, 1, (pad(nh * a.rank) + pad(np * a.rank) + 2 * np) * sizeof(float), 1);
@@ -323,17 +536,143 @@ int run(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs& all, uin
         a.pm = a.po + pad(np * a.rank);
         a.pl = a.pm + np;
         a.absorb_ctas = a.heads * slices;
-        e = prepare<WT>(s, a, kv->elem_f32, one);
+        e = prepare<WT>(s, a, kv->elem_f32, append);
         M40_COUNT_LAUNCH(ctx);
         if (e != cudaSuccess) return -6;
         const dim3 grid(a.heads, a.rows, a.splits);
-        e = kv->elem_f32 ? m40_launch_dependent(latent_rows_kernel<float>, grid, dim3(128), 0, s, a)
-                         : m40_launch_dependent(latent_rows_kernel<__half>, grid, dim3(128), 0, s, a);
+        if (tiles)
+            e = a.rank <= 128 ? launch_tiles<1>(ctx, a) : (a.rank <= 256 ? launch_tiles<2>(ctx, a) : launch_tiles<4>(ctx, a));
+        else
+            e = kv->elem_f32 ? m40_launch_dependent(latent_rows_kernel<float>, grid, dim3(128), 0, s, a)
+                             : m40_launch_dependent(latent_rows_kernel<__half>, grid, dim3(128), 0, s, a);
         M40_COUNT_LAUNCH(ctx);
         if (e != cudaSuccess) return -6;
         e = launch_merge<WT>(ctx, a);
         M40_COUNT_LAUNCH(ctx);
         if (e != cudaSuccess || cudaGetLastError() != cudaSuccess) return -6;
+    }
+    return 0;
+}
+
+bool takes_expanded(const M40llmKVCache* kv, const LatArgs& a, uint32_t w_dtype) {
+    return !kv->elem_f32 && w_dtype != M40LLM_DT_F32 && a.dim <= 128 && a.vdim <= 128 && a.dim % 2 == 0 && a.vdim % 2 == 0 &&
+           a.ld % 2 == 0 && (((uintptr_t)a.packed | (uintptr_t)a.out) & 7u) == 0 && (a.heads * a.vdim) % 2 == 0 &&
+           m40_gemm_tc_grouped_supported(a.uk, a.heads * a.dim, a.rank, a.rank, 0) &&
+           m40_gemm_tc_grouped_supported(a.uv, a.heads * a.vdim, a.rank, a.rank, 0);
+}
+size_t expanded_bytes(const LatArgs& a, uint32_t kv_len, uint32_t hd) {
+    return (size_t)kv_len * ((size_t)a.heads * hd * 4 + (size_t)a.rank * 4) + 1024;
+}
+
+// One portion (its latents are in the cache): the heads' keys and values, then the prompt kernel. seg is on the device.
+int run_expanded(M40llmCudaContext* ctx, const LatArgs& a, uint32_t w_dtype, const uint32_t* seg, const uint32_t* seg_host) {
+    cudaStream_t s = ctx->decode_stream;
+    const uint32_t hd = a.dim <= 64 && a.vdim <= 64 ? 64u : 128u, n = seg_host[3] + seg_host[1];
+    const uint32_t slot = seg_host[2] * a.slot_mul + a.slot_add;
+    const __half* C = reinterpret_cast<const __half*>(a.C) + (size_t)slot * a.max_seq_len * a.rank;
+    const size_t kv_elems = (size_t)n * a.heads * hd, c_elems = (size_t)n * a.rank;
+    unsigned char* work = (unsigned char*)m40_ensure_scratch(ctx, 1, expanded_bytes(a, n, hd), 1);
+    if (!work) return -5;
+    work = (unsigned char*)(((uintptr_t)work + 255) & ~(uintptr_t)255);
+    __half *K = (__half*)work, *V = K + kv_elems;
+    const bool bf16 = w_dtype == M40LLM_DT_BF16;
+    M40GroupedCall c = {};
+    c.x[0] = C;
+    c.parts = 1;
+    cudaError_t e;
+    if (bf16) {
+        __nv_bfloat16 *hi = (__nv_bfloat16*)(((uintptr_t)(V + kv_elems) + 127) & ~(uintptr_t)127), *lo = hi + c_elems;
+        const size_t blocks = (c_elems + 2047) / 2048;
+        e = m40_launch_dependent(latent_split_kernel, dim3((unsigned)(blocks < 4096 ? blocks : 4096)), dim3(256), 0, s, C, hi, lo, c_elems);
+        M40_COUNT_LAUNCH(ctx);
+        if (e != cudaSuccess) return -6;
+        c.x[0] = hi, c.x[1] = lo;
+        c.parts = 2;
+    }
+    // dimensions beyond a head's own are zeros
+    if (a.dim < hd && cudaMemsetAsync(K, 0, kv_elems * 2, s) != cudaSuccess) return -6;
+    if (a.vdim < hd && cudaMemsetAsync(V, 0, kv_elems * 2, s) != cudaSuccess) return -6;
+    c.bf16 = bf16;
+    c.groups = 1;
+    c.K = c.ldx = a.rank;
+    c.x_rows = n;
+    c.tile_rows = 128;
+    c.kind = M40_GROUPED_HEADS;
+    c.head_pitch = hd;
+    c.w = a.uk;
+    c.N = a.heads * a.dim;
+    c.head_dim = a.dim;
+    c.heads = K;
+    int rc = m40_gemm_tc_grouped(ctx, s, c);
+    if (rc != 0) return rc;
+    c.w = a.uv;
+    c.N = a.heads * a.vdim;
+    c.head_dim = a.vdim;
+    c.heads = V;
+    if ((rc = m40_gemm_tc_grouped(ctx, s, c)) != 0) return rc;
+    M40PrefillCall p = {};
+    p.K = K;
+    p.V = V;
+    p.q = a.packed;
+    p.out = a.out;
+    p.seg = seg;
+    p.sink = a.sink;
+    p.segments = 1;
+    p.max_segment_rows = seg_host[1];
+    p.rows = a.rows;
+    p.hd = hd;
+    p.q_heads = p.kv_heads = a.heads;
+    p.q_ld = a.ld;
+    p.q_dim = a.dim;
+    p.out_ld = a.heads * a.vdim;
+    p.v_dim = a.vdim;
+    p.slots = 1;
+    p.max_seq_len = n;
+    p.scale = a.scale;
+    rc = m40_attention_prefill(ctx, p);
+    return rc > 0 ? -6 : rc;
+}
+
+template <typename WT>
+int run(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs& all, uint32_t bound, uint32_t w_dtype, const M40llmStepRows& r) {
+    const uint32_t hd = all.dim <= 64 && all.vdim <= 64 ? 64u : 128u;
+    // the portion's host copy decides its form; out-of-range portions take the absorbed form, which checks them on the device
+    auto expands = [&](const uint32_t* sg) {
+        return sg[1] >= EXPAND_ROWS && (uint64_t)sg[0] + sg[1] <= all.rows && (uint64_t)sg[3] + sg[1] <= all.max_seq_len &&
+               (uint64_t)sg[2] * all.slot_mul + all.slot_add < all.slots && expanded_bytes(all, sg[3] + sg[1], hd) <= EXPAND_BYTES;
+    };
+    bool any = false;
+    if (r.seg_host && r.seg && r.max_segment_rows >= EXPAND_ROWS && takes_expanded(kv, all, w_dtype))
+        for (uint32_t i = 0; i < r.segments; ++i) any = any || expands(r.seg_host + 4 * i);
+    // several launches read the cache: every latent of the step is appended first
+    const bool first = any || all.rows > RUN_ROWS;
+    if (first) {
+        LatArgs a = all;
+        a.absorb_ctas = 0;
+        const cudaError_t e = prepare<WT>(ctx->decode_stream, a, kv->elem_f32, true);
+        M40_COUNT_LAUNCH(ctx);
+        if (e != cudaSuccess) return -6;
+    }
+    if (!any) return run_absorbed<WT>(ctx, kv, all, bound, !first);
+    uint32_t run0 = 0;  // first row of the absorbed run that is being gathered
+    for (uint32_t i = 0; i <= r.segments; ++i) {
+        const uint32_t* sg = i < r.segments ? r.seg_host + 4 * i : nullptr;
+        if (sg && !expands(sg)) continue;
+        const uint32_t end = sg ? sg[0] : all.rows;
+        if (end > run0) {
+            LatArgs a = all;
+            a.rows = end - run0;
+            a.packed += (size_t)run0 * a.ld;
+            a.out += (size_t)run0 * a.heads * a.vdim;
+            a.row_seq += run0;
+            a.row_pos += run0;
+            const int rc = run_absorbed<WT>(ctx, kv, a, bound, false);
+            if (rc != 0) return rc;
+        }
+        if (!sg) break;
+        const int rc = run_expanded(ctx, all, w_dtype, r.seg + 4 * i, sg);
+        if (rc != 0) return rc;
+        run0 = sg[0] + sg[1];
     }
     return 0;
 }
@@ -374,6 +713,6 @@ extern "C" int m40llm_attention_latent_async(M40llmCudaContext* ctx, M40llmKVCac
     a.scale = c->scale;
     a.wide = c->w_dtype != M40LLM_DT_F32 && a.rank % 8 == 0 && (((uintptr_t)c->uk | (uintptr_t)c->uv) & 15u) == 0;
     const uint32_t bound = r->max_len && r->max_len < kv->max_seq_len ? r->max_len : kv->max_seq_len;
-    if (c->w_dtype == M40LLM_DT_F32) return run<float>(ctx, kv, a, bound);
-    return c->w_dtype == M40LLM_DT_BF16 ? run<__nv_bfloat16>(ctx, kv, a, bound) : run<__half>(ctx, kv, a, bound);
+    if (c->w_dtype == M40LLM_DT_F32) return run<float>(ctx, kv, a, bound, c->w_dtype, *r);
+    return c->w_dtype == M40LLM_DT_BF16 ? run<__nv_bfloat16>(ctx, kv, a, bound, c->w_dtype, *r) : run<__half>(ctx, kv, a, bound, c->w_dtype, *r);
 }

@@ -38,11 +38,8 @@ __global__ void __launch_bounds__(256) prefill_pack_kv_kernel(const float* __res
 }
 
 struct PrefillCache {
-    const uint32_t* seg;  // [segments][4]: first row, rows, sequence, position of the first row
-    const float2* turn_back;
-    const float* gate;
+    M40PrefillCall c;
     uint32_t* status;
-    uint32_t slot_mul, slot_add, slots, max_seq_len, gate_ld, rows;
 };
 
 template <int HD, bool CACHE>
@@ -52,7 +49,7 @@ __global__ void __launch_bounds__(128, 2) prefill_varlen_kernel(const float* __r
                                                                 const uint32_t* __restrict__ kv_offsets,
                                                                 const uint32_t* __restrict__ q_lens,
                                                                 const uint32_t* __restrict__ kv_lens, uint32_t q_heads,
-                                                                uint32_t kv_heads, float inv_sqrt, float* __restrict__ Out, PrefillCache pc) {
+                                                                uint32_t kv_heads, float inv_sqrt, float* __restrict__ Out, PrefillCache cache) {
     constexpr int KS = HD / 16;      // k-steps of Q K^T
     constexpr int NT = HD / 8;       // n8 tiles of the output
     constexpr int CHUNKS = HD / 8;   // 16-byte f16 pieces per row
@@ -64,6 +61,7 @@ __global__ void __launch_bounds__(128, 2) prefill_varlen_kernel(const float* __r
         pdl_wait();
         pdl_trigger();
     }
+    const M40PrefillCall& pc = cache.c;
     const uint32_t q_len = CACHE ? pc.seg[4 * b + 1] : q_lens[b];
     const uint32_t kv_len = CACHE ? pc.seg[4 * b + 3] + q_len : kv_lens[b];
     if (r0 >= q_len || q_len == 0 || kv_len == 0 || q_len > kv_len) return;
@@ -72,7 +70,7 @@ __global__ void __launch_bounds__(128, 2) prefill_varlen_kernel(const float* __r
     const uint32_t kvh = qh / (q_heads / kv_heads);
     const uint32_t slot = CACHE ? pc.seg[4 * b + 2] * pc.slot_mul + pc.slot_add : 0u;
     if (CACHE && (slot >= pc.slots || kv_len > pc.max_seq_len || (uint64_t)pc.seg[4 * b] + q_len > pc.rows)) {
-        if (threadIdx.x == 0) atomicOr(pc.status, 1u);
+        if (threadIdx.x == 0) atomicOr(cache.status, 1u);
         return;
     }
     const size_t q_row0 = (size_t)(CACHE ? pc.seg[4 * b] : q_offsets[b]) + r0;
@@ -88,19 +86,22 @@ __global__ void __launch_bounds__(128, 2) prefill_varlen_kernel(const float* __r
     uint32_t qhi[KS][4], qlo[KS][4];
     {
         const float qs = inv_sqrt * LOG2E;
-        const float* qa = Q + ((q_row0 + warp * 16u + g) * q_heads + qh) * HD;
-        const float* qb = qa + (size_t)8 * q_heads * HD;
+        const size_t q_ld = CACHE ? pc.q_ld : q_heads * HD;
+        const uint32_t q_dim = CACHE ? pc.q_dim : HD;
+        const float* qa = Q + (q_row0 + warp * 16u + g) * q_ld + qh * q_dim;
+        const float* qb = qa + 8 * q_ld;
 #pragma unroll
         for (int ks = 0; ks < KS; ++ks) {
             const int k0 = ks * 16 + 2 * t4;
             float2 x0 = make_float2(0.f, 0.f), x1 = x0, x2 = x0, x3 = x0;
+            const bool lo_in = !CACHE || (uint32_t)k0 < q_dim, hi_in = !CACHE || (uint32_t)k0 + 8u < q_dim;
             if (row_a < q_len) {
-                x0 = *reinterpret_cast<const float2*>(qa + k0);
-                x2 = *reinterpret_cast<const float2*>(qa + k0 + 8);
+                if (lo_in) x0 = *reinterpret_cast<const float2*>(qa + k0);
+                if (hi_in) x2 = *reinterpret_cast<const float2*>(qa + k0 + 8);
             }
             if (row_b < q_len) {
-                x1 = *reinterpret_cast<const float2*>(qb + k0);
-                x3 = *reinterpret_cast<const float2*>(qb + k0 + 8);
+                if (lo_in) x1 = *reinterpret_cast<const float2*>(qb + k0);
+                if (hi_in) x3 = *reinterpret_cast<const float2*>(qb + k0 + 8);
             }
             split_h2(x0.x * qs, x0.y * qs, &qhi[ks][0], &qlo[ks][0]);
             split_h2(x1.x * qs, x1.y * qs, &qhi[ks][1], &qlo[ks][1]);
@@ -112,6 +113,10 @@ __global__ void __launch_bounds__(128, 2) prefill_varlen_kernel(const float* __r
 #pragma unroll
     for (int n = 0; n < NT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.0f;
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};
+    if (CACHE && pc.sink) {  // a sink is a key whose score is known from the start and whose value is zero
+        m_run[0] = m_run[1] = pc.sink[qh] * LOG2E;
+        l_run[0] = l_run[1] = 1.0f;
+    }
 
     // kv rows this q tile may see: 0 .. shift + (last q row of the tile)
     const uint32_t last_q = min(r0 + PF_TILE, q_len) - 1u;
@@ -249,10 +254,13 @@ __global__ void __launch_bounds__(128, 2) prefill_varlen_kernel(const float* __r
             if (row_b < q_len) inv_b *= m40_sigmoid(pc.gate[(ra + 8u) * pc.gate_ld + qh]);
         }
     }
-    float* oa = Out + ((q_row0 + warp * 16u + g) * q_heads + qh) * HD;
-    float* ob = oa + (size_t)8 * q_heads * HD;
+    const size_t out_ld = CACHE ? pc.out_ld : q_heads * HD;
+    const uint32_t v_dim = CACHE ? pc.v_dim : HD;
+    float* oa = Out + (q_row0 + warp * 16u + g) * out_ld + qh * v_dim;
+    float* ob = oa + 8 * out_ld;
 #pragma unroll
     for (int n = 0; n < NT; ++n) {
+        if (CACHE && n * 8u + 2u * t4 >= v_dim) break;
         if (row_a < q_len) *reinterpret_cast<float2*>(oa + n * 8 + 2 * t4) = make_float2(o[n][0] * inv_a, o[n][1] * inv_a);
         if (row_b < q_len) *reinterpret_cast<float2*>(ob + n * 8 + 2 * t4) = make_float2(o[n][2] * inv_b, o[n][3] * inv_b);
     }
@@ -273,23 +281,20 @@ bool prefill_configure(int device_id) {
 
 }  // namespace
 
-int m40_attention_prefill_cache(M40llmCudaContext* ctx, const M40llmKVCache* kv, const float* q, float* out,
-                                const M40llmStepRows& rows, uint32_t q_heads, float scale, const float2* turn_back,
-                                const float* gate, uint32_t gate_ld) {
-    const uint32_t hd = kv->head_dim;
-    if ((hd != 64 && hd != 128) || !kv->d_k || !kv->d_v || !rows.seg) return 1;
-    if ((((uintptr_t)q) & 7u) != 0u || (((uintptr_t)out) & 7u) != 0u) return 1;
+int m40_attention_prefill(M40llmCudaContext* ctx, const M40PrefillCall& c) {
+    if ((c.hd != 64 && c.hd != 128) || !c.K || !c.V || !c.seg) return 1;
+    if (c.q_dim > c.hd || c.v_dim > c.hd || ((c.q_dim | c.v_dim | c.q_ld | c.out_ld) & 1u)) return 1;
+    if ((((uintptr_t)c.q) & 7u) != 0u || (((uintptr_t)c.out) & 7u) != 0u) return 1;
     if (!prefill_configure(ctx->device_id)) return -4;
-    const PrefillCache pc = {rows.seg, turn_back, gate, ctx->d_status, rows.slot_mul, rows.slot_add, kv->max_batch_size,
-                             kv->max_seq_len, gate_ld, rows.rows};
-    const dim3 grid((rows.max_segment_rows + PF_TILE - 1) / PF_TILE, q_heads, rows.segments);
-    const size_t smem = (size_t)2 * 2 * PF_TILE * hd * sizeof(__half);
+    const PrefillCache pc = {c, ctx->d_status};
+    const dim3 grid((c.max_segment_rows + PF_TILE - 1) / PF_TILE, c.q_heads, c.segments);
+    const size_t smem = (size_t)2 * 2 * PF_TILE * c.hd * sizeof(__half);
     const uint32_t* none = nullptr;
     const cudaError_t e =
-        hd == 128 ? m40_launch_dependent(prefill_varlen_kernel<128, true>, grid, dim3(128), smem, ctx->decode_stream, q, kv->d_k,
-                                         kv->d_v, none, none, none, none, q_heads, kv->num_heads, scale, out, pc)
-                  : m40_launch_dependent(prefill_varlen_kernel<64, true>, grid, dim3(128), smem, ctx->decode_stream, q, kv->d_k,
-                                         kv->d_v, none, none, none, none, q_heads, kv->num_heads, scale, out, pc);
+        c.hd == 128 ? m40_launch_dependent(prefill_varlen_kernel<128, true>, grid, dim3(128), smem, ctx->decode_stream, c.q, c.K,
+                                           c.V, none, none, none, none, c.q_heads, c.kv_heads, c.scale, c.out, pc)
+                    : m40_launch_dependent(prefill_varlen_kernel<64, true>, grid, dim3(128), smem, ctx->decode_stream, c.q, c.K,
+                                           c.V, none, none, none, none, c.q_heads, c.kv_heads, c.scale, c.out, pc);
     M40_COUNT_LAUNCH(ctx);
     return e == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

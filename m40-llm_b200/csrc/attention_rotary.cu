@@ -384,8 +384,28 @@ extern "C" int m40llm_attention_rotary_async(M40llmCudaContext* ctx, M40llmKVCac
     }
     if (tiles) {
         const float* gate = c->has_gate ? a.packed + (size_t)c->q_heads * kd + (size_t)kv->num_heads * (kd + vd) : nullptr;
-        const int rc = m40_attention_prefill_cache(ctx, kv, a.q, a.out, *r, c->q_heads, c->scale, a.v_turns ? a.turn : nullptr,
-                                                   gate, c->ld);
+        M40PrefillCall p = {};
+        p.K = kv->d_k;
+        p.V = kv->d_v;
+        p.q = a.q;
+        p.out = a.out;
+        p.seg = r->seg;
+        p.turn_back = a.v_turns ? a.turn : nullptr;
+        p.gate = gate;
+        p.gate_ld = c->ld;
+        p.segments = r->segments;
+        p.max_segment_rows = r->max_segment_rows;
+        p.rows = r->rows;
+        p.hd = p.q_dim = p.v_dim = kd;
+        p.q_heads = c->q_heads;
+        p.kv_heads = kv->num_heads;
+        p.q_ld = p.out_ld = c->q_heads * kd;
+        p.slot_mul = r->slot_mul;
+        p.slot_add = r->slot_add;
+        p.slots = kv->max_batch_size;
+        p.max_seq_len = kv->max_seq_len;
+        p.scale = c->scale;
+        const int rc = m40_attention_prefill(ctx, p);
         if (rc <= 0) return rc;
     }
     const size_t smem = (size_t)kd * sizeof(float);

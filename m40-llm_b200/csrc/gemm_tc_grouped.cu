@@ -27,6 +27,8 @@ struct GArgs {
     uint32_t* status;
     uint32_t N, K, x_rows, group_k, tile_rows, parts, kblocks, stages, fmt_bits, bf16;
     int act;
+    __half* heads;
+    uint32_t head_dim, head_pitch;
     M40RgArgs rg;
 };
 
@@ -196,6 +198,8 @@ __global__ void __launch_bounds__(192, 1) gemm_tc_grouped_kernel(const __grid_co
             }
         } else {
             const uint32_t n = n0 + row_of_tile;
+            __half* heads = KIND == M40_GROUPED_HEADS
+                                ? a.heads + (size_t)(n / a.head_dim) * a.x_rows * a.head_pitch + n % a.head_dim : nullptr;
             for (uint32_t c = 0; c < a.tile_rows && c < m_live; c += 8) {
                 float v[8];
                 sums(c, v);
@@ -204,6 +208,7 @@ __global__ void __launch_bounds__(192, 1) gemm_tc_grouped_kernel(const __grid_co
                     if (n >= a.N || c + j >= m_live) continue;
                     const size_t at = (size_t)(m_base + c + j) * a.N + n;
                     if (KIND == M40_GROUPED_F32) a.out[at] = v[j];
+                    else if (KIND == M40_GROUPED_HEADS) heads[(size_t)(m_base + c + j) * a.head_pitch] = __float2half_rn(v[j]);
                     else if (a.bf16) store_split((__nv_bfloat16*)a.hi, (__nv_bfloat16*)a.lo, at, m40_act(a.act, v[j]));
                     else store_split((__half*)a.hi, (__half*)a.lo, at, m40_act(a.act, v[j]));
                 }
@@ -266,6 +271,9 @@ int m40_gemm_tc_grouped(M40llmCudaContext* ctx, cudaStream_t s, const M40Grouped
     a.fmt_bits = c.bf16 ? tc::idesc_bf16() : 0u;
     a.bf16 = c.bf16;
     a.act = c.act;
+    a.heads = c.heads;
+    a.head_dim = c.head_dim;
+    a.head_pitch = c.head_pitch;
     a.rg = c.rg;
     const uint32_t stage = tc::BLOCK_N * tc::BLOCK_K * 2 + c.parts * c.tile_rows * tc::BLOCK_K * 2;
     uint32_t stages = 100u * 1024u / stage;
@@ -280,6 +288,7 @@ int m40_gemm_tc_grouped(M40llmCudaContext* ctx, cudaStream_t s, const M40Grouped
     switch (c.kind) {
         case M40_GROUPED_F32: return launch<M40_GROUPED_F32>(ctx, s, grid, smem, m, a);
         case M40_GROUPED_ACT_SPLIT: return launch<M40_GROUPED_ACT_SPLIT>(ctx, s, grid, smem, m, a);
+        case M40_GROUPED_HEADS: return launch<M40_GROUPED_HEADS>(ctx, s, grid, smem, m, a);
         default: return launch<M40_GROUPED_RG>(ctx, s, grid, smem, m, a);
     }
 }

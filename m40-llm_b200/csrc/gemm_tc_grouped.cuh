@@ -7,7 +7,7 @@ struct M40GroupTile {
     uint32_t group, row0, live, pad;
 };
 
-enum { M40_GROUPED_F32 = 0, M40_GROUPED_ACT_SPLIT = 1, M40_GROUPED_RG = 2 };
+enum { M40_GROUPED_F32 = 0, M40_GROUPED_ACT_SPLIT = 1, M40_GROUPED_RG = 2, M40_GROUPED_HEADS = 3 };
 
 // D[m][n] = sum_k X[m][group * group_k + k] * W[group * N + n][k] for the rows m of every tile.
 // X is given as `parts` 16-bit arrays of the weights' type, [x_rows][ldx] each, whose sum is the activation.
@@ -26,6 +26,8 @@ struct M40GroupedCall {
     float* out;                // F32: [x_rows][N]
     void* hi;                  // ACT_SPLIT: act(D) as hi + lo of the weights' type, [x_rows][N]
     void* lo;
+    __half* heads;             // HEADS: f16 [N / head_dim][x_rows][head_pitch], one row of D dealt to heads of head_dim values
+    uint32_t head_dim, head_pitch;
     M40RgArgs rg;              // RG: a and b of every (row, channel)
 };
 // Whether the shapes and pointers are ones the kernel takes.

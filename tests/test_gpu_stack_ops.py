@@ -103,7 +103,8 @@ def test_linear_rejects(nat):
     assert call(mk(ldx=63)) == -2
     assert call(mk(act=9)) == -3
     assert call(mk(pre=N.Norm(N.NORM_RMS, 1e-5, 0.0, None, None))) == -4
-    assert call(mk(post=N.Norm(N.NORM_RMS, 1e-5, 0.0, b.ptr, None))) == -4
+    assert call(mk(post=N.Norm(N.NORM_RMS, 1e-5, 0.0, None, None))) == -4
+    assert call(mk(post=N.Norm(N.NORM_POLY, 1e-5, 0.0, b.ptr, None))) == -4
     assert nat.lib.m40llm_linear_async(nat.ctx, C.byref(N.Linear()), 1) == -1
     nat.free_all()
 
