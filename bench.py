@@ -1221,7 +1221,8 @@ def main():
     ap.add_argument("--workload", default="layer", choices=["layer", "splitk", "stack", "sidalorn"],
                     help="layer: the batched decode layer (the contract's line); splitk: one 32K sequence, split-K over "
                          "the ranks (its own JSON line); stack: the Lamutar layer stack at several sizes beside the Llama "
-                         "stack of equal size, whole models and single calls (its own JSON line, one GPU)")
+                         "stack of equal size, whole models and single calls (its own JSON line, one GPU); sidalorn: Sidalorn "
+                         "models beside the Lamutar stack of equal size, likewise")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
     rank = int(os.environ.get("RANK", "0"))

@@ -20,7 +20,6 @@
 namespace {
 
 constexpr uint32_t MAX_RANK = 1024;
-constexpr uint32_t COLS = 64;        // latent columns per absorbing CTA
 constexpr uint32_t RUN_ROWS = 512;   // rows per pass of the absorbed form (bounds the work space)
 constexpr uint32_t EXPAND_ROWS = 64;
 constexpr size_t EXPAND_BYTES = (size_t)1 << 30;  // work space for one portion's keys and values
@@ -57,54 +56,59 @@ __device__ __forceinline__ float block_sum_256(float v, float* red) {
     return t;
 }
 
-// grid (absorb_ctas + 1 or 0, row groups of RG). CTAs below absorb_ctas: (head, 64 latent columns) of the absorbed query;
-// the last one, when present: norm and append of the group's latents.
-template <typename WT, typename ET, int RG>
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+
+// grid (absorb_ctas + RG or 0, row groups of RG). CTAs below absorb_ctas: (head, COLS latent columns) of the group's absorbed
+// queries; the others, when present: norm and append of one row's latent.
+template <typename WT, typename ET, int RG, int COLS>
 __global__ void __launch_bounds__(256) latent_prepare_kernel(LatArgs a) {
     extern __shared__ __align__(16) float sq[];  // [RG][dim]
+    constexpr uint32_t CG = COLS / 8, KG = 256 / CG;  // groups of 8 columns, groups of query dimensions
     __shared__ float part[8][RG][COLS];
     __shared__ float red[8];
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u, row0 = blockIdx.y * RG;
+    const uint32_t slices = (a.rank + COLS - 1u) / COLS, head = blockIdx.x / slices, c0 = (blockIdx.x % slices) * COLS;
+    const WT* w = reinterpret_cast<const WT*>(a.uk) + (size_t)head * a.dim * a.rank;
+    if (blockIdx.x < a.absorb_ctas)  // the weights do not depend on the previous kernel
+        for (uint32_t d = tid; d < a.dim; d += 256u) prefetch_l2(w + (size_t)d * a.rank + c0);
     pdl_wait();
     pdl_trigger();
-    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u, row0 = blockIdx.y * RG;
     if (blockIdx.x >= a.absorb_ctas) {
-        for (uint32_t r = 0; r < RG && row0 + r < a.rows; ++r) {
-            const uint32_t row = row0 + r, pos = a.row_pos[row], slot = a.row_seq[row] * a.slot_mul + a.slot_add;
-            if (slot >= a.slots || pos >= a.max_seq_len) {
-                if (tid == 0) atomicOr(a.status, 2u);
-                continue;
-            }
-            const float* c = a.packed + (size_t)row * a.ld + (size_t)a.heads * a.dim;
-            float v[MAX_RANK / 256], ss = 0.0f;
-#pragma unroll
-            for (int i = 0; i < (int)MAX_RANK / 256; ++i) {
-                const uint32_t k = tid + 256u * i;
-                v[i] = k < a.rank ? c[k] : 0.0f;
-                ss = fmaf(v[i], v[i], ss);
-            }
-            const float n = 1.0f / sqrtf(block_sum_256(ss, red) / (float)a.rank + a.eps);
-            ET* dst = reinterpret_cast<ET*>(a.C) + ((size_t)slot * a.max_seq_len + pos) * a.rank;
-#pragma unroll
-            for (int i = 0; i < (int)MAX_RANK / 256; ++i) {
-                const uint32_t k = tid + 256u * i;
-                if (k < a.rank) m40_store_elem(dst + k, v[i] * n * a.c_norm[k]);
-            }
-            if (tid == 0 && a.seq_map) a.seq_map[slot] = pos + 1u;
+        const uint32_t row = row0 + blockIdx.x - a.absorb_ctas;
+        if (row >= a.rows) return;
+        const uint32_t pos = a.row_pos[row], slot = a.row_seq[row] * a.slot_mul + a.slot_add;
+        if (slot >= a.slots || pos >= a.max_seq_len) {
+            if (tid == 0) atomicOr(a.status, 2u);
+            return;
         }
+        const float* c = a.packed + (size_t)row * a.ld + (size_t)a.heads * a.dim;
+        float v[MAX_RANK / 256], ss = 0.0f;
+#pragma unroll
+        for (int i = 0; i < (int)MAX_RANK / 256; ++i) {
+            const uint32_t k = tid + 256u * i;
+            v[i] = k < a.rank ? c[k] : 0.0f;
+            ss = fmaf(v[i], v[i], ss);
+        }
+        const float n = 1.0f / sqrtf(block_sum_256(ss, red) / (float)a.rank + a.eps);
+        ET* dst = reinterpret_cast<ET*>(a.C) + ((size_t)slot * a.max_seq_len + pos) * a.rank;
+#pragma unroll
+        for (int i = 0; i < (int)MAX_RANK / 256; ++i) {
+            const uint32_t k = tid + 256u * i;
+            if (k < a.rank) m40_store_elem(dst + k, v[i] * n * a.c_norm[k]);
+        }
+        if (tid == 0 && a.seq_map) a.seq_map[slot] = pos + 1u;
         return;
     }
-    const uint32_t slices = (a.rank + COLS - 1u) / COLS, head = blockIdx.x / slices, c0 = (blockIdx.x % slices) * COLS;
     for (uint32_t i = tid; i < RG * a.dim; i += 256u) {
         const uint32_t row = min(row0 + i / a.dim, a.rows - 1u);
         sq[i] = a.packed[(size_t)row * a.ld + (size_t)head * a.dim + i % a.dim];
     }
     __syncthreads();
-    const uint32_t cg = c0 + (lane & 7u) * 8u, kg = warp * 4u + (lane >> 3);
-    const WT* w = reinterpret_cast<const WT*>(a.uk) + (size_t)head * a.dim * a.rank;
+    const uint32_t cg = c0 + (lane % CG) * 8u, kg = warp * (32u / CG) + lane / CG;
     float acc[RG][8] = {};
     if (cg < a.rank) {
 #pragma unroll 4
-        for (uint32_t d = kg; d < a.dim; d += 32u) {
+        for (uint32_t d = kg; d < a.dim; d += KG) {
             float wv[8];
             if (a.wide) {
                 m40_load8(w + (size_t)d * a.rank + cg, wv);
@@ -123,10 +127,17 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(LatArgs a) {
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
             float v = acc[r][i];
-            v += __shfl_xor_sync(0xffffffffu, v, 8);
-            v += __shfl_xor_sync(0xffffffffu, v, 16);
-            if (lane < 8u) part[warp][r][lane * 8u + i] = v;
+#pragma unroll
+            for (uint32_t o = CG; o < 32u; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+            acc[r][i] = v;
         }
+    if (lane < CG) {
+#pragma unroll
+        for (int r = 0; r < RG; ++r) {
+            *reinterpret_cast<float4*>(&part[warp][r][lane * 8u]) = make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]);
+            *reinterpret_cast<float4*>(&part[warp][r][lane * 8u + 4u]) = make_float4(acc[r][4], acc[r][5], acc[r][6], acc[r][7]);
+        }
+    }
     __syncthreads();
     for (uint32_t i = tid; i < RG * COLS; i += 256u) {
         const uint32_t r = i / COLS, c = i % COLS;
@@ -206,23 +217,29 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(LatArgs a) {
     }
 }
 
-// Tensor-core form. Eight warps; warp w owns UW units of 16 latent columns. Per tile of 64 tokens: every warp multiplies the
+// Tensor-core form. Eight warps; warp w owns UW units of 16 latent columns. Per tile of 64 or 32 tokens: every warp multiplies the
 // absorbed queries of 16 heads with the tile over its own columns (mma.sync, query split into f16 hi + lo), the eight partial
 // score tiles are added in shared memory, two heads per warp run the online softmax (base 2), and every warp adds P c for its
 // columns. So a latent is read from shared memory once as key and once as value, whatever the number of heads.
-constexpr int LT = 64;
-constexpr int SC_PITCH = 72, P_PITCH = 72;
-__host__ __device__ constexpr size_t latent_tile_bytes(uint32_t rank) { return (size_t)LT * (rank + 8u) * 2u; }
-constexpr size_t LT_FIXED = (size_t)8 * 16 * SC_PITCH * 4 + (size_t)16 * P_PITCH * 2 + 16 * 4;
+// Two CTAs share an SM, so that one's barriers and softmax hide behind the other's products.
+template <int UW>
+struct LatTile {
+    static constexpr int TOKENS = UW <= 2 ? 64 : 32;
+    static constexpr int PITCH = TOKENS + 8;  // of scores (f32) and weights (f16): no bank conflicts
+    static constexpr size_t FIXED = ((size_t)8 * 16 * PITCH * 4 + (size_t)16 * PITCH * 2 + 16 * 4 + 127) / 128 * 128;
+    static constexpr size_t bytes(uint32_t rank) { return (size_t)TOKENS * (rank + 8u) * 2u; }
+};
+constexpr size_t TILE_SMEM = 112u * 1024u;
 
 template <int UW>
-__global__ void __launch_bounds__(256, UW <= 2 ? 2 : 1) latent_tiles_kernel(LatArgs a, uint32_t stages) {
+__global__ void __launch_bounds__(256, 2) latent_tiles_kernel(LatArgs a, uint32_t stages) {
     using namespace attn_mma;
+    constexpr int LT = LatTile<UW>::TOKENS, SC_PITCH = LatTile<UW>::PITCH, P_PITCH = SC_PITCH, TPL = LT / 32;
     extern __shared__ __align__(128) unsigned char lt_smem[];
     float* sc = reinterpret_cast<float*>(lt_smem);                              // [8][16][SC_PITCH]
     __half* sp = reinterpret_cast<__half*>(sc + 8 * 16 * SC_PITCH);             // [16][P_PITCH]
     float* scorr = reinterpret_cast<float*>(sp + 16 * P_PITCH);                 // [16]
-    __half* ring = reinterpret_cast<__half*>(lt_smem + (LT_FIXED + 127) / 128 * 128);
+    __half* ring = reinterpret_cast<__half*>(lt_smem + LatTile<UW>::FIXED);
     pdl_wait();
     pdl_trigger();
     const uint32_t split = blockIdx.x, h0 = blockIdx.y * 16u, row = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
@@ -284,15 +301,15 @@ __global__ void __launch_bounds__(256, UW <= 2 ? 2 : 1) latent_tiles_kernel(LatA
         cp_async_commit();
         const __half* tc = ring + (size_t)(tile % stages) * LT * pitch;
         if (warp < busy) {
-            float s[8][4];
+            float s[LT / 8][4];
 #pragma unroll
-            for (int j = 0; j < 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.0f;
+            for (int j = 0; j < LT / 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.0f;
 #pragma unroll
             for (int i = 0; i < UW; ++i) {
                 const uint32_t u = warp * UW + i;
                 if (u >= NU) break;
 #pragma unroll
-                for (int p = 0; p < 4; ++p) {
+                for (int p = 0; p < LT / 16; ++p) {
                     const uint32_t r = p * 16 + (jm >> 1) * 8 + (lane & 7u);
                     uint32_t b[4];
                     ldmatrix_x4(b, tc + r * pitch + u * 16u + (jm & 1u) * 8u);
@@ -304,7 +321,7 @@ __global__ void __launch_bounds__(256, UW <= 2 ? 2 : 1) latent_tiles_kernel(LatA
             }
             float* mine = sc + (size_t)warp * 16 * SC_PITCH;
 #pragma unroll
-            for (int j = 0; j < 8; ++j) {
+            for (int j = 0; j < LT / 8; ++j) {
                 *reinterpret_cast<float2*>(mine + g * SC_PITCH + j * 8 + 2 * t4) = make_float2(s[j][0], s[j][1]);
                 *reinterpret_cast<float2*>(mine + (g + 8) * SC_PITCH + j * 8 + 2 * t4) = make_float2(s[j][2], s[j][3]);
             }
@@ -313,20 +330,28 @@ __global__ void __launch_bounds__(256, UW <= 2 ? 2 : 1) latent_tiles_kernel(LatA
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
             const uint32_t h = 2u * warp + e;
-            float v0 = 0.0f, v1 = 0.0f;
-            for (uint32_t w = 0; w < busy; ++w) {
-                v0 += sc[((size_t)w * 16 + h) * SC_PITCH + lane];
-                v1 += sc[((size_t)w * 16 + h) * SC_PITCH + lane + 32u];
+            float v[TPL] = {}, mx = -INFINITY, ps = 0.0f;
+#pragma unroll
+            for (uint32_t w = 0; w < 8u; ++w)
+                if (w < busy) {
+#pragma unroll
+                    for (int j = 0; j < TPL; ++j) v[j] += sc[((size_t)w * 16 + h) * SC_PITCH + lane + 32u * j];
+                }
+#pragma unroll
+            for (int j = 0; j < TPL; ++j) {
+                if (lo + tile * LT + lane + 32u * j >= hi) v[j] = -INFINITY;
+                mx = fmaxf(mx, v[j]);
             }
-            const uint32_t t = lo + tile * LT + lane;
-            if (t >= hi) v0 = -INFINITY;
-            if (t + 32u >= hi) v1 = -INFINITY;
-            const float m_new = fmaxf(m_run[e], warp_max(fmaxf(v0, v1)));  // the tile's first token is visible: finite
-            const float corr = fast_exp2(m_run[e] - m_new), p0 = fast_exp2(v0 - m_new), p1 = fast_exp2(v1 - m_new);
-            l_run[e] = l_run[e] * corr + warp_sum(p0 + p1);
+            const float m_new = fmaxf(m_run[e], warp_max(mx));  // the tile's first token is visible: finite
+            const float corr = fast_exp2(m_run[e] - m_new);
+#pragma unroll
+            for (int j = 0; j < TPL; ++j) {
+                const float p = fast_exp2(v[j] - m_new);
+                ps += p;
+                sp[h * P_PITCH + lane + 32u * j] = __float2half_rn(p);
+            }
+            l_run[e] = l_run[e] * corr + warp_sum(ps);
             m_run[e] = m_new;
-            sp[h * P_PITCH + lane] = __float2half_rn(p0);
-            sp[h * P_PITCH + lane + 32u] = __float2half_rn(p1);
             if (lane == 0) scorr[h] = corr;
         }
         __syncthreads();
@@ -337,7 +362,7 @@ __global__ void __launch_bounds__(256, UW <= 2 ? 2 : 1) latent_tiles_kernel(LatA
 #pragma unroll
                 for (int n = 0; n < 2; ++n) o[i][n][0] *= ca, o[i][n][1] *= ca, o[i][n][2] *= cb, o[i][n][3] *= cb;
 #pragma unroll
-            for (int kk = 0; kk < 4; ++kk) {
+            for (int kk = 0; kk < LT / 16; ++kk) {
                 uint32_t pa[4];
                 ldmatrix_x4(pa, sp + (lane & 15u) * P_PITCH + kk * 16 + (lane >> 4) * 8u);
                 const uint32_t r = kk * 16 + (jm & 1u) * 8 + (lane & 7u);
@@ -397,15 +422,23 @@ __global__ void __launch_bounds__(256) latent_split_kernel(const __half* __restr
     }
 }
 
-// grid (heads, row groups of RG, slices of the values): splits and sink -> the head's weighted latent, then uv.
+// grid (heads, row groups of RG, slices of the values): splits and sink -> the head's weighted latent, then uv. Every slice
+// merges for itself: the partials are in L2.
 template <typename WT, int RG>
 __global__ void __launch_bounds__(256) latent_merge_kernel(LatArgs a) {
-    extern __shared__ __align__(16) float so[];  // [RG][rank padded to 4], then [RG][splits] weights
+    extern __shared__ __align__(16) float so[];  // [RG][rank padded to 8], [RG][splits] weights, [256][RG] float4
+    const uint32_t head = blockIdx.x, row0 = blockIdx.y * RG, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
+    const uint32_t rp = (a.rank + 7u) & ~7u, live = min((uint32_t)RG, a.rows - row0);
+    float* sw = so + RG * rp;
+    const uint32_t per = (a.vdim + gridDim.z - 1u) / gridDim.z, n_lo = blockIdx.z * per, n_hi = min(n_lo + per, a.vdim);
+    const WT* uv = reinterpret_cast<const WT*>(a.uv) + (size_t)head * a.vdim * a.rank;
+    if (n_lo < n_hi) {  // the weights do not depend on the previous kernel
+        const char* p = reinterpret_cast<const char*>(uv + (size_t)n_lo * a.rank);
+        const size_t bytes = (size_t)(n_hi - n_lo) * a.rank * sizeof(WT);
+        for (size_t i = (size_t)tid * 128u; i < bytes; i += 256u * 128u) prefetch_l2(p + i);
+    }
     pdl_wait();
     pdl_trigger();
-    const uint32_t head = blockIdx.x, row0 = blockIdx.y * RG, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
-    const uint32_t rp = (a.rank + 3u) & ~3u, live = min((uint32_t)RG, a.rows - row0);
-    float* sw = so + RG * rp;
     if (warp < RG && warp < live) {  // one warp per row: the splits' weights
         const size_t base = ((size_t)(row0 + warp) * a.heads + head) * a.splits;
         const float sink = a.sink ? a.sink[head] : -INFINITY;
@@ -425,64 +458,119 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(LatArgs a) {
         for (uint32_t s = lane; s < a.splits; s += 32u) sw[warp * a.splits + s] *= inv;
     }
     __syncthreads();
-    for (uint32_t i = tid; i < RG * rp; i += 256u) {
-        const uint32_t r = i / rp, c = i % rp;
-        float t = 0.0f;
-        if (r < live && c < a.rank) {
-            const float* w = sw + r * a.splits;
-            const float* o = a.po + ((size_t)(row0 + r) * a.heads + head) * a.splits * a.rank + c;
+    // where column k of the weighted latent lies: the halves of every 8 columns apart, so that 16-byte reads of neighbouring
+    // lanes fall into different banks
+    auto place = [&](uint32_t k) { return ((k & 4u) ? rp / 2u : 0u) + (k >> 3) * 4u + (k & 3u); };
+    if (a.rank % 4u == 0u) {
+        const uint32_t c4 = a.rank / 4u, teams = 256u / c4 ? 256u / c4 : 1u, team = tid / c4, col = tid % c4;  // rank <= 1024
+        float4* st = reinterpret_cast<float4*>(sw + ((RG * a.splits + 3u) & ~3u));
+        float4 acc[RG];
+#pragma unroll
+        for (int r = 0; r < RG; ++r) {
+            acc[r] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (team < teams && (uint32_t)r < live) {
+                const float* w = sw + r * a.splits;
+                const float4* o = reinterpret_cast<const float4*>(a.po + ((size_t)(row0 + r) * a.heads + head) * a.splits * a.rank) + col;
 #pragma unroll 8
-            for (uint32_t s = 0; s < a.splits; ++s) {
-                const float ws = w[s], x = ws != 0.0f ? o[(size_t)s * a.rank] : 0.0f;  // empty splits may hold anything
-                t = fmaf(ws, x, t);
+                for (uint32_t s = team; s < a.splits; s += teams) {
+                    const float ws = w[s];
+                    const float4 x = o[(size_t)s * c4];
+                    if (ws != 0.0f) {  // empty splits may hold anything
+                        acc[r].x = fmaf(ws, x.x, acc[r].x), acc[r].y = fmaf(ws, x.y, acc[r].y);
+                        acc[r].z = fmaf(ws, x.z, acc[r].z), acc[r].w = fmaf(ws, x.w, acc[r].w);
+                    }
+                }
             }
+            st[tid * RG + r] = acc[r];
         }
-        so[i] = t;
+        __syncthreads();
+        for (uint32_t i = tid; i < RG * c4; i += 256u) {
+            const uint32_t r = i / c4, c = i % c4;
+            float4 t = st[c * RG + r];
+            for (uint32_t k = 1; k < teams; ++k) {
+                const float4 u = st[(k * c4 + c) * RG + r];
+                t.x += u.x, t.y += u.y, t.z += u.z, t.w += u.w;
+            }
+            *reinterpret_cast<float4*>(so + r * rp + place(4u * c)) = t;
+        }
+    } else {
+        for (uint32_t i = tid; i < RG * rp; i += 256u) {
+            const uint32_t r = i / rp, c = i % rp;
+            float t = 0.0f;
+            if (r < live && c < a.rank) {
+                const float* w = sw + r * a.splits;
+                const float* o = a.po + ((size_t)(row0 + r) * a.heads + head) * a.splits * a.rank + c;
+                for (uint32_t s = 0; s < a.splits; ++s) {
+                    const float ws = w[s], x = ws != 0.0f ? o[(size_t)s * a.rank] : 0.0f;
+                    t = fmaf(ws, x, t);
+                }
+            }
+            so[r * rp + place(c)] = t;
+        }
     }
     __syncthreads();
-    const uint32_t per = (a.vdim + gridDim.z - 1u) / gridDim.z, n1 = min((blockIdx.z + 1u) * per, a.vdim);
-    const WT* uv = reinterpret_cast<const WT*>(a.uv) + (size_t)head * a.vdim * a.rank;
-#pragma unroll 2
-    for (uint32_t n = blockIdx.z * per + warp; n < n1; n += 8u) {
-        const WT* w = uv + (size_t)n * a.rank;
-        float acc[RG] = {};
+    for (uint32_t n0 = n_lo + 2u * warp; n0 < n_hi; n0 += 16u) {  // two values at a time
+        const uint32_t n1 = min(n0 + 1u, n_hi - 1u);
+        const WT *w0 = uv + (size_t)n0 * a.rank, *w1 = uv + (size_t)n1 * a.rank;
+        float acc[2][RG] = {};
         if (a.wide) {
 #pragma unroll 2
             for (uint32_t k = lane * 8u; k < a.rank; k += 256u) {
-                float wv[8];
-                m40_load8(w + k, wv);
+                float v0[8], v1[8];
+                m40_load8(w0 + k, v0);
+                m40_load8(w1 + k, v1);
 #pragma unroll
-                for (int r = 0; r < RG; ++r)
+                for (int r = 0; r < RG; ++r) {
+                    const float4 x0 = *reinterpret_cast<const float4*>(so + r * rp + (k >> 1));
+                    const float4 x1 = *reinterpret_cast<const float4*>(so + r * rp + rp / 2u + (k >> 1));
+                    const float x[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
 #pragma unroll
-                    for (int i = 0; i < 8; ++i) acc[r] = fmaf(wv[i], so[r * rp + k + i], acc[r]);
+                    for (int i = 0; i < 8; ++i) acc[0][r] = fmaf(v0[i], x[i], acc[0][r]), acc[1][r] = fmaf(v1[i], x[i], acc[1][r]);
+                }
             }
         } else {
-            for (uint32_t k = lane; k < a.rank; k += 32u)
+            for (uint32_t k = lane; k < a.rank; k += 32u) {
+                const float v0 = m40_load_elem(w0 + k), v1 = m40_load_elem(w1 + k);
 #pragma unroll
-                for (int r = 0; r < RG; ++r) acc[r] = fmaf(m40_load_elem(w + k), so[r * rp + k], acc[r]);
+                for (int r = 0; r < RG; ++r) {
+                    const float x = so[r * rp + place(k)];
+                    acc[0][r] = fmaf(v0, x, acc[0][r]), acc[1][r] = fmaf(v1, x, acc[1][r]);
+                }
+            }
         }
 #pragma unroll
-        for (int r = 0; r < RG; ++r) {
-            const float v = warp_sum(acc[r]);
-            if (lane == 0 && (uint32_t)r < live) a.out[((size_t)(row0 + r) * a.heads + head) * a.vdim + n] = v;
-        }
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int r = 0; r < RG; ++r) {
+                const float v = warp_sum(acc[j][r]);
+                if (lane == 0 && (uint32_t)r < live && n0 + j < n_hi) a.out[((size_t)(row0 + r) * a.heads + head) * a.vdim + n0 + j] = v;
+            }
     }
+}
+
+// Rows per prepare CTA: 8 when there are several (their queries fit shared memory), and the latent columns that go with it.
+uint32_t prepare_rows(const LatArgs& a) { return a.rows > 1 && a.dim <= 256 ? 8u : 1u; }
+uint32_t absorb_ctas(const LatArgs& a) {
+    const uint32_t cols = prepare_rows(a) == 8 ? 128u : 64u;
+    return a.heads * ((a.rank + cols - 1) / cols);
 }
 
 template <typename WT, typename ET>
 cudaError_t launch_prepare(cudaStream_t s, const LatArgs& a, bool append) {
-    const uint32_t x = a.absorb_ctas + (append ? 1u : 0u);
-    if (a.rows == 1) return m40_launch_dependent(latent_prepare_kernel<WT, ET, 1>, dim3(x, 1), dim3(256), a.dim * sizeof(float), s, a);
-    return m40_launch_dependent(latent_prepare_kernel<WT, ET, 4>, dim3(x, (a.rows + 3) / 4), dim3(256), 4 * a.dim * sizeof(float), s, a);
+    const uint32_t rg = prepare_rows(a);
+    const dim3 grid(a.absorb_ctas + (append ? rg : 0u), (a.rows + rg - 1) / rg);
+    const size_t smem = (size_t)rg * a.dim * sizeof(float);
+    return rg == 8 ? m40_launch_dependent(latent_prepare_kernel<WT, ET, 8, 128>, grid, dim3(256), smem, s, a)
+                   : m40_launch_dependent(latent_prepare_kernel<WT, ET, 1, 64>, grid, dim3(256), smem, s, a);
 }
 
 template <typename WT>
 cudaError_t launch_merge(M40llmCudaContext* ctx, const LatArgs& a) {
-    const uint32_t rp = (a.rank + 3u) & ~3u, rg = a.rows == 1 ? 1u : 4u, groups = (a.rows + rg - 1) / rg;
+    const uint32_t rp = (a.rank + 7u) & ~7u, rg = a.rows == 1 ? 1u : 4u, groups = (a.rows + rg - 1) / rg;
     uint32_t z = (uint32_t)ctx->sm_count / (a.heads * groups);
     const uint32_t z_max = (a.vdim + 15u) / 16u;
     z = z < 1u ? 1u : (z > z_max ? z_max : z);
-    const size_t smem = (size_t)rg * (rp + a.splits) * sizeof(float);
+    const size_t smem = ((size_t)rg * rp + (((size_t)rg * a.splits + 3) & ~(size_t)3) + (size_t)256 * 4 * rg) * sizeof(float);
     const dim3 grid(a.heads, groups, z);
     return rg == 1 ? m40_launch_dependent(latent_merge_kernel<WT, 1>, grid, dim3(256), smem, ctx->decode_stream, a)
                    : m40_launch_dependent(latent_merge_kernel<WT, 4>, grid, dim3(256), smem, ctx->decode_stream, a);
@@ -497,26 +585,36 @@ template <int UW>
 cudaError_t launch_tiles(M40llmCudaContext* ctx, const LatArgs& a) {
     static unsigned long long configured = 0ull;
     const unsigned long long bit = 1ull << (ctx->device_id & 63);
-    constexpr size_t fixed = (LT_FIXED + 127) / 128 * 128, budget = UW <= 2 ? 112u * 1024u : 200u * 1024u;
     if (!(configured & bit)) {
-        const cudaError_t e = cudaFuncSetAttribute(latent_tiles_kernel<UW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)budget);
+        const cudaError_t e = cudaFuncSetAttribute(latent_tiles_kernel<UW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TILE_SMEM);
         if (e != cudaSuccess) return e;
         configured |= bit;
     }
-    size_t stages = (budget - fixed) / latent_tile_bytes(a.rank);
+    size_t stages = (TILE_SMEM - LatTile<UW>::FIXED) / LatTile<UW>::bytes(a.rank);
     if (stages > 4) stages = 4;
     const dim3 grid(a.splits, (a.heads + 15) / 16, a.rows);
-    return m40_launch_dependent(latent_tiles_kernel<UW>, grid, dim3(256), fixed + stages * latent_tile_bytes(a.rank),
+    return m40_launch_dependent(latent_tiles_kernel<UW>, grid, dim3(256), LatTile<UW>::FIXED + stages * LatTile<UW>::bytes(a.rank),
                                 ctx->decode_stream, a, (uint32_t)stages);
 }
-static_assert((LT_FIXED + 127) / 128 * 128 + 2 * latent_tile_bytes(256) <= 112u * 1024u, "two tiles of rank 256, two CTAs per SM");
-static_assert((LT_FIXED + 127) / 128 * 128 + 2 * latent_tile_bytes(512) <= 200u * 1024u, "two tiles of rank 512");
+static_assert(LatTile<2>::FIXED + 2 * LatTile<2>::bytes(256) <= TILE_SMEM && LatTile<4>::FIXED + 2 * LatTile<4>::bytes(512) <= TILE_SMEM,
+              "two tiles of the largest rank");
+
+// Tokens per split: as many splits as keep every CTA of the launch resident (two per SM), at least 128 tokens each; at most
+// 1024, because the bound may be the cache's capacity when the lengths are not known.
+void pick_splits(const M40llmCudaContext* ctx, uint32_t ctas_per_split, uint32_t bound, uint32_t* chunk, uint32_t* splits) {
+    uint32_t n = 2u * (uint32_t)ctx->sm_count / ctas_per_split;
+    n = n < 1u ? 1u : (n > 128u ? 128u : n);
+    uint32_t c = ((bound + n - 1) / n + 63u) & ~63u;
+    c = c < 128u ? 128u : (c > 1024u ? 1024u : c);
+    if ((bound + c - 1) / c > 128u) c = ((bound + 127u) / 128u + 63u) & ~63u;
+    *chunk = c;
+    *splits = (bound + c - 1) / c;
+}
 
 // Absorbed form over the rows of `all`; append: the latents are not in the cache yet.
 template <typename WT>
 int run_absorbed(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs& all, uint32_t bound, bool append) {
     cudaStream_t s = ctx->decode_stream;
-    const uint32_t slices = (all.rank + COLS - 1) / COLS;
     const bool tiles = !kv->elem_f32 && all.rank % 16 == 0 && all.rank <= 512;
     cudaError_t e;
     for (uint32_t at = 0; at < all.rows; at += RUN_ROWS) {
@@ -526,7 +624,7 @@ int run_absorbed(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs&
         a.out += (size_t)at * a.heads * a.vdim;
         a.row_seq += at;
         a.row_pos += at;
-        m40_attn_pick_chunk(ctx, a.rows, tiles ? (a.heads + 15) / 16 : a.heads, bound, &a.chunk, &a.splits);
+        pick_splits(ctx, a.rows * (tiles ? (a.heads + 15) / 16 : a.heads), bound, &a.chunk, &a.splits);
         const size_t nh = (size_t)a.rows * a.heads, np = nh * a.splits;
         auto pad = [](size_t v) { return (v + 3) & ~(size_t)3; };
         float* work = (float*)m40_ensure_scratch(ctx, 1, (pad(nh * a.rank) + pad(np * a.rank) + 2 * np) * sizeof(float), 1);
@@ -535,7 +633,7 @@ int run_absorbed(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs&
         a.po = work + pad(nh * a.rank);
         a.pm = a.po + pad(np * a.rank);
         a.pl = a.pm + np;
-        a.absorb_ctas = a.heads * slices;
+        a.absorb_ctas = absorb_ctas(a);
         e = prepare<WT>(s, a, kv->elem_f32, append);
         M40_COUNT_LAUNCH(ctx);
         if (e != cudaSuccess) return -6;

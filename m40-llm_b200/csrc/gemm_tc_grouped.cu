@@ -186,6 +186,19 @@ __global__ void __launch_bounds__(192, 1) gemm_tc_grouped_kernel(const __grid_co
                 sums(c, v);
 #pragma unroll
                 for (int j = 0; j < 8; ++j) u[j] = g.u[(size_t)(m_base + min(c + j, m_live - 1u)) * g.width + chan];
+                if (g.step) {
+                    M40RgStep st[8];
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) st[j] = m40_rg_fetch(g, m_base + min(c + j, m_live - 1u), chan);
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) {
+                        if (!n_ok || c + j >= m_live) continue;
+                        const float o = xs[(c + j) * 64u + ch];
+                        m40_rg_store(g, m_base + c + j, chan, st[j],
+                                     m40_rg_gated(g, (is_i ? o : v[j]) + rb, (is_i ? v[j] : o) + ib, sp, u[j]));
+                    }
+                    continue;
+                }
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
                     if (!n_ok || c + j >= m_live) continue;

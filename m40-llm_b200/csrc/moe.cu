@@ -6,9 +6,10 @@
 //                      are read once), the exact mode and the shapes the tensor path does not take;
 //   tensor path          moe_sort_kernel deals the chosen slots to experts (rows sorted by expert, each expert's share padded to
 //                      whole tiles) and writes the tile table, moe_scatter_kernel copies the rows there as hi + lo, two grouped
-//                      GEMMs (gemm_tc_grouped.cu; act and the next split in the first one's epilogue), moe_gather_kernel adds a
-//                      row's slots up. No host round trip: the table and its length stay on the device;
-//   then post norm and residual (norm_rows.cu).
+//                      GEMMs (gemm_tc_grouped.cu; act and the next split in the first one's epilogue). No host round trip: the table
+//                      and its length stay on the device;
+//   then post norm and residual (norm_rows.cu), after the tensor path together with adding a row's slots up (or, for shapes
+//   that pass does not take, after moe_gather_kernel).
 #include "moe.cuh"
 
 #include "gemm_tc_grouped.cuh"
@@ -288,7 +289,8 @@ uint32_t pick_tile_rows(uint32_t slots, uint32_t experts) {
     return avg <= 16 ? 16 : (avg <= 32 ? 32 : (avg <= 96 ? 64 : 128));
 }
 
-int run_tensor(M40llmCudaContext* ctx, cudaStream_t s, const M40MoeArgs& a, uint32_t max_tiles) {
+// `after`: the norm of these rows.
+int run_tensor(M40llmCudaContext* ctx, cudaStream_t s, const M40MoeArgs& a, uint32_t max_tiles, M40NormRows after) {
     cudaError_t e = m40_launch_dependent(moe_sort_kernel, dim3(1), dim3(1024), a.experts * sizeof(uint32_t), s, a);
     M40_COUNT_LAUNCH(ctx);
     if (e != cudaSuccess) return -6;
@@ -321,9 +323,14 @@ int run_tensor(M40llmCudaContext* ctx, cudaStream_t s, const M40MoeArgs& a, uint
     c.kind = M40_GROUPED_F32;
     c.out = a.ys;
     if ((rc = m40_gemm_tc_grouped(ctx, s, c)) != 0) return rc;
+    after.x = a.add;
+    const M40NormGather y = {a.ys, a.x, a.weights, a.ids, a.place, a.top, a.experts};
+    if (m40_norm_gather_rows_takes(after, y)) return m40_norm_gather_rows(ctx, s, after, y);
     e = m40_launch_dependent(moe_gather_kernel, dim3((a.K + 1023) / 1024, a.rows), dim3(256), 0, s, a);
     M40_COUNT_LAUNCH(ctx);
-    return e == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -6;
+    if (e != cudaSuccess || cudaGetLastError() != cudaSuccess) return -6;
+    after.x = a.y;
+    return m40_norm_rows(ctx, s, after);
 }
 
 template <typename WT>
@@ -426,11 +433,17 @@ extern "C" int m40llm_moe_async(M40llmCudaContext* ctx, const M40llmMoe* c, uint
         p.y += (size_t)at * c->K;
         p.ids += (size_t)at * c->top;
         p.weights += (size_t)at * c->top;
-        const int rc = tensor ? run_tensor(ctx, s, p, max_tiles)
-                       : c->w_dtype == M40LLM_DT_F32 ? run_rows<float>(ctx, s, p)
+        const M40NormRows after = {p.y, (float*)c->out + (size_t)at * c->K, c->residual ? (const float*)c->residual + (size_t)at * c->K : nullptr,
+                             c->post, p.rows, c->K, c->K, 0.0f};
+        if (tensor) {
+            const int rc = run_tensor(ctx, s, p, max_tiles, after);
+            if (rc != 0) return rc;
+            continue;
+        }
+        int rc = c->w_dtype == M40LLM_DT_F32 ? run_rows<float>(ctx, s, p)
                        : c->w_dtype == M40LLM_DT_BF16 ? run_rows<__nv_bfloat16>(ctx, s, p) : run_rows<__half>(ctx, s, p);
+        if (rc == 0) rc = m40_norm_rows(ctx, s, after);
         if (rc != 0) return rc;
     }
-    const M40NormRows after = {a.y, (float*)c->out, (const float*)c->residual, c->post, c->rows, c->K, c->K, 0.0f};
-    return m40_norm_rows(ctx, s, after);
+    return 0;
 }

@@ -11,5 +11,19 @@ struct M40NormRows {
     uint32_t rows, K, ldx;
     float soft_cap;
 };
+// The normed value is x[r] (may be null: zeros) plus a weighted sum of `slots` rows of K values: slot j of row r adds
+// weights[r][j] times row place[r][j] of `values`, or times row r of `x` when ids[r][j] >= experts.
+constexpr uint32_t M40_NORM_SLOTS = 32;
+struct M40NormGather {
+    const float* values;
+    const float* x;
+    const float* weights;
+    const uint32_t* ids;
+    const uint32_t* place;
+    uint32_t slots, experts;
+};
+bool m40_norm_gather_rows_takes(const M40NormRows& a, const M40NormGather& y);
+int m40_norm_gather_rows(M40llmCudaContext* ctx, cudaStream_t s, const M40NormRows& a, const M40NormGather& y);
+
 bool m40_norm_valid(const M40llmNorm& n, uint32_t K);
 int m40_norm_rows(M40llmCudaContext* ctx, cudaStream_t s, const M40NormRows& a);

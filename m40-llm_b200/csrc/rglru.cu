@@ -2,14 +2,15 @@
 //
 //   S <- a S + sqrt(1 - a^2) i u,  log a = -decay r softplus(lam),  r, i = sigmoid of block-diagonal maps of u.
 //
-//   rglru_decode_kernel   one token per sequence: CTA = (32 channels of a block, up to RG rows) does the convolution, the
-//                         gates, the state and the output gate in one launch; a weight row is read once per RG rows.
-//   portions:
+//   rglru_decode_kernel   one token: CTA = 32 channels of a block does the convolution, the gates, the state and the output
+//                         gate in one launch.
+//   several rows:
 //     short convolution   u (short_conv.cu);
 //     gates               a and b = sqrt(1 - a^2) i u per (row, channel). The block-diagonal products run on the tensor cores
 //                         (gemm_tc_grouped.cu) with u cut into three bf16 parts, whose sum is the f32 value and whose products
 //                         with bf16 weights are exact in f32, or on f32 multiply-adds: 32-bit arithmetic either way;
-//     rglru_scan_kernel   CTA = (32 channels, segment), a warp per piece of the portion: every piece is folded into one
+//     one token per sequence: the gates' epilogue makes the step and the output;
+//     portions: rglru_scan_kernel, CTA = (32 channels, segment), a warp per piece of the portion: every piece is folded into one
 //                         (product of a, sum) pair, the pairs are chained from the slot's state, and the pieces are walked
 //                         again from their starting states.
 // 1 - a^2 is taken as -expm1(2 log a), which keeps its accuracy when a is close to one.
@@ -24,13 +25,13 @@ constexpr uint32_t SLICE = 32;  // output channels per decode CTA
 
 using RgArgs = M40RgArgs;
 
-template <typename WT, int RG>
+template <typename WT>
 __global__ void __launch_bounds__(256) rglru_decode_kernel(RgArgs g) {
-    extern __shared__ __align__(16) float su[];  // [RG][bs padded to 8]
-    __shared__ float sz[2][RG][SLICE];
+    extern __shared__ __align__(16) float su[];  // [bs padded to 8]
+    __shared__ float sz[2][SLICE];
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
     const uint32_t slices = (g.bs + SLICE - 1u) / SLICE, blk = blockIdx.x / slices, o0 = (blockIdx.x % slices) * SLICE;
-    const uint32_t row0 = blockIdx.y * RG, bsp = (g.bs + 7u) & ~7u;
+    const uint32_t bsp = (g.bs + 7u) & ~7u;
     const WT* ra = reinterpret_cast<const WT*>(g.ra) + (size_t)blk * g.bs * g.bs;
     const WT* ri = reinterpret_cast<const WT*>(g.ri) + (size_t)blk * g.bs * g.bs;
     // this warp's first weight pieces do not depend on the previous kernel
@@ -47,43 +48,34 @@ __global__ void __launch_bounds__(256) rglru_decode_kernel(RgArgs g) {
     }
     pdl_wait();
     pdl_trigger();
-    // the finishing thread's inputs: row row0 + warp, channel o0 + lane of the block
-    const uint32_t frow = row0 + warp, fo = o0 + lane, fc = blk * g.bs + fo;
-    const bool live_row = warp < RG && frow < g.rows;
-    uint32_t fslot = 0, fpos = 0;
-    bool ok = false;
-    float s_old = 0.0f, fy = 0.0f, fx = 0.0f;
-    if (live_row) {
-        fslot = g.row_seq[frow] * g.slot_mul + g.slot_add;
-        fpos = g.row_pos[frow];
-        ok = fslot < g.slots;
-        if (!ok && lane == 0 && blockIdx.x == 0) atomicOr(g.status, 2u);
-        if (ok && fo < g.bs) {
-            if (fpos > 0) s_old = g.state[fslot * g.slot_stride + fc];
-            fy = g.packed[(size_t)frow * g.ld + fc];
-            fx = g.packed[(size_t)frow * g.ld + g.width + fc];
-        }
+    const uint32_t slot = g.row_seq[0] * g.slot_mul + g.slot_add, pos = g.row_pos[0];
+    const bool ok = slot < g.slots;
+    // the finishing warp's inputs
+    const uint32_t fo = o0 + lane, fc = blk * g.bs + fo;
+    const bool mine = warp == 0 && fo < g.bs;
+    M40RgStep step = {0.0f, 0.0f, ~(size_t)0};
+    float fx = 0.0f;
+    if (mine) {
+        step = m40_rg_fetch(g, 0, fc);
+        fx = g.packed[g.width + fc];
     }
-    // u of the whole block for every row
-    for (uint32_t i = tid; i < RG * bsp; i += 256u) {
-        const uint32_t r = i / bsp, ch = i % bsp, row = row0 + r;
+    // u of the whole block
+    for (uint32_t ch = tid; ch < bsp; ch += 256u) {
         float y = 0.0f;
-        if (ch < g.bs && row < g.rows) {
-            const uint32_t c = blk * g.bs + ch, slot = g.row_seq[row] * g.slot_mul + g.slot_add, pos = g.row_pos[row];
-            if (slot < g.slots) {
-                const float* w = g.conv_w + (size_t)c * g.taps;
-                const float* ring = g.state + slot * g.slot_stride + g.width + c;
-                y = g.conv_b ? g.conv_b[c] : 0.0f;
+        if (ch < g.bs && ok) {
+            const uint32_t c = blk * g.bs + ch;
+            const float* w = g.conv_w + (size_t)c * g.taps;
+            const float* ring = g.state + slot * g.slot_stride + g.width + c;
+            y = g.conv_b ? g.conv_b[c] : 0.0f;
 #pragma unroll 4
-                for (uint32_t back = g.taps - 1u; back > 0u; --back)
-                    if (back <= pos) y = fmaf(w[g.taps - 1u - back], ring[(size_t)((pos - back) % g.taps) * g.width], y);
-                y = fmaf(w[g.taps - 1u], g.packed[(size_t)row * g.ld + g.width + c], y);
-            }
+            for (uint32_t back = g.taps - 1u; back > 0u; --back)
+                if (back <= pos) y = fmaf(w[g.taps - 1u - back], ring[(size_t)((pos - back) % g.taps) * g.width], y);
+            y = fmaf(w[g.taps - 1u], g.packed[g.width + c], y);
         }
-        su[i] = y;
+        su[ch] = y;
     }
     __syncthreads();
-    float ar[PER][RG] = {}, ai[PER][RG] = {};
+    float ar[PER] = {}, ai[PER] = {};
     if (g.wide) {
         for (uint32_t k = lane * 8u; k < g.bs; k += 256u) {
             if (k >= 256u) {
@@ -94,54 +86,32 @@ __global__ void __launch_bounds__(256) rglru_decode_kernel(RgArgs g) {
                     m40_load8(ri + (size_t)o * g.bs + k, wi[j]);
                 }
             }
+            const float4 x0 = *reinterpret_cast<const float4*>(su + k), x1 = *reinterpret_cast<const float4*>(su + k + 4);
+            const float x[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
 #pragma unroll
-            for (int r = 0; r < RG; ++r) {
-                const float4 x0 = *reinterpret_cast<const float4*>(su + r * bsp + k);
-                const float4 x1 = *reinterpret_cast<const float4*>(su + r * bsp + k + 4);
-                const float x[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
+            for (int j = 0; j < PER; ++j)
 #pragma unroll
-                for (int j = 0; j < PER; ++j)
-#pragma unroll
-                    for (int i = 0; i < 8; ++i) {
-                        ar[j][r] = fmaf(wr[j][i], x[i], ar[j][r]);
-                        ai[j][r] = fmaf(wi[j][i], x[i], ai[j][r]);
-                    }
-            }
+                for (int i = 0; i < 8; ++i) ar[j] = fmaf(wr[j][i], x[i], ar[j]), ai[j] = fmaf(wi[j][i], x[i], ai[j]);
         }
     } else {
         for (uint32_t k = lane; k < g.bs; k += 32u)
 #pragma unroll
             for (int j = 0; j < PER; ++j) {
                 const uint32_t o = min(ow + j, g.bs - 1u);
-                const float vr = m40_load_elem(ra + (size_t)o * g.bs + k), vi = m40_load_elem(ri + (size_t)o * g.bs + k);
-#pragma unroll
-                for (int r = 0; r < RG; ++r) {
-                    ar[j][r] = fmaf(vr, su[r * bsp + k], ar[j][r]);
-                    ai[j][r] = fmaf(vi, su[r * bsp + k], ai[j][r]);
-                }
+                ar[j] = fmaf(m40_load_elem(ra + (size_t)o * g.bs + k), su[k], ar[j]);
+                ai[j] = fmaf(m40_load_elem(ri + (size_t)o * g.bs + k), su[k], ai[j]);
             }
     }
 #pragma unroll
-    for (int j = 0; j < PER; ++j)
-#pragma unroll
-        for (int r = 0; r < RG; ++r) {
-            const float zr = warp_sum(ar[j][r]), zi = warp_sum(ai[j][r]);
-            if (lane == 0) sz[0][r][warp * PER + j] = zr, sz[1][r][warp * PER + j] = zi;
-        }
-    __syncthreads();
-    if (!live_row || fo >= g.bs) return;
-    float* out = g.out + (size_t)frow * g.width + fc;
-    if (!ok) {
-        *out = 0.0f;
-        return;
+    for (int j = 0; j < PER; ++j) {
+        const float zr = warp_sum(ar[j]), zi = warp_sum(ai[j]);
+        if (lane == 0) sz[0][warp * PER + j] = zr, sz[1][warp * PER + j] = zi;
     }
-    const float2 ab = m40_rg_gated(g, sz[0][warp][lane] + g.ra_b[fc], sz[1][warp][lane] + g.ri_b[fc], m40_softplus(g.lam[fc]),
-                                   su[warp * bsp + fo]);
-    const float s = fmaf(ab.x, s_old, ab.y);
-    float* st = g.state + fslot * g.slot_stride;
-    st[fc] = s;
-    if (g.taps > 1u) st[g.width + (size_t)(fpos % g.taps) * g.width + fc] = fx;
-    *out = s * m40_act((int)M40LLM_ACT_GELU_TANH, fy);
+    __syncthreads();
+    if (!mine) return;
+    m40_rg_store(g, 0, fc, step,
+                 m40_rg_gated(g, sz[0][lane] + g.ra_b[fc], sz[1][lane] + g.ri_b[fc], m40_softplus(g.lam[fc]), su[fo]));
+    if (ok && g.taps > 1u) g.state[slot * g.slot_stride + g.width + (size_t)(pos % g.taps) * g.width + fc] = fx;
 }
 
 // a and b of 64 rows x 64 channels of one block, f32 multiply-adds. A k tile is summed on its own before it joins the
@@ -196,6 +166,10 @@ __global__ void __launch_bounds__(256) rglru_gates_f32_kernel(RgArgs g) {
             if (m >= g.rows) continue;
             const size_t at = (size_t)m * g.width + c;
             const float2 ab = m40_rg_gated(g, ar[i][j] + rb, ai[i][j] + ib, sp, g.u[at]);
+            if (g.step) {
+                m40_rg_store(g, m, c, m40_rg_fetch(g, m, c), ab);
+                continue;
+            }
             g.a[at] = ab.x;
             g.b[at] = ab.y;
         }
@@ -272,21 +246,16 @@ __global__ void __launch_bounds__(1024) rglru_scan_kernel(RgArgs g) {
 }
 
 template <typename WT>
-int run_decode(M40llmCudaContext* ctx, const RgArgs& g, uint32_t blocks) {
+int run_one(M40llmCudaContext* ctx, const RgArgs& g, uint32_t blocks) {
     const uint32_t bsp = (g.bs + 7u) & ~7u, slices = (g.bs + SLICE - 1) / SLICE;
-    cudaError_t e;
-    if (g.rows == 1)
-        e = m40_launch_dependent(rglru_decode_kernel<WT, 1>, dim3(blocks * slices, 1), dim3(256), bsp * sizeof(float),
-                                 ctx->decode_stream, g);
-    else
-        e = m40_launch_dependent(rglru_decode_kernel<WT, 8>, dim3(blocks * slices, (g.rows + 7) / 8), dim3(256),
-                                 8 * bsp * sizeof(float), ctx->decode_stream, g);
+    const cudaError_t e =
+        m40_launch_dependent(rglru_decode_kernel<WT>, dim3(blocks * slices), dim3(256), bsp * sizeof(float), ctx->decode_stream, g);
     M40_COUNT_LAUNCH(ctx);
     return e == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -6;
 }
 
 template <typename WT>
-int run_portion(M40llmCudaContext* ctx, RgArgs g, uint32_t blocks, const M40llmStepRows& rows) {
+int run_rows(M40llmCudaContext* ctx, RgArgs g, uint32_t blocks, const M40llmStepRows& rows) {
     cudaStream_t s = ctx->decode_stream;
     const size_t n = ((size_t)g.rows * g.width + 3) & ~(size_t)3;
     const bool tensor = g.tensor && m40_gemm_tc_grouped_supported(g.ra, g.bs, g.bs, g.width, g.bs) &&
@@ -332,6 +301,7 @@ int run_portion(M40llmCudaContext* ctx, RgArgs g, uint32_t blocks, const M40llmS
         M40_COUNT_LAUNCH(ctx);
         if (e != cudaSuccess) return -6;
     }
+    if (g.step) return cudaGetLastError() == cudaSuccess ? 0 : -6;
     e = m40_launch_dependent(rglru_scan_kernel, dim3((g.width + 31) / 32, rows.segments), dim3(1024), 0, s, g);
     M40_COUNT_LAUNCH(ctx);
     return e == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : -6;
@@ -339,7 +309,7 @@ int run_portion(M40llmCudaContext* ctx, RgArgs g, uint32_t blocks, const M40llmS
 
 template <typename WT>
 int run(M40llmCudaContext* ctx, const RgArgs& g, uint32_t blocks, const M40llmStepRows& rows) {
-    return rows.max_segment_rows == 1 ? run_decode<WT>(ctx, g, blocks) : run_portion<WT>(ctx, g, blocks, rows);
+    return g.step && g.rows == 1 ? run_one<WT>(ctx, g, blocks) : run_rows<WT>(ctx, g, blocks, rows);
 }
 
 }  // namespace
@@ -377,6 +347,7 @@ extern "C" int m40llm_rglru_async(M40llmCudaContext* ctx, M40llmStateCache* stat
     g.slot_add = r->slot_add;
     g.slots = state->slots;
     g.rows = r->rows;
+    g.step = r->max_segment_rows == 1;
     g.decay = c->decay;
     g.wide = c->w_dtype != M40LLM_DT_F32 && g.bs % 8 == 0 && (((uintptr_t)c->ra | (uintptr_t)c->ri) & 15u) == 0;
     g.tensor = c->w_dtype == M40LLM_DT_BF16 && !c->exact;

@@ -22,10 +22,34 @@ struct M40RgArgs {
     const uint32_t* row_pos;
     const uint32_t* seg;
     uint32_t ld, width, bs, taps, slot_mul, slot_add, slots, rows, wide, tensor;
+    uint32_t step;       // every row is the next token of its own sequence: whoever has a and b makes the step
     float decay;
 };
 
 __device__ __forceinline__ float m40_softplus(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
+
+// What one row's channel needs from memory before its step: state (0 at a sequence's start) and output gate input.
+struct M40RgStep {
+    float s_old, y;
+    size_t slot;  // or ~0: not a valid row
+};
+__device__ __forceinline__ M40RgStep m40_rg_fetch(const M40RgArgs& g, uint32_t row, uint32_t c) {
+    M40RgStep t = {0.0f, 0.0f, g.row_seq[row] * g.slot_mul + g.slot_add};
+    if (t.slot >= g.slots) {
+        if (c == 0) atomicOr(g.status, 2u);
+        t.slot = ~(size_t)0;
+        return t;
+    }
+    if (g.row_pos[row] > 0) t.s_old = g.state[t.slot * g.slot_stride + c];
+    t.y = g.packed[(size_t)row * g.ld + c];
+    return t;
+}
+__device__ __forceinline__ void m40_rg_store(const M40RgArgs& g, uint32_t row, uint32_t c, const M40RgStep& t, const float2& ab) {
+    const float s = fmaf(ab.x, t.s_old, ab.y);
+    const bool ok = t.slot != ~(size_t)0;
+    if (ok) g.state[t.slot * g.slot_stride + c] = s;
+    g.out[(size_t)row * g.width + c] = ok ? s * m40_act((int)M40LLM_ACT_GELU_TANH, t.y) : 0.0f;
+}
 
 // gate sums (biases added) -> (a, sqrt(1 - a^2) i u); sp = softplus(lam)
 __device__ __forceinline__ float2 m40_rg_gated(const M40RgArgs& g, float zr, float zi, float sp, float u) {
