@@ -734,6 +734,9 @@ def _torch_stack_weights(pkg, nat, rank):
                 self._mat[names] = t.data_ptr()
             return self._mat[names]
 
+        def blocks_transposed(self, name, shape, blocks):
+            return self.matrix(name + " transposed", shapes=[(blocks * shape[1], shape[0] // blocks)])
+
         def vectors(self, names, sizes, total):
             return self.vector(names, total)
 
@@ -1002,12 +1005,13 @@ def sidalorn_ops_case(nat, ev, name, reps=20):
     bf = torch.bfloat16
     cases = ((T, [(0, 0, T)], "prompt 2048"), (1, [(0, 8191, 1)], "decode 1 x 8192"), (32, [(s, 2047, 1) for s in range(32)], "decode 32 x 2048"))
     # ---- latent attention beside rotary attention
-    cn, uk, uv, sink = dev(R), dev(H * D, R, dtype=bf, std=R ** -0.5), dev(H * D, R, dtype=bf, std=R ** -0.5), dev(H)
+    cn, sink = dev(R), dev(H)
+    uk, ukt, uv = (dev(*sh, dtype=bf, std=R ** -0.5) for sh in ((H * D, R), (H * R, D), (H * D, R)))
     for rows, segs, key in cases:
         max_len, tokens = (8192 if rows == 1 else 2048), sum(p0 + n for _, p0, n in segs)
         r, host = step_rows(segs)
         kv = L.m40llm_kvcache_create_typed(ctx, max_len, len(segs), 1, R, 0, N.DT_F16)
-        c = N.LatentAttention(dev(rows, H * D + R), cn, uk, uv, sink, dev(rows, H * D), H * D + R, H, D, D, N.DT_BF16, 1e-5, D ** -0.5)
+        c = N.LatentAttention(dev(rows, H * D + R), cn, uk, ukt, uv, sink, dev(rows, H * D), H * D + R, H, D, D, N.DT_BF16, 1e-5, D ** -0.5)
         ms = timed(lambda i: L.m40llm_attention_latent_async(ctx, kv, C.byref(c), C.byref(r)))
         if rows == T:   # scores and values, and making the heads' keys and values once
             put(f"latent attention, {key}", ms, 4.0 * D * H * T * (T + 1) / 2 + 4.0 * T * R * H * D)

@@ -676,11 +676,13 @@ int m40llm_rglru_async(M40llmCudaContext* ctx, M40llmStateCache* state, const M4
  *   out = sum_j p_j v_j, p = exp(scale * q . k_j) / (sum over positions 0 .. pos + exp(sink[head])); sink f32 or null.
  * out f32 [rows][heads * vdim]. The cache is m40llm_kvcache_create_typed with one head, k_dim = rank and v_dim = 0. Keys and
  * values of the heads are made only for long portions; otherwise uk meets the query and uv the weighted latents.
- * rank <= 1024. */
+ * uk_t: uk with every head's matrix transposed, [heads * rank][dim], or null: lets the queries of several rows meet uk on the
+ * tensor cores. rank <= 1024. */
 typedef struct {
     const void* packed;
     const void* c_norm;
     const void* uk;
+    const void* uk_t;
     const void* uv;
     const void* sink;
     void* out;

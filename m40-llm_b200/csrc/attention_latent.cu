@@ -3,12 +3,13 @@
 // A head's key and value are uk c and uv c of the cached latent c, so  q . k = (uk^T q) . c  and  sum p v = uv (sum p c):
 // with uk folded into the query every head attends the same rows c, which are key and value at once.
 //
-//   latent_prepare_kernel  uk^T q per head (absorbed query), and the latent's norm and append;
+//   latent_prepare_kernel  uk^T q per head (absorbed query), and the latent's norm and append; with several rows on the tensor
+//                          path latent_append_kernel (append, and the queries cut into hi + lo) and a grouped tcgen05 GEMM;
 //   attention over latents, one of
 //     latent_tiles_kernel  f16 cache, rank a multiple of 16 up to 512: CTA = (row, 16 heads, token split). The tokens' latents
 //                          stream once through shared memory and serve all 16 heads, as keys and as values;
 //     latent_rows_kernel   any rank, f16 or f32 cache, f32 arithmetic: CTA = (head, row, token split);
-//   latent_merge_kernel    merges the token splits and the sink, then uv.
+//   latent_merge_kernel    merges the token splits and the sink, then uv (itself, or as a grouped GEMM of several rows).
 // Long portions (segments of EXPAND_ROWS rows or more, f16 cache) do less work with the heads' keys and values in hand: they
 // are made once per portion from the cached latents by the grouped tcgen05 GEMM, f16 and head-major, and the prompt kernel of
 // attention_prefill.cu attends them.
@@ -22,15 +23,18 @@ namespace {
 constexpr uint32_t MAX_RANK = 1024;
 constexpr uint32_t RUN_ROWS = 512;   // rows per pass of the absorbed form (bounds the work space)
 constexpr uint32_t EXPAND_ROWS = 64;
+constexpr uint32_t GROUPED_ROWS = 8;    // rows from which uk and uv go through the grouped GEMM
 constexpr size_t EXPAND_BYTES = (size_t)1 << 30;  // work space for one portion's keys and values
 
 struct LatArgs {
     const float* packed;   // of the pass's first row
     const float* c_norm;
     const void* uk;
+    const void* uk_t;
     const void* uv;
     const float* sink;
     void* C;
+    __nv_bfloat16* part[2];  // tensor path: hi and lo of the queries [rows][heads * dim], then of the weighted latents
     uint32_t* seq_map;
     float* qa;             // absorbed queries [rows][heads][rank]
     float* pm;             // [rows][heads][splits]
@@ -56,6 +60,58 @@ __device__ __forceinline__ float block_sum_256(float v, float* red) {
     return t;
 }
 
+// Norm and append of one row's latent by the whole CTA.
+template <typename ET>
+__device__ __forceinline__ void append_row(const LatArgs& a, uint32_t row, float* red) {
+    const uint32_t tid = threadIdx.x, pos = a.row_pos[row], slot = a.row_seq[row] * a.slot_mul + a.slot_add;
+    if (slot >= a.slots || pos >= a.max_seq_len) {
+        if (tid == 0) atomicOr(a.status, 2u);
+        return;
+    }
+    const float* c = a.packed + (size_t)row * a.ld + (size_t)a.heads * a.dim;
+    float v[MAX_RANK / 256], ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < (int)MAX_RANK / 256; ++i) {
+        const uint32_t k = tid + 256u * i;
+        v[i] = k < a.rank ? c[k] : 0.0f;
+        ss = fmaf(v[i], v[i], ss);
+    }
+    const float n = 1.0f / sqrtf(block_sum_256(ss, red) / (float)a.rank + a.eps);
+    ET* dst = reinterpret_cast<ET*>(a.C) + ((size_t)slot * a.max_seq_len + pos) * a.rank;
+#pragma unroll
+    for (int i = 0; i < (int)MAX_RANK / 256; ++i) {
+        const uint32_t k = tid + 256u * i;
+        if (k < a.rank) m40_store_elem(dst + k, v[i] * n * a.c_norm[k]);
+    }
+    if (tid == 0 && a.seq_map) a.seq_map[slot] = pos + 1u;
+}
+
+__device__ __forceinline__ void split_store4(__nv_bfloat16* hi, __nv_bfloat16* lo, size_t at, const float4& x) {
+    const float v[4] = {x.x, x.y, x.z, x.w};
+    __nv_bfloat16 h[4], l[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        h[i] = __float2bfloat16_rn(v[i]);
+        l[i] = __float2bfloat16_rn(v[i] - __bfloat162float(h[i]));
+    }
+    *reinterpret_cast<uint2*>(hi + at) = *reinterpret_cast<const uint2*>(h);
+    *reinterpret_cast<uint2*>(lo + at) = *reinterpret_cast<const uint2*>(l);
+}
+
+// grid (rows, 1 + shares of the query): CTA (row, 0) appends the row's latent (when asked to), the others cut its queries.
+__global__ void __launch_bounds__(256) latent_append_kernel(LatArgs a, uint32_t append) {
+    __shared__ float red[8];
+    pdl_wait();
+    pdl_trigger();
+    const uint32_t row = blockIdx.x, n = a.heads * a.dim;
+    if (blockIdx.y == 0) {
+        if (append) append_row<__half>(a, row, red);
+        return;
+    }
+    for (uint32_t k = ((blockIdx.y - 1u) * 256u + threadIdx.x) * 4u; k < n; k += (gridDim.y - 1u) * 1024u)
+        split_store4(a.part[0], a.part[1], (size_t)row * n + k, *reinterpret_cast<const float4*>(a.packed + (size_t)row * a.ld + k));
+}
+
 __device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
 
 // grid (absorb_ctas + RG or 0, row groups of RG). CTAs below absorb_ctas: (head, COLS latent columns) of the group's absorbed
@@ -75,28 +131,7 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(LatArgs a) {
     pdl_trigger();
     if (blockIdx.x >= a.absorb_ctas) {
         const uint32_t row = row0 + blockIdx.x - a.absorb_ctas;
-        if (row >= a.rows) return;
-        const uint32_t pos = a.row_pos[row], slot = a.row_seq[row] * a.slot_mul + a.slot_add;
-        if (slot >= a.slots || pos >= a.max_seq_len) {
-            if (tid == 0) atomicOr(a.status, 2u);
-            return;
-        }
-        const float* c = a.packed + (size_t)row * a.ld + (size_t)a.heads * a.dim;
-        float v[MAX_RANK / 256], ss = 0.0f;
-#pragma unroll
-        for (int i = 0; i < (int)MAX_RANK / 256; ++i) {
-            const uint32_t k = tid + 256u * i;
-            v[i] = k < a.rank ? c[k] : 0.0f;
-            ss = fmaf(v[i], v[i], ss);
-        }
-        const float n = 1.0f / sqrtf(block_sum_256(ss, red) / (float)a.rank + a.eps);
-        ET* dst = reinterpret_cast<ET*>(a.C) + ((size_t)slot * a.max_seq_len + pos) * a.rank;
-#pragma unroll
-        for (int i = 0; i < (int)MAX_RANK / 256; ++i) {
-            const uint32_t k = tid + 256u * i;
-            if (k < a.rank) m40_store_elem(dst + k, v[i] * n * a.c_norm[k]);
-        }
-        if (tid == 0 && a.seq_map) a.seq_map[slot] = pos + 1u;
+        if (row < a.rows) append_row<ET>(a, row, red);
         return;
     }
     for (uint32_t i = tid; i < RG * a.dim; i += 256u) {
@@ -229,7 +264,7 @@ struct LatTile {
     static constexpr size_t FIXED = ((size_t)8 * 16 * PITCH * 4 + (size_t)16 * PITCH * 2 + 16 * 4 + 127) / 128 * 128;
     static constexpr size_t bytes(uint32_t rank) { return (size_t)TOKENS * (rank + 8u) * 2u; }
 };
-constexpr size_t TILE_SMEM = 112u * 1024u;
+constexpr size_t TILE_SMEM = 112u * 1024u, TILE_SMEM_ALONE = 200u * 1024u;
 
 template <int UW>
 __global__ void __launch_bounds__(256, 2) latent_tiles_kernel(LatArgs a, uint32_t stages) {
@@ -255,17 +290,22 @@ __global__ void __launch_bounds__(256, 2) latent_tiles_kernel(LatArgs a, uint32_
     }
     const __half* C = reinterpret_cast<const __half*>(a.C) + (size_t)slot * a.max_seq_len * a.rank;
     const uint32_t n_tiles = (hi - lo + LT - 1u) / LT, pieces = a.rank / 8u;
-    auto load_tile = [&](uint32_t tile) {
-        __half* dst = ring + (size_t)(tile % stages) * LT * pitch;
+    // this thread's 16-byte pieces of a tile: every 256th, as (token, piece) pairs that are stepped, not divided for
+    const uint32_t r_first = tid / pieces, ch_first = tid % pieces, r_step = 256u / pieces, ch_step = 256u % pieces;
+    auto load_tile = [&](uint32_t tile, uint32_t slot_of_ring) {
+        __half* dst = ring + (size_t)slot_of_ring * LT * pitch;
         const uint32_t base = lo + tile * LT;
-        for (uint32_t i = tid; i < LT * pieces; i += 256u) {
-            const uint32_t r = i / pieces, ch = i % pieces;
+        const __half* src = C + (size_t)base * a.rank;
+        const uint32_t last = hi - 1u - base;
+        for (uint32_t r = r_first, ch = ch_first; r < LT;) {
             // rows past the end repeat the last visible one: masked below, and their bytes are finite
-            cp_async16(dst + r * pitch + ch * 8u, C + (size_t)min(base + r, hi - 1u) * a.rank + ch * 8u);
+            cp_async16(dst + r * pitch + ch * 8u, src + min(r, last) * a.rank + ch * 8u);
+            r += r_step, ch += ch_step;
+            if (ch >= pieces) ch -= pieces, ++r;
         }
     };
     for (uint32_t t = 0; t + 1u < stages; ++t) {
-        if (t < n_tiles) load_tile(t);
+        if (t < n_tiles) load_tile(t, t);
         cp_async_commit();
     }
     // query fragments of this warp's columns
@@ -292,14 +332,18 @@ __global__ void __launch_bounds__(256, 2) latent_tiles_kernel(LatArgs a, uint32_
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};  // heads 2 * warp and 2 * warp + 1
     const uint32_t busy = (NU + UW - 1u) / UW;                         // warps that own columns
 
-    for (uint32_t tile = 0; tile < n_tiles; ++tile) {
-        if (stages == 2u) cp_async_wait<0>();
-        else if (stages == 3u) cp_async_wait<1>();
-        else cp_async_wait<2>();
+    uint32_t here = 0;  // ring slot of this tile
+    for (uint32_t tile = 0; tile < n_tiles; ++tile, here = here + 1u < stages ? here + 1u : 0u) {
+        switch (stages) {  // all but the newest stages - 2 groups have landed
+            case 2: cp_async_wait<0>(); break;
+            case 3: cp_async_wait<1>(); break;
+            case 4: cp_async_wait<2>(); break;
+            default: cp_async_wait<3>();
+        }
         __syncthreads();
-        if (tile + stages - 1u < n_tiles) load_tile(tile + stages - 1u);
+        if (tile + stages - 1u < n_tiles) load_tile(tile + stages - 1u, here ? here - 1u : stages - 1u);
         cp_async_commit();
-        const __half* tc = ring + (size_t)(tile % stages) * LT * pitch;
+        const __half* tc = ring + (size_t)here * LT * pitch;
         if (warp < busy) {
             float s[LT / 8][4];
 #pragma unroll
@@ -423,8 +467,8 @@ __global__ void __launch_bounds__(256) latent_split_kernel(const __half* __restr
 }
 
 // grid (heads, row groups of RG, slices of the values): splits and sink -> the head's weighted latent, then uv. Every slice
-// merges for itself: the partials are in L2.
-template <typename WT, int RG>
+// merges for itself: the partials are in L2. SPLIT: the weighted latents are the result, as hi + lo (the caller applies uv).
+template <typename WT, int RG, bool SPLIT>
 __global__ void __launch_bounds__(256) latent_merge_kernel(LatArgs a) {
     extern __shared__ __align__(16) float so[];  // [RG][rank padded to 8], [RG][splits] weights, [256][RG] float4
     const uint32_t head = blockIdx.x, row0 = blockIdx.y * RG, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
@@ -432,56 +476,84 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(LatArgs a) {
     float* sw = so + RG * rp;
     const uint32_t per = (a.vdim + gridDim.z - 1u) / gridDim.z, n_lo = blockIdx.z * per, n_hi = min(n_lo + per, a.vdim);
     const WT* uv = reinterpret_cast<const WT*>(a.uv) + (size_t)head * a.vdim * a.rank;
-    if (n_lo < n_hi) {  // the weights do not depend on the previous kernel
+    // The weights do not depend on the previous kernel. One row of 16-bit weights: a warp's first four rows of uv go to
+    // registers (their part of columns below 512), everything else to L2.
+    constexpr bool HOLD = RG == 1 && !SPLIT && sizeof(WT) == 2;
+    uint4 held[HOLD ? 4 : 1][2];
+    if (!SPLIT && n_lo < n_hi) {
+        if (HOLD && a.wide) {
+#pragma unroll
+            for (int j = 0; j < (HOLD ? 4 : 0); ++j) {
+                const WT* w = uv + (size_t)min(n_lo + 2u * warp + (j >> 1) * 16u + (j & 1), n_hi - 1u) * a.rank;
+#pragma unroll
+                for (int i = 0; i < 2; ++i) held[j][i] = *reinterpret_cast<const uint4*>(w + min(lane * 8u + 256u * i, a.rank - 8u));
+            }
+        }
         const char* p = reinterpret_cast<const char*>(uv + (size_t)n_lo * a.rank);
         const size_t bytes = (size_t)(n_hi - n_lo) * a.rank * sizeof(WT);
         for (size_t i = (size_t)tid * 128u; i < bytes; i += 256u * 128u) prefetch_l2(p + i);
     }
     pdl_wait();
     pdl_trigger();
-    if (warp < RG && warp < live) {  // one warp per row: the splits' weights
+    if (warp < RG && warp < live) {  // one warp per row: the splits' weights (at most 128 splits)
         const size_t base = ((size_t)(row0 + warp) * a.heads + head) * a.splits;
         const float sink = a.sink ? a.sink[head] : -INFINITY;
-        float M = sink;
-        for (uint32_t s = lane; s < a.splits; s += 32u)
-            if (a.pl[base + s] > 0.0f) M = fmaxf(M, a.pm[base + s]);
+        float l[4], m[4], M = sink, L = 0.0f;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const uint32_t s = lane + 32u * i;
+            l[i] = s < a.splits ? a.pl[base + s] : 0.0f;
+            m[i] = s < a.splits ? a.pm[base + s] : 0.0f;
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+            if (l[i] > 0.0f) M = fmaxf(M, m[i]);
         M = warp_max(M);
-        float L = 0.0f;
-        for (uint32_t s = lane; s < a.splits; s += 32u) {
-            const float l = a.pl[base + s], e = l > 0.0f ? expf(a.pm[base + s] - M) : 0.0f;
-            sw[warp * a.splits + s] = e;
-            L = fmaf(l, e, L);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            m[i] = l[i] > 0.0f ? expf(m[i] - M) : 0.0f;
+            L = fmaf(l[i], m[i], L);
         }
         L = warp_sum(L);
         if (a.sink) L += expf(sink - M);
         const float inv = 1.0f / (L > 0.0f ? L : 1.0f);
-        for (uint32_t s = lane; s < a.splits; s += 32u) sw[warp * a.splits + s] *= inv;
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+            if (lane + 32u * i < a.splits) sw[warp * a.splits + lane + 32u * i] = m[i] * inv;
     }
-    __syncthreads();
     // where column k of the weighted latent lies: the halves of every 8 columns apart, so that 16-byte reads of neighbouring
     // lanes fall into different banks
     auto place = [&](uint32_t k) { return ((k & 4u) ? rp / 2u : 0u) + (k >> 3) * 4u + (k & 3u); };
     if (a.rank % 4u == 0u) {
-        const uint32_t c4 = a.rank / 4u, teams = 256u / c4 ? 256u / c4 : 1u, team = tid / c4, col = tid % c4;  // rank <= 1024
+        const uint32_t c4 = a.rank / 4u, teams = 256u / c4, team = tid / c4, col = tid % c4;  // rank <= 1024
+        const bool busy = team < teams;
         float4* st = reinterpret_cast<float4*>(sw + ((RG * a.splits + 3u) & ~3u));
-        float4 acc[RG];
+        constexpr int AHEAD = RG == 1 ? 16 : 4;  // partials requested before the weights are known, per row
+        float4 x[RG][AHEAD];
+        const float4* o0 = reinterpret_cast<const float4*>(a.po + ((size_t)row0 * a.heads + head) * a.splits * a.rank) + (busy ? col : 0u);
+        const size_t row_step = (size_t)a.heads * a.splits * c4;
+#pragma unroll
+        for (int r = 0; r < RG; ++r)
+#pragma unroll
+            for (int i = 0; i < AHEAD; ++i)
+                x[r][i] = o0[min((uint32_t)r, live - 1u) * row_step + (size_t)min((busy ? team : 0u) + i * teams, a.splits - 1u) * c4];
+        __syncthreads();
+        auto add = [](float4& t, float w, const float4& v) {
+            if (w != 0.0f)  // empty splits may hold anything
+                t.x = fmaf(w, v.x, t.x), t.y = fmaf(w, v.y, t.y), t.z = fmaf(w, v.z, t.z), t.w = fmaf(w, v.w, t.w);
+        };
 #pragma unroll
         for (int r = 0; r < RG; ++r) {
-            acc[r] = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (team < teams && (uint32_t)r < live) {
+            float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (busy && (uint32_t)r < live) {
                 const float* w = sw + r * a.splits;
-                const float4* o = reinterpret_cast<const float4*>(a.po + ((size_t)(row0 + r) * a.heads + head) * a.splits * a.rank) + col;
+#pragma unroll
+                for (int i = 0; i < AHEAD; ++i)
+                    if (team + i * teams < a.splits) add(acc, w[team + i * teams], x[r][i]);
 #pragma unroll 8
-                for (uint32_t s = team; s < a.splits; s += teams) {
-                    const float ws = w[s];
-                    const float4 x = o[(size_t)s * c4];
-                    if (ws != 0.0f) {  // empty splits may hold anything
-                        acc[r].x = fmaf(ws, x.x, acc[r].x), acc[r].y = fmaf(ws, x.y, acc[r].y);
-                        acc[r].z = fmaf(ws, x.z, acc[r].z), acc[r].w = fmaf(ws, x.w, acc[r].w);
-                    }
-                }
+                for (uint32_t s = team + AHEAD * teams; s < a.splits; s += teams) add(acc, w[s], o0[r * row_step + (size_t)s * c4]);
             }
-            st[tid * RG + r] = acc[r];
+            st[tid * RG + r] = acc;
         }
         __syncthreads();
         for (uint32_t i = tid; i < RG * c4; i += 256u) {
@@ -491,9 +563,11 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(LatArgs a) {
                 const float4 u = st[(k * c4 + c) * RG + r];
                 t.x += u.x, t.y += u.y, t.z += u.z, t.w += u.w;
             }
-            *reinterpret_cast<float4*>(so + r * rp + place(4u * c)) = t;
+            if (!SPLIT) *reinterpret_cast<float4*>(so + r * rp + place(4u * c)) = t;
+            else if (r < live) split_store4(a.part[0], a.part[1], ((size_t)(row0 + r) * a.heads + head) * a.rank + 4u * c, t);
         }
     } else {
+        __syncthreads();
         for (uint32_t i = tid; i < RG * rp; i += 256u) {
             const uint32_t r = i / rp, c = i % rp;
             float t = 0.0f;
@@ -508,17 +582,14 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(LatArgs a) {
             so[r * rp + place(c)] = t;
         }
     }
+    if (SPLIT) return;
     __syncthreads();
-    for (uint32_t n0 = n_lo + 2u * warp; n0 < n_hi; n0 += 16u) {  // two values at a time
+    for (uint32_t n0 = n_lo + 2u * warp, it = 0; n0 < n_hi; n0 += 16u, ++it) {  // two values at a time
         const uint32_t n1 = min(n0 + 1u, n_hi - 1u);
         const WT *w0 = uv + (size_t)n0 * a.rank, *w1 = uv + (size_t)n1 * a.rank;
         float acc[2][RG] = {};
         if (a.wide) {
-#pragma unroll 2
-            for (uint32_t k = lane * 8u; k < a.rank; k += 256u) {
-                float v0[8], v1[8];
-                m40_load8(w0 + k, v0);
-                m40_load8(w1 + k, v1);
+            auto piece = [&](uint32_t k, const float* v0, const float* v1) {
 #pragma unroll
                 for (int r = 0; r < RG; ++r) {
                     const float4 x0 = *reinterpret_cast<const float4*>(so + r * rp + (k >> 1));
@@ -527,6 +598,25 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(LatArgs a) {
 #pragma unroll
                     for (int i = 0; i < 8; ++i) acc[0][r] = fmaf(v0[i], x[i], acc[0][r]), acc[1][r] = fmaf(v1[i], x[i], acc[1][r]);
                 }
+            };
+            uint32_t k = lane * 8u;
+            if (HOLD && it < 2u) {
+#pragma unroll
+                for (int i = 0; i < 2; ++i, k += 256u) {
+                    if (k >= a.rank) break;
+                    float v0[8], v1[8];
+                    const uint4 h0 = it == 0u ? held[0][i] : held[HOLD ? 2 : 0][i], h1 = it == 0u ? held[HOLD ? 1 : 0][i] : held[HOLD ? 3 : 0][i];
+                    m40_load8(reinterpret_cast<const WT*>(&h0), v0);
+                    m40_load8(reinterpret_cast<const WT*>(&h1), v1);
+                    piece(k, v0, v1);
+                }
+            }
+#pragma unroll 2
+            for (; k < a.rank; k += 256u) {
+                float v0[8], v1[8];
+                m40_load8(w0 + k, v0);
+                m40_load8(w1 + k, v1);
+                piece(k, v0, v1);
             }
         } else {
             for (uint32_t k = lane; k < a.rank; k += 32u) {
@@ -565,15 +655,16 @@ cudaError_t launch_prepare(cudaStream_t s, const LatArgs& a, bool append) {
 }
 
 template <typename WT>
-cudaError_t launch_merge(M40llmCudaContext* ctx, const LatArgs& a) {
+cudaError_t launch_merge(M40llmCudaContext* ctx, const LatArgs& a, bool split) {
     const uint32_t rp = (a.rank + 7u) & ~7u, rg = a.rows == 1 ? 1u : 4u, groups = (a.rows + rg - 1) / rg;
     uint32_t z = (uint32_t)ctx->sm_count / (a.heads * groups);
     const uint32_t z_max = (a.vdim + 15u) / 16u;
     z = z < 1u ? 1u : (z > z_max ? z_max : z);
     const size_t smem = ((size_t)rg * rp + (((size_t)rg * a.splits + 3) & ~(size_t)3) + (size_t)256 * 4 * rg) * sizeof(float);
-    const dim3 grid(a.heads, groups, z);
-    return rg == 1 ? m40_launch_dependent(latent_merge_kernel<WT, 1>, grid, dim3(256), smem, ctx->decode_stream, a)
-                   : m40_launch_dependent(latent_merge_kernel<WT, 4>, grid, dim3(256), smem, ctx->decode_stream, a);
+    const dim3 grid(a.heads, groups, split ? 1 : z);
+    if (split) return m40_launch_dependent(latent_merge_kernel<WT, 4, true>, grid, dim3(256), smem, ctx->decode_stream, a);
+    return rg == 1 ? m40_launch_dependent(latent_merge_kernel<WT, 1, false>, grid, dim3(256), smem, ctx->decode_stream, a)
+                   : m40_launch_dependent(latent_merge_kernel<WT, 4, false>, grid, dim3(256), smem, ctx->decode_stream, a);
 }
 
 template <typename WT>
@@ -586,13 +677,15 @@ cudaError_t launch_tiles(M40llmCudaContext* ctx, const LatArgs& a) {
     static unsigned long long configured = 0ull;
     const unsigned long long bit = 1ull << (ctx->device_id & 63);
     if (!(configured & bit)) {
-        const cudaError_t e = cudaFuncSetAttribute(latent_tiles_kernel<UW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TILE_SMEM);
+        const cudaError_t e = cudaFuncSetAttribute(latent_tiles_kernel<UW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TILE_SMEM_ALONE);
         if (e != cudaSuccess) return e;
         configured |= bit;
     }
-    size_t stages = (TILE_SMEM - LatTile<UW>::FIXED) / LatTile<UW>::bytes(a.rank);
-    if (stages > 4) stages = 4;
     const dim3 grid(a.splits, (a.heads + 15) / 16, a.rows);
+    // a launch that gives every SM at most one CTA lets it have the shared memory of two: a deeper ring
+    const bool alone = (uint64_t)grid.x * grid.y * grid.z <= (uint64_t)ctx->sm_count;
+    size_t stages = ((alone ? TILE_SMEM_ALONE : TILE_SMEM) - LatTile<UW>::FIXED) / LatTile<UW>::bytes(a.rank);
+    if (stages > 5) stages = 5;
     return m40_launch_dependent(latent_tiles_kernel<UW>, grid, dim3(256), LatTile<UW>::FIXED + stages * LatTile<UW>::bytes(a.rank),
                                 ctx->decode_stream, a, (uint32_t)stages);
 }
@@ -611,9 +704,36 @@ void pick_splits(const M40llmCudaContext* ctx, uint32_t ctas_per_split, uint32_t
     *splits = (bound + c - 1) / c;
 }
 
+// Whether uk and uv of several rows go through the grouped GEMM.
+bool takes_grouped(const M40llmKVCache* kv, const LatArgs& a, uint32_t w_dtype) {
+    return !kv->elem_f32 && w_dtype == M40LLM_DT_BF16 && a.uk_t && a.ld % 4 == 0 && (((uintptr_t)a.packed | (uintptr_t)a.out) & 15u) == 0 &&
+           m40_gemm_tc_grouped_supported(a.uk_t, a.rank, a.dim, a.heads * a.dim, a.dim) &&
+           m40_gemm_tc_grouped_supported(a.uv, a.vdim, a.rank, a.heads * a.rank, a.rank);
+}
+
+// out[row][head * N ..] = the head's matrix [N][K] times x[row][head * K ..], x as hi + lo.
+int per_head(M40llmCudaContext* ctx, const LatArgs& a, const void* w, uint32_t N, uint32_t K, float* out) {
+    M40GroupedCall c = {};
+    c.w = w;
+    c.x[0] = a.part[0], c.x[1] = a.part[1];
+    c.parts = 2;
+    c.bf16 = 1;
+    c.groups = a.heads;
+    c.N = N;
+    c.K = c.group_k = K;
+    c.x_rows = a.rows;
+    c.ldx = a.heads * K;
+    c.tile_rows = a.rows <= 16 ? 16 : (a.rows <= 32 ? 32 : (a.rows <= 64 ? 64 : 128));
+    c.kind = M40_GROUPED_F32;
+    c.out = out;
+    c.out_ld = a.heads * N;
+    c.out_group = N;
+    return m40_gemm_tc_grouped(ctx, ctx->decode_stream, c);
+}
+
 // Absorbed form over the rows of `all`; append: the latents are not in the cache yet.
 template <typename WT>
-int run_absorbed(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs& all, uint32_t bound, bool append) {
+int run_absorbed(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs& all, uint32_t bound, bool append, uint32_t w_dtype) {
     cudaStream_t s = ctx->decode_stream;
     const bool tiles = !kv->elem_f32 && all.rank % 16 == 0 && all.rank <= 512;
     cudaError_t e;
@@ -624,19 +744,33 @@ int run_absorbed(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs&
         a.out += (size_t)at * a.heads * a.vdim;
         a.row_seq += at;
         a.row_pos += at;
+        const bool grouped = a.rows >= GROUPED_ROWS && takes_grouped(kv, a, w_dtype);
         pick_splits(ctx, a.rows * (tiles ? (a.heads + 15) / 16 : a.heads), bound, &a.chunk, &a.splits);
         const size_t nh = (size_t)a.rows * a.heads, np = nh * a.splits;
-        auto pad = [](size_t v) { return (v + 3) & ~(size_t)3; };
-        float* work = (float*)m40_ensure_scratch(ctx, 1, (pad(nh * a.rank) + pad(np * a.rank) + 2 * np) * sizeof(float), 1);
+        auto pad = [](size_t v) { return (v + 63) & ~(size_t)63; };
+        const size_t part = grouped ? pad(nh * (a.rank > a.dim ? a.rank : a.dim)) : 0;  // 16-bit values
+        float* work = (float*)m40_ensure_scratch(ctx, 1, (pad(nh * a.rank) + pad(np * a.rank) + 2 * pad(np) + part) * sizeof(float) + 256, 1);
         if (!work) return -5;
+        work = (float*)(((uintptr_t)work + 255) & ~(uintptr_t)255);
         a.qa = work;
         a.po = work + pad(nh * a.rank);
         a.pm = a.po + pad(np * a.rank);
-        a.pl = a.pm + np;
-        a.absorb_ctas = absorb_ctas(a);
-        e = prepare<WT>(s, a, kv->elem_f32, append);
-        M40_COUNT_LAUNCH(ctx);
-        if (e != cudaSuccess) return -6;
+        a.pl = a.pm + pad(np);
+        a.part[0] = (__nv_bfloat16*)(a.pl + pad(np));
+        a.part[1] = a.part[0] + part;
+        int rc;
+        if (grouped) {
+            const uint32_t shares = (a.heads * a.dim + 1023) / 1024;
+            e = m40_launch_dependent(latent_append_kernel, dim3(a.rows, 1 + (shares < 4 ? shares : 4)), dim3(256), 0, s, a, append ? 1u : 0u);
+            M40_COUNT_LAUNCH(ctx);
+            if (e != cudaSuccess) return -6;
+            if ((rc = per_head(ctx, a, a.uk_t, a.rank, a.dim, a.qa)) != 0) return rc;
+        } else {
+            a.absorb_ctas = absorb_ctas(a);
+            e = prepare<WT>(s, a, kv->elem_f32, append);
+            M40_COUNT_LAUNCH(ctx);
+            if (e != cudaSuccess) return -6;
+        }
         const dim3 grid(a.heads, a.rows, a.splits);
         if (tiles)
             e = a.rank <= 128 ? launch_tiles<1>(ctx, a) : (a.rank <= 256 ? launch_tiles<2>(ctx, a) : launch_tiles<4>(ctx, a));
@@ -645,9 +779,10 @@ int run_absorbed(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs&
                              : m40_launch_dependent(latent_rows_kernel<__half>, grid, dim3(128), 0, s, a);
         M40_COUNT_LAUNCH(ctx);
         if (e != cudaSuccess) return -6;
-        e = launch_merge<WT>(ctx, a);
+        e = launch_merge<WT>(ctx, a, grouped);
         M40_COUNT_LAUNCH(ctx);
         if (e != cudaSuccess || cudaGetLastError() != cudaSuccess) return -6;
+        if (grouped && (rc = per_head(ctx, a, a.uv, a.vdim, a.rank, a.out)) != 0) return rc;
     }
     return 0;
 }
@@ -751,7 +886,7 @@ int run(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs& all, uin
         M40_COUNT_LAUNCH(ctx);
         if (e != cudaSuccess) return -6;
     }
-    if (!any) return run_absorbed<WT>(ctx, kv, all, bound, !first);
+    if (!any) return run_absorbed<WT>(ctx, kv, all, bound, !first, w_dtype);
     uint32_t run0 = 0;  // first row of the absorbed run that is being gathered
     for (uint32_t i = 0; i <= r.segments; ++i) {
         const uint32_t* sg = i < r.segments ? r.seg_host + 4 * i : nullptr;
@@ -764,7 +899,7 @@ int run(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs& all, uin
             a.out += (size_t)run0 * a.heads * a.vdim;
             a.row_seq += run0;
             a.row_pos += run0;
-            const int rc = run_absorbed<WT>(ctx, kv, a, bound, false);
+            const int rc = run_absorbed<WT>(ctx, kv, a, bound, false, w_dtype);
             if (rc != 0) return rc;
         }
         if (!sg) break;
@@ -789,6 +924,7 @@ extern "C" int m40llm_attention_latent_async(M40llmCudaContext* ctx, M40llmKVCac
     a.packed = (const float*)c->packed;
     a.c_norm = (const float*)c->c_norm;
     a.uk = c->uk;
+    a.uk_t = c->uk_t;
     a.uv = c->uv;
     a.sink = (const float*)c->sink;
     a.C = kv->d_typed_k;

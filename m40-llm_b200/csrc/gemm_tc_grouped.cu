@@ -27,6 +27,7 @@ struct GArgs {
     uint32_t* status;
     uint32_t N, K, x_rows, group_k, tile_rows, parts, kblocks, stages, fmt_bits, bf16;
     int act;
+    uint32_t out_ld, out_group;
     __half* heads;
     uint32_t head_dim, head_pitch;
     M40RgArgs rg;
@@ -220,7 +221,7 @@ __global__ void __launch_bounds__(192, 1) gemm_tc_grouped_kernel(const __grid_co
                 for (int j = 0; j < 8; ++j) {
                     if (n >= a.N || c + j >= m_live) continue;
                     const size_t at = (size_t)(m_base + c + j) * a.N + n;
-                    if (KIND == M40_GROUPED_F32) a.out[at] = v[j];
+                    if (KIND == M40_GROUPED_F32) a.out[(size_t)(m_base + c + j) * a.out_ld + group * a.out_group + n] = v[j];
                     else if (KIND == M40_GROUPED_HEADS) heads[(size_t)(m_base + c + j) * a.head_pitch] = __float2half_rn(v[j]);
                     else if (a.bf16) store_split((__nv_bfloat16*)a.hi, (__nv_bfloat16*)a.lo, at, m40_act(a.act, v[j]));
                     else store_split((__half*)a.hi, (__half*)a.lo, at, m40_act(a.act, v[j]));
@@ -284,6 +285,8 @@ int m40_gemm_tc_grouped(M40llmCudaContext* ctx, cudaStream_t s, const M40Grouped
     a.fmt_bits = c.bf16 ? tc::idesc_bf16() : 0u;
     a.bf16 = c.bf16;
     a.act = c.act;
+    a.out_ld = c.out_ld ? c.out_ld : c.N;
+    a.out_group = c.out_group;
     a.heads = c.heads;
     a.head_dim = c.head_dim;
     a.head_pitch = c.head_pitch;

@@ -23,7 +23,8 @@ struct M40GroupedCall {
     uint32_t max_tiles;
     // result
     int kind, act;
-    float* out;                // F32: [x_rows][N]
+    float* out;                // F32: [x_rows][out_ld], group g's values from column g * out_group on (0, 0: N, 0)
+    uint32_t out_ld, out_group;
     void* hi;                  // ACT_SPLIT: act(D) as hi + lo of the weights' type, [x_rows][N]
     void* lo;
     __half* heads;             // HEADS: f16 [N / head_dim][x_rows][head_pitch], one row of D dealt to heads of head_dim values

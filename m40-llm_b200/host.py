@@ -56,7 +56,7 @@ class StackLayerDesc(C.Structure):
                 [("router_scale", C.c_float), ("shared_ff", C.c_uint32), ("n_router", C.c_uint32)] +
                 [(n, C.c_void_p) for n in ("w_router", "shared_down", "correction")] +
                 [("conv_taps", C.c_uint32), ("conv_w", C.c_void_p), ("in_bias", C.c_void_p), ("rank_kv", C.c_uint32)] +
-                [(n, C.c_void_p) for n in ("c_norm", "uk", "uv", "sink")] +
+                [(n, C.c_void_p) for n in ("c_norm", "uk", "uk_t", "uv", "sink")] +
                 [(n, C.c_uint32) for n in ("rg_width", "rg_blocks", "rg_taps")] + [("rg_decay", C.c_float)] +
                 [(n, C.c_void_p) for n in ("rg_conv", "rg_conv_b", "ra", "ra_b", "ri", "ri_b", "lam")])
 

@@ -165,6 +165,7 @@ int StackLayer::enqueue_mixer(M40llmCudaContext* ctx, const M40llmStepRows& rows
         m.ld = d_.n_in;
         m.c_norm = d_.c_norm;
         m.uk = d_.uk;
+        m.uk_t = d_.uk_t;
         m.uv = d_.uv;
         m.sink = d_.sink;
         m.out = b.att;

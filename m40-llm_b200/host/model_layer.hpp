@@ -109,7 +109,7 @@ struct StackLayerDesc {
     const void* in_bias; // of w_in, f32, or null
     // latent attention (q_heads, k_dim, v_dim and scale above)
     uint32_t rank_kv;
-    const void *c_norm, *uk, *uv, *sink;
+    const void *c_norm, *uk, *uk_t, *uv, *sink;
     // real-gated linear recurrence
     uint32_t rg_width, rg_blocks, rg_taps;
     float rg_decay;

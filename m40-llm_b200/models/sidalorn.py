@@ -64,6 +64,7 @@ class SidalornSpec:
             d.q_heads, d.k_dim, d.v_dim, d.rank_kv, d.scale = H, K, V, R, float(m["scale"])
             d.c_norm, d.sink = w.vector(mix + "dkv.norm", R), w.vector(mix + "sink", H)
             d.uk, d.uv = w.matrix(mix + "uk", shapes=[(H * K, R)]), w.matrix(mix + "uv", shapes=[(H * V, R)])
+            d.uk_t = w.blocks_transposed(mix + "uk", (H * K, R), H)
         else:
             D, B, T = int(m["width"]), int(m["blocks"]), int(m["conv"])
             if D % B:

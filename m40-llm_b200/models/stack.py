@@ -56,6 +56,16 @@ class StackWeights:
             self._mat[names] = self.nat.buf(np.concatenate(parts)).ptr
         return self._mat[names]
 
+    def blocks_transposed(self, name: str, shape, blocks: int) -> int:
+        """bf16 copy of a matrix [blocks * n][k] with every block of n rows transposed: [blocks * k][n]."""
+        key = (name, "transposed", blocks)
+        if key not in self._mat:
+            if self.t.shape(name) != tuple(shape):
+                raise ValueError(f"tensor {name}: shape {self.t.shape(name)}, expected {tuple(shape)}")
+            a = self.t.bf16(name).reshape(blocks, shape[0] // blocks, shape[1])
+            self._mat[key] = self.nat.buf(np.ascontiguousarray(a.transpose(0, 2, 1))).ptr
+        return self._mat[key]
+
     def vectors(self, names, sizes, total: int) -> int:
         """f32 copies of several vectors, one after the other, zeros up to `total` values."""
         key = ("vectors", *names)

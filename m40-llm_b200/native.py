@@ -71,7 +71,7 @@ class RgLru(C.Structure):
 
 class LatentAttention(C.Structure):
     """M40llmLatentAttention."""
-    _fields_ = ([(n, C.c_void_p) for n in ("packed", "c_norm", "uk", "uv", "sink", "out")] +
+    _fields_ = ([(n, C.c_void_p) for n in ("packed", "c_norm", "uk", "uk_t", "uv", "sink", "out")] +
                 [(n, C.c_uint32) for n in ("ld", "heads", "dim", "vdim", "w_dtype")] + [("eps", C.c_float), ("scale", C.c_float)])
 
 

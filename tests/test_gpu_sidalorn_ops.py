@@ -156,7 +156,8 @@ class Latent:
         self.sink = rng.uniform(-1, 4, H).astype(np.float32) if sink else None
         self.kv = nat.lib.m40llm_kvcache_create_typed(nat.ctx, max_len, slots, 1, R, 0, N.DT_F32 if fp32 else N.DT_F16)
         self.ld = (H * D + R + 7) // 8 * 8
-        self.dev = [f32(nat, self.cn), bits(nat, self.uk), bits(nat, self.uv), f32(nat, self.sink) if sink else None]
+        ukt = self.uk.reshape(H, D, R).transpose(0, 2, 1).reshape(H * R, D)
+        self.dev = [f32(nat, self.cn), bits(nat, self.uk), bits(nat, ukt), bits(nat, self.uv), f32(nat, self.sink) if sink else None]
 
     def oracle(self, q, c):
         """q [T, H * D], c [T, R] of one sequence from position 0 -> [T, H * V]."""
@@ -218,7 +219,7 @@ def test_latent_attention(nat, H, D, V, R, fp32):
                 at[s] += n
     # without a sink, without the host's copy of the segments and without a known length
     t.sink = None
-    t.dev[3] = None
+    t.dev[4] = None
     got = t.run([(0, 0, 300)], q[0, :300], c[0, :300], host=False)
     close(got, t.oracle(q[0, :300], c[0, :300]), tol, "no sink")
     no_status(nat)
@@ -232,7 +233,7 @@ def test_latent_attention_finds_one_far_token(nat, H, D, V, R, fp32):
     token to the newest one, past tile and chunk edges, and from nowhere before it is there."""
     t = Latent(nat, H, D, V, R, fp32, seed=3, max_len=1400)
     t.sink[:] = 0.0
-    t.dev[3] = f32(nat, t.sink)
+    t.dev[4] = f32(nat, t.sink)
     rng = np.random.default_rng(2)
     T = 1300
     key = rng.standard_normal(R)
@@ -270,6 +271,9 @@ def test_latent_attention_batch_decode_lengths(nat):
         c.append(cc[-1])
     got = t.run([(s, n - 1, 1) for s, n in enumerate(lens)], np.array(q), np.array(c), host=False)
     close(got, np.array(want), 3e-3)
+    t.dev[2] = None       # and without the transposed matrix
+    got = t.run([(s, n - 1, 1) for s, n in enumerate(lens)], np.array(q), np.array(c), host=False)
+    close(got, np.array(want), 3e-3)
     no_status(nat)
     t.close()
 
@@ -285,7 +289,7 @@ def test_latent_attention_rejects(nat):
     plain = nat.lib.m40llm_kvcache_create_typed(nat.ctx, 8, 3, 1, 32, 16, N.DT_F16)
     rows = Rows(nat, [(0, 0, 1)])
     b = nat.buf(4096).ptr
-    call = N.LatentAttention(b, b, b, b, None, b, 64, 2, 16, 16, N.DT_BF16, 1e-5, 1.0)
+    call = N.LatentAttention(b, b, b, None, b, None, b, 64, 2, 16, 16, N.DT_BF16, 1e-5, 1.0)
     assert nat.lib.m40llm_attention_latent_async(nat.ctx, plain, C.byref(call), C.byref(rows.c)) == -4
     call.ld = 63
     assert nat.lib.m40llm_attention_latent_async(nat.ctx, t.kv, C.byref(call), C.byref(rows.c)) == -2
