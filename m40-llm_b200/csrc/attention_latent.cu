@@ -266,19 +266,32 @@ struct LatTile {
 };
 constexpr size_t TILE_SMEM = 112u * 1024u, TILE_SMEM_ALONE = 200u * 1024u;
 
-template <int UW>
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm4_trans(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src));
+}
+
+// RANK: the latent size when it is 128 * UW (addresses are then constants), or 0 for any other.
+template <int UW, int RANK>
 __global__ void __launch_bounds__(256, 2) latent_tiles_kernel(LatArgs a, uint32_t stages) {
     using namespace attn_mma;
-    constexpr int LT = LatTile<UW>::TOKENS, SC_PITCH = LatTile<UW>::PITCH, P_PITCH = SC_PITCH, TPL = LT / 32;
+    constexpr int LT = LatTile<UW>::TOKENS, PITCH = LatTile<UW>::PITCH, TPL = LT / 32;
     extern __shared__ __align__(128) unsigned char lt_smem[];
-    float* sc = reinterpret_cast<float*>(lt_smem);                              // [8][16][SC_PITCH]
-    __half* sp = reinterpret_cast<__half*>(sc + 8 * 16 * SC_PITCH);             // [16][P_PITCH]
-    float* scorr = reinterpret_cast<float*>(sp + 16 * P_PITCH);                 // [16]
-    __half* ring = reinterpret_cast<__half*>(lt_smem + LatTile<UW>::FIXED);
+    float* sc = reinterpret_cast<float*>(lt_smem);                  // [8][16][PITCH]
+    __half* sp = reinterpret_cast<__half*>(sc + 8 * 16 * PITCH);    // [16][PITCH]
+    float* scorr = reinterpret_cast<float*>(sp + 16 * PITCH);       // [16]
+    const uint32_t ring = (uint32_t)__cvta_generic_to_shared(lt_smem + LatTile<UW>::FIXED);
     pdl_wait();
     pdl_trigger();
+    const uint32_t rank = RANK ? (uint32_t)RANK : a.rank;
     const uint32_t split = blockIdx.x, h0 = blockIdx.y * 16u, row = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
-    const uint32_t g = lane >> 2, t4 = lane & 3u, jm = lane >> 3, NU = a.rank / 16u, pitch = a.rank + 8u;
+    const uint32_t g = lane >> 2, t4 = lane & 3u, jm = lane >> 3, NU = rank / 16u, pitch = (rank + 8u) * 2u, tile_bytes = LT * pitch;
     const uint32_t pos = a.row_pos[row], slot = a.row_seq[row] * a.slot_mul + a.slot_add;
     const uint32_t lo = split * a.chunk, hi = min(lo + a.chunk, pos + 1u), heads = min(16u, a.heads - h0);
     if (slot >= a.slots || pos >= a.max_seq_len || lo >= hi) {  // empty partials
@@ -288,18 +301,25 @@ __global__ void __launch_bounds__(256, 2) latent_tiles_kernel(LatArgs a, uint32_
         }
         return;
     }
-    const __half* C = reinterpret_cast<const __half*>(a.C) + (size_t)slot * a.max_seq_len * a.rank;
-    const uint32_t n_tiles = (hi - lo + LT - 1u) / LT, pieces = a.rank / 8u;
+    const __half* C = reinterpret_cast<const __half*>(a.C) + (size_t)slot * a.max_seq_len * rank;
+    const uint32_t n_tiles = (hi - lo + LT - 1u) / LT, pieces = rank / 8u;
     // this thread's 16-byte pieces of a tile: every 256th, as (token, piece) pairs that are stepped, not divided for
     const uint32_t r_first = tid / pieces, ch_first = tid % pieces, r_step = 256u / pieces, ch_step = 256u % pieces;
     auto load_tile = [&](uint32_t tile, uint32_t slot_of_ring) {
-        __half* dst = ring + (size_t)slot_of_ring * LT * pitch;
-        const uint32_t base = lo + tile * LT;
-        const __half* src = C + (size_t)base * a.rank;
+        const uint32_t dst = ring + slot_of_ring * tile_bytes, base = lo + tile * LT;
+        const __half* src = C + (size_t)base * rank;
+        if (RANK && base + LT <= hi) {
+            constexpr uint32_t RS = RANK ? 2048u / RANK : 1u;  // tokens per 256 pieces
+            const __half* p = src + (size_t)r_first * rank + ch_first * 8u;
+            const uint32_t d = dst + r_first * pitch + ch_first * 16u;
+#pragma unroll
+            for (uint32_t i = 0; i < LT / RS; ++i) cp16(d + i * RS * pitch, p + (size_t)i * RS * rank);
+            return;
+        }
         const uint32_t last = hi - 1u - base;
         for (uint32_t r = r_first, ch = ch_first; r < LT;) {
             // rows past the end repeat the last visible one: masked below, and their bytes are finite
-            cp_async16(dst + r * pitch + ch * 8u, src + min(r, last) * a.rank + ch * 8u);
+            cp16(dst + r * pitch + ch * 16u, src + min(r, last) * rank + ch * 8u);
             r += r_step, ch += ch_step;
             if (ch >= pieces) ch -= pieces, ++r;
         }
@@ -314,14 +334,13 @@ __global__ void __launch_bounds__(256, 2) latent_tiles_kernel(LatArgs a, uint32_
 #pragma unroll
     for (int i = 0; i < UW; ++i) {
         const uint32_t u = warp * UW + i, k0 = u * 16u + 2u * t4;
-        float2 x[4];
 #pragma unroll
         for (int j = 0; j < 4; ++j) {  // rows g, g + 8 of columns k0, then of k0 + 8
             const uint32_t h = g + (j & 1) * 8u;
-            x[j] = u < NU && h < heads
-                       ? *reinterpret_cast<const float2*>(a.qa + ((size_t)row * a.heads + h0 + h) * a.rank + k0 + (j >> 1) * 8u)
-                       : make_float2(0.f, 0.f);
-            split_h2(x[j].x * qs, x[j].y * qs, &qhi[i][j], &qlo[i][j]);
+            const float2 x = (RANK || u < NU) && h < heads
+                                 ? *reinterpret_cast<const float2*>(a.qa + ((size_t)row * a.heads + h0 + h) * rank + k0 + (j >> 1) * 8u)
+                                 : make_float2(0.f, 0.f);
+            split_h2(x.x * qs, x.y * qs, &qhi[i][j], &qlo[i][j]);
         }
     }
     float o[UW][2][4];
@@ -330,7 +349,13 @@ __global__ void __launch_bounds__(256, 2) latent_tiles_kernel(LatArgs a, uint32_
 #pragma unroll
         for (int j = 0; j < 8; ++j) o[i][j >> 2][j & 3] = 0.0f;
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};  // heads 2 * warp and 2 * warp + 1
-    const uint32_t busy = (NU + UW - 1u) / UW;                         // warps that own columns
+    const uint32_t busy = RANK ? 8u : (NU + UW - 1u) / UW;             // warps that own columns
+    // this lane's ldmatrix rows: tokens (jm / 2) * 8 + lane % 8 as keys, (jm % 2) * 8 + lane % 8 as values, P's row lane % 16
+    const uint32_t key_at = ((jm >> 1) * 8u + (lane & 7u)) * pitch + (jm & 1u) * 16u + warp * UW * 32u;
+    const uint32_t val_at = ((jm & 1u) * 8u + (lane & 7u)) * pitch + (jm >> 1) * 16u + warp * UW * 32u;
+    const uint32_t p_at = (uint32_t)__cvta_generic_to_shared(sp) + ((lane & 15u) * PITCH + (lane >> 4) * 8u) * 2u;
+    float* sc_out = sc + ((size_t)warp * 16 + g) * PITCH + 2 * t4;
+    const float* sc_in = sc + 2u * warp * PITCH + lane;
 
     uint32_t here = 0;  // ring slot of this tile
     for (uint32_t tile = 0; tile < n_tiles; ++tile, here = here + 1u < stages ? here + 1u : 0u) {
@@ -343,79 +368,92 @@ __global__ void __launch_bounds__(256, 2) latent_tiles_kernel(LatArgs a, uint32_
         __syncthreads();
         if (tile + stages - 1u < n_tiles) load_tile(tile + stages - 1u, here ? here - 1u : stages - 1u);
         cp_async_commit();
-        const __half* tc = ring + (size_t)here * LT * pitch;
+        const uint32_t tile_at = ring + here * tile_bytes;
         if (warp < busy) {
             float s[LT / 8][4];
 #pragma unroll
             for (int j = 0; j < LT / 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.0f;
 #pragma unroll
             for (int i = 0; i < UW; ++i) {
-                const uint32_t u = warp * UW + i;
-                if (u >= NU) break;
+                if (!RANK && warp * UW + i >= NU) break;
 #pragma unroll
                 for (int p = 0; p < LT / 16; ++p) {
-                    const uint32_t r = p * 16 + (jm >> 1) * 8 + (lane & 7u);
                     uint32_t b[4];
-                    ldmatrix_x4(b, tc + r * pitch + u * 16u + (jm & 1u) * 8u);
+                    ldsm4(b, tile_at + key_at + p * 16u * pitch + i * 32u);
                     mma16816(s[2 * p], qhi[i][0], qhi[i][1], qhi[i][2], qhi[i][3], b[0], b[1]);
-                    mma16816(s[2 * p], qlo[i][0], qlo[i][1], qlo[i][2], qlo[i][3], b[0], b[1]);
                     mma16816(s[2 * p + 1], qhi[i][0], qhi[i][1], qhi[i][2], qhi[i][3], b[2], b[3]);
+                    mma16816(s[2 * p], qlo[i][0], qlo[i][1], qlo[i][2], qlo[i][3], b[0], b[1]);
                     mma16816(s[2 * p + 1], qlo[i][0], qlo[i][1], qlo[i][2], qlo[i][3], b[2], b[3]);
                 }
             }
-            float* mine = sc + (size_t)warp * 16 * SC_PITCH;
 #pragma unroll
             for (int j = 0; j < LT / 8; ++j) {
-                *reinterpret_cast<float2*>(mine + g * SC_PITCH + j * 8 + 2 * t4) = make_float2(s[j][0], s[j][1]);
-                *reinterpret_cast<float2*>(mine + (g + 8) * SC_PITCH + j * 8 + 2 * t4) = make_float2(s[j][2], s[j][3]);
+                *reinterpret_cast<float2*>(sc_out + j * 8) = make_float2(s[j][0], s[j][1]);
+                *reinterpret_cast<float2*>(sc_out + 8 * PITCH + j * 8) = make_float2(s[j][2], s[j][3]);
             }
         }
         __syncthreads();
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-            const uint32_t h = 2u * warp + e;
-            float v[TPL] = {}, mx = -INFINITY, ps = 0.0f;
+        {
+            float v[2][TPL] = {}, mx[2], ps[2] = {0.0f, 0.0f};
 #pragma unroll
             for (uint32_t w = 0; w < 8u; ++w)
-                if (w < busy) {
+                if (RANK || w < busy) {
 #pragma unroll
-                    for (int j = 0; j < TPL; ++j) v[j] += sc[((size_t)w * 16 + h) * SC_PITCH + lane + 32u * j];
+                    for (int e = 0; e < 2; ++e)
+#pragma unroll
+                        for (int j = 0; j < TPL; ++j) v[e][j] += sc_in[(w * 16 + e) * PITCH + 32 * j];
                 }
 #pragma unroll
-            for (int j = 0; j < TPL; ++j) {
-                if (lo + tile * LT + lane + 32u * j >= hi) v[j] = -INFINITY;
-                mx = fmaxf(mx, v[j]);
-            }
-            const float m_new = fmaxf(m_run[e], warp_max(mx));  // the tile's first token is visible: finite
-            const float corr = fast_exp2(m_run[e] - m_new);
+            for (int e = 0; e < 2; ++e) {
+                mx[e] = -INFINITY;
 #pragma unroll
-            for (int j = 0; j < TPL; ++j) {
-                const float p = fast_exp2(v[j] - m_new);
-                ps += p;
-                sp[h * P_PITCH + lane + 32u * j] = __float2half_rn(p);
+                for (int j = 0; j < TPL; ++j) {
+                    if (lo + tile * LT + lane + 32u * j >= hi) v[e][j] = -INFINITY;
+                    mx[e] = fmaxf(mx[e], v[e][j]);
+                }
             }
-            l_run[e] = l_run[e] * corr + warp_sum(ps);
-            m_run[e] = m_new;
-            if (lane == 0) scorr[h] = corr;
+#pragma unroll
+            for (int d = 16; d > 0; d >>= 1)  // the two heads' chains side by side
+#pragma unroll
+                for (int e = 0; e < 2; ++e) mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], d));
+            float corr[2];
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const float m_new = fmaxf(m_run[e], mx[e]);  // the tile's first token is visible: finite
+                corr[e] = fast_exp2(m_run[e] - m_new);
+                m_run[e] = m_new;
+#pragma unroll
+                for (int j = 0; j < TPL; ++j) {
+                    const float p = fast_exp2(v[e][j] - m_new);
+                    ps[e] += p;
+                    sp[(2u * warp + e) * PITCH + lane + 32u * j] = __float2half_rn(p);
+                }
+            }
+            // a lane keeps its own share of the sum; the shares meet at the end
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                l_run[e] = l_run[e] * corr[e] + ps[e];
+                if (lane == 0) scorr[2u * warp + e] = corr[e];
+            }
         }
         __syncthreads();
         if (warp < busy) {
             const float ca = scorr[g], cb = scorr[g + 8];
+            if (!__all_sync(0xffffffffu, ca == 1.0f && cb == 1.0f)) {
 #pragma unroll
-            for (int i = 0; i < UW; ++i)
+                for (int i = 0; i < UW; ++i)
 #pragma unroll
-                for (int n = 0; n < 2; ++n) o[i][n][0] *= ca, o[i][n][1] *= ca, o[i][n][2] *= cb, o[i][n][3] *= cb;
+                    for (int n = 0; n < 2; ++n) o[i][n][0] *= ca, o[i][n][1] *= ca, o[i][n][2] *= cb, o[i][n][3] *= cb;
+            }
 #pragma unroll
             for (int kk = 0; kk < LT / 16; ++kk) {
                 uint32_t pa[4];
-                ldmatrix_x4(pa, sp + (lane & 15u) * P_PITCH + kk * 16 + (lane >> 4) * 8u);
-                const uint32_t r = kk * 16 + (jm & 1u) * 8 + (lane & 7u);
+                ldsm4(pa, p_at + kk * 32u);
 #pragma unroll
                 for (int i = 0; i < UW; ++i) {
-                    const uint32_t u = warp * UW + i;
-                    if (u >= NU) break;
+                    if (!RANK && warp * UW + i >= NU) break;
                     uint32_t b[4];
-                    ldmatrix_x4_trans(b, tc + r * pitch + u * 16u + (jm >> 1) * 8u);
+                    ldsm4_trans(b, tile_at + val_at + kk * 16u * pitch + i * 32u);
                     mma16816(o[i][0], pa[0], pa[1], pa[2], pa[3], b[0], b[1]);
                     mma16816(o[i][1], pa[0], pa[1], pa[2], pa[3], b[2], b[3]);
                 }
@@ -426,21 +464,22 @@ __global__ void __launch_bounds__(256, 2) latent_tiles_kernel(LatArgs a, uint32_
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
         const uint32_t h = 2u * warp + e;
+        const float l = warp_sum(l_run[e]);
         if (lane == 0 && h < heads) {
             const size_t pi = ((size_t)row * a.heads + h0 + h) * a.splits + split;
             a.pm[pi] = m_run[e] * LN2;  // natural-log domain, as in the other form
-            a.pl[pi] = l_run[e];
+            a.pl[pi] = l;
         }
     }
 #pragma unroll
     for (int i = 0; i < UW; ++i) {
         const uint32_t u = warp * UW + i;
-        if (u >= NU) break;
+        if (!RANK && u >= NU) break;
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
             const uint32_t h = g + 8u * j;
             if (h >= heads) continue;
-            float* dst = a.po + (((size_t)row * a.heads + h0 + h) * a.splits + split) * a.rank + u * 16u + 2u * t4;
+            float* dst = a.po + (((size_t)row * a.heads + h0 + h) * a.splits + split) * rank + u * 16u + 2u * t4;
 #pragma unroll
             for (int n = 0; n < 2; ++n) *reinterpret_cast<float2*>(dst + n * 8) = make_float2(o[i][n][2 * j], o[i][n][2 * j + 1]);
         }
@@ -672,12 +711,13 @@ cudaError_t prepare(cudaStream_t s, const LatArgs& a, bool f32, bool append) {
     return f32 ? launch_prepare<WT, float>(s, a, append) : launch_prepare<WT, __half>(s, a, append);
 }
 
-template <int UW>
-cudaError_t launch_tiles(M40llmCudaContext* ctx, const LatArgs& a) {
+template <int UW, int RANK>
+cudaError_t launch_tiles_as(M40llmCudaContext* ctx, const LatArgs& a) {
     static unsigned long long configured = 0ull;
     const unsigned long long bit = 1ull << (ctx->device_id & 63);
+    auto kernel = latent_tiles_kernel<UW, RANK>;
     if (!(configured & bit)) {
-        const cudaError_t e = cudaFuncSetAttribute(latent_tiles_kernel<UW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TILE_SMEM_ALONE);
+        const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TILE_SMEM_ALONE);
         if (e != cudaSuccess) return e;
         configured |= bit;
     }
@@ -686,8 +726,12 @@ cudaError_t launch_tiles(M40llmCudaContext* ctx, const LatArgs& a) {
     const bool alone = (uint64_t)grid.x * grid.y * grid.z <= (uint64_t)ctx->sm_count;
     size_t stages = ((alone ? TILE_SMEM_ALONE : TILE_SMEM) - LatTile<UW>::FIXED) / LatTile<UW>::bytes(a.rank);
     if (stages > 5) stages = 5;
-    return m40_launch_dependent(latent_tiles_kernel<UW>, grid, dim3(256), LatTile<UW>::FIXED + stages * LatTile<UW>::bytes(a.rank),
-                                ctx->decode_stream, a, (uint32_t)stages);
+    return m40_launch_dependent(kernel, grid, dim3(256), LatTile<UW>::FIXED + stages * LatTile<UW>::bytes(a.rank), ctx->decode_stream, a,
+                                (uint32_t)stages);
+}
+template <int UW>
+cudaError_t launch_tiles(M40llmCudaContext* ctx, const LatArgs& a) {
+    return a.rank == 128u * UW ? launch_tiles_as<UW, 128 * UW>(ctx, a) : launch_tiles_as<UW, 0>(ctx, a);
 }
 static_assert(LatTile<2>::FIXED + 2 * LatTile<2>::bytes(256) <= TILE_SMEM && LatTile<4>::FIXED + 2 * LatTile<4>::bytes(512) <= TILE_SMEM,
               "two tiles of the largest rank");
