@@ -23,6 +23,7 @@ namespace {
 constexpr uint32_t MAX_RANK = 1024;
 constexpr uint32_t RUN_ROWS = 512;   // rows per pass of the absorbed form (bounds the work space)
 constexpr uint32_t EXPAND_ROWS = 64;
+constexpr uint32_t TEAM_ROWS = 4;
 constexpr uint32_t GROUPED_ROWS = 8;    // rows from which uk and uv go through the grouped GEMM
 constexpr size_t EXPAND_BYTES = (size_t)1 << 30;  // work space for one portion's keys and values
 
@@ -277,23 +278,31 @@ __device__ __forceinline__ void cp16(uint32_t dst, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src));
 }
 
-// RANK: the latent size when it is 128 * UW (addresses are then constants), or 0 for any other.
-template <int UW, int RANK>
-__global__ void __launch_bounds__(256, 2) latent_tiles_kernel(LatArgs a, uint32_t stages) {
+// RANK: the latent size when it is 128 * UW (addresses are then constants), or 0 for any other. TEAMS = 2: two teams of eight
+// warps with 16 heads each share one ring (one CTA per SM), so that the latents are fetched once for 32 heads.
+template <int UW, int RANK, int TEAMS>
+__global__ void __launch_bounds__(256 * TEAMS, TEAMS == 2 ? 1 : 2) latent_tiles_kernel(LatArgs a, uint32_t stages) {
     using namespace attn_mma;
     constexpr int LT = LatTile<UW>::TOKENS, PITCH = LatTile<UW>::PITCH, TPL = LT / 32;
     extern __shared__ __align__(128) unsigned char lt_smem[];
-    float* sc = reinterpret_cast<float*>(lt_smem);                  // [8][16][PITCH]
+    constexpr uint32_t NT = 256u * TEAMS;
+    const uint32_t team = TEAMS == 2 ? threadIdx.x >> 8 : 0u;
+    float* sc = reinterpret_cast<float*>(lt_smem + team * LatTile<UW>::FIXED);  // [8][16][PITCH]
     __half* sp = reinterpret_cast<__half*>(sc + 8 * 16 * PITCH);    // [16][PITCH]
     float* scorr = reinterpret_cast<float*>(sp + 16 * PITCH);       // [16]
-    const uint32_t ring = (uint32_t)__cvta_generic_to_shared(lt_smem + LatTile<UW>::FIXED);
+    const uint32_t ring = (uint32_t)__cvta_generic_to_shared(lt_smem + TEAMS * LatTile<UW>::FIXED);
+    auto team_barrier = [&]() {
+        if (TEAMS == 1) __syncthreads();
+        else asm volatile("bar.sync %0, 256;" ::"r"(team + 1u) : "memory");
+    };
     pdl_wait();
     pdl_trigger();
     const uint32_t rank = RANK ? (uint32_t)RANK : a.rank;
-    const uint32_t split = blockIdx.x, h0 = blockIdx.y * 16u, row = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
+    const uint32_t split = blockIdx.x, h0 = (blockIdx.y * TEAMS + team) * 16u, row = blockIdx.z;
+    const uint32_t tid = threadIdx.x & 255u, warp = tid >> 5, lane = tid & 31u;
     const uint32_t g = lane >> 2, t4 = lane & 3u, jm = lane >> 3, NU = rank / 16u, pitch = (rank + 8u) * 2u, tile_bytes = LT * pitch;
     const uint32_t pos = a.row_pos[row], slot = a.row_seq[row] * a.slot_mul + a.slot_add;
-    const uint32_t lo = split * a.chunk, hi = min(lo + a.chunk, pos + 1u), heads = min(16u, a.heads - h0);
+    const uint32_t lo = split * a.chunk, hi = min(lo + a.chunk, pos + 1u), heads = h0 < a.heads ? min(16u, a.heads - h0) : 0u;
     if (slot >= a.slots || pos >= a.max_seq_len || lo >= hi) {  // empty partials
         if (tid < heads) {
             const size_t pi = ((size_t)row * a.heads + h0 + tid) * a.splits + split;
@@ -303,13 +312,13 @@ __global__ void __launch_bounds__(256, 2) latent_tiles_kernel(LatArgs a, uint32_
     }
     const __half* C = reinterpret_cast<const __half*>(a.C) + (size_t)slot * a.max_seq_len * rank;
     const uint32_t n_tiles = (hi - lo + LT - 1u) / LT, pieces = rank / 8u;
-    // this thread's 16-byte pieces of a tile: every 256th, as (token, piece) pairs that are stepped, not divided for
-    const uint32_t r_first = tid / pieces, ch_first = tid % pieces, r_step = 256u / pieces, ch_step = 256u % pieces;
+    // this thread's 16-byte pieces of a tile: every NT-th, as (token, piece) pairs that are stepped, not divided for
+    const uint32_t r_first = threadIdx.x / pieces, ch_first = threadIdx.x % pieces, r_step = NT / pieces, ch_step = NT % pieces;
     auto load_tile = [&](uint32_t tile, uint32_t slot_of_ring) {
         const uint32_t dst = ring + slot_of_ring * tile_bytes, base = lo + tile * LT;
         const __half* src = C + (size_t)base * rank;
         if (RANK && base + LT <= hi) {
-            constexpr uint32_t RS = RANK ? 2048u / RANK : 1u;  // tokens per 256 pieces
+            constexpr uint32_t RS = RANK ? NT * 8u / RANK : 1u;  // tokens per NT pieces
             const __half* p = src + (size_t)r_first * rank + ch_first * 8u;
             const uint32_t d = dst + r_first * pitch + ch_first * 16u;
 #pragma unroll
@@ -392,7 +401,7 @@ __global__ void __launch_bounds__(256, 2) latent_tiles_kernel(LatArgs a, uint32_
                 *reinterpret_cast<float2*>(sc_out + 8 * PITCH + j * 8) = make_float2(s[j][2], s[j][3]);
             }
         }
-        __syncthreads();
+        team_barrier();
         {
             float v[2][TPL] = {}, mx[2], ps[2] = {0.0f, 0.0f};
 #pragma unroll
@@ -436,7 +445,7 @@ __global__ void __launch_bounds__(256, 2) latent_tiles_kernel(LatArgs a, uint32_
                 if (lane == 0) scorr[2u * warp + e] = corr[e];
             }
         }
-        __syncthreads();
+        team_barrier();
         if (warp < busy) {
             const float ca = scorr[g], cb = scorr[g + 8];
             if (!__all_sync(0xffffffffu, ca == 1.0f && cb == 1.0f)) {
@@ -711,35 +720,38 @@ cudaError_t prepare(cudaStream_t s, const LatArgs& a, bool f32, bool append) {
     return f32 ? launch_prepare<WT, float>(s, a, append) : launch_prepare<WT, __half>(s, a, append);
 }
 
-template <int UW, int RANK>
+template <int UW, int RANK, int TEAMS>
 cudaError_t launch_tiles_as(M40llmCudaContext* ctx, const LatArgs& a) {
     static unsigned long long configured = 0ull;
     const unsigned long long bit = 1ull << (ctx->device_id & 63);
-    auto kernel = latent_tiles_kernel<UW, RANK>;
+    auto kernel = latent_tiles_kernel<UW, RANK, TEAMS>;
     if (!(configured & bit)) {
         const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TILE_SMEM_ALONE);
         if (e != cudaSuccess) return e;
         configured |= bit;
     }
-    const dim3 grid(a.splits, (a.heads + 15) / 16, a.rows);
+    const dim3 grid(a.splits, (a.heads + 16 * TEAMS - 1) / (16 * TEAMS), a.rows);
     // a launch that gives every SM at most one CTA lets it have the shared memory of two: a deeper ring
-    const bool alone = (uint64_t)grid.x * grid.y * grid.z <= (uint64_t)ctx->sm_count;
-    size_t stages = ((alone ? TILE_SMEM_ALONE : TILE_SMEM) - LatTile<UW>::FIXED) / LatTile<UW>::bytes(a.rank);
+    const bool alone = TEAMS == 2 || (uint64_t)grid.x * grid.y * grid.z <= (uint64_t)ctx->sm_count;
+    constexpr size_t fixed = TEAMS * LatTile<UW>::FIXED;
+    size_t stages = ((alone ? TILE_SMEM_ALONE : TILE_SMEM) - fixed) / LatTile<UW>::bytes(a.rank);
     if (stages > 5) stages = 5;
-    return m40_launch_dependent(kernel, grid, dim3(256), LatTile<UW>::FIXED + stages * LatTile<UW>::bytes(a.rank), ctx->decode_stream, a,
+    return m40_launch_dependent(kernel, grid, dim3(256 * TEAMS), fixed + stages * LatTile<UW>::bytes(a.rank), ctx->decode_stream, a,
                                 (uint32_t)stages);
 }
 template <int UW>
-cudaError_t launch_tiles(M40llmCudaContext* ctx, const LatArgs& a) {
-    return a.rank == 128u * UW ? launch_tiles_as<UW, 128 * UW>(ctx, a) : launch_tiles_as<UW, 0>(ctx, a);
+cudaError_t launch_tiles(M40llmCudaContext* ctx, const LatArgs& a, uint32_t teams) {
+    if (teams == 2) return a.rank == 128u * UW ? launch_tiles_as<UW, 128 * UW, 2>(ctx, a) : launch_tiles_as<UW, 0, 2>(ctx, a);
+    return a.rank == 128u * UW ? launch_tiles_as<UW, 128 * UW, 1>(ctx, a) : launch_tiles_as<UW, 0, 1>(ctx, a);
 }
 static_assert(LatTile<2>::FIXED + 2 * LatTile<2>::bytes(256) <= TILE_SMEM && LatTile<4>::FIXED + 2 * LatTile<4>::bytes(512) <= TILE_SMEM,
               "two tiles of the largest rank");
+static_assert(2 * LatTile<4>::FIXED + 2 * LatTile<4>::bytes(512) <= TILE_SMEM_ALONE, "two teams");
 
-// Tokens per split: as many splits as keep every CTA of the launch resident (two per SM), at least 128 tokens each; at most
+// Tokens per split: as many splits as keep every CTA of the launch resident (`slots` of them), at least 128 tokens each; at most
 // 1024, because the bound may be the cache's capacity when the lengths are not known.
-void pick_splits(const M40llmCudaContext* ctx, uint32_t ctas_per_split, uint32_t bound, uint32_t* chunk, uint32_t* splits) {
-    uint32_t n = 2u * (uint32_t)ctx->sm_count / ctas_per_split;
+void pick_splits(uint32_t slots, uint32_t ctas_per_split, uint32_t bound, uint32_t* chunk, uint32_t* splits) {
+    uint32_t n = slots / ctas_per_split;
     n = n < 1u ? 1u : (n > 128u ? 128u : n);
     uint32_t c = ((bound + n - 1) / n + 63u) & ~63u;
     c = c < 128u ? 128u : (c > 1024u ? 1024u : c);
@@ -789,7 +801,10 @@ int run_absorbed(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs&
         a.row_seq += at;
         a.row_pos += at;
         const bool grouped = a.rows >= GROUPED_ROWS && takes_grouped(kv, a, w_dtype);
-        pick_splits(ctx, a.rows * (tiles ? (a.heads + 15) / 16 : a.heads), bound, &a.chunk, &a.splits);
+        // two teams per CTA where there are heads for them and rows enough to give every SM work
+        const uint32_t teams = tiles && a.heads > 16 && a.rows >= TEAM_ROWS ? 2 : 1, sms = (uint32_t)ctx->sm_count;
+        if (teams == 2) pick_splits(sms, a.rows * ((a.heads + 31) / 32), bound, &a.chunk, &a.splits);
+        else pick_splits(2u * sms, a.rows * (tiles ? (a.heads + 15) / 16 : a.heads), bound, &a.chunk, &a.splits);
         const size_t nh = (size_t)a.rows * a.heads, np = nh * a.splits;
         auto pad = [](size_t v) { return (v + 63) & ~(size_t)63; };
         const size_t part = grouped ? pad(nh * (a.rank > a.dim ? a.rank : a.dim)) : 0;  // 16-bit values
@@ -817,7 +832,8 @@ int run_absorbed(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs&
         }
         const dim3 grid(a.heads, a.rows, a.splits);
         if (tiles)
-            e = a.rank <= 128 ? launch_tiles<1>(ctx, a) : (a.rank <= 256 ? launch_tiles<2>(ctx, a) : launch_tiles<4>(ctx, a));
+            e = a.rank <= 128 ? launch_tiles<1>(ctx, a, teams)
+                              : (a.rank <= 256 ? launch_tiles<2>(ctx, a, teams) : launch_tiles<4>(ctx, a, teams));
         else
             e = kv->elem_f32 ? m40_launch_dependent(latent_rows_kernel<float>, grid, dim3(128), 0, s, a)
                              : m40_launch_dependent(latent_rows_kernel<__half>, grid, dim3(128), 0, s, a);
