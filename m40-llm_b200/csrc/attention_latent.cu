@@ -752,7 +752,12 @@ static_assert(2 * LatTile<4>::FIXED + 2 * LatTile<4>::bytes(512) <= TILE_SMEM_AL
 // 1024, because the bound may be the cache's capacity when the lengths are not known.
 void pick_splits(uint32_t slots, uint32_t ctas_per_split, uint32_t bound, uint32_t* chunk, uint32_t* splits) {
     uint32_t n = slots / ctas_per_split;
-    n = n < 1u ? 1u : (n > 128u ? 128u : n);
+    if (n <= 1u) {  // rows enough: no splits, whatever the length
+        *chunk = bound;
+        *splits = 1u;
+        return;
+    }
+    n = n > 128u ? 128u : n;
     uint32_t c = ((bound + n - 1) / n + 63u) & ~63u;
     c = c < 128u ? 128u : (c > 1024u ? 1024u : c);
     if ((bound + c - 1) / c > 128u) c = ((bound + 127u) / 128u + 63u) & ~63u;
