@@ -12,6 +12,8 @@
 //   that pass does not take, after moe_gather_kernel).
 #include "moe.cuh"
 
+#include <math.h>
+
 #include "gemm_tc_grouped.cuh"
 #include "norm_rows.cuh"
 
@@ -283,10 +285,13 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(M40MoeArgs a) {
     *reinterpret_cast<float4*>(a.y + at) = y;
 }
 
-// Rows of a tile: about the rows an expert gets, so that an expert's weights are read once and tiles are mostly full.
-uint32_t pick_tile_rows(uint32_t slots, uint32_t experts) {
-    const uint32_t avg = (slots + experts - 1) / experts;
-    return avg <= 16 ? 16 : (avg <= 32 ? 32 : (avg <= 96 ? 64 : 128));
+// Rows of a tile: the rows that all but the most crowded experts get (their mean and two standard deviations of an even
+// routing), dealt to as few tiles of at most 128 as hold them. So tiles are mostly full and weights mostly read once.
+uint32_t pick_tile_rows(uint64_t slots, uint32_t outputs) {
+    const double avg = (double)slots / outputs, most = avg + 2.0 * sqrt(avg);
+    const uint32_t n = (uint32_t)ceil(most), tiles = (n + 127u) / 128u;
+    const uint32_t rows = ((n + tiles - 1u) / tiles + 15u) / 16u * 16u;
+    return rows < 16u ? 16u : (rows > 128u ? 128u : rows);
 }
 
 // `after`: the norm of these rows.
@@ -391,7 +396,7 @@ extern "C" int m40llm_moe_async(M40llmCudaContext* ctx, const M40llmMoe* c, uint
     if (tensor && pass > PASS_SLOTS / c->top) pass = PASS_SLOTS / c->top;
     if (pass > c->rows) pass = c->rows;
     const uint64_t slots = pass * c->top;
-    a.tile_rows = pick_tile_rows((uint32_t)slots, c->experts);
+    a.tile_rows = pick_tile_rows(slots, (uint32_t)n);
     const uint32_t max_tiles = (uint32_t)(slots / a.tile_rows + (c->experts < slots ? c->experts : slots));
     const uint64_t sorted = (uint64_t)max_tiles * a.tile_rows;
     size_t used = 0;
