@@ -292,8 +292,9 @@ int m40_gemm_tc_grouped(M40llmCudaContext* ctx, cudaStream_t s, const M40Grouped
     a.head_pitch = c.head_pitch;
     a.rg = c.rg;
     const uint32_t stage = tc::BLOCK_N * tc::BLOCK_K * 2 + c.parts * c.tile_rows * tc::BLOCK_K * 2;
-    uint32_t stages = 100u * 1024u / stage;
-    if (stages > 8) stages = 8;
+    // a short ring and three CTAs per SM where the tile allows it: their prologues and epilogues cover one another
+    uint32_t stages = 66u * 1024u / stage;
+    if (stages < 2) stages = 2;
     if (stages > a.kblocks) stages = a.kblocks;
     // the paired epilogue passes tile_rows * 64 f32 through the ring
     const uint32_t least = paired ? (c.tile_rows * 64u * 4u + stage - 1) / stage : 1u;

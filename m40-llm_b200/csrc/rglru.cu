@@ -291,7 +291,7 @@ int run_rows(M40llmCudaContext* ctx, RgArgs g, uint32_t blocks, const M40llmStep
         q.N = q.K = q.group_k = g.bs;
         q.x_rows = g.rows;
         q.ldx = g.width;
-        q.tile_rows = g.rows > 32 ? 64 : 32;
+        q.tile_rows = 32;
         q.kind = M40_GROUPED_RG;
         q.rg = g;
         if ((rc = m40_gemm_tc_grouped(ctx, s, q)) != 0) return rc;
