@@ -17,6 +17,7 @@
 #include "attention_mma.cuh"
 #include "gemm_tc_grouped.cuh"
 #include "stack_math.cuh"
+#include "tc_ptx.cuh"
 
 namespace {
 
@@ -257,7 +258,10 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(LatArgs a) {
 // absorbed queries of 16 heads with the tile over its own columns (mma.sync, query split into f16 hi + lo), the eight partial
 // score tiles are added in shared memory, two heads per warp run the online softmax (base 2), and every warp adds P c for its
 // columns. So a latent is read from shared memory once as key and once as value, whatever the number of heads.
-// Two CTAs share an SM, so that one's barriers and softmax hide behind the other's products.
+// Two CTAs, or two teams of warps, share an SM, so that one's barriers and softmax hide behind the other's products. The ring
+// of tiles is handed over by mbarriers (every thread copies its pieces with cp.async, every warp releases a tile when it has
+// used it), so that the teams need not keep step. Every wait is bounded: one that runs out raises status bit 4, and from then
+// on nothing waits.
 template <int UW>
 struct LatTile {
     static constexpr int TOKENS = UW <= 2 ? 64 : 32;
@@ -265,6 +269,7 @@ struct LatTile {
     static constexpr size_t FIXED = ((size_t)8 * 16 * PITCH * 4 + (size_t)16 * PITCH * 2 + 16 * 4 + 127) / 128 * 128;
     static constexpr size_t bytes(uint32_t rank) { return (size_t)TOKENS * (rank + 8u) * 2u; }
 };
+constexpr uint32_t MAX_STAGES = 6;
 constexpr size_t TILE_SMEM = 112u * 1024u, TILE_SMEM_ALONE = 200u * 1024u;
 
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
@@ -274,6 +279,7 @@ __device__ __forceinline__ void ldsm4_trans(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
+__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 __device__ __forceinline__ void cp16(uint32_t dst, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src));
 }
@@ -287,6 +293,8 @@ __global__ void __launch_bounds__(256 * TEAMS, TEAMS == 2 ? 1 : 2) latent_tiles_
     extern __shared__ __align__(128) unsigned char lt_smem[];
     constexpr uint32_t NT = 256u * TEAMS;
     const uint32_t team = TEAMS == 2 ? threadIdx.x >> 8 : 0u;
+    __shared__ uint64_t full[MAX_STAGES], empty[MAX_STAGES];
+    __shared__ volatile uint32_t abort_flag;
     float* sc = reinterpret_cast<float*>(lt_smem + team * LatTile<UW>::FIXED);  // [8][16][PITCH]
     __half* sp = reinterpret_cast<__half*>(sc + 8 * 16 * PITCH);    // [16][PITCH]
     float* scorr = reinterpret_cast<float*>(sp + 16 * PITCH);       // [16]
@@ -295,6 +303,15 @@ __global__ void __launch_bounds__(256 * TEAMS, TEAMS == 2 ? 1 : 2) latent_tiles_
         if (TEAMS == 1) __syncthreads();
         else asm volatile("bar.sync %0, 256;" ::"r"(team + 1u) : "memory");
     };
+    if (threadIdx.x == 0) {
+        for (uint32_t i = 0; i < stages; ++i) {
+            tc::mbar_init(&full[i], NT);
+            tc::mbar_init(&empty[i], NT / 32u);
+        }
+        abort_flag = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncthreads();
     pdl_wait();
     pdl_trigger();
     const uint32_t rank = RANK ? (uint32_t)RANK : a.rank;
@@ -333,9 +350,20 @@ __global__ void __launch_bounds__(256 * TEAMS, TEAMS == 2 ? 1 : 2) latent_tiles_
             if (ch >= pieces) ch -= pieces, ++r;
         }
     };
-    for (uint32_t t = 0; t + 1u < stages; ++t) {
-        if (t < n_tiles) load_tile(t, t);
-        cp_async_commit();
+    auto wait = [&](uint64_t* bar, uint32_t parity) {
+        if (!abort_flag && !tc::mbar_wait(bar, parity)) {
+            abort_flag = 1;
+            atomicOr(a.status, 4u);
+        }
+    };
+    auto landed_on = [&](uint64_t* bar) {  // this thread's copies so far arrive on the barrier when they have landed
+        asm volatile("cp.async.mbarrier.arrive.noinc.shared::cta.b64 [%0];" ::"r"(tc::smem_u32(bar)) : "memory");
+    };
+    // tiles in flight ahead of the one in use; with four slots or more, one stays free so that a team may lag by a tile
+    const uint32_t ahead = stages >= 4u ? stages - 2u : stages - 1u;
+    for (uint32_t t = 0; t < ahead && t < n_tiles; ++t) {
+        load_tile(t, t);
+        landed_on(&full[t]);
     }
     // query fragments of this warp's columns
     uint32_t qhi[UW][4], qlo[UW][4];
@@ -366,17 +394,16 @@ __global__ void __launch_bounds__(256 * TEAMS, TEAMS == 2 ? 1 : 2) latent_tiles_
     float* sc_out = sc + ((size_t)warp * 16 + g) * PITCH + 2 * t4;
     const float* sc_in = sc + 2u * warp * PITCH + lane;
 
-    uint32_t here = 0;  // ring slot of this tile
-    for (uint32_t tile = 0; tile < n_tiles; ++tile, here = here + 1u < stages ? here + 1u : 0u) {
-        switch (stages) {  // all but the newest stages - 2 groups have landed
-            case 2: cp_async_wait<0>(); break;
-            case 3: cp_async_wait<1>(); break;
-            case 4: cp_async_wait<2>(); break;
-            default: cp_async_wait<3>();
+    // ring slots and use numbers of this tile and of the one to be requested
+    uint32_t here = 0, here_use = 0, next = ahead % stages, next_use = ahead / stages;
+    for (uint32_t tile = 0; tile < n_tiles; ++tile) {
+        if (tile + ahead < n_tiles) {
+            if (next_use > 0u) wait(&empty[next], (next_use - 1u) & 1u);
+            load_tile(tile + ahead, next);
+            landed_on(&full[next]);
         }
-        __syncthreads();
-        if (tile + stages - 1u < n_tiles) load_tile(tile + stages - 1u, here ? here - 1u : stages - 1u);
-        cp_async_commit();
+        if (++next == stages) next = 0, ++next_use;
+        wait(&full[here], here_use & 1u);
         const uint32_t tile_at = ring + here * tile_bytes;
         if (warp < busy) {
             float s[LT / 8][4];
@@ -468,8 +495,11 @@ __global__ void __launch_bounds__(256 * TEAMS, TEAMS == 2 ? 1 : 2) latent_tiles_
                 }
             }
         }
+        __syncwarp();
+        if (lane == 0) tc::mbar_arrive(&empty[here]);
+        if (++here == stages) here = 0, ++here_use;
     }
-    cp_async_wait<0>();
+    cp_async_wait_all();
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
         const uint32_t h = 2u * warp + e;
@@ -735,7 +765,7 @@ cudaError_t launch_tiles_as(M40llmCudaContext* ctx, const LatArgs& a) {
     const bool alone = TEAMS == 2 || (uint64_t)grid.x * grid.y * grid.z <= (uint64_t)ctx->sm_count;
     constexpr size_t fixed = TEAMS * LatTile<UW>::FIXED;
     size_t stages = ((alone ? TILE_SMEM_ALONE : TILE_SMEM) - fixed) / LatTile<UW>::bytes(a.rank);
-    if (stages > 5) stages = 5;
+    if (stages > MAX_STAGES) stages = MAX_STAGES;
     return m40_launch_dependent(kernel, grid, dim3(256 * TEAMS), fixed + stages * LatTile<UW>::bytes(a.rank), ctx->decode_stream, a,
                                 (uint32_t)stages);
 }
