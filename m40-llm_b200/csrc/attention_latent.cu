@@ -6,13 +6,17 @@
 //   latent_prepare_kernel  uk^T q per head (absorbed query), and the latent's norm and append; with several rows on the tensor
 //                          path latent_append_kernel (append, and the queries cut into hi + lo) and a grouped tcgen05 GEMM;
 //   attention over latents, one of
-//     latent_tiles_kernel  f16 cache, rank a multiple of 16 up to 512: CTA = (row, 16 heads, token split). The tokens' latents
-//                          stream once through shared memory and serve all 16 heads, as keys and as values;
+//     latent_tc_kernel     (attention_latent_tc.cu) f16 cache, rank a multiple of 128 up to 512: tcgen05, CTA = (row, 32 heads,
+//                          token split);
+//     latent_tiles_kernel  f16 cache, rank a multiple of 16 up to 512: mma.sync, CTA = (row, 16 heads, token split). In both the
+//                          tokens' latents stream once through shared memory and serve all the heads, as keys and as values;
 //     latent_rows_kernel   any rank, f16 or f32 cache, f32 arithmetic: CTA = (head, row, token split);
 //   latent_merge_kernel    merges the token splits and the sink, then uv (itself, or as a grouped GEMM of several rows).
 // Long portions (segments of EXPAND_ROWS rows or more, f16 cache) do less work with the heads' keys and values in hand: they
 // are made once per portion from the cached latents by the grouped tcgen05 GEMM, f16 and head-major, and the prompt kernel of
 // attention_prefill.cu attends them.
+#include "attention_latent.cuh"
+
 #include "attention.cuh"
 #include "attention_mma.cuh"
 #include "gemm_tc_grouped.cuh"
@@ -28,28 +32,7 @@ constexpr uint32_t TEAM_ROWS = 4;
 constexpr uint32_t GROUPED_ROWS = 8;    // rows from which uk and uv go through the grouped GEMM
 constexpr size_t EXPAND_BYTES = (size_t)1 << 30;  // work space for one portion's keys and values
 
-struct LatArgs {
-    const float* packed;   // of the pass's first row
-    const float* c_norm;
-    const void* uk;
-    const void* uk_t;
-    const void* uv;
-    const float* sink;
-    void* C;
-    __nv_bfloat16* part[2];  // tensor path: hi and lo of the queries [rows][heads * dim], then of the weighted latents
-    uint32_t* seq_map;
-    float* qa;             // absorbed queries [rows][heads][rank]
-    float* pm;             // [rows][heads][splits]
-    float* pl;
-    float* po;             // [rows][heads][splits][rank]
-    float* out;
-    uint32_t* status;
-    const uint32_t* row_seq;
-    const uint32_t* row_pos;
-    uint32_t ld, heads, dim, vdim, rank, slot_mul, slot_add, slots, max_seq_len, rows, splits, chunk;
-    uint32_t absorb_ctas, wide;
-    float eps, scale;
-};
+using LatArgs = M40LatArgs;
 
 __device__ __forceinline__ float block_sum_256(float v, float* red) {
     v = warp_sum(v);
@@ -780,7 +763,8 @@ static_assert(2 * LatTile<4>::FIXED + 2 * LatTile<4>::bytes(512) <= TILE_SMEM_AL
 
 // Tokens per split: as many splits as keep every CTA of the launch resident (`slots` of them), at least 128 tokens each; at most
 // 1024, because the bound may be the cache's capacity when the lengths are not known.
-void pick_splits(uint32_t slots, uint32_t ctas_per_split, uint32_t bound, uint32_t* chunk, uint32_t* splits) {
+// A split is a multiple of `unit` tokens.
+void pick_splits(uint32_t slots, uint32_t ctas_per_split, uint32_t bound, uint32_t unit, uint32_t* chunk, uint32_t* splits) {
     uint32_t n = slots / ctas_per_split;
     if (n <= 1u) {  // rows enough: no splits, whatever the length
         *chunk = bound;
@@ -788,9 +772,10 @@ void pick_splits(uint32_t slots, uint32_t ctas_per_split, uint32_t bound, uint32
         return;
     }
     n = n > 128u ? 128u : n;
-    uint32_t c = ((bound + n - 1) / n + 63u) & ~63u;
+    auto whole = [&](uint32_t v) { return (v + unit - 1) / unit * unit; };
+    uint32_t c = whole((bound + n - 1) / n);
     c = c < 128u ? 128u : (c > 1024u ? 1024u : c);
-    if ((bound + c - 1) / c > 128u) c = ((bound + 127u) / 128u + 63u) & ~63u;
+    if ((bound + c - 1) / c > 128u) c = whole((bound + 127u) / 128u);
     *chunk = c;
     *splits = (bound + c - 1) / c;
 }
@@ -837,9 +822,11 @@ int run_absorbed(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs&
         a.row_pos += at;
         const bool grouped = a.rows >= GROUPED_ROWS && takes_grouped(kv, a, w_dtype);
         // two teams per CTA where there are heads for them and rows enough to give every SM work
+        const bool tc = tiles && m40_latent_tc_takes(a);
         const uint32_t teams = tiles && a.heads > 16 && a.rows >= TEAM_ROWS ? 2 : 1, sms = (uint32_t)ctx->sm_count;
-        if (teams == 2) pick_splits(sms, a.rows * ((a.heads + 31) / 32), bound, &a.chunk, &a.splits);
-        else pick_splits(2u * sms, a.rows * (tiles ? (a.heads + 15) / 16 : a.heads), bound, &a.chunk, &a.splits);
+        const uint32_t g16 = (a.heads + 15) / 16, g32 = (a.heads + 31) / 32;
+        if (tc || teams == 2) pick_splits(sms, a.rows * g32, bound, tc ? 128u : 64u, &a.chunk, &a.splits);
+        else pick_splits(2u * sms, a.rows * (tiles ? g16 : a.heads), bound, 64u, &a.chunk, &a.splits);
         const size_t nh = (size_t)a.rows * a.heads, np = nh * a.splits;
         auto pad = [](size_t v) { return (v + 63) & ~(size_t)63; };
         const size_t part = grouped ? pad(nh * (a.rank > a.dim ? a.rank : a.dim)) : 0;  // 16-bit values
@@ -866,13 +853,17 @@ int run_absorbed(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs&
             if (e != cudaSuccess) return -6;
         }
         const dim3 grid(a.heads, a.rows, a.splits);
-        if (tiles)
+        if (tc) {
+            if ((rc = m40_latent_tc(ctx, a)) != 0) return rc;
+        } else if (tiles) {
             e = a.rank <= 128 ? launch_tiles<1>(ctx, a, teams)
                               : (a.rank <= 256 ? launch_tiles<2>(ctx, a, teams) : launch_tiles<4>(ctx, a, teams));
-        else
+            M40_COUNT_LAUNCH(ctx);
+        } else {
             e = kv->elem_f32 ? m40_launch_dependent(latent_rows_kernel<float>, grid, dim3(128), 0, s, a)
                              : m40_launch_dependent(latent_rows_kernel<__half>, grid, dim3(128), 0, s, a);
-        M40_COUNT_LAUNCH(ctx);
+            M40_COUNT_LAUNCH(ctx);
+        }
         if (e != cudaSuccess) return -6;
         e = launch_merge<WT>(ctx, a, grouped);
         M40_COUNT_LAUNCH(ctx);
