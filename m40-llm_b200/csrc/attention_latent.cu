@@ -28,7 +28,7 @@ namespace {
 constexpr uint32_t MAX_RANK = 1024;
 constexpr uint32_t RUN_ROWS = 512;   // rows per pass of the absorbed form (bounds the work space)
 constexpr uint32_t EXPAND_ROWS = 64;
-constexpr uint32_t TEAM_ROWS = 4;
+constexpr uint32_t TEAM_ROWS = 4;       // rows from which a CTA takes 32 heads
 constexpr uint32_t GROUPED_ROWS = 8;    // rows from which uk and uv go through the grouped GEMM
 constexpr size_t EXPAND_BYTES = (size_t)1 << 30;  // work space for one portion's keys and values
 
@@ -821,8 +821,8 @@ int run_absorbed(M40llmCudaContext* ctx, const M40llmKVCache* kv, const LatArgs&
         a.row_seq += at;
         a.row_pos += at;
         const bool grouped = a.rows >= GROUPED_ROWS && takes_grouped(kv, a, w_dtype);
-        // two teams per CTA where there are heads for them and rows enough to give every SM work
-        const bool tc = tiles && m40_latent_tc_takes(a);
+        // a few rows: smaller CTAs start sooner; else tcgen05, or two teams per CTA where there are heads for them
+        const bool tc = tiles && a.rows >= TEAM_ROWS && m40_latent_tc_takes(a);
         const uint32_t teams = tiles && a.heads > 16 && a.rows >= TEAM_ROWS ? 2 : 1, sms = (uint32_t)ctx->sm_count;
         const uint32_t g16 = (a.heads + 15) / 16, g32 = (a.heads + 31) / 32;
         if (tc || teams == 2) pick_splits(sms, a.rows * g32, bound, tc ? 128u : 64u, &a.chunk, &a.splits);

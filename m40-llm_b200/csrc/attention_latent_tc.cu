@@ -199,7 +199,7 @@ __global__ void __launch_bounds__(192, 1) latent_tc_kernel(const __grid_constant
         {
             const float qs = a.scale * LOG2E;
             const uint32_t pieces = a.rank / 8u;
-#pragma unroll 4
+#pragma unroll 8
             for (uint32_t i = tid; i < HP * pieces; i += 128u) {
                 const uint32_t h = i / pieces, pc = i % pieces;
                 float4 x0 = make_float4(0.f, 0.f, 0.f, 0.f), x1 = x0;
