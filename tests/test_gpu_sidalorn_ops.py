@@ -193,7 +193,7 @@ class Latent:
 
 
 LATENT = [(6, 64, 64, 128), (2, 128, 128, 512), (16, 64, 64, 64), (20, 32, 48, 80), (3, 96, 16, 256), (3, 10, 14, 21), (33, 16, 16, 48),
-          (1, 128, 128, 1024), (5, 128, 64, 192)]
+          (1, 128, 128, 1024), (5, 128, 64, 192), (40, 64, 64, 384)]
 
 
 @pytest.mark.parametrize("fp32", [0, 1])
@@ -250,6 +250,8 @@ def test_latent_attention_finds_one_far_token(nat, H, D, V, R, fp32):
         got = np.concatenate([t.run([(0, 0, 1290)], q[:1290], c[:1290], 1290)] +
                              [t.run([(0, p, 1)], q[p:p + 1], c[p:p + 1], p + 1) for p in range(1290, T)])
         close(got, want, 2e-4 if fp32 else 2e-2, f"token {place}")
+        # the last rows again, together: the form of several rows over cached latents
+        close(t.run([(0, 1290, T - 1290)], q[1290:], c[1290:], T), want[1290:], 2e-4 if fp32 else 2e-2, f"token {place}, ten rows")
         if place < T - 1:
             value = (t.uv.astype(np.float64) @ (t.cn * c[place]))
             assert np.abs(want[-1] - value).max() < 0.3 * np.abs(value).max()      # it is that token's value that comes back
