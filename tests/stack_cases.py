@@ -239,5 +239,5 @@ SIDALORN = {
     "unaligned": sidalorn([rglru(42, 3, 3, mlp=experts(7, 1, 2, 19, groups=(2, 1), scale=0.5, shared=13)),
                            latent(3, 10, 14, 21, mlp=dense(33))], width=54, vocab=61, taps=7, groups=6),
     # recurrent layers only
-    "recurrent": sidalorn([rglru(256, 4, 4, mlp=dense(144)), rglru(64, 8, 6)], width=128, vocab=150, taps=2, groups=8),
+    "recurrent": sidalorn([rglru(288, 4, 5, mlp=dense(144)), rglru(64, 8, 6)], width=128, vocab=150, taps=2, groups=8),
 }
